@@ -361,6 +361,8 @@ int ktb200_mla_kv_write(void* kv_cache, int page_size, const void* ckv, const vo
  *   `groups` equal consecutive parts times weight, and with `shift` != NULL  hs_t = h_t + (prev - h_t) * shift  where prev is the
  *   h of row prev_idx[t] of this launch (>= 0), else state row rd_row[t] (>= 0), else zero; h_t is stored to state row
  *   wr_row[t] when >= 0 (the caller double-buffers the state rows so that no launch reads a row it writes).
+ * ktb200_residual_layernorm: row r = rows ? rows[t] : t of x_in, delta_a, delta_b (each may be NULL): x = x_in + mult * (a + b) to x_out[t] (NULL: not
+ *   kept), h_out[t] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight * h_scale (NULL: the sum alone).
  * ktb200_latent_prep: proj row = [q latent | kv latent | rotated key part | ...]; writes RMS-normed q latent to cq_out and the
  *   RMS-normed kv latent + the rotated key part (over the first rot_dims; rot_layout 0: columns 2i and 2i + 1 pair up, 1: column i
  *   pairs with column i + rot_dims / 2; angle pos * inv_freq[i]; q_rank = 0: no query latent) into the
@@ -377,6 +379,8 @@ int ktb200_mla_kv_write(void* kv_cache, int page_size, const void* ckv, const vo
 int ktb200_group_rmsnorm_shift(const float* x_in, const void* delta_a, int a_type, const void* delta_b, int b_type, float mult, const float* row_add, float* x_out,
                                const void* weight, int groups, float eps, const void* shift, const int* prev_idx, const int* rd_row,
                                const int* wr_row, float* state, void* h_out, void* hs_out, int n_tokens, int width, int dtype, void* stream);
+int ktb200_residual_layernorm(const float* x_in, const void* delta_a, int a_type, const void* delta_b, int b_type, float mult, const int64_t* rows,
+                              float* x_out, const void* weight, float eps, float h_scale, void* h_out, int n_tokens, int width, int dtype, void* stream);
 int ktb200_latent_prep(const void* proj, long proj_stride, int q_rank, int kv_rank, int rot_dim, int rot_dims, int rot_layout, const double* inv_freq,
                        const void* q_norm_w, const void* kv_norm_w, float eps, const int* pos, const int* slot, const int* page_table,
                        int max_pages, int page_size, void* cache, void* cq_out, int n_tokens, int dtype, void* stream);
@@ -398,19 +402,21 @@ int ktb200_sigmoid_gate_mul(const void* heads, const void* gate, long gate_strid
                             int dtype, void* stream);
 int ktb200_poly_norm(const void* z, void* out, const float* coef, float eps, int n_tokens, int ff, int dtype, void* stream);
 int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top, const void* w_gate, const void* w_up, void* act, int n_tokens,
-                           int width, int ff, int act_kind, float limit, int dtype, void* stream);
+                           int width, int ff, int act_kind, float limit, const float* in_weights, int dtype, void* stream);
 int ktb200_experts_down(const void* act, const int64_t* ids, const float* weights, int top, const void* w_down, float* out, int n_tokens,
                         int width, int ff, int dtype, void* stream);
 /* the same for batches of a few tokens, by expert: each expert's rows are streamed once per `staged` (2 or 4; 0: chosen from the
  *   batch) pairs routed to it instead of once per pair; pair_rows [T*top][width] fp32 is scratch for the per-pair down rows
  *   before the weighted sum in slot order. */
 int ktb200_experts_gate_up_by_expert(const void* x, const int64_t* ids, int top, int n_experts, const void* w_gate, const void* w_up, void* act,
-                                     int n_tokens, int width, int ff, int staged, int act_kind, float limit, int dtype, void* stream);
+                                     int n_tokens, int width, int ff, int staged, int act_kind, float limit, const float* in_weights, int dtype,
+                                     void* stream);
 int ktb200_experts_down_by_expert(const void* act, const int64_t* ids, const float* weights, int top, int n_experts, const void* w_down,
                                   float* pair_rows, float* out, int n_tokens, int width, int ff, int staged, int dtype, void* stream);
 /* w_gate == NULL in the four calls above: experts of two matrices, act = relu(W_up x)^2.  Otherwise act_kind picks what becomes of
  * g = W_gate x and u = W_up x: 0 silu(g) u; 1 gelu(g) u (tanh form); 2 g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit),
- * u' = clamp(u, -limit, limit).
+ * u' = clamp(u, -limit, limit).  in_weights [T*top] (NULL: none): an expert sees in_weights[pair] * x; the down calls take weights == NULL
+ * as ones.
  *
  * Layers with norms on both sides of every sublayer, sigmoid attention and gated linear attention (csrc/seq_mixers.cu):
  *   ktb200_group_rmsnorm_sandwich   x_out = x_in + gnorm(y) * (w_post + weight_offset) + row_add ; h = gnorm(x_out) * (w_pre + weight_offset).
@@ -448,9 +454,10 @@ int ktb200_gla_scan(const void* proj, long proj_stride, int q_off, int k_off, in
 int ktb200_gla_out(const float* o, const void* norm_w, float eps, const void* gate, long gate_stride, void* out, int n_tokens, int heads,
                    int vdim, int dtype, void* stream);
 int ktb200_xielu(const void* z, void* out, const float* pq, long n, int dtype, void* stream);
-/* out[t][i] = that activation (act, limit as act_kind above) of gate[t * in_stride + i] and up[t * in_stride + i]; rows [gate | up]: up = gate + ff,
+/* out[t][i] = that activation (act, limit as act_kind above) of row_scale[t] (NULL: 1) times gate[t * in_stride + i] and up[t * in_stride + i]; rows [gate | up]: up = gate + ff,
  * in_stride = 2 ff.  ktb200_relu_squared: out = relu(z)^2.  ktb200_softcap: out (fp32) = cap tanh(z / cap). */
-int ktb200_gated_act_mul(const void* gate, const void* up, long in_stride, void* out, int n_tokens, int ff, int act, float limit, int dtype, void* stream);
+int ktb200_gated_act_mul(const void* gate, const void* up, long in_stride, void* out, int n_tokens, int ff, int act, float limit, const float* row_scale,
+                         int dtype, void* stream);
 int ktb200_relu_squared(const void* z, void* out, long n, int dtype, void* stream);
 int ktb200_softcap(const void* z, float* out, long n, float cap, int dtype, void* stream);
 
@@ -489,6 +496,91 @@ int ktb200_delta_prep(const void* proj, long proj_stride, int qkv_off, int b_off
                       int dtype, void* stream);
 int ktb200_delta_scan(const float* qn, const float* kn, const float* vv, const float* beta, const float* decay, int heads, int kv_heads, int dim,
                       int vdim, const int* seqs, int seqs_stride, int n_seqs, float* state, long state_stride, float* o_out, void* stream);
+
+/* The two calls above with every option of their kernels (csrc/softmax_attn.cu), arguments in a struct; unused pointers are NULL.
+ *   ktb200_qkv_prep: `maps` rows of `dim` columns per query and key head ([head][map][dim]; the values have one row per key/value head); conv_w
+ *     [channels q | k | v][taps]: a causal filter along time on every channel ahead of everything else, whose last taps - 1 inputs per
+ *     portion live at conv_off of its state rows (seqs / seq_of as for ktb200_delta_prep).
+ *   ktb200_softmax_attn: scores also lose dist_r1[h] ln(1 + dist_r2[h] (pos - j)); exp(sink[h]) joins the denominator; maps 2: two attentions per
+ *     head over the same values, o = (a1 - lambda[0] a2) / sqrt(mean_vdim(.^2) + rms_eps); out[t * out_stride + h vdim + c] =
+ *     out_scale * o * sigmoid(gate[t * gate_stride + h vdim + c]) (gate NULL: without).  Cache row: [k kv_heads*maps*dim | v kv_heads*vdim]. */
+typedef struct {
+    const void* proj;
+    long proj_stride;
+    int q_off, k_off, v_off, heads, kv_heads, maps, dim, vdim, rot_dims, rot_layout;
+    const double* inv_freq;
+    int qk_norm;
+    const void *q_weight, *k_weight;
+    int v_unit_rms;
+    float eps;
+    const void* v_other;
+    long v_other_stride;
+    const float* blend;
+    const void* conv_w;
+    int taps;
+    const int *seq_of, *seqs;
+    int seqs_stride;
+    float* state;
+    long state_stride, conv_off;
+    const int *pos, *slot, *page_table;
+    int max_pages, page_size;
+    void *cache, *q_out;
+} ktb200_qkv_prep_params;
+int ktb200_qkv_prep(const ktb200_qkv_prep_params* params, int n_tokens, int dtype, void* stream);
+typedef struct {
+    const void* q;
+    int heads, kv_heads, maps, dim, vdim;
+    float scale;
+    const float* head_scale;
+    float softcap;
+    int window, chunk;
+    const float *dist_r1, *dist_r2, *sink;
+    const void* gate;
+    long gate_stride;
+    float out_scale;
+    const float* lambda;
+    float rms_eps;
+    const int *pos, *slot, *seqs;
+    int seqs_stride, n_seqs;
+    const int* page_table;
+    int max_pages, page_size;
+    const void* cache;
+    void* out;
+    long out_stride;
+} ktb200_softmax_attn_params;
+int ktb200_softmax_attn(const ktb200_softmax_attn_params* params, int n_tokens, int splits, float* workspace, int dtype, int allow_tensor_cores,
+                        void* stream);
+size_t ktb200_softmax_attn_workspace(int n_tokens, int heads, int maps, int vdim, int splits, int tensor_cores);
+int ktb200_softmax_attn_uses_tensor_cores(int heads, int kv_heads, int maps, int dim, int vdim, int dtype);
+int ktb200_softmax_attn_tiles(int heads, int kv_heads, int maps, int n_tokens, int n_seqs);
+
+/* Mamba-2 (csrc/ssd.cu): proj rows hold [x heads*vdim | B groups*state_size | C groups*state_size] at xbc_off and one step logit per head at
+ * dt_off; conv_w [channels][taps] (last column = current token), conv_b [channels]; state rows [S heads*state_size*vdim | filter inputs
+ * (taps - 1)*channels] fp32, row stride state_stride; portions seqs[0..3][s] and seq_of as for ktb200_delta_prep.
+ *   ktb200_ssd_conv   xbc [n_tokens][channels] = silu(filter + conv_b), the portions' last taps - 1 inputs to their state rows
+ *   ktb200_ssd_scan   per portion and head p (group p / (heads / groups)), dt = softplus(logit + dt_bias[p]):
+ *                     S <- exp(-exp(a_log[p]) dt) S + dt B x^T, y [n_tokens][heads*vdim] = S^T C + d_skip[p] x; state_size <= 256
+ *   ktb200_ssd_step   both for decode steps, where every portion has one token (n_tokens = n_seqs)
+ *   ktb200_gated_group_norm   out[t * out_stride + c] = u / sqrt(mean(u^2) + eps) * weight[c] * out_scale, u = y silu(z), the mean over each of
+ *                     `groups` equal parts */
+typedef struct {
+    const void* proj;
+    long proj_stride;
+    int xbc_off, dt_off;
+    const void *conv_w, *conv_b;
+    int taps;
+    const float *dt_bias, *a_log, *d_skip;
+    int heads, groups, state_size, vdim;
+    const int *seq_of, *seqs;
+    int seqs_stride, n_seqs;
+    float* state;
+    long state_stride;
+} ktb200_ssd_params;
+int ktb200_ssd_conv(const ktb200_ssd_params* params, void* xbc, int n_tokens, int dtype, void* stream);
+int ktb200_ssd_scan(const ktb200_ssd_params* params, const void* xbc, float* y, int dtype, void* stream);
+int ktb200_ssd_step(const ktb200_ssd_params* params, float* y, int dtype, void* stream);
+int ktb200_gated_group_norm(const float* y, const void* z, long z_stride, const void* weight, int groups, float eps, float out_scale, void* out,
+                            long out_stride, int n_tokens, int width, int dtype, void* stream);
 
 /* Diagnostics (bench.py --probe): time a plain read-only stream over `bytes` of device memory.
  * mode 0 = grid-stride coalesced 16-byte loads; mode 1 = every warp reads chunk_bytes pieces at hashed offsets

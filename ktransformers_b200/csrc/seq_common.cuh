@@ -100,6 +100,31 @@ __device__ __forceinline__ float rot_turn(float own, float other, int c, int rot
     return second ? own * (float)cs + other * (float)sn : own * (float)cs - other * (float)sn;
 }
 
+// A causal filter along time on the channels of one sequence portion: channel c of the token at offset `off` becomes
+// sum_j w[c][j] u[off - taps + 1 + j][c], w's last column meeting the token itself; inputs ahead of the portion come from the state row
+// `before` ([taps - 1][C], oldest first; nullptr: zeros).  `store_tail` keeps the last taps - 1 inputs up to this token in `after`.
+template <typename T> struct ConvRows {
+    const T* rows;           // the portion's first row
+    long stride;
+    const T* w;              // [C][taps]
+    int taps, C;
+    const float* before;
+    float* after;
+    int off;
+    __device__ __forceinline__ float input(int i, int col, int c) const {      // i: offset in the portion; col: column in the rows; c: channel
+        if (i >= 0) return to_f(rows[(long)i * stride + col]);
+        return before ? before[(long)(taps - 1 + i) * C + c] : 0.f;
+    }
+    __device__ __forceinline__ float value(int col, int c) const {
+        float a = 0.f;
+        for (int j = 0; j < taps; j++) a = fmaf(to_f(w[(long)c * taps + j]), input(off - (taps - 1) + j, col, c), a);
+        return a;
+    }
+    __device__ __forceinline__ void store_tail(int col, int c) const {
+        for (int j = 0; j < taps - 1; j++) after[(long)j * C + c] = input(off + 1 - (taps - 1) + j, col, c);
+    }
+};
+
 // Gated feed-forward activations, fp32: what becomes of a (gate, up) pair of pre-activations.
 //   kActSilu        silu(g) * u
 //   kActGeluTanh    gelu(g) * u, gelu in its tanh form

@@ -590,14 +590,16 @@ __global__ void xielu_kernel(const T* __restrict__ z, T* __restrict__ out, const
 }
 
 // ------------------------------------------------------------------------------------------------ gated activation
-// out[t][i] = gated_act(gate[t * stride + i], up[t * stride + i]) (seq_common.cuh); rows [gate F | up F]: up = gate + F, stride = 2 F
+// out[t][i] = gated_act(r gate[t * stride + i], r up[t * stride + i]) (seq_common.cuh), r = row_scale ? row_scale[t] : 1; rows [gate F | up F]:
+// up = gate + F, stride = 2 F
 template <typename T>
-__global__ void gated_act_mul_kernel(const T* __restrict__ gate, const T* __restrict__ up, long stride, T* __restrict__ out, long n_rows, int F, int act, float limit) {
+__global__ void gated_act_mul_kernel(const T* __restrict__ gate, const T* __restrict__ up, long stride, T* __restrict__ out, long n_rows, int F, int act, float limit, const float* __restrict__ row_scale) {
     const long n = n_rows * F;
     for (long i = blockIdx.x * (long)blockDim.x + threadIdx.x; i < n; i += (long)gridDim.x * blockDim.x) {
         const long t = i / F;
         const int c = (int)(i - t * F);
-        out[i] = from_f<T>(gated_act(to_f(gate[t * stride + c]), to_f(up[t * stride + c]), act, limit));
+        const float r = row_scale ? row_scale[t] : 1.0f;
+        out[i] = from_f<T>(gated_act(r * to_f(gate[t * stride + c]), r * to_f(up[t * stride + c]), act, limit));
     }
 }
 // out = relu(z)^2, element by element
@@ -776,11 +778,11 @@ extern "C" int ktb200_xielu(const void* z, void* out, const float* pq, long n, i
     return KTB200_OK;
 }
 
-extern "C" int ktb200_gated_act_mul(const void* gate, const void* up, long in_stride, void* out, int n_tokens, int ff, int act, float limit, int dtype, void* stream) {
+extern "C" int ktb200_gated_act_mul(const void* gate, const void* up, long in_stride, void* out, int n_tokens, int ff, int act, float limit, const float* row_scale, int dtype, void* stream) {
     if (!gate || !up || !out || ff <= 0 || in_stride < ff || act < kActSilu || act > kActClampedGlu) { set_error("gated_act_mul: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
     SEQ_DISPATCH(dtype, (gated_act_mul_kernel<T><<<grid_for((long)n_tokens * ff, 256 * 4), 256, 0, (cudaStream_t)stream>>>((const T*)gate, (const T*)up, in_stride, (T*)out,
-                                                                                                                         n_tokens, ff, act, limit)));
+                                                                                                                         n_tokens, ff, act, limit, row_scale)));
     KTB_LAUNCH_CHECK();
     return KTB200_OK;
 }

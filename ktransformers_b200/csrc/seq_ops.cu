@@ -3,6 +3,7 @@
 //   ktb200_group_rmsnorm_shift   x_out = x_in + mult * (a + b) + row   (each optional; row: one vector for all tokens), then RMS norm in `groups` equal parts, then an
 //                                optional token shift  hs_t = h_t + (h_{t-1} - h_t) * mu  whose h_{t-1} comes from the same
 //                                step (recomputed from the previous row) or from the per-sequence state rows
+//   ktb200_residual_layernorm    x_out = x_in + mult * (a + b), then layer norm (mean taken off, weight without bias); rows picked by an index
 //   ktb200_latent_prep           what follows the fused down-projections of latent attention: RMS norm of the query latent,
 //                                RMS norm of the key/value latent, rotation of the shared rotated key part, paged cache write
 //   ktb200_sigmoid_gate_mul      heads [H][T][dv] * sigmoid(gate [T][H*dv]) -> [T][H*dv]
@@ -192,6 +193,72 @@ __global__ void __launch_bounds__(256) group_norm_shift_kernel(const float* __re
     }
 }
 
+// ------------------------------------------------------------------------------------------------ residual sum + layer norm
+// One CTA per token.  Row r = rows ? rows[t] : t of x_in, a and b:  x = x_in + mult * (a + b)  (each optional: an embedding lookup has only a),
+// x_out[t] = x, h[t] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w * h_scale.  A thread keeps its NV float4 of the row in registers through
+// both sums (NV = 0: rows of any width, staged in shared memory).
+template <typename T, int NV>
+__global__ void __launch_bounds__(NV == 0 || NV > 4 ? 256 : (NV > 2 ? 512 : 1024)) residual_layernorm_kernel(const float* __restrict__ x_in, const void* __restrict__ da, int a_type, const void* __restrict__ db, int b_type,
+                                                                                 float mult, const int64_t* __restrict__ rows, float* __restrict__ x_out, const T* __restrict__ w, float eps,
+                                                                                 float h_scale, T* __restrict__ h_out, int D) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[32];
+    const long t = blockIdx.x, r = (rows ? (long)rows[t] : t) * D;
+    const int tid = threadIdx.x;
+    if (NV > 0) {
+        float4 v[NV > 0 ? NV : 1], wv[NV > 0 ? NV : 1];
+        float s = 0.f;
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (k * blockDim.x + tid) * 4;
+            v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < D) {
+                float4 u = make_float4(0.f, 0.f, 0.f, 0.f), z = u, x = u;
+                if (x_in) x = load4(x_in + r + i);
+                if (da) u = load4_hidden(da, r + i, a_type);
+                if (db) z = load4_hidden(db, r + i, b_type);
+                if (h_out) wv[k] = load4(w + i);
+                v[k] = make_float4(fmaf(mult, u.x + z.x, x.x), fmaf(mult, u.y + z.y, x.y), fmaf(mult, u.z + z.z, x.z), fmaf(mult, u.w + z.w, x.w));
+                if (x_out) store4(x_out + t * D + i, v[k]);
+            }
+            s += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+        }
+        if (!h_out) return;
+        const float mean = block_sum(s, red) / (float)D;
+        float s2 = 0.f;
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            if ((k * (int)blockDim.x + tid) * 4 < D) {
+                v[k].x -= mean; v[k].y -= mean; v[k].z -= mean; v[k].w -= mean;
+                s2 += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+            }
+        }
+        const float inv = h_scale / sqrtf(block_sum(s2, red) / (float)D + eps);
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (k * blockDim.x + tid) * 4;
+            if (i < D) store4(h_out + t * D + i, make_float4(v[k].x * inv * wv[k].x, v[k].y * inv * wv[k].y, v[k].z * inv * wv[k].z, v[k].w * inv * wv[k].w));
+        }
+        return;
+    }
+    float s = 0.f;
+    for (int i = tid; i < D; i += blockDim.x) {
+        float u = 0.f;
+        if (da) u += load_hidden(da, r + i, a_type);
+        if (db) u += load_hidden(db, r + i, b_type);
+        const float v = fmaf(mult, u, x_in ? x_in[r + i] : 0.f);
+        if (x_out) x_out[t * D + i] = v;
+        sm[i] = v;      // read back by the same thread only
+        s += v;
+    }
+    if (!h_out) return;
+    const float mean = block_sum(s, red) / (float)D;
+    float s2 = 0.f;
+    for (int i = tid; i < D; i += blockDim.x) { const float c = sm[i] - mean; s2 += c * c; }
+    const float inv = h_scale / sqrtf(block_sum(s2, red) / (float)D + eps);
+    for (int i = tid; i < D; i += blockDim.x) h_out[t * D + i] = from_f<T>((sm[i] - mean) * inv * to_f(w[i]));
+}
+
 // ------------------------------------------------------------------------------------------------ latent prep
 // One CTA per token.  proj row = [ q latent (q_rank) | kv latent (kv_rank) | rotated key part (rot_dim) | ... ].
 template <typename T>
@@ -273,11 +340,13 @@ __global__ void __launch_bounds__(256) poly_norm_kernel(const T* __restrict__ z,
 
 // ------------------------------------------------------------------------------------------------ dense experts, per pair
 // Two kinds of expert: gated (gated_act(W_gate x, W_up x), seq_common.cuh) and, with no gate matrix (Wg == nullptr), relu(W_up x)^2.
+// in_wts (optional, one per pair): the expert sees in_wts[p] * x, i.e. both pre-activations are multiplied by it (fp32); the down kernels
+// then take no weights.
 __device__ __forceinline__ float act_relu_sq(float x) { const float r = fmaxf(x, 0.f); return r * r; }
 // grid (pairs, row blocks); a warp owns ff rows r = blockIdx.y * nw + warp (+ stride); the token's row sits in shared memory.
 template <typename T>
 __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restrict__ x, const int64_t* __restrict__ ids, int top, const T* __restrict__ Wg, const T* __restrict__ Wu,
-                                                              T* __restrict__ act, int D, int F, int act_kind, float limit) {
+                                                              T* __restrict__ act, int D, int F, int act_kind, float limit, const float* __restrict__ in_wts) {
     extern __shared__ __align__(16) float xs[];
     const long p = blockIdx.x;
     const long t = p / top;
@@ -290,7 +359,7 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
         const bool vec = rows_vectorise(Wu, D);
         for (int r = blockIdx.y * nw + warp; r < F; r += gridDim.y * nw) {
             const float su = warp_sum(lane_dot(u + (long)r * D, xs, D, lane, vec));
-            if (lane == 0) act[p * F + r] = from_f<T>(act_relu_sq(su));
+            if (lane == 0) act[p * F + r] = from_f<T>(act_relu_sq(in_wts ? su * in_wts[p] : su));
         }
         return;
     }
@@ -301,6 +370,7 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
         float su = lane_dot(u + (long)r * D, xs, D, lane, vec);
         sg = warp_sum(sg);
         su = warp_sum(su);
+        if (in_wts) { sg *= in_wts[p]; su *= in_wts[p]; }
         if (lane == 0) act[p * F + r] = from_f<T>(gated_act(sg, su, act_kind, limit));
     }
 }
@@ -319,7 +389,7 @@ __global__ void __launch_bounds__(256) experts_down_kernel(const T* __restrict__
         float acc = 0.f;      // this lane's share of sum_j w_j * (row . act_j): ONE warp reduction per output row, and the
         for (int j = 0; j < top; j++) {   // next expert's loads are not held up behind a shuffle chain
             const T* wd = Wd + (ids[t * top + j] * (long)D + d) * F;
-            acc = fmaf(wts[t * top + j], lane_dot(wd, as + j * F, F, lane, vec), acc);
+            acc = fmaf(wts ? wts[t * top + j] : 1.0f, lane_dot(wd, as + j * F, F, lane, vec), acc);
         }
         acc = warp_sum(acc);
         if (lane == 0) out[t * D + d] = acc;
@@ -452,7 +522,7 @@ __device__ __forceinline__ void lane_dot_rows(const float* const (&w)[NW], const
 // shared memory: list[P + 1] ints (padded to 16 bytes) | rows [NT][D] of T.  A warp takes two ff rows at a time (gate and up of each).
 template <typename T, int NT>
 __global__ void __launch_bounds__(256) experts_gate_up_by_expert_kernel(const T* __restrict__ x, const int64_t* __restrict__ ids, int top, int P, const T* __restrict__ Wg,
-                                                                        const T* __restrict__ Wu, T* __restrict__ act, int D, int F, int act_kind, float limit) {
+                                                                        const T* __restrict__ Wu, T* __restrict__ act, int D, int F, int act_kind, float limit, const float* __restrict__ in_wts) {
     extern __shared__ __align__(16) unsigned char sm_raw[];
     int* list = reinterpret_cast<int*>(sm_raw);
     T* xs = reinterpret_cast<T*>(sm_raw + (((size_t)(P + 1) * sizeof(int) + 15) & ~(size_t)15));
@@ -481,7 +551,8 @@ __global__ void __launch_bounds__(256) experts_gate_up_by_expert_kernel(const T*
                     if (k < m) {
 #pragma unroll
                         for (int q = 0; q < 4; q++) {
-                            const float a = warp_sum(s[q][k]);
+                            float a = warp_sum(s[q][k]);
+                            if (in_wts) a *= in_wts[list[c + k]];
                             if (lane == q && r + q < F) act[(long)list[c + k] * F + r + q] = from_f<T>(act_relu_sq(a));
                         }
                     }
@@ -501,7 +572,11 @@ __global__ void __launch_bounds__(256) experts_gate_up_by_expert_kernel(const T*
 #pragma unroll
             for (int k = 0; k < NT; k++) {
                 if (k < m) {
-                    const float a0 = warp_sum(s[0][k]), b0 = warp_sum(s[1][k]), a1 = warp_sum(s[2][k]), b1 = warp_sum(s[3][k]);
+                    float a0 = warp_sum(s[0][k]), b0 = warp_sum(s[1][k]), a1 = warp_sum(s[2][k]), b1 = warp_sum(s[3][k]);
+                    if (in_wts) {
+                        const float iw = in_wts[list[c + k]];
+                        a0 *= iw; b0 *= iw; a1 *= iw; b1 *= iw;
+                    }
                     if (lane == 0) {
                         T* o = act + (long)list[c + k] * F;
                         o[r] = from_f<T>(gated_act(a0, b0, act_kind, limit));
@@ -561,7 +636,7 @@ __global__ void __launch_bounds__(256) experts_combine_kernel(const float* __res
         const long t = i / D;
         const int d = (int)(i - t * D);
         float acc = 0.f;
-        for (int j = 0; j < top; j++) acc = fmaf(wts[t * top + j], y[(t * top + j) * D + d], acc);
+        for (int j = 0; j < top; j++) acc = fmaf(wts ? wts[t * top + j] : 1.0f, y[(t * top + j) * D + d], acc);
         out[i] = acc;
     }
 }
@@ -596,6 +671,38 @@ extern "C" int ktb200_group_rmsnorm_shift(const float* x_in, const void* delta_a
         group_norm_shift_kernel<T><<<n_tokens, 256, smem, (cudaStream_t)stream>>>(x_in, delta_a, a_type, delta_b, b_type, mult, row_add, x_out, (const T*)weight, groups, eps,
                                                                                   (const T*)shift, prev_idx, rd_row, wr_row, state, (T*)h_out, (T*)hs_out, width, stash, vec);
     });
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
+extern "C" int ktb200_residual_layernorm(const float* x_in, const void* delta_a, int a_type, const void* delta_b, int b_type, float mult, const int64_t* rows, float* x_out,
+                                         const void* weight, float eps, float h_scale, void* h_out, int n_tokens, int width, int dtype, void* stream) {
+    if ((!x_in && !delta_a) || (!x_out && !h_out) || (h_out && !weight) || width <= 0 || (x_out && x_out == x_in)) { set_error("residual_layernorm: bad argument"); return KTB200_EINVAL; }
+    if (n_tokens <= 0) return KTB200_OK;
+    auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const bool vec = width % 8 == 0 && al(x_in) && al(delta_a) && al(delta_b) && al(x_out) && al(weight) && al(h_out);
+    // wide CTAs when there are few tokens: one round of loads per thread
+    int threads = n_tokens >= 296 ? 256 : 1024;
+    while (threads > 64 && threads * 2 > width) threads >>= 1;
+    int nv = (width / 4 + threads - 1) / threads;
+    while ((nv > 2 && threads > 512) || (nv > 4 && threads > 256)) { threads >>= 1; nv = (width / 4 + threads - 1) / threads; }
+#define LN_LAUNCH(NV, TH, SM)                                                                                                                                             \
+    residual_layernorm_kernel<T, NV><<<n_tokens, TH, SM, (cudaStream_t)stream>>>(x_in, delta_a, a_type, delta_b, b_type, mult, rows, x_out, (const T*)weight, eps, h_scale, \
+                                                                                 (T*)h_out, width)
+    SEQ_DISPATCH(dtype, {
+        if (vec && nv <= 1) LN_LAUNCH(1, threads, 0);
+        else if (vec && nv <= 2) LN_LAUNCH(2, threads, 0);
+        else if (vec && nv <= 4) LN_LAUNCH(4, threads, 0);
+        else if (vec && nv <= 8) LN_LAUNCH(8, threads, 0);
+        else {
+            const size_t smem = (size_t)width * sizeof(float);
+            if (smem > 200 * 1024) { set_error("residual_layernorm: row too wide"); return KTB200_EINVAL; }
+            static size_t granted = 48 * 1024;
+            if (smem > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(residual_layernorm_kernel<T, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
+            LN_LAUNCH(0, 256, smem);
+        }
+    });
+#undef LN_LAUNCH
     KTB_LAUNCH_CHECK();
     return KTB200_OK;
 }
@@ -650,7 +757,7 @@ extern "C" int ktb200_poly_norm(const void* z, void* out, const float* coef, flo
 }
 
 extern "C" int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top, const void* w_gate, const void* w_up, void* act, int n_tokens, int width, int ff, int act_kind,
-                                      float limit, int dtype, void* stream) {
+                                      float limit, const float* in_weights, int dtype, void* stream) {
     if (!x || !ids || !w_up || !act || top <= 0 || width <= 0 || ff <= 0 || width * sizeof(float) > 200 * 1024 || act_kind < kActSilu || act_kind > kActClampedGlu) { set_error("experts_gate_up: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
     const size_t smem = (size_t)width * sizeof(float);
@@ -659,7 +766,7 @@ extern "C" int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top
     SEQ_DISPATCH(dtype, {
         static size_t granted = 48 * 1024;
         if (smem > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(experts_gate_up_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
-        experts_gate_up_kernel<T><<<dim3(n_tokens * top, ry), 256, smem, (cudaStream_t)stream>>>((const T*)x, ids, top, (const T*)w_gate, (const T*)w_up, (T*)act, width, ff, act_kind, limit);
+        experts_gate_up_kernel<T><<<dim3(n_tokens * top, ry), 256, smem, (cudaStream_t)stream>>>((const T*)x, ids, top, (const T*)w_gate, (const T*)w_up, (T*)act, width, ff, act_kind, limit, in_weights);
     });
     KTB_LAUNCH_CHECK();
     return KTB200_OK;
@@ -667,7 +774,7 @@ extern "C" int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top
 
 extern "C" int ktb200_experts_down(const void* act, const int64_t* ids, const float* weights, int top, const void* w_down, float* out, int n_tokens, int width, int ff, int dtype,
                                    void* stream) {
-    if (!act || !ids || !weights || !w_down || !out || top <= 0 || width <= 0 || ff <= 0 || (size_t)top * ff * sizeof(float) > 200 * 1024) { set_error("experts_down: bad argument"); return KTB200_EINVAL; }
+    if (!act || !ids || !w_down || !out || top <= 0 || width <= 0 || ff <= 0 || (size_t)top * ff * sizeof(float) > 200 * 1024) { set_error("experts_down: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
     const size_t smem = (size_t)top * ff * sizeof(float);
     int ry = (width + 7) / 8;
@@ -702,16 +809,16 @@ static int by_expert_staged(int staged, int pairs, int n_experts) { return stage
     })
 
 extern "C" int ktb200_experts_gate_up_by_expert(const void* x, const int64_t* ids, int top, int n_experts, const void* w_gate, const void* w_up, void* act, int n_tokens, int width,
-                                                int ff, int staged, int act_kind, float limit, int dtype, void* stream) {
+                                                int ff, int staged, int act_kind, float limit, const float* in_weights, int dtype, void* stream) {
     if (!x || !ids || !w_up || !act || top <= 0 || n_experts <= 0 || width <= 0 || ff <= 0 || act_kind < kActSilu || act_kind > kActClampedGlu) { set_error("experts_gate_up_by_expert: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
     const int P = n_tokens * top;
     if (by_expert_staged(staged, P, n_experts) == 4) {
         constexpr int NT = 4;
-        BY_EXPERT_LAUNCH(experts_gate_up_by_expert_kernel, ff, 2, (size_t)width, (const T*)x, ids, top, P, (const T*)w_gate, (const T*)w_up, (T*)act, width, ff, act_kind, limit);
+        BY_EXPERT_LAUNCH(experts_gate_up_by_expert_kernel, ff, 2, (size_t)width, (const T*)x, ids, top, P, (const T*)w_gate, (const T*)w_up, (T*)act, width, ff, act_kind, limit, in_weights);
     } else {
         constexpr int NT = 2;
-        BY_EXPERT_LAUNCH(experts_gate_up_by_expert_kernel, ff, 2, (size_t)width, (const T*)x, ids, top, P, (const T*)w_gate, (const T*)w_up, (T*)act, width, ff, act_kind, limit);
+        BY_EXPERT_LAUNCH(experts_gate_up_by_expert_kernel, ff, 2, (size_t)width, (const T*)x, ids, top, P, (const T*)w_gate, (const T*)w_up, (T*)act, width, ff, act_kind, limit, in_weights);
     }
     KTB_LAUNCH_CHECK();
     return KTB200_OK;
@@ -719,7 +826,7 @@ extern "C" int ktb200_experts_gate_up_by_expert(const void* x, const int64_t* id
 
 extern "C" int ktb200_experts_down_by_expert(const void* act, const int64_t* ids, const float* weights, int top, int n_experts, const void* w_down, float* pair_rows, float* out,
                                              int n_tokens, int width, int ff, int staged, int dtype, void* stream) {
-    if (!act || !ids || !weights || !w_down || !pair_rows || !out || top <= 0 || n_experts <= 0 || width <= 0 || ff <= 0) {
+    if (!act || !ids || !w_down || !pair_rows || !out || top <= 0 || n_experts <= 0 || width <= 0 || ff <= 0) {
         set_error("experts_down_by_expert: bad argument");
         return KTB200_EINVAL;
     }

@@ -1,0 +1,438 @@
+// Mamba-2 (state-space duality): a recurrent mixer whose matrix state per head decays by one number per token and head
+// (libktb200_seq.so).
+//
+//   ktb200_ssd_conv   prompt portions: causal filter of `taps` taps along time with bias on the [x | B | C] channels, then SiLU; the last taps - 1
+//                     inputs of every portion go to its state row
+//   ktb200_ssd_scan   per portion and head p (group j = p / (P / J)), tokens in order, fp32:
+//                         dt = softplus(. + dt_bias_p), S <- exp(-exp(A_log_p) dt) S + dt B_j x_p^T, y = S^T C_j + D_p x_p
+//   ktb200_ssd_step   decode steps (one token per portion): the filter, SiLU and the recurrence in one launch
+//   ktb200_gated_group_norm   y silu(z), every one of `groups` equal parts to unit rms, times a weight and a constant
+//
+// State row of a sequence and layer (fp32): [ S heads x state x vdim | filter inputs (taps - 1) x channels, oldest first ], read from the row
+// seqs[2][s] (or zeros when -1) and written to the row seqs[3][s]: the caller double-buffers the rows.  Storage type T (bf16 or float) for
+// projections, filter weights and the filtered channels; steps, decays, the state and everything read from it are fp32.
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+#include "seq_common.cuh"
+
+namespace ktb {
+
+__device__ __forceinline__ float ssd_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+
+// ------------------------------------------------------------------------------------------------ filter + SiLU over prompt portions
+// grid (token blocks, channel blocks); a thread owns VEC consecutive channels and runs over kConvTokens tokens with the last TAPS - 1 inputs
+// in registers (TAPS = 0: any number of taps, one channel, inputs read again per token).
+constexpr int kConvTokens = 16, kConvThreads = 128;
+template <typename T, int VEC> __device__ __forceinline__ void load_vec(float (&v)[VEC], const T* p) {
+    if (VEC == 4) {
+        const float4 u = load4(p);
+        v[0] = u.x; v[VEC > 1 ? 1 : 0] = u.y; v[VEC > 2 ? 2 : 0] = u.z; v[VEC > 3 ? 3 : 0] = u.w;
+    } else {
+        v[0] = to_f(p[0]);
+    }
+}
+template <typename T, int VEC, int TAPS>
+__global__ void __launch_bounds__(kConvThreads) ssd_conv_kernel(const T* __restrict__ in, long stride, const T* __restrict__ w, const T* __restrict__ bias, int taps_rt, int C,
+                                                                const int* __restrict__ seq_of, const int* __restrict__ seqs, int seqs_stride, float* __restrict__ state,
+                                                                long state_stride, long conv_off, T* __restrict__ out, int n_tokens) {
+    const int c = (blockIdx.y * kConvThreads + threadIdx.x) * VEC;
+    if (c >= C) return;
+    const int t0 = blockIdx.x * kConvTokens, t1 = min(n_tokens, t0 + kConvTokens);
+    constexpr int BACK = TAPS > 1 ? TAPS - 1 : 1;
+    float win[BACK][VEC], wv[TAPS > 0 ? TAPS : 1][VEC], bv[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) {
+        bv[e] = bias ? to_f(bias[c + e]) : 0.f;
+        if (TAPS > 0)
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) wv[j][e] = to_f(w[(long)(c + e) * TAPS + j]);
+    }
+    int cur = -1, start = 0, len = 0, rd = -1, wr = -1;
+    for (int t = t0; t < t1; t++) {
+        const int s = seq_of[t];
+        const bool fresh = s != cur;      // another portion, or this thread's first token: fetch the inputs ahead of it
+        if (fresh) {
+            cur = s;
+            start = seqs[s]; len = seqs[seqs_stride + s]; rd = seqs[2 * seqs_stride + s]; wr = seqs[3 * seqs_stride + s];
+        }
+        const int off = t - start;
+        const ConvRows<T> cv{in + (long)start * stride, stride, w, TAPS > 0 ? TAPS : taps_rt, C, rd >= 0 ? state + (long)rd * state_stride + conv_off : nullptr,
+                             wr >= 0 ? state + (long)wr * state_stride + conv_off : nullptr, off};
+        if (TAPS == 0) {
+            out[(long)t * C + c] = from_f<T>(act_silu(cv.value(c, c) + bv[0]));
+            if (off == len - 1 && wr >= 0) cv.store_tail(c, c);
+            continue;
+        }
+        if (fresh && TAPS > 1) {
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; j++)
+#pragma unroll
+                for (int e = 0; e < VEC; e++) win[j][e] = cv.input(off - (TAPS - 1) + j, c + e, c + e);
+        }
+        float u[VEC], y[VEC];
+        load_vec<T, VEC>(u, in + (long)t * stride + c);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) {
+            float a = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; j++) a = fmaf(wv[j][e], win[j][e], a);
+            y[e] = act_silu(fmaf(wv[TAPS - 1 > 0 ? TAPS - 1 : 0][e], u[e], a) + bv[e]);
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS - 1; j++) win[j][e] = win[j + 1][e];
+            if (TAPS > 1) win[BACK - 1][e] = u[e];
+        }
+        if (VEC == 4) store4(out + (long)t * C + c, make_float4(y[0], y[VEC > 1 ? 1 : 0], y[VEC > 2 ? 2 : 0], y[VEC > 3 ? 3 : 0]));
+        else out[(long)t * C + c] = from_f<T>(y[0]);
+        if (TAPS > 1 && off == len - 1 && wr >= 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; j++)
+#pragma unroll
+                for (int e = 0; e < VEC; e++) cv.after[(long)j * C + c + e] = win[j][e];
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ the recurrence over prompt portions
+// grid (portions, heads, column blocks of 32 value columns); 8 warps; thread (warp w, lane) keeps S[n][col] for a contiguous run of state
+// rows n in registers.  Tokens run in order in chunks of kSsdChunk staged in shared memory, the next chunk's inputs fetched into registers
+// while the current one runs; per token every warp leaves its part of y in shared memory, summed in warp order once per chunk.
+constexpr int kSsdChunk = 16, kSsdWarps = 8, kSsdRows = 32;      // state size <= 256
+template <typename T, int ROWS>
+__global__ void __launch_bounds__(256, 2) ssd_scan_kernel(const T* __restrict__ xbc, const T* __restrict__ dt_in, long dt_stride, const float* __restrict__ dt_bias,
+                                                          const float* __restrict__ a_log, const float* __restrict__ Dv, int P, int J, int N, int dv, const int* __restrict__ seqs,
+                                                          int seqs_stride, float* __restrict__ state, long state_stride, float* __restrict__ y_out) {
+    extern __shared__ __align__(16) float sm[];
+    const int rpt = (((N + kSsdWarps - 1) / kSsdWarps) + 3) & ~3, np = rpt * kSsdWarps;
+    float* Bs = sm;                              // [chunk][np]
+    float* Cs = Bs + kSsdChunk * np;             // [chunk][np]
+    float* xs = Cs + kSsdChunk * np;             // [chunk][32]
+    float* sc = xs + kSsdChunk * 32;             // [chunk][2]: decay, dt
+    float* part = sc + kSsdChunk * 2;            // [chunk][warps][32]
+    const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * 32, j = h / (P / J), inner = P * dv, C = inner + 2 * J * N;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, col = c0 + lane;
+    const int start = seqs[s], len = seqs[seqs_stride + s], rd = seqs[2 * seqs_stride + s], wr = seqs[3 * seqs_stride + s];
+    float S[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; r++) {
+        const int n = warp * rpt + r;
+        S[r] = (rd >= 0 && r < rpt && n < N && col < dv) ? state[(long)rd * state_stride + ((long)h * N + n) * dv + col] : 0.f;
+    }
+    const float rate = expf(a_log[h]), bias = dt_bias[h], Dh = Dv[h];
+    constexpr int E = kSsdChunk * ROWS * kSsdWarps / 256;      // staged state-row values per thread and array, at most
+    float rb[E], rc[E], rx[2], rdt = 0.f;
+    auto fetch = [&](int t0) {
+        const int nt = min(kSsdChunk, len - t0);
+#pragma unroll
+        for (int e = 0; e < E; e++) {
+            const int i = threadIdx.x + e * 256;
+            rb[e] = rc[e] = 0.f;
+            if (i < nt * np) {
+                const int tt = i / np, n = i - tt * np;
+                if (n < N) {
+                    const T* row = xbc + (long)(start + t0 + tt) * C + inner + j * N + n;
+                    rb[e] = to_f(row[0]);
+                    rc[e] = to_f(row[J * N]);
+                }
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int i = threadIdx.x + e * 256, c = c0 + (i & 31);
+            rx[e] = (i < nt * 32 && c < dv) ? to_f(xbc[(long)(start + t0 + (i >> 5)) * C + h * dv + c]) : 0.f;
+        }
+        if (threadIdx.x < nt) rdt = to_f(dt_in[(long)(start + t0 + threadIdx.x) * dt_stride + h]);
+    };
+    if (len > 0) fetch(0);
+    for (int t0 = 0; t0 < len; t0 += kSsdChunk) {
+        const int nt = min(kSsdChunk, len - t0);
+        __syncthreads();      // the previous chunk is consumed
+#pragma unroll
+        for (int e = 0; e < E; e++) {
+            const int i = threadIdx.x + e * 256;
+            if (i < nt * np) { Bs[i] = rb[e]; Cs[i] = rc[e]; }
+        }
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int i = threadIdx.x + e * 256;
+            if (i < nt * 32) xs[i] = rx[e];
+        }
+        if (threadIdx.x < nt) {
+            const float dt = ssd_softplus(rdt + bias);
+            sc[2 * threadIdx.x] = expf(-rate * dt);
+            sc[2 * threadIdx.x + 1] = dt;
+        }
+        __syncthreads();
+        if (t0 + kSsdChunk < len) fetch(t0 + kSsdChunk);
+#pragma unroll 2
+        for (int tt = 0; tt < nt; tt++) {
+            const float a = sc[2 * tt], xd = xs[tt * 32 + lane] * sc[2 * tt + 1];
+            const float4* br = reinterpret_cast<const float4*>(Bs + tt * np + warp * rpt);
+            const float4* cr = reinterpret_cast<const float4*>(Cs + tt * np + warp * rpt);
+            float y0 = 0.f, y1 = 0.f;
+#pragma unroll
+            for (int r4 = 0; r4 < ROWS / 4; r4++) {
+                if (4 * r4 < rpt) {
+                    const float4 b = br[r4], c = cr[r4];
+                    S[4 * r4] = fmaf(a, S[4 * r4], b.x * xd);
+                    y0 = fmaf(S[4 * r4], c.x, y0);
+                    S[4 * r4 + 1] = fmaf(a, S[4 * r4 + 1], b.y * xd);
+                    y1 = fmaf(S[4 * r4 + 1], c.y, y1);
+                    S[4 * r4 + 2] = fmaf(a, S[4 * r4 + 2], b.z * xd);
+                    y0 = fmaf(S[4 * r4 + 2], c.z, y0);
+                    S[4 * r4 + 3] = fmaf(a, S[4 * r4 + 3], b.w * xd);
+                    y1 = fmaf(S[4 * r4 + 3], c.w, y1);
+                }
+            }
+            part[(tt * kSsdWarps + warp) * 32 + lane] = y0 + y1;
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < nt * 32; i += blockDim.x) {
+            const int tt = i >> 5, c = c0 + (i & 31);
+            float y = 0.f;
+#pragma unroll
+            for (int w = 0; w < kSsdWarps; w++) y += part[(tt * kSsdWarps + w) * 32 + (i & 31)];
+            if (c < dv) y_out[(long)(start + t0 + tt) * inner + h * dv + c] = fmaf(Dh, xs[i], y);
+        }
+    }
+    if (wr >= 0) {
+#pragma unroll
+        for (int r = 0; r < ROWS; r++) {
+            const int n = warp * rpt + r;
+            if (r < rpt && n < N && col < dv) state[(long)wr * state_stride + ((long)h * N + n) * dv + col] = S[r];
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ one token per portion
+// grid (portions, heads, column blocks of `cpb` columns); a thread owns VEC columns of every `rows_par`-th state row, kStepRows of which it
+// requests before the filter of this head's x columns and its group's B and C runs.  The group's first head keeps the filter inputs of B and C.
+constexpr int kStepRows = 8;
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) ssd_step_kernel(const T* __restrict__ proj, long stride, int xbc_off, int dt_off, const T* __restrict__ w, const T* __restrict__ bias, int taps,
+                                                       const float* __restrict__ dt_bias, const float* __restrict__ a_log, const float* __restrict__ Dv, int P, int J, int N, int dv,
+                                                       const int* __restrict__ seqs, int seqs_stride, float* __restrict__ state, long state_stride, long conv_off,
+                                                       float* __restrict__ y_out, int cpb) {
+    extern __shared__ __align__(16) float sm[];
+    const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * cpb, ncol = min(cpb, dv - c0), j = h / (P / J), inner = P * dv, C = inner + 2 * J * N;
+    const int t = seqs[s], rd = seqs[2 * seqs_stride + s], wr = seqs[3 * seqs_stride + s];
+    float* xs = sm;                         // [cpb]
+    float* Bs = xs + cpb;                   // [N]
+    float* Cs = Bs + N;                     // [N]
+    float* red = Cs + N;                    // [rows_par][cpb]
+    const int tcol = cpb / VEC, rows_par = blockDim.x / tcol;      // (cpb <= 256, a multiple of VEC)
+    const int tc = threadIdx.x % tcol, tr = threadIdx.x / tcol, cc = tc * VEC;
+    const bool mine = tr < rows_par && cc < ncol;
+    const float* Sr = state + (long)rd * state_stride + (long)h * N * dv + c0 + cc;
+    float* Sw = state + (long)wr * state_stride + (long)h * N * dv + c0 + cc;
+    float v[kStepRows][VEC];
+    auto request = [&](int base) {
+#pragma unroll
+        for (int k = 0; k < kStepRows; k++) {
+            const int n = base + k * rows_par + tr;
+            if (mine && rd >= 0 && n < N) {
+                load_vec<float, VEC>(v[k], Sr + (long)n * dv);
+            } else {
+#pragma unroll
+                for (int e = 0; e < VEC; e++) v[k][e] = 0.f;
+            }
+        }
+    };
+    request(0);
+    const ConvRows<T> cv{proj + (long)t * stride + xbc_off, stride, w, taps, C, rd >= 0 ? state + (long)rd * state_stride + conv_off : nullptr,
+                         wr >= 0 ? state + (long)wr * state_stride + conv_off : nullptr, 0};
+    const bool keeps_bc = h % (P / J) == 0 && blockIdx.z == 0;
+    for (int i = threadIdx.x; i < ncol + 2 * N; i += blockDim.x) {
+        const bool is_x = i < ncol;
+        const int c = is_x ? h * dv + c0 + i : inner + (i - ncol < N ? j * N + i - ncol : J * N + j * N + i - ncol - N);
+        const float y = act_silu(cv.value(c, c) + to_f(bias[c]));
+        if (is_x) xs[i] = y;
+        else Bs[i - ncol] = y;      // (Cs follows Bs)
+        if (wr >= 0 && (is_x || keeps_bc)) cv.store_tail(c, c);
+    }
+    const float dt = ssd_softplus(to_f(proj[(long)t * stride + dt_off + h]) + dt_bias[h]);
+    const float a = expf(-expf(a_log[h]) * dt);
+    __syncthreads();
+    float xd[VEC], y[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) {
+        xd[e] = mine ? xs[cc + e] * dt : 0.f;
+        y[e] = 0.f;
+    }
+    for (int base = 0; base < N; base += kStepRows * rows_par) {
+        if (base) request(base);
+#pragma unroll
+        for (int k = 0; k < kStepRows; k++) {
+            const int n = base + k * rows_par + tr;
+            if (mine && n < N) {
+                const float b = Bs[n], c = Cs[n];
+#pragma unroll
+                for (int e = 0; e < VEC; e++) {
+                    v[k][e] = fmaf(a, v[k][e], b * xd[e]);
+                    y[e] = fmaf(v[k][e], c, y[e]);
+                }
+                if (wr >= 0) {
+                    if (VEC == 4) store4(Sw + (long)n * dv, make_float4(v[k][0], v[k][VEC > 1 ? 1 : 0], v[k][VEC > 2 ? 2 : 0], v[k][VEC > 3 ? 3 : 0]));
+                    else Sw[(long)n * dv] = v[k][0];
+                }
+            }
+        }
+    }
+    if (mine) {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) red[tr * cpb + cc + e] = y[e];
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < ncol; i += blockDim.x) {
+        float o = 0.f;
+        for (int r = 0; r < rows_par; r++) o += red[r * cpb + i];
+        y_out[(long)t * inner + h * dv + c0 + i] = fmaf(Dv[h], xs[i], o);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ gate, then grouped norm
+// grid (tokens, groups): u = y silu(z) of one part in shared memory, its mean square, out = u inv w out_scale into rows of any stride
+template <typename T>
+__global__ void __launch_bounds__(512) gated_group_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, long z_stride, const T* __restrict__ w, float eps, float out_scale,
+                                                               T* __restrict__ out, long out_stride, int n, int vec) {
+    extern __shared__ __align__(16) float u[];
+    __shared__ float red[32];
+    const long t = blockIdx.x;
+    const int lo = blockIdx.y * n;
+    const float* yr = y + t * (long)gridDim.y * n + lo;
+    const T* zr = z + t * z_stride + lo;
+    const T* wr = w + lo;
+    T* o = out + t * out_stride + lo;
+    float s = 0.f;
+    if (vec) {
+        for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+            const float4 a = load4(yr + i), g = load4(zr + i);
+            const float4 v = make_float4(a.x * act_silu(g.x), a.y * act_silu(g.y), a.z * act_silu(g.z), a.w * act_silu(g.w));
+            store4(u + i, v);
+            s += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+        }
+        const float inv = out_scale / sqrtf(block_sum(s, red) / (float)n + eps);
+        for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+            const float4 v = load4(u + i), g = load4(wr + i);
+            store4(o + i, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float v = yr[i] * act_silu(to_f(zr[i]));
+        u[i] = v;
+        s += v * v;
+    }
+    const float inv = out_scale / sqrtf(block_sum(s, red) / (float)n + eps);
+    for (int i = threadIdx.x; i < n; i += blockDim.x) o[i] = from_f<T>(u[i] * inv * to_f(wr[i]));
+}
+
+}  // namespace ktb
+
+using namespace ktb;
+
+#define SEQ_DISPATCH(dtype, ...)                                                           \
+    do {                                                                                   \
+        if ((dtype) == KTB200_TYPE_BF16) { using T = __nv_bfloat16; __VA_ARGS__; }         \
+        else if ((dtype) == KTB200_TYPE_F32) { using T = float; __VA_ARGS__; }             \
+        else { set_error("dtype must be bf16 or f32"); return KTB200_EINVAL; }             \
+    } while (0)
+#define GRANT_SMEM(kernel, smem)                                                                                                       \
+    do {                                                                                                                               \
+        static size_t granted = 48 * 1024;                                                                                             \
+        if ((smem) > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(smem))); granted = (smem); } \
+    } while (0)
+
+static bool ssd_aligned(const void* p, size_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
+static bool ssd_bad(const ktb200_ssd_params* c) {
+    return !c || !c->proj || !c->conv_w || !c->conv_b || !c->dt_bias || !c->a_log || !c->d_skip || !c->seqs || !c->state || c->heads <= 0 || c->groups <= 0 || c->heads % c->groups ||
+           c->state_size <= 0 || c->vdim <= 0 || c->taps < 1;
+}
+
+extern "C" int ktb200_ssd_conv(const ktb200_ssd_params* c, void* xbc, int n_tokens, int dtype, void* stream) {
+    if (ssd_bad(c) || !c->seq_of || !xbc) { set_error("ssd_conv: bad argument"); return KTB200_EINVAL; }
+    if (n_tokens <= 0) return KTB200_OK;
+    const int C = c->heads * c->vdim + 2 * c->groups * c->state_size;
+    const long conv_off = (long)c->heads * c->state_size * c->vdim;
+    const size_t esz = dtype == KTB200_TYPE_BF16 ? 2 : 4;
+    const bool vec = C % 4 == 0 && c->xbc_off % 4 == 0 && c->proj_stride % 4 == 0 && ssd_aligned(c->proj, 4 * esz) && ssd_aligned(xbc, 4 * esz);
+#define CONV_LAUNCH(VEC, TAPS)                                                                                                                                        \
+    ssd_conv_kernel<T, VEC, TAPS><<<dim3((n_tokens + kConvTokens - 1) / kConvTokens, (C + kConvThreads * VEC - 1) / (kConvThreads * VEC)), kConvThreads, 0,           \
+                                    (cudaStream_t)stream>>>((const T*)c->proj + c->xbc_off, c->proj_stride, (const T*)c->conv_w, (const T*)c->conv_b, c->taps, C,      \
+                                                            c->seq_of, c->seqs, c->seqs_stride, c->state, c->state_stride, conv_off, (T*)xbc, n_tokens)
+    SEQ_DISPATCH(dtype, {
+        if (vec && c->taps == 4) CONV_LAUNCH(4, 4);
+        else if (vec && c->taps == 3) CONV_LAUNCH(4, 3);
+        else if (vec && c->taps == 2) CONV_LAUNCH(4, 2);
+        else CONV_LAUNCH(1, 0);
+    });
+#undef CONV_LAUNCH
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
+extern "C" int ktb200_ssd_scan(const ktb200_ssd_params* c, const void* xbc, float* y, int dtype, void* stream) {
+    if (ssd_bad(c) || !xbc || !y || c->state_size > kSsdWarps * kSsdRows) { set_error("ssd_scan: bad argument (state size <= %d)", kSsdWarps * kSsdRows); return KTB200_EINVAL; }
+    if (c->n_seqs <= 0) return KTB200_OK;
+    const int N = c->state_size, rpt = (((N + kSsdWarps - 1) / kSsdWarps) + 3) & ~3, np = rpt * kSsdWarps;
+    const size_t smem = ((size_t)2 * kSsdChunk * np + kSsdChunk * 34 + (size_t)kSsdChunk * kSsdWarps * 32) * sizeof(float);
+    const dim3 grid(c->n_seqs, c->heads, (c->vdim + 31) / 32);
+#define SSD_LAUNCH(ROWS)                                                                                                                                                 \
+    SEQ_DISPATCH(dtype, {                                                                                                                                                \
+        GRANT_SMEM((ssd_scan_kernel<T, ROWS>), smem);                                                                                                                    \
+        ssd_scan_kernel<T, ROWS><<<grid, kSsdWarps * 32, smem, (cudaStream_t)stream>>>((const T*)xbc, (const T*)c->proj + c->dt_off, c->proj_stride, c->dt_bias, c->a_log, \
+                                                                                      c->d_skip, c->heads, c->groups, N, c->vdim, c->seqs, c->seqs_stride, c->state,     \
+                                                                                      c->state_stride, y);                                                              \
+    })
+    if (rpt <= 8) SSD_LAUNCH(8);
+    else if (rpt <= 16) SSD_LAUNCH(16);
+    else SSD_LAUNCH(32);
+#undef SSD_LAUNCH
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
+extern "C" int ktb200_ssd_step(const ktb200_ssd_params* c, float* y, int dtype, void* stream) {
+    if (ssd_bad(c) || !y) { set_error("ssd_step: bad argument"); return KTB200_EINVAL; }
+    if (c->n_seqs <= 0) return KTB200_OK;
+    const int N = c->state_size, dv = c->vdim;
+    const long conv_off = (long)c->heads * N * dv;
+    const bool vec = dv % 4 == 0 && c->state_stride % 4 == 0 && ssd_aligned(c->state, 16);
+    // columns per CTA: a head's, or 32 when that leaves SMs idle; never more than 256 threads own
+    int cpb = vec ? (dv + 3) / 4 * 4 : dv;
+    if (cpb > 256) cpb = 256;
+    if ((long)c->n_seqs * c->heads < 2 * 148 && cpb > 32) cpb = 32;
+    const int tcol = vec ? cpb / 4 : cpb, rows_par = 256 / tcol;
+    const size_t smem = ((size_t)cpb + 2 * N + (size_t)rows_par * cpb) * sizeof(float);
+    if (smem > 200 * 1024) { set_error("ssd_step: state too large for shared memory"); return KTB200_EINVAL; }
+    const dim3 grid(c->n_seqs, c->heads, (dv + cpb - 1) / cpb);
+#define STEP_LAUNCH(VEC)                                                                                                                                                \
+    SEQ_DISPATCH(dtype, {                                                                                                                                               \
+        GRANT_SMEM((ssd_step_kernel<T, VEC>), smem);                                                                                                                    \
+        ssd_step_kernel<T, VEC><<<grid, 256, smem, (cudaStream_t)stream>>>((const T*)c->proj, c->proj_stride, c->xbc_off, c->dt_off, (const T*)c->conv_w, (const T*)c->conv_b, \
+                                                                          c->taps, c->dt_bias, c->a_log, c->d_skip, c->heads, c->groups, N, dv, c->seqs, c->seqs_stride,  \
+                                                                          c->state, c->state_stride, conv_off, y, cpb);                                                \
+    })
+    if (vec) STEP_LAUNCH(4);
+    else STEP_LAUNCH(1);
+#undef STEP_LAUNCH
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
+extern "C" int ktb200_gated_group_norm(const float* y, const void* z, long z_stride, const void* weight, int groups, float eps, float out_scale, void* out, long out_stride, int n_tokens,
+                                       int width, int dtype, void* stream) {
+    if (!y || !z || !weight || !out || groups <= 0 || width <= 0 || width % groups || out_stride < width) { set_error("gated_group_norm: bad argument"); return KTB200_EINVAL; }
+    if (n_tokens <= 0) return KTB200_OK;
+    const int n = width / groups;
+    const size_t smem = (size_t)n * sizeof(float), esz = dtype == KTB200_TYPE_BF16 ? 2 : 4;
+    if (smem > 200 * 1024) { set_error("gated_group_norm: part too wide for shared memory"); return KTB200_EINVAL; }
+    const int vec = n % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0 && ssd_aligned(y, 16) && ssd_aligned(z, 4 * esz) && ssd_aligned(out, 4 * esz) && ssd_aligned(weight, 4 * esz);
+    const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : 128);
+    SEQ_DISPATCH(dtype, {
+        GRANT_SMEM(gated_group_norm_kernel<T>, smem);
+        gated_group_norm_kernel<T><<<dim3(n_tokens, groups), threads, smem, (cudaStream_t)stream>>>(y, (const T*)z, z_stride, (const T*)weight, eps, out_scale, (T*)out, out_stride, n, vec);
+    });
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}

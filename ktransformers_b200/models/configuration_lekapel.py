@@ -14,13 +14,24 @@ class RotarySpec:
     base: float
     dims: int                      # leading dimensions of the rotated part that are actually turned
     layout: str = "interleaved"    # "interleaved": columns 2i and 2i + 1 turn together; "halves": column i with column i + dims / 2
-    factor: float = 1.0            # linear scaling: every frequency is divided by this
+    factor: float = 1.0            # scaling: every frequency is divided by this, or with `original` only the slow ones (Llama 3.1):
+    low: float = 1.0               # wavelengths above original / low are stretched by factor, those below original / high are kept,
+    high: float = 1.0              # and between the two the frequency moves linearly in original / wavelength
+    original: Optional[float] = None
 
     def inv_freq(self, device):
-        """base^(-2 i / dims) / factor for the dims / 2 pairs, float64 (the kernels take the angle in fp64)"""
+        """base^(-2 i / dims) for the dims / 2 pairs, scaled, float64 (the kernels take the angle in fp64)"""
+        import math
+
         import torch
         i = torch.arange(self.dims // 2, dtype=torch.float64)
-        return (float(self.base) ** (-2.0 * i / max(self.dims, 1)) / float(self.factor)).to(device)
+        f = float(self.base) ** (-2.0 * i / max(self.dims, 1))
+        if self.original is None:
+            return (f / float(self.factor)).to(device)
+        turns = float(self.original) * f / (2.0 * math.pi)            # original / wavelength
+        span = float(self.high) - float(self.low)
+        s = ((turns - self.low) / span).clamp(0.0, 1.0) if span else (turns > self.low).to(f.dtype)
+        return ((1.0 - s) * f / float(self.factor) + s * f).to(device)
 
     @property
     def layout_code(self) -> int:

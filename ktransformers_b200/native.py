@@ -102,6 +102,31 @@ SYMBOLS = {
 }
 
 
+def _fields(text):
+    """ctypes fields of a header struct of scalars and pointers: "p": pointer, "i": int, "l": long, "f": float"""
+    kinds = {"p": C.c_void_p, "i": C.c_int, "l": C.c_long, "f": C.c_float}
+    return [(n, kinds[k]) for k, names in (part.split(":") for part in text.split()) for n in names.split(",")]
+
+
+class QkvPrepParams(C.Structure):
+    """ktb200_qkv_prep_params (include/ktb200.h)"""
+    _fields_ = _fields("p:proj l:proj_stride i:q_off,k_off,v_off,heads,kv_heads,maps,dim,vdim,rot_dims,rot_layout p:inv_freq i:qk_norm p:q_weight,k_weight i:v_unit_rms f:eps "
+                       "p:v_other l:v_other_stride p:blend p:conv_w i:taps p:seq_of,seqs i:seqs_stride p:state l:state_stride,conv_off p:pos,slot,page_table i:max_pages,page_size "
+                       "p:cache,q_out")
+
+
+class SoftmaxAttnParams(C.Structure):
+    """ktb200_softmax_attn_params (include/ktb200.h)"""
+    _fields_ = _fields("p:q i:heads,kv_heads,maps,dim,vdim f:scale p:head_scale f:softcap i:window,chunk p:dist_r1,dist_r2,sink p:gate l:gate_stride f:out_scale p:lambda_ f:rms_eps "
+                       "p:pos,slot,seqs i:seqs_stride,n_seqs p:page_table i:max_pages,page_size p:cache,out l:out_stride")
+
+
+class SsdParams(C.Structure):
+    """ktb200_ssd_params (include/ktb200.h)"""
+    _fields_ = _fields("p:proj l:proj_stride i:xbc_off,dt_off p:conv_w,conv_b i:taps p:dt_bias,a_log,d_skip i:heads,groups,state_size,vdim p:seq_of,seqs i:seqs_stride,n_seqs p:state "
+                       "l:state_stride")
+
+
 # libktb200_seq.so: the token-major operators (csrc/seq_ops.cu, csrc/window_attn.cu) + the router (csrc/gate.cu)
 _F, _D = C.c_float, C.POINTER(C.c_double)
 SEQ_SYMBOLS = {
@@ -110,6 +135,7 @@ SEQ_SYMBOLS = {
     "ktb200_moe_gate_forward": (_I, [C.POINTER(GateConfig), _I, _VP, _VP, _VP, _VP, _VP, _VP]),
     "ktb200_moe_gate_select": (_I, [C.POINTER(GateConfig), _I, _VP, _VP, _VP, _VP]),
     "ktb200_group_rmsnorm_shift": (_I, [_VP, _VP, _I, _VP, _I, _F, _VP, _VP, _VP, _I, _F, _VP, _VP, _VP, _VP, _VP, _VP, _VP, _I, _I, _I, _VP]),
+    "ktb200_residual_layernorm": (_I, [_VP, _VP, _I, _VP, _I, _F, _VP, _VP, _VP, _F, _F, _VP, _I, _I, _I, _VP]),
     "ktb200_latent_prep": (_I, [_VP, _L, _I, _I, _I, _I, _I, _VP, _VP, _VP, _F, _VP, _VP, _VP, _I, _I, _VP, _VP, _I, _I, _VP]),
     "ktb200_latent_window_attn_workspace": (C.c_size_t, [_I, _I, _I, _I]),
     "ktb200_latent_window_attn": (_I, [_VP, _VP, _I, _I, _I, _I, _I, _I, _VP, _F, _VP, _I, _VP, _VP, _VP, _I, _I, _VP, _VP, _I, _I, _VP, _I, _VP]),
@@ -118,9 +144,9 @@ SEQ_SYMBOLS = {
     "ktb200_rope_rows": (_I, [_VP, _I, _I, _I, _I, _I, _VP, _VP, _VP, _I, _I, _VP]),
     "ktb200_sigmoid_gate_mul": (_I, [_VP, _VP, _L, _VP, _I, _I, _I, _I, _VP]),
     "ktb200_poly_norm": (_I, [_VP, _VP, _VP, _F, _I, _I, _I, _VP]),
-    "ktb200_experts_gate_up": (_I, [_VP, _VP, _I, _VP, _VP, _VP, _I, _I, _I, _I, _F, _I, _VP]),
+    "ktb200_experts_gate_up": (_I, [_VP, _VP, _I, _VP, _VP, _VP, _I, _I, _I, _I, _F, _VP, _I, _VP]),
     "ktb200_experts_down": (_I, [_VP, _VP, _VP, _I, _VP, _VP, _I, _I, _I, _I, _VP]),
-    "ktb200_experts_gate_up_by_expert": (_I, [_VP, _VP, _I, _I, _VP, _VP, _VP, _I, _I, _I, _I, _I, _F, _I, _VP]),
+    "ktb200_experts_gate_up_by_expert": (_I, [_VP, _VP, _I, _I, _VP, _VP, _VP, _I, _I, _I, _I, _I, _F, _VP, _I, _VP]),
     "ktb200_experts_down_by_expert": (_I, [_VP, _VP, _VP, _I, _I, _VP, _VP, _VP, _I, _I, _I, _I, _I, _VP]),
     # csrc/seq_mixers.cu
     "ktb200_group_rmsnorm_sandwich": (_I, [_VP, _VP, _I, _VP, _VP, _VP, _VP, _VP, _I, _F, _F, _I, _I, _I, _VP]),
@@ -132,7 +158,7 @@ SEQ_SYMBOLS = {
     "ktb200_gla_scan": (_I, [_VP, _L, _I, _I, _I, _VP, _L, _VP, _F, _I, _I, _I, _VP, _I, _I, _I, _VP, _VP, _I, _VP]),
     "ktb200_gla_out": (_I, [_VP, _VP, _F, _VP, _L, _VP, _I, _I, _I, _I, _VP]),
     "ktb200_xielu": (_I, [_VP, _VP, _VP, _L, _I, _VP]),
-    "ktb200_gated_act_mul": (_I, [_VP, _VP, _L, _VP, _I, _I, _I, _F, _I, _VP]),
+    "ktb200_gated_act_mul": (_I, [_VP, _VP, _L, _VP, _I, _I, _I, _F, _VP, _I, _VP]),
     "ktb200_relu_squared": (_I, [_VP, _VP, _L, _I, _VP]),
     "ktb200_softcap": (_I, [_VP, _VP, _L, _F, _I, _VP]),
     # csrc/softmax_attn.cu, csrc/delta_rule.cu
@@ -143,6 +169,16 @@ SEQ_SYMBOLS = {
     "ktb200_window_softmax_attn_tiles": (_I, [_I, _I, _I, _I]),
     "ktb200_delta_prep": (_I, [_VP, _L, _I, _I, _I, _VP, _I, _VP, _VP, _I, _I, _I, _I, _F, _VP, _VP, _I, _VP, _L, _VP, _VP, _VP, _VP, _VP, _I, _I, _VP]),
     "ktb200_delta_scan": (_I, [_VP, _VP, _VP, _VP, _VP, _I, _I, _I, _I, _VP, _I, _I, _VP, _L, _VP, _VP]),
+    "ktb200_qkv_prep": (_I, [C.POINTER(QkvPrepParams), _I, _I, _VP]),
+    "ktb200_softmax_attn": (_I, [C.POINTER(SoftmaxAttnParams), _I, _I, _VP, _I, _I, _VP]),
+    "ktb200_softmax_attn_workspace": (C.c_size_t, [_I, _I, _I, _I, _I, _I]),
+    "ktb200_softmax_attn_uses_tensor_cores": (_I, [_I, _I, _I, _I, _I, _I]),
+    "ktb200_softmax_attn_tiles": (_I, [_I, _I, _I, _I, _I]),
+    # csrc/ssd.cu
+    "ktb200_ssd_conv": (_I, [C.POINTER(SsdParams), _VP, _I, _I, _VP]),
+    "ktb200_ssd_scan": (_I, [C.POINTER(SsdParams), _VP, _VP, _I, _VP]),
+    "ktb200_ssd_step": (_I, [C.POINTER(SsdParams), _VP, _I, _VP]),
+    "ktb200_gated_group_norm": (_I, [_VP, _VP, _L, _VP, _I, _F, _F, _VP, _L, _I, _I, _I, _VP]),
 }
 SEQ_LIB_PATH = os.path.join(_HERE, "libktb200_seq.so")
 _seq_lib = None

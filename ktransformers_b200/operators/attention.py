@@ -8,6 +8,7 @@ TMEM + TMA, csrc/mla.cu); the cache write is ktb200_mla_kv_write; the projection
 GEMVs over the bf16 halves of kv_b_proj; torch.matmul for other dtypes).  Prefill (q_len > 1 without absorb) is outside this path and raises."""
 from __future__ import annotations
 
+import ctypes as C
 import math
 from typing import Optional, Tuple
 
@@ -306,13 +307,13 @@ class KSigmoidBiasAttention(torch.nn.Module):
         return torch.nn.functional.linear(o, self.o, self.o_b)
 
 
-def softmax_attention_splits(heads: int, kv_heads: int, keys: int, n_tokens: int, n_seqs: int = 0, tensor_cores: bool = False) -> int:
-    """Into how many parts `ktb200_window_softmax_attn` cuts a key range of up to `keys` keys: more than one when a small batch
-    would leave most SMs idle on a long range."""
+def softmax_attention_splits(heads: int, kv_heads: int, keys: int, n_tokens: int, n_seqs: int = 0, tensor_cores: bool = False, maps: int = 1) -> int:
+    """Into how many parts `ktb200_softmax_attn` cuts a key range of up to `keys` keys: more than one when a small batch would leave most
+    SMs idle on a long range."""
     if tensor_cores:
-        ctas = native.seq_lib().ktb200_window_softmax_attn_tiles(heads, kv_heads, n_tokens, n_seqs) * kv_heads
+        ctas = native.seq_lib().ktb200_softmax_attn_tiles(heads, kv_heads, maps, n_tokens, n_seqs) * kv_heads
     else:
-        ctas = n_tokens * kv_heads * ((heads // kv_heads + 7) // 8)
+        ctas = n_tokens * kv_heads * maps * ((heads // kv_heads + 7) // 8)
     if ctas >= 148 or keys <= 256:
         return 1
     if tensor_cores:      # four CTAs per SM; parts of 64 keys or more
@@ -322,24 +323,56 @@ def softmax_attention_splits(heads: int, kv_heads: int, keys: int, n_tokens: int
 
 def paged_softmax_attention(q: torch.Tensor, kv: torch.Tensor, batch, cache, heads: int, kv_heads: int, dim: int, vdim: int, scale: float,
                             head_scale: Optional[torch.Tensor] = None, softcap: Optional[float] = None, window: Optional[int] = None, chunk: Optional[int] = None,
-                            tensor_cores: bool = True) -> torch.Tensor:
-    """o [T, heads * vdim] = soft-max attention of the prepared queries q [T, heads, dim] over the [k | v] rows of cache layer `kv`
-    (`ktb200_window_softmax_attn`, csrc/softmax_attn.cu): the key at position j is seen from position i when j <= i,
-    i - j < window (if a window is given) and floor(j / chunk) == floor(i / chunk) (if a chunk length is given, chunks counted from the
-    sequence's position 0); scores scale * head_scale[h] * q.k, squashed to c tanh(s / c) with c = softcap; fp32 scores and weights."""
+                            tensor_cores: bool = True, maps: int = 1, dist_bias: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, sink: Optional[torch.Tensor] = None,
+                            gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, out_scale: float = 1.0, lam: Optional[torch.Tensor] = None,
+                            rms_eps: float = 0.0) -> torch.Tensor:
+    """o [T, heads * vdim] = soft-max attention of the prepared queries q [T, heads, maps * dim] over the [k | v] rows of cache layer `kv`
+    (`ktb200_softmax_attn`, csrc/softmax_attn.cu): the key at position j is seen from position i when j <= i, i - j < window (if a window is
+    given) and floor(j / chunk) == floor(i / chunk) (if a chunk length is given, chunks counted from the sequence's position 0); scores
+    scale * head_scale[h] * q.k, squashed to c tanh(s / c) with c = softcap, less r1[h] ln(1 + r2[h] (i - j)) with dist_bias = (r1, r2); exp(sink[h])
+    joins the denominator; fp32 scores and weights.  maps = 2: two attentions per head over the same values, combined as
+    unit rms of (first - lam[0] second), `rms_eps` inside the root.  The result times out_scale times sigmoid(gate), element by element
+    (gate [T, heads * vdim], a view of any row stride), goes to `out` (a view of any row stride) or a new tensor."""
     T, dev, dt = q.shape[0], q.device, q.dtype
     lib, code, st = native.seq_lib(), native.GGML_BF16 if dt == torch.bfloat16 else native.GGML_F32, torch.cuda.current_stream(dev).cuda_stream
-    o = torch.empty((T, heads * vdim), dtype=dt, device=dev)
-    tc = bool(tensor_cores and batch.seqs is not None and lib.ktb200_window_softmax_attn_uses_tensor_cores(heads, kv_heads, dim, vdim, code))
+    o = torch.empty((T, heads * vdim), dtype=dt, device=dev) if out is None else out
+    tc = bool(tensor_cores and batch.seqs is not None and lib.ktb200_softmax_attn_uses_tensor_cores(heads, kv_heads, maps, dim, vdim, code))
+    for view in (o, gate):      # the tensor-core tiles store and read pairs of columns
+        if view is not None and (view.data_ptr() % 4 or view.stride(0) % 2):
+            tc = False
     keys = min(x for x in (window, chunk, batch.max_kv) if x)
-    splits = softmax_attention_splits(heads, kv_heads, keys, T, batch.n_seqs, tc)
-    ws = torch.empty(lib.ktb200_window_softmax_attn_workspace(T, heads, vdim, splits) // 4, dtype=torch.float32, device=dev) if splits > 1 else None
-    native.check_seq(lib.ktb200_window_softmax_attn(q.data_ptr(), heads, kv_heads, dim, vdim, float(scale), head_scale.data_ptr() if head_scale is not None else None,
-                                                    float(softcap or 0.0), int(window or 0), int(chunk or 0), batch.pos.data_ptr(), batch.slot.data_ptr(),
-                                                    batch.seqs.data_ptr() if tc else None, batch.seqs.stride(0) if tc else 0, batch.n_seqs if tc else 0,
-                                                    cache.page_table.data_ptr(), cache.max_pages_per_seq, cache.page_size, kv.data_ptr(), o.data_ptr(), T, splits,
-                                                    ws.data_ptr() if ws is not None else None, code, int(tc), st))
+    splits = softmax_attention_splits(heads, kv_heads, keys, T, batch.n_seqs, tc, maps)
+    ws_bytes = lib.ktb200_softmax_attn_workspace(T, heads, maps, vdim, splits, int(tc))
+    ws = torch.empty(ws_bytes // 4, dtype=torch.float32, device=dev) if ws_bytes else None
+    ptr = lambda t: t.data_ptr() if t is not None else None
+    r1, r2 = dist_bias if dist_bias is not None else (None, None)
+    a = native.SoftmaxAttnParams(q=q.data_ptr(), heads=heads, kv_heads=kv_heads, maps=maps, dim=dim, vdim=vdim, scale=float(scale), head_scale=ptr(head_scale),
+                                 softcap=float(softcap or 0.0), window=int(window or 0), chunk=int(chunk or 0), dist_r1=ptr(r1), dist_r2=ptr(r2), sink=ptr(sink), gate=ptr(gate),
+                                 gate_stride=gate.stride(0) if gate is not None else 0, out_scale=float(out_scale), lambda_=ptr(lam), rms_eps=float(rms_eps), pos=batch.pos.data_ptr(),
+                                 slot=batch.slot.data_ptr(), seqs=batch.seqs.data_ptr() if tc else None, seqs_stride=batch.seqs.stride(0) if tc else 0,
+                                 n_seqs=batch.n_seqs if tc else 0, page_table=cache.page_table.data_ptr(), max_pages=cache.max_pages_per_seq, page_size=cache.page_size,
+                                 cache=kv.data_ptr(), out=o.data_ptr(), out_stride=o.stride(0))
+    native.check_seq(lib.ktb200_softmax_attn(C.byref(a), T, splits, ptr(ws), code, int(tc), st))
     return o
+
+
+def qkv_prep(proj: torch.Tensor, batch, cache, kv: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, offsets, maps: int = 1, rot=None, inv_freq: Optional[torch.Tensor] = None,
+             qk_norm: int = 0, eps: float = 0.0, conv_w: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """From a projection's q, k and v columns (`offsets`) to the queries [T, heads, maps * dim] and the [k | v] rows of cache layer `kv`, one
+    `ktb200_qkv_prep` launch (csrc/softmax_attn.cu): a short causal filter on every channel (conv_w [channels, taps]; its last inputs per
+    sequence live at the front of the `state` rows), the rotation, unit rms per row (qk_norm = 1)."""
+    T, dt = proj.shape[0], proj.dtype
+    q = torch.empty((T, heads, maps * dim), dtype=dt, device=proj.device)
+    ptr = lambda t: t.data_ptr() if t is not None else None
+    rot_dims = rot.dims if rot is not None else 0
+    a = native.QkvPrepParams(proj=proj.data_ptr(), proj_stride=proj.stride(0), q_off=offsets[0], k_off=offsets[1], v_off=offsets[2], heads=heads, kv_heads=kv_heads, maps=maps, dim=dim,
+                             vdim=vdim, rot_dims=rot_dims, rot_layout=rot.layout_code if rot_dims else 0, inv_freq=ptr(inv_freq) if rot_dims else None, qk_norm=qk_norm, eps=float(eps),
+                             conv_w=ptr(conv_w), taps=conv_w.shape[1] if conv_w is not None else 0, seq_of=batch.seq_of.data_ptr(), seqs=batch.seqs.data_ptr(),
+                             seqs_stride=batch.seqs.stride(0), state=ptr(state), state_stride=state.stride(0) if state is not None else 0, conv_off=0, pos=batch.pos.data_ptr(),
+                             slot=batch.slot.data_ptr(), page_table=cache.page_table.data_ptr(), max_pages=cache.max_pages_per_seq, page_size=cache.page_size, cache=kv.data_ptr(),
+                             q_out=q.data_ptr())
+    native.check_seq(native.seq_lib().ktb200_qkv_prep(C.byref(a), T, native.GGML_BF16 if dt == torch.bfloat16 else native.GGML_F32, torch.cuda.current_stream(proj.device).cuda_stream))
+    return q
 
 
 class KCappedWindowAttention(torch.nn.Module):
@@ -472,3 +505,115 @@ class KChunkedSoftmaxAttention(torch.nn.Module):
         o = paged_softmax_attention(q, kv, batch, cache, s.heads, s.kv_heads, s.dim, s.vdim, s.scale, head_scale=self.temp, softcap=s.softcap, chunk=s.chunk,
                                     tensor_cores=self.use_tensor_cores)
         return torch.nn.functional.linear(o, self.o, self.o_b)
+
+
+class KBiasedSinkAttention(torch.nn.Module):
+    """Causal soft-max attention over grouped key/value heads inside chunks of the sequence, with unit-rms queries and keys (no weight), no
+    rotation, a logarithmic distance bias and a sink per query head, and an element-wise output gate read from the mixer's input:
+
+        P       = [W_q ; W_k ; W_v ; W_g] h                     one GEMM over the matrices that read the mixer input
+        q, k    = x / sqrt(mean(x^2) + eps) per head of P[q], P[k] ; [k | v] -> paged cache          ktb200_qkv_prep
+        s_ij    = scale q_i . k_j - r1_h ln(1 + r2_h (i - j))   for j <= i with floor(j / C) == floor(i / C), C = chunk
+        o_i     = sum_j exp(s_ij) v_j / (exp(sink_h) + sum_j exp(s_ij)) * sigmoid(P[g])              ktb200_softmax_attn
+        out     = W_o o                                         GEMM
+
+    Alone (`forward`), or side by side with another mixer of the same input (operators/side_by_side.py): `load_in` gives the rows this mixer
+    contributes to a stacked input matrix, `mix` runs everything between the two GEMMs on its columns of P and leaves `out_scale * o` in
+    a view of the stacked output operand.  Sizes, scale and the chunk length are constructor parameters
+    (models/configuration_rununex.BiasedSinkAttentionSpec).  (The reference's attention operators:
+    archive/ktransformers/operators/attention.py.)"""
+
+    use_tensor_cores = True
+
+    def __init__(self, width: int, spec, eps: float, dtype=torch.bfloat16, device="cuda", stacked: bool = False):
+        """`stacked`: the input and output matrices belong to whoever stacks this mixer with others."""
+        super().__init__()
+        P = lambda *shape, dt=dtype: torch.nn.Parameter(torch.zeros(shape, dtype=dt, device=device), requires_grad=False)
+        s = self.spec = spec
+        if s.heads % s.kv_heads:
+            raise ValueError("query heads must divide into the key/value heads")
+        self.width, self.eps = width, eps
+        self.n_q, self.n_k, self.n_v = s.heads * s.dim, s.kv_heads * s.dim, s.kv_heads * s.vdim
+        self.n_out = s.heads * s.vdim
+        self.n_rows = self.n_q + self.n_k + self.n_v + self.n_out       # rows of the input matrix
+        self.n_in = (self.n_rows + 7) // 8 * 8                           # padded so that every row of P starts 16-byte aligned
+        self.w_in, self.o = (None, None) if stacked else (P(self.n_in, width), P(width, self.n_out))
+        self.r1, self.r2, self.sink = P(s.heads, dt=torch.float32), P(s.heads, dt=torch.float32), P(s.heads, dt=torch.float32)
+
+    def load_in(self, loader, prefix: str) -> torch.Tensor:
+        return torch.cat([loader.load_tensor(prefix + n, "cpu") for n in ("q", "k", "v", "g")], 0)
+
+    def load_rest(self, loader, prefix: str):
+        for p, n in ((self.r1, "r1"), (self.r2, "r2"), (self.sink, "sink")):
+            p.data.copy_(loader.load_tensor(prefix + n, "cpu").float())
+
+    def load(self, loader, prefix: str):
+        self.w_in.data[:self.n_rows].copy_(self.load_in(loader, prefix))
+        self.load_rest(loader, prefix)
+        self.o.data.copy_(loader.load_tensor(prefix + "o", "cpu"))
+
+    def mix(self, proj: torch.Tensor, off: int, batch, cache, cache_idx: int, out: torch.Tensor, out_scale: float = 1.0) -> torch.Tensor:
+        """proj [T, >= off + n_rows]; out [T, n_out], a view of any row stride"""
+        s, T = self.spec, proj.shape[0]
+        kv = cache.key_cache[cache_idx]
+        q = qkv_prep(proj, batch, cache, kv, s.heads, s.kv_heads, s.dim, s.vdim, offsets=(off, off + self.n_q, off + self.n_q + self.n_k), qk_norm=1, eps=self.eps)
+        g_off = off + self.n_q + self.n_k + self.n_v
+        return paged_softmax_attention(q, kv, batch, cache, s.heads, s.kv_heads, s.dim, s.vdim, s.scale, chunk=s.chunk, tensor_cores=self.use_tensor_cores, dist_bias=(self.r1, self.r2),
+                                       sink=self.sink, gate=proj[:, g_off:g_off + self.n_out], out=out, out_scale=out_scale)
+
+    def forward(self, h: torch.Tensor, batch, cache, cache_idx: int) -> torch.Tensor:
+        proj = torch.nn.functional.linear(h, self.w_in)
+        o = torch.empty((h.shape[0], self.n_out), dtype=h.dtype, device=h.device)
+        return torch.nn.functional.linear(self.mix(proj, 0, batch, cache, cache_idx, o), self.o)
+
+
+class KDifferentialAttention(torch.nn.Module):
+    """Differential soft-max attention inside chunks of the sequence: every head runs two attention maps over the same values and keeps their
+    difference; q, k and v pass a short causal filter along time, q and k a partial rotation:
+
+        P        = [W_q ; W_k ; W_v] h                          one GEMM; rows of q and k head by head as [map 1 | map 2]
+        q, k, v  = filter(P) (conv taps per channel), q and k turned per map ; [k | v] -> paged cache       ktb200_qkv_prep
+        a_m      = softmax over j <= i with floor(j / C) == floor(i / C) of scale q_i,m . k_j,m, times v    (m = 1, 2)
+        o        = (1 - diff) u / sqrt(mean(u^2) + eps) , u = a_1 - lambda a_2 , per head                   ktb200_softmax_attn
+        lambda   = exp(lq1 . lk1) - exp(lq2 . lk2) + diff        one number per layer, made when the weights arrive
+        out      = W_o o                                        GEMM
+
+    The tensor-core tiles run both maps in one CTA over shared value tiles.  A sequence's state is the last conv - 1 projected inputs of every
+    channel (the cache manager's double-buffered fp32 state rows).  Sizes, scale, chunk length, taps, rotation constants and `diff` are
+    constructor parameters (models/configuration_rununex.DifferentialAttentionSpec).  (The reference's attention operators:
+    archive/ktransformers/operators/attention.py.)"""
+
+    use_tensor_cores = True
+
+    def __init__(self, width: int, spec, eps: float, dtype=torch.bfloat16, device="cuda"):
+        super().__init__()
+        P = lambda *shape, dt=dtype: torch.nn.Parameter(torch.zeros(shape, dtype=dt, device=device), requires_grad=False)
+        s = self.spec = spec
+        if s.heads % s.kv_heads:
+            raise ValueError("query heads must divide into the key/value heads")
+        self.width, self.eps = width, eps
+        self.n_q, self.n_k, self.n_v = s.heads * 2 * s.dim, s.kv_heads * 2 * s.dim, s.kv_heads * s.vdim
+        self.n_in = (self.n_q + self.n_k + self.n_v + 7) // 8 * 8       # rows padded so that every row of P starts 16-byte aligned
+        self.w_in = P(self.n_in, width)
+        self.conv_w = P(s.channels, s.conv)
+        self.lam = P(1, dt=torch.float32)
+        self.o = P(width, s.heads * s.vdim)
+        self.register_buffer("inv_freq", s.rot.inv_freq(device) if s.rot is not None and s.rot.dims else torch.zeros(1, dtype=torch.float64, device=device), persistent=False)
+
+    def load(self, loader, prefix: str):
+        t = lambda n: loader.load_tensor(prefix + n, "cpu")
+        self.w_in.data[:self.n_q + self.n_k + self.n_v].copy_(torch.cat([t("q"), t("k"), t("v")], 0))
+        self.conv_w.data.copy_(torch.cat([t("q.conv"), t("k.conv"), t("v.conv")], 0))
+        dot = lambda a, b: float((t(a).double() * t(b).double()).sum())
+        self.lam.data.fill_(math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + self.spec.diff)
+        self.o.data.copy_(t("o"))
+
+    def forward(self, h: torch.Tensor, batch, cache, cache_idx: int) -> torch.Tensor:
+        s = self.spec
+        kv = cache.key_cache[cache_idx]
+        proj = torch.nn.functional.linear(h, self.w_in)
+        q = qkv_prep(proj, batch, cache, kv, s.heads, s.kv_heads, s.dim, s.vdim, offsets=(0, self.n_q, self.n_q + self.n_k), maps=2, rot=s.rot, inv_freq=self.inv_freq,
+                     conv_w=self.conv_w, state=cache.state[cache_idx])
+        o = paged_softmax_attention(q, kv, batch, cache, s.heads, s.kv_heads, s.dim, s.vdim, s.scale, chunk=s.chunk, tensor_cores=self.use_tensor_cores, maps=2, lam=self.lam,
+                                    rms_eps=self.eps, out_scale=1.0 - s.diff)
+        return torch.nn.functional.linear(o, self.o)

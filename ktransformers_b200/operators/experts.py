@@ -586,54 +586,60 @@ class KExpertsDense(nn.Module):
         passes = T * top / (4.0 * self.experts) + 0.5
         return (passes - 1.0) * all_bytes / 5e12 > 300e-6
 
-    def forward(self, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor) -> torch.Tensor:
-        """x [T, width], ids [T, top] int64, weights [T, top] fp32 -> [T, width] fp32"""
+    def forward(self, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, on_input: bool = False) -> torch.Tensor:
+        """x [T, width], ids [T, top] int64, weights [T, top] fp32 -> [T, width] fp32.  A weight multiplies its expert's output, or with
+        `on_input` the expert's input (in fp32, as a factor of both pre-activations), and the outputs are summed as they are."""
         T, top = ids.shape
         fits = 4 * top * self.ff <= 200 * 1024 and 4 * self.width <= 200 * 1024      # the per-pair kernels stage these rows in shared memory
         staged = 4 * (T * top + 4) + self.by_expert_rows * x.element_size() * max(self.width, self.ff)
         by_expert = T >= self.by_expert_min_tokens and staged <= 200 * 1024
         if self.prefers_grouped(T, top, x.dtype) or not (fits or by_expert):
-            return self.forward_grouped(x, ids, weights)
+            return self.forward_grouped(x, ids, weights, on_input)
         act = torch.empty((T * top, self.ff), dtype=x.dtype, device=x.device)
         out = torch.empty((T, self.width), dtype=torch.float32, device=x.device)
         lib, dt, st = native.seq_lib(), TORCH_TO_GGML_HIDDEN[x.dtype], _stream(x.device)
         gate_ptr = self.gate.data_ptr() if self.gated else None
+        in_w, out_w = (weights.data_ptr(), None) if on_input else (None, weights.data_ptr())
         if by_expert:
             pair_rows = torch.empty((T * top, self.width), dtype=torch.float32, device=x.device)
             native.check_seq(lib.ktb200_experts_gate_up_by_expert(x.data_ptr(), ids.data_ptr(), top, self.experts, gate_ptr, self.up.data_ptr(),
-                                                                  act.data_ptr(), T, self.width, self.ff, self.by_expert_staged, self.act, self.limit, dt, st))
-            native.check_seq(lib.ktb200_experts_down_by_expert(act.data_ptr(), ids.data_ptr(), weights.data_ptr(), top, self.experts, self.down.data_ptr(),
+                                                                  act.data_ptr(), T, self.width, self.ff, self.by_expert_staged, self.act, self.limit, in_w, dt, st))
+            native.check_seq(lib.ktb200_experts_down_by_expert(act.data_ptr(), ids.data_ptr(), out_w, top, self.experts, self.down.data_ptr(),
                                                                pair_rows.data_ptr(), out.data_ptr(), T, self.width, self.ff, self.by_expert_staged, dt, st))
             return out
         native.check_seq(lib.ktb200_experts_gate_up(x.data_ptr(), ids.data_ptr(), top, gate_ptr, self.up.data_ptr(), act.data_ptr(), T, self.width,
-                                                    self.ff, self.act, self.limit, dt, st))
-        native.check_seq(lib.ktb200_experts_down(act.data_ptr(), ids.data_ptr(), weights.data_ptr(), top, self.down.data_ptr(), out.data_ptr(), T, self.width,
+                                                    self.ff, self.act, self.limit, in_w, dt, st))
+        native.check_seq(lib.ktb200_experts_down(act.data_ptr(), ids.data_ptr(), out_w, top, self.down.data_ptr(), out.data_ptr(), T, self.width,
                                                  self.ff, dt, st))
         return out
 
 
-    def _activate(self, g: Optional[torch.Tensor], u: torch.Tensor) -> torch.Tensor:
-        """the experts' activation over whole GEMM outputs [pairs, ff]: one elementwise launch, fp32 inside"""
+    def _activate(self, g: Optional[torch.Tensor], u: torch.Tensor, row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """the experts' activation over whole GEMM outputs [pairs, ff]: one elementwise launch, fp32 inside; row_scale [pairs] fp32
+        multiplies g and u first"""
         lib, st, out = native.seq_lib(), _stream(u.device), torch.empty_like(u)
         if g is None:
+            if row_scale is not None:
+                u = (u.float() * row_scale.unsqueeze(-1)).to(u.dtype)
             native.check_seq(lib.ktb200_relu_squared(u.data_ptr(), out.data_ptr(), u.numel(), TORCH_TO_GGML_HIDDEN[u.dtype], st))
         else:
             native.check_seq(lib.ktb200_gated_act_mul(g.data_ptr(), u.data_ptr(), self.ff, out.data_ptr(), u.shape[0], self.ff, self.act, self.limit,
-                                                      TORCH_TO_GGML_HIDDEN[u.dtype], st))
+                                                      row_scale.data_ptr() if row_scale is not None else None, TORCH_TO_GGML_HIDDEN[u.dtype], st))
         return out
 
-    def forward_grouped(self, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor) -> torch.Tensor:
+    def forward_grouped(self, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, on_input: bool = False) -> torch.Tensor:
         T, top = ids.shape
         F = nn.functional
         flat = ids.reshape(-1)
         order = torch.argsort(flat, stable=True)
         counts = torch.bincount(flat, minlength=self.experts)
         xs = x.index_select(0, torch.div(order, top, rounding_mode="floor"))
+        rs = weights.reshape(-1).index_select(0, order) if on_input else None            # the weights in the order of the sorted pairs
         if x.dtype == torch.bfloat16 and self.width % 8 == 0 and self.ff % 8 == 0 and hasattr(F, "grouped_mm"):
             # the library's grouped GEMM takes the segment ends on the device: no host read of the routing, three launches
             offs = counts.cumsum(0).to(torch.int32)
             u = F.grouped_mm(xs, self.up.transpose(1, 2), offs=offs)
-            a = self._activate(F.grouped_mm(xs, self.gate.transpose(1, 2), offs=offs) if self.gated else None, u)
+            a = self._activate(F.grouped_mm(xs, self.gate.transpose(1, 2), offs=offs) if self.gated else None, u, rs)
             y = F.grouped_mm(a, self.down.transpose(1, 2), offs=offs)
         else:
             y = torch.empty((T * top, self.width), dtype=x.dtype, device=x.device)
@@ -641,12 +647,13 @@ class KExpertsDense(nn.Module):
             for e, n in enumerate(counts.tolist()):                              # one host read of a step's routing
                 if n:
                     seg = xs[lo:lo + n]
-                    a = self._activate(F.linear(seg, self.gate[e]) if self.gated else None, F.linear(seg, self.up[e]))
+                    a = self._activate(F.linear(seg, self.gate[e]) if self.gated else None, F.linear(seg, self.up[e]), rs[lo:lo + n] if on_input else None)
                     y[lo:lo + n] = F.linear(a, self.down[e])
                     lo += n
         pairs = torch.empty_like(y)
         pairs[order] = y
-        return (pairs.view(T, top, self.width).float() * weights.unsqueeze(-1)).sum(1)
+        pairs = pairs.view(T, top, self.width).float()
+        return pairs.sum(1) if on_input else (pairs * weights.unsqueeze(-1)).sum(1)
 
 
 class KSoftmaxTopKMoE(nn.Module):
@@ -704,3 +711,27 @@ class KGroupedSigmoidMoE(nn.Module):
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         ids, w = self.router(h)
         return self.experts(h, ids, w)
+
+
+class KSharedSigmoidMoE(nn.Module):
+    """router (operators/gate.KSigmoidTopKGate: the `top` largest sigmoid scores, which are the weights as they are) -> dense gated experts whose
+    weight multiplies their INPUT, plus a shared gated expert that every token uses (operators/mlp.KGatedMLP).  Returns the two parts
+    (routed sum fp32, shared output in the compute dtype): the next residual sum takes both."""
+
+    def __init__(self, width: int, ff: int, experts: int, top: int, shared_ff: Optional[int], act: str = "silu", dtype=torch.bfloat16, device="cuda"):
+        super().__init__()
+        from .gate import KSigmoidTopKGate
+        from .mlp import KGatedMLP
+        self.router = KSigmoidTopKGate(width, experts, top, device=device)
+        self.experts = KExpertsDense(width, ff, experts, dtype=dtype, device=device, act=act)
+        self.shared = KGatedMLP(width, shared_ff, act=act, dtype=dtype, device=device) if shared_ff else None
+
+    def load(self, loader, prefix: str):
+        self.router.load(loader, prefix + "router")
+        self.experts.load(loader, prefix)
+        if self.shared is not None:
+            self.shared.load(loader, prefix + "shared.")
+
+    def forward(self, h: torch.Tensor):
+        ids, w = self.router(h)
+        return self.experts(h, ids, w, on_input=True), self.shared(h) if self.shared is not None else None

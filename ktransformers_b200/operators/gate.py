@@ -197,3 +197,38 @@ class KGroupedSigmoidGate(nn.Module):
         else:
             native.check_seq(native.seq_lib().ktb200_moe_gate_forward(C.byref(cfg), n, x.data_ptr(), idx.data_ptr(), wt.data_ptr(), None, None, st))
         return idx, wt
+
+
+class KSigmoidTopKGate(nn.Module):
+    """Sigmoid scores s = sigmoid(W x) in fp32, the `top` largest chosen, their scores the weights as they are (no correction, no groups, not
+    normalised): the router kernel's `scoring = sigmoid, topk_method = greedy, norm_topk_prob = 0, routed_scaling_factor = 1` case.  As for
+    KGroupedSigmoidGate, decode-sized batches run the one-launch kernel, and batches from `gemm_min_tokens` tokens an fp32 library GEMM (TF32
+    off) and `ktb200_moe_gate_select`; more than 512 experts or 32 choices select with torch's top-k."""
+
+    gemm_min_tokens = 48
+
+    def __init__(self, width: int, experts: int, top: int, device="cuda"):
+        super().__init__()
+        if not 1 <= top <= experts:
+            raise ValueError(f"router: {top} choices among {experts} experts")
+        self.width, self.experts, self.top = width, experts, top
+        self.weight = nn.Parameter(torch.empty((experts, width), dtype=torch.float32, device=device), requires_grad=False)
+
+    def load(self, loader, key: str):
+        self.weight.data.copy_(loader.load_tensor(key, "cpu").float())
+
+    def forward(self, x: torch.Tensor):
+        n = x.shape[0]
+        if self.experts > 512 or self.top > 32:
+            wt, idx = torch.topk(torch.sigmoid(nn.functional.linear(x.float(), self.weight)), self.top, dim=-1)
+            return idx, wt.contiguous()
+        idx = torch.empty((n, self.top), dtype=torch.int64, device=x.device)
+        wt = torch.empty((n, self.top), dtype=torch.float32, device=x.device)
+        cfg = native.GateConfig(self.experts, self.width, self.top, 1, 1, _SCORING["sigmoid"], _TOPK["greedy"], 0, 1.0, self.weight.data_ptr(), None, TORCH_TO_GGML_HIDDEN[x.dtype])
+        st = torch.cuda.current_stream(x.device).cuda_stream
+        if n >= self.gemm_min_tokens or self.width % 4:
+            logits = nn.functional.linear(x.float(), self.weight)
+            native.check_seq(native.seq_lib().ktb200_moe_gate_select(C.byref(cfg), n, logits.data_ptr(), idx.data_ptr(), wt.data_ptr(), st))
+        else:
+            native.check_seq(native.seq_lib().ktb200_moe_gate_forward(C.byref(cfg), n, x.data_ptr(), idx.data_ptr(), wt.data_ptr(), None, None, st))
+        return idx, wt

@@ -1,4 +1,5 @@
 """Recurrent mixers with a matrix state per head.  KGatedDeltaRule (below) — the gated delta rule behind short convolutions.
+KStateSpace (below) — Mamba-2 (state-space duality): one decay per token and head.
 KGatedLinearAttention — linear attention with a decay per key channel and a recurrent matrix state per head:
 
     q = W_q h / sqrt(dim) ,  k = W_k h ,  v = W_v h ,  a = sigmoid(W_a2 (W_a1 h) + b) ** (1 / tau)        (a per head and key channel)
@@ -17,6 +18,8 @@ result does not depend on where the prompt was cut.  `cache_idx` picks the cache
 can run several times per step with separate states.  (The reference has no recurrent mixer; its caches are per-token:
 archive/ktransformers/models/custom_cache.py:26-200.)"""
 from __future__ import annotations
+
+import ctypes as C
 
 import torch
 from torch import nn
@@ -136,3 +139,80 @@ class KGatedDeltaRule(nn.Module):
         native.check_seq(lib.ktb200_gla_out(o.data_ptr(), self.norm.data_ptr(), float(self.eps), proj[:, self.g_off:].data_ptr(), self.n_in, og.data_ptr(), T,
                                             s.heads, s.vdim, code, st))
         return torch.nn.functional.linear(og, self.o)
+
+
+class KStateSpace(nn.Module):
+    """Mamba-2 (state-space duality), a recurrent mixer with a state_size x vdim matrix per head whose decay is one number per token and head:
+
+        [z | x | B | C | dt] = W_in h                          x: heads x vdim; B, C: groups x state_size, shared by heads / groups heads each
+        x, B, C = silu(filter(x, B, C) + b)                     a causal filter of `conv` taps along time on every channel
+        dt      = softplus(dt + dt_bias) ;  S <- exp(-exp(A_log) dt) S + dt B x^T ;  y = S^T C + D x      per head, S in fp32
+        out     = W_o (norm(y silu(z)) w)                       norm: `norm_groups` equal parts, each divided by its own rms
+
+        P     = W_in h                                          one GEMM
+        y     = prompt portions: ktb200_ssd_conv + ktb200_ssd_scan; decode steps (one token per sequence): ktb200_ssd_step
+        o     = ktb200_gated_group_norm                         (the gate comes before the norm)
+        out   = W_o o                                           GEMM
+
+    A sequence's state — the matrices and the last conv - 1 inputs of every filtered channel — lives in the cache manager's double-buffered
+    fp32 state rows (models/custom_cache.PagedStateCache).  Alone (`forward`), or side by side with another mixer of the same input
+    (operators/side_by_side.py) through `load_in` and `mix`, as KBiasedSinkAttention.  Sizes are constructor parameters
+    (models/configuration_rununex.StateSpaceSpec).  (The reference has no recurrent mixer.)"""
+
+    def __init__(self, width: int, spec, eps: float, dtype=torch.bfloat16, device="cuda", stacked: bool = False):
+        """`stacked`: the input and output matrices belong to whoever stacks this mixer with others."""
+        super().__init__()
+        P = lambda *shape, dt=dtype: nn.Parameter(torch.zeros(shape, dtype=dt, device=device), requires_grad=False)
+        s = self.spec = spec
+        if s.heads % s.groups or s.inner % s.norm_groups:
+            raise ValueError("state-space heads must divide into the groups, and the inner size into the norm groups")
+        self.width, self.eps = width, eps
+        self.n_out = s.inner
+        self.n_rows = s.inner + s.channels + s.heads
+        self.n_in = (self.n_rows + 7) // 8 * 8
+        self.w_in, self.o = (None, None) if stacked else (P(self.n_in, width), P(width, self.n_out))
+        self.conv_w, self.conv_b = P(s.channels, s.conv), P(s.channels)
+        self.dt_bias, self.a_log, self.d_skip = P(s.heads, dt=torch.float32), P(s.heads, dt=torch.float32), P(s.heads, dt=torch.float32)
+        self.norm = P(s.inner)
+
+    def load_in(self, loader, prefix: str) -> torch.Tensor:
+        return loader.load_tensor(prefix + "in", "cpu")
+
+    def load_rest(self, loader, prefix: str):
+        t = lambda n: loader.load_tensor(prefix + n, "cpu")
+        self.conv_w.data.copy_(t("conv"))
+        self.conv_b.data.copy_(t("conv.b"))
+        self.dt_bias.data.copy_(t("dt_bias").float())
+        self.a_log.data.copy_(t("A_log").float())
+        self.d_skip.data.copy_(t("D").float())
+        self.norm.data.copy_(t("norm"))
+
+    def load(self, loader, prefix: str):
+        self.w_in.data[:self.n_rows].copy_(self.load_in(loader, prefix))
+        self.load_rest(loader, prefix)
+        self.o.data.copy_(loader.load_tensor(prefix + "o", "cpu"))
+
+    def mix(self, proj: torch.Tensor, off: int, batch, cache, cache_idx: int, out: torch.Tensor, out_scale: float = 1.0) -> torch.Tensor:
+        """proj [T, >= off + n_rows]; out [T, n_out], a view of any row stride"""
+        s, T, dev, dt = self.spec, proj.shape[0], proj.device, proj.dtype
+        lib, code, st = native.seq_lib(), native.GGML_BF16 if dt == torch.bfloat16 else native.GGML_F32, torch.cuda.current_stream(dev).cuda_stream
+        state = cache.state[cache_idx]
+        a = native.SsdParams(proj=proj.data_ptr(), proj_stride=proj.stride(0), xbc_off=off + s.inner, dt_off=off + s.inner + s.channels, conv_w=self.conv_w.data_ptr(),
+                             conv_b=self.conv_b.data_ptr(), taps=s.conv, dt_bias=self.dt_bias.data_ptr(), a_log=self.a_log.data_ptr(), d_skip=self.d_skip.data_ptr(), heads=s.heads,
+                             groups=s.groups, state_size=s.state_size, vdim=s.vdim, seq_of=batch.seq_of.data_ptr(), seqs=batch.seqs.data_ptr(), seqs_stride=batch.seqs.stride(0),
+                             n_seqs=batch.n_seqs, state=state.data_ptr(), state_stride=state.stride(0))
+        y = torch.empty((T, s.inner), dtype=torch.float32, device=dev)
+        if T == batch.n_seqs:
+            native.check_seq(lib.ktb200_ssd_step(C.byref(a), y.data_ptr(), code, st))
+        else:
+            xbc = torch.empty((T, s.channels), dtype=dt, device=dev)
+            native.check_seq(lib.ktb200_ssd_conv(C.byref(a), xbc.data_ptr(), T, code, st))
+            native.check_seq(lib.ktb200_ssd_scan(C.byref(a), xbc.data_ptr(), y.data_ptr(), code, st))
+        native.check_seq(lib.ktb200_gated_group_norm(y.data_ptr(), proj[:, off:].data_ptr(), proj.stride(0), self.norm.data_ptr(), s.norm_groups, float(self.eps), float(out_scale),
+                                                     out.data_ptr(), out.stride(0), T, s.inner, code, st))
+        return out
+
+    def forward(self, h: torch.Tensor, batch, cache, cache_idx: int) -> torch.Tensor:
+        proj = nn.functional.linear(h, self.w_in)
+        o = torch.empty((h.shape[0], self.n_out), dtype=h.dtype, device=h.device)
+        return nn.functional.linear(self.mix(proj, 0, batch, cache, cache_idx, o), self.o)

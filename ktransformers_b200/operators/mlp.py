@@ -86,7 +86,7 @@ class KGatedMLP(nn.Module):
         gu = F.linear(h, self.gate_up)
         a = torch.empty((h.shape[0], self.ff), dtype=gu.dtype, device=gu.device)
         native.check_seq(native.seq_lib().ktb200_gated_act_mul(gu.data_ptr(), gu.data_ptr() + self.ff * gu.element_size(), 2 * self.ff, a.data_ptr(), gu.shape[0], self.ff,
-                                                               self.act, 0.0, GGML_OF[gu.dtype], torch.cuda.current_stream(gu.device).cuda_stream))
+                                                               self.act, 0.0, None, GGML_OF[gu.dtype], torch.cuda.current_stream(gu.device).cuda_stream))
         return F.linear(a, self.down)
 
 

@@ -103,3 +103,36 @@ class KGroupRMSNorm(nn.Module):
         if cast_h and pre is None and not plain_h:
             h = x_out
         return x_out, h
+
+
+class KLayerNorm(nn.Module):
+    """Layer norm with a weight and no bias, fused with the residual sum before it: one `ktb200_residual_layernorm` launch (csrc/seq_ops.cu) for
+
+        x = x_in + mult * (a + b)                            (every term optional; an embedding lookup is a = table, rows = token ids)
+        h = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight * h_scale
+
+    The residual stream stays fp32; h is rounded once to the compute dtype.  `rows` [T] int64 picks the rows of x_in, a and b."""
+
+    def __init__(self, width: int, eps: float, dtype=torch.bfloat16, device="cuda"):
+        super().__init__()
+        self.width, self.eps = width, float(eps)
+        self.weight = nn.Parameter(torch.ones(width, dtype=dtype, device=device), requires_grad=False)
+
+    def load(self, loader, key: str):
+        self.weight.data.copy_(loader.load_tensor(key, "cpu"))
+
+    def forward(self, x: Optional[torch.Tensor], a: Optional[torch.Tensor] = None, b: Optional[torch.Tensor] = None, mult: float = 1.0, rows: Optional[torch.Tensor] = None,
+                keep_x: bool = True, want_h: bool = True, h_scale: float = 1.0):
+        """Returns (x after the sum in fp32 or None, h or None)."""
+        ref = x if x is not None else a
+        T, dt, dev = (ref.shape[0] if rows is None else rows.shape[0]), self.weight.dtype, ref.device
+        for d in (x, a, b):
+            assert d is None or (d.is_contiguous() and d.shape[-1] == self.width)
+        assert rows is None or (rows.dtype == torch.int64 and rows.is_contiguous())
+        plain = rows is None and a is None and b is None and x is not None      # nothing to add: the stream stays where it is
+        x_out = torch.empty((T, self.width), dtype=torch.float32, device=dev) if keep_x and not plain else None
+        h = torch.empty((T, self.width), dtype=dt, device=dev) if want_h else None
+        native.check_seq(native.seq_lib().ktb200_residual_layernorm(
+            _ptr(x), _ptr(a), GGML_OF[a.dtype] if a is not None else 0, _ptr(b), GGML_OF[b.dtype] if b is not None else 0, float(mult), _ptr(rows), _ptr(x_out), self.weight.data_ptr(),
+            self.eps, float(h_scale), _ptr(h), T, self.width, GGML_OF[dt], torch.cuda.current_stream(dev).cuda_stream))
+        return (x if plain else x_out), h

@@ -314,7 +314,7 @@ def kernel_leg(flush, peak_gbs, have_main_lib):
         ids = torch.stack([torch.randperm(E, generator=g, device=dev)[:top] for _ in range(T)]).to(torch.int64)
         wts = torch.rand(T, top, generator=g, device=dev)
         act, out = torch.empty(T * top, ff, dtype=bf, device=dev), torch.empty(T, D, device=dev)
-        f1 = lambda: native.check_seq(seq.ktb200_experts_gate_up(x.data_ptr(), ids.data_ptr(), top, Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0.0, 30, S()))
+        f1 = lambda: native.check_seq(seq.ktb200_experts_gate_up(x.data_ptr(), ids.data_ptr(), top, Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0.0, None, 30, S()))
         f2 = lambda: native.check_seq(seq.ktb200_experts_down(act.data_ptr(), ids.data_ptr(), wts.data_ptr(), top, Wd.data_ptr(), out.data_ptr(), T, D, ff, 30, S()))
         uniq = len(set(ids.flatten().tolist()))                            # every chosen expert is read from HBM at least once
         row("experts_gate_up_kernel", f"T={T} top={top} width={D} ff={ff} bf16", timed(f1, flush), uniq * 2 * ff * D * 2,
@@ -326,7 +326,7 @@ def kernel_leg(flush, peak_gbs, have_main_lib):
         ids = torch.stack([torch.randperm(E, generator=g, device=dev)[:top] for _ in range(T)]).to(torch.int64)
         wts = torch.rand(T, top, generator=g, device=dev)
         act, out, pair_rows = torch.empty(T * top, ff, dtype=bf, device=dev), torch.empty(T, D, device=dev), torch.empty(T * top, D, device=dev)
-        f1 = lambda: native.check_seq(seq.ktb200_experts_gate_up_by_expert(x.data_ptr(), ids.data_ptr(), top, E, Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0, 0.0, 30, S()))
+        f1 = lambda: native.check_seq(seq.ktb200_experts_gate_up_by_expert(x.data_ptr(), ids.data_ptr(), top, E, Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0, 0.0, None, 30, S()))
         f2 = lambda: native.check_seq(seq.ktb200_experts_down_by_expert(act.data_ptr(), ids.data_ptr(), wts.data_ptr(), top, E, Wd.data_ptr(), pair_rows.data_ptr(), out.data_ptr(),
                                                                         T, D, ff, 0, 30, S()))
         uniq = len(set(ids.flatten().tolist()))
@@ -468,8 +468,8 @@ def mabidra_kernel_leg(flush, peak_gbs, peak_tflops):
         ids = torch.stack([torch.randperm(E, generator=g, device=dev)[:top] for _ in range(T)]).to(torch.int64)
         act = torch.empty(T * top, ff, dtype=bf, device=dev)
         uniq = len(set(ids.flatten().tolist()))
-        ours = timed(lambda: native.check_seq(seq.ktb200_experts_gate_up_by_expert(x.data_ptr(), ids.data_ptr(), top, E, None, Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0, 0.0, 30, S())), flush)
-        ms = timed(lambda: native.check_seq(seq.ktb200_experts_gate_up_by_expert(x.data_ptr(), ids.data_ptr(), top, E, Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0, 0.0, 30, S())), flush)
+        ours = timed(lambda: native.check_seq(seq.ktb200_experts_gate_up_by_expert(x.data_ptr(), ids.data_ptr(), top, E, None, Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0, 0.0, None, 30, S())), flush)
+        ms = timed(lambda: native.check_seq(seq.ktb200_experts_gate_up_by_expert(x.data_ptr(), ids.data_ptr(), top, E, Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0, 0.0, None, 30, S())), flush)
         row("experts_gate_up_by_expert_kernel (no gate, relu^2)", f"T={T} top={top} width={D} ff={ff} bf16", ours, nbytes=uniq * ff * D * 2,
             peer={"kernel": "experts_gate_up_by_expert_kernel (gated)", "us": ms * 1e3, "frac_of_measured_hbm": uniq * 2 * ff * D * 2 / ms / 1e6 / peak_gbs})
     return rows
@@ -621,7 +621,7 @@ def zivulix_kernel_leg(flush, peak_gbs, peak_tflops):
     # ---- activation
     for T, ff in ((8, 18432), (2048, 18432)):
         gu, oo, zz, pq = rn(T, 2 * ff), torch.empty(T, ff, dtype=bf, device=dev), rn(T, ff), torch.tensor([0.3, -0.2], device=dev)
-        ours = timed(lambda: native.check_seq(seq.ktb200_gated_act_mul(gu.data_ptr(), gu.data_ptr() + 2 * ff, 2 * ff, oo.data_ptr(), T, ff, 1, 0.0, 30, S())), flush)
+        ours = timed(lambda: native.check_seq(seq.ktb200_gated_act_mul(gu.data_ptr(), gu.data_ptr() + 2 * ff, 2 * ff, oo.data_ptr(), T, ff, 1, 0.0, None, 30, S())), flush)
         ms = timed(lambda: native.check_seq(seq.ktb200_xielu(zz.data_ptr(), oo.data_ptr(), pq.data_ptr(), zz.numel(), 30, S())), flush)
         row("gated_act_mul_kernel (gelu_tanh)", f"T={T} ff={ff}", ours, nbytes=T * ff * 6, peer=peer_of("xielu_kernel", ms, T * ff * 4))
     return rows
@@ -752,7 +752,7 @@ def bilurax_kernel_leg(flush, peak_gbs, peak_tflops):
         ids = torch.stack([torch.randperm(E, generator=g, device=dev)[:top] for _ in range(T)])
         uniq = int(ids.unique().numel())
         fn = lambda kind, lim: native.check_seq(seq.ktb200_experts_gate_up_by_expert(x.data_ptr(), ids.data_ptr(), top, E, Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, kind,
-                                                                                     lim, 30, S()))
+                                                                                     lim, None, 30, S()))
         ours, ms = timed(lambda: fn(2, 7.0), flush), timed(lambda: fn(0, 0.0), flush)
         nb = uniq * 2 * ff * D * 2
         row("experts_gate_up_by_expert_kernel (clamped sigmoid form)", f"T={T} top={top} width={D} ff={ff} bf16", ours, nbytes=nb,
@@ -761,8 +761,8 @@ def bilurax_kernel_leg(flush, peak_gbs, peak_tflops):
     for P in (64, 2048 * 8):
         gg, uu, oo = rn(P, ff), rn(P, ff), torch.empty(P, ff, dtype=bf, device=dev)
         gu = rn(P, 2 * ff)
-        ours = timed(lambda: native.check_seq(seq.ktb200_gated_act_mul(gg.data_ptr(), uu.data_ptr(), ff, oo.data_ptr(), P, ff, 2, 7.0, 30, S())), flush)
-        ms = timed(lambda: native.check_seq(seq.ktb200_gated_act_mul(gu.data_ptr(), gu.data_ptr() + 2 * ff, 2 * ff, oo.data_ptr(), P, ff, 1, 0.0, 30, S())), flush)
+        ours = timed(lambda: native.check_seq(seq.ktb200_gated_act_mul(gg.data_ptr(), uu.data_ptr(), ff, oo.data_ptr(), P, ff, 2, 7.0, None, 30, S())), flush)
+        ms = timed(lambda: native.check_seq(seq.ktb200_gated_act_mul(gu.data_ptr(), gu.data_ptr() + 2 * ff, 2 * ff, oo.data_ptr(), P, ff, 1, 0.0, None, 30, S())), flush)
         row("gated_act_mul_kernel (clamped sigmoid form, separate gate and up rows)", f"pairs={P} ff={ff}", ours, nbytes=P * ff * 6,
             peer=peer_of("gated_act_mul_kernel (gelu_tanh, stacked rows)", ms, P * ff * 6))
     for T, F_ in ((8, 18432), (2048, 18432)):
