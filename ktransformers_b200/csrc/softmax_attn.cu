@@ -190,6 +190,145 @@ __global__ void __launch_bounds__(256) rope_norm_cache_write_kernel(const QkvPre
     }
 }
 
+// The same behind a filter, by column pairs: grid (tiles of `tile` consecutive tokens, unit blocks), a warp per unit walks over the tile's tokens with
+// the filter's last TAPS - 1 inputs in registers, a lane owning the column pairs 2 lane + 64 e: every input is read once per tile instead of TAPS
+// times, a rotated pair (interleaved layout) lies in one lane, loads and stores take two columns.  Loads of kPairBatch tokens are in flight
+// together.  Even head sizes and offsets; no row-wide norm, value blend or value norm (those take the kernel above).
+constexpr int kPairTile = 16, kPairBatch = 4;
+__device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 load2(const __nv_bfloat16* p) {
+    const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
+    return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
+}
+__device__ __forceinline__ void store2(float* p, float x, float y) { *reinterpret_cast<float2*>(p) = make_float2(x, y); }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float x, float y) { *reinterpret_cast<uint32_t*>(p) = pack_bf16(x, y); }
+
+template <typename T, int TAPS, int PAIRS>
+__global__ void __launch_bounds__(256, PAIRS > 2 ? 1 : 2) conv_rope_cache_write_kernel(const QkvPrep a, int n_tokens, int tile) {
+    extern __shared__ __align__(16) float2 turn_s[];      // [tile][rot_dims / 2] (cos, sin)
+    __shared__ int info[kPairTile][5];                    // per token: first row, tokens, row to read, row to write of its portion; cache row
+    constexpr int BACK = TAPS - 1;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    const int H = a.Hq, G = a.Gk, d = a.d, dv = a.dv, half = a.rot_dims >> 1, C = (H + G) * d + a.Gv * dv;
+    const int t0 = blockIdx.x * tile, nt = min(tile, n_tokens - t0);
+    const int units = H + G + a.Gv, u0 = blockIdx.y * a.units_per_cta, u1 = min(units, u0 + a.units_per_cta);
+    if (threadIdx.x < nt) {
+        const int t = t0 + threadIdx.x, s = a.seq_of[t], p = a.pos[t];
+#pragma unroll
+        for (int k = 0; k < 4; k++) info[threadIdx.x][k] = a.seqs[k * a.seqs_stride + s];
+        info[threadIdx.x][4] = a.page_table[(long)a.slot[t] * a.max_pages + (p / a.page_size) % a.max_pages] * a.page_size + p % a.page_size;
+    }
+    if (u0 < H + G)
+        for (int i = threadIdx.x; i < nt * half; i += blockDim.x) {
+            const int tt = i / half;
+            double sn, cs;
+            sincos((double)a.pos[t0 + tt] * a.inv_freq[i - tt * half], &sn, &cs);
+            turn_s[i] = make_float2((float)cs, (float)sn);
+        }
+    __syncthreads();
+    const T* proj = (const T*)a.proj;
+    const T* cw = (const T*)a.conv_w;
+    T* cache = (T*)a.cache;
+    const long row_width = (long)G * d + (long)a.Gv * dv;
+    for (int u = u0 + warp; u < u1; u += nw) {
+        const bool is_v = u >= H + G, is_q = u < H;
+        const int n = is_v ? dv : d, ch0 = is_v ? (H + G) * d + (u - H - G) * dv : u * d;
+        const int col0 = is_q ? a.q_off + u * d : (is_v ? a.v_off + (u - H - G) * dv : a.k_off + (u - H) * d);
+        float w[TAPS][PAIRS][2], win[BACK][PAIRS][2];
+#pragma unroll
+        for (int e = 0; e < PAIRS; e++) {
+            const int i = 2 * lane + 64 * e;
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) {
+                w[j][e][0] = i < n ? to_f(cw[(long)(ch0 + i) * TAPS + j]) : 0.f;
+                w[j][e][1] = i < n ? to_f(cw[(long)(ch0 + i + 1) * TAPS + j]) : 0.f;
+            }
+        }
+        int cur = -1;
+        for (int b = 0; b < nt; b += kPairBatch) {
+            float2 in[kPairBatch][PAIRS];
+#pragma unroll
+            for (int k = 0; k < kPairBatch; k++)
+#pragma unroll
+                for (int e = 0; e < PAIRS; e++) {
+                    const int i = 2 * lane + 64 * e;
+                    in[k][e] = b + k < nt && i < n ? load2(proj + (long)(t0 + b + k) * a.proj_stride + col0 + i) : make_float2(0.f, 0.f);
+                }
+#pragma unroll
+            for (int k = 0; k < kPairBatch; k++) {
+                const int tt = b + k;
+                if (tt >= nt) break;
+                const int start = info[tt][0], len = info[tt][1], rd = info[tt][2], wr = info[tt][3], off = t0 + tt - start;
+                if (start != cur) {      // another portion, or the tile's first token: fetch the inputs ahead of it
+                    cur = start;
+#pragma unroll
+                    for (int j = 0; j < BACK; j++)
+#pragma unroll
+                        for (int e = 0; e < PAIRS; e++) {
+                            const int i = 2 * lane + 64 * e, at = off - BACK + j;
+                            float2 v = make_float2(0.f, 0.f);
+                            if (i < n) {
+                                if (at >= 0) v = load2(proj + (long)(start + at) * a.proj_stride + col0 + i);
+                                else if (rd >= 0) {
+                                    const float* st = a.state + (long)rd * a.state_stride + a.conv_off + (long)(BACK + at) * C + ch0 + i;
+                                    v = make_float2(st[0], st[1]);
+                                }
+                            }
+                            win[j][e][0] = v.x;
+                            win[j][e][1] = v.y;
+                        }
+                }
+                float y[PAIRS][2], ss = 0.f;
+#pragma unroll
+                for (int e = 0; e < PAIRS; e++) {
+                    const int i = 2 * lane + 64 * e;
+                    float x0 = 0.f, x1 = 0.f;
+#pragma unroll
+                    for (int j = 0; j < BACK; j++) {
+                        x0 = fmaf(w[j][e][0], win[j][e][0], x0);
+                        x1 = fmaf(w[j][e][1], win[j][e][1], x1);
+                    }
+                    x0 = fmaf(w[BACK][e][0], in[k][e].x, x0);
+                    x1 = fmaf(w[BACK][e][1], in[k][e].y, x1);
+#pragma unroll
+                    for (int j = 0; j + 1 < BACK; j++) {
+                        win[j][e][0] = win[j + 1][e][0];
+                        win[j][e][1] = win[j + 1][e][1];
+                    }
+                    win[BACK - 1][e][0] = in[k][e].x;
+                    win[BACK - 1][e][1] = in[k][e].y;
+                    if (!is_v && i < a.rot_dims) {
+                        const float2 cs = turn_s[tt * half + (i >> 1)];
+                        const float z = x0;
+                        x0 = z * cs.x - x1 * cs.y;
+                        x1 = x1 * cs.x + z * cs.y;
+                    }
+                    y[e][0] = x0;
+                    y[e][1] = x1;
+                    ss += x0 * x0 + x1 * x1;
+                }
+                const float inv = !is_v && a.qk_norm == kQkNormHead ? 1.0f / sqrtf(warp_sum(ss) / (float)d + a.eps) : 1.0f;
+                T* dst = is_q ? (T*)a.q_out + ((long)(t0 + tt) * H + u) * d : cache + (long)info[tt][4] * row_width + (is_v ? (long)G * d + (u - H - G) * dv : (long)(u - H) * d);
+#pragma unroll
+                for (int e = 0; e < PAIRS; e++) {
+                    const int i = 2 * lane + 64 * e;
+                    if (i < n) {
+                        store2(dst + i, y[e][0] * inv, y[e][1] * inv);
+                        if (off == len - 1 && wr >= 0) {
+#pragma unroll
+                            for (int j = 0; j < BACK; j++) {
+                                float* st = a.state + (long)wr * a.state_stride + a.conv_off + (long)j * C + ch0 + i;
+                                st[0] = win[j][e][0];
+                                st[1] = win[j][e][1];
+                            }
+                        }
+                    }
+                }
+            }
+        }
+    }
+}
+
 // ------------------------------------------------------------------------------------------------ soft-max attention, CUDA cores
 // grid (tokens, G * head blocks, splits); a warp per query head (HB = blockDim / 32 heads of ONE key/value head per CTA).  Tiles of
 // 32 keys in shared memory as fp32: lane = key for the scores, lane = value column for the weighted sum; running maximum and sum per
@@ -345,7 +484,7 @@ __device__ __forceinline__ float cap_score_fast(float s, float two_over_cap, flo
 }
 
 template <int D16MAX, int DV16MAX, int MAPS, bool BIAS>
-__global__ void __launch_bounds__(kMmaRows * 2, (MAPS == 1 && !BIAS) || DV16MAX <= 4 ? 4 : 3) window_softmax_attn_mma_kernel(const SmAttn a) {
+__global__ void __launch_bounds__(kMmaRows * 2, 4) window_softmax_attn_mma_kernel(const SmAttn a) {
     constexpr int ROWS = kMmaRows / MAPS, KEYS = kMmaKeys, WPM = 4 / MAPS;      // (token, head) rows; warps per map
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ int tile_info[3];
@@ -622,54 +761,63 @@ __global__ void __launch_bounds__(kMmaRows * 2, (MAPS == 1 && !BIAS) || DV16MAX 
     }
 }
 
-// one CTA of 128 threads per (token, head): per map the parts' weights exp(m_s - m) / l once in shared memory (parts without a key have
+// one CTA of 128 threads per map for each (token, head): the parts' weights exp(m_s - m) / l once in shared memory (parts without a key have
 // m = -inf and weigh nothing; the sink joins l), then the columns in parallel, parts in order; two maps are combined and the row normed here
 constexpr int kMergeMaxSplits = 128;
-template <typename T>
-__global__ void __launch_bounds__(128) softmax_merge_kernel(const SmAttn a) {
-    __shared__ float wgt[kMergeMaxSplits];
-    __shared__ float red[4];
+template <typename T, int MAPS>
+__global__ void __launch_bounds__(128 * MAPS) softmax_merge_kernel(const SmAttn a) {
+    __shared__ float wgt_s[MAPS][kMergeMaxSplits];
+    __shared__ float red_s[MAPS][4];
+    __shared__ float second[MAPS == 2 ? 256 : 1];
     const long row = blockIdx.x, t = row / a.H;
     const int h = (int)(row - t * a.H), splits = a.splits, dv = a.dv;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int map = MAPS == 1 ? 0 : threadIdx.x >> 7, tid = threadIdx.x & 127, lane = tid & 31, warp = tid >> 5;
+    float *wgt = wgt_s[map], *red = red_s[map];
     float acc[2] = {0.f, 0.f};      // columns tid and tid + 128
-    for (int map = 0; map < a.M; map++) {
-        const float* part = a.partial + (row * a.M + map) * splits * (dv + 2);
-        const float ms = tid < splits ? part[(long)tid * (dv + 2)] : -INFINITY;
-        const float ls = tid < splits ? part[(long)tid * (dv + 2) + 1] : 0.f;
-        float m = warp_max(ms);
-        if (lane == 0) red[warp] = m;
-        __syncthreads();
-        m = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
-        if (a.sink) m = fmaxf(m, a.sink[h]);
-        __syncthreads();
-        const float e = ms > -INFINITY ? expf(ms - m) : 0.f;
-        float l = warp_sum(ls * e);
-        if (lane == 0) red[warp] = l;
-        __syncthreads();
-        l = (red[0] + red[1]) + (red[2] + red[3]);
-        if (a.sink) l += expf(a.sink[h] - m);
-        if (tid < splits) wgt[tid] = e / l;
-        __syncthreads();
-        const float sign = map ? -a.lambda[0] : 1.0f;
+    const float* part = a.partial + (row * MAPS + map) * splits * (dv + 2);
+    const float ms = tid < splits ? part[(long)tid * (dv + 2)] : -INFINITY;
+    const float ls = tid < splits ? part[(long)tid * (dv + 2) + 1] : 0.f;
+    float m = warp_max(ms);
+    if (lane == 0) red[warp] = m;
+    __syncthreads();
+    m = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+    if (a.sink) m = fmaxf(m, a.sink[h]);
+    __syncthreads();
+    const float e = ms > -INFINITY ? expf(ms - m) : 0.f;
+    float l = warp_sum(ls * e);
+    if (lane == 0) red[warp] = l;
+    __syncthreads();
+    l = (red[0] + red[1]) + (red[2] + red[3]);
+    if (a.sink) l += expf(a.sink[h] - m);
+    if (tid < splits) wgt[tid] = e / l;
+    __syncthreads();
 #pragma unroll
-        for (int k = 0; k < 2; k++) {
-            const int c = tid + 128 * k;
-            if (c < dv) {
-                float v = 0.f;
-                for (int s = 0; s < splits; s++) v = fmaf(wgt[s], part[(long)s * (dv + 2) + 2 + c], v);
-                acc[k] = map ? fmaf(sign, v, acc[k]) : v;
-            }
+    for (int k = 0; k < 2; k++) {
+        const int c = tid + 128 * k;
+        if (c < dv) {
+#pragma unroll 8
+            for (int s = 0; s < splits; s++) acc[k] = fmaf(wgt[s], part[(long)s * (dv + 2) + 2 + c], acc[k]);
         }
-        __syncthreads();      // the weights and the partial sums are read before the next map's are written
     }
     float inv = a.out_scale;
-    if (a.M == 2) {
-        float ss = warp_sum(acc[0] * acc[0] + acc[1] * acc[1]);
-        if (lane == 0) red[warp] = ss;
+    if (MAPS == 2) {
+        const float lam = a.lambda[0];
+        if (map == 1) {
+#pragma unroll
+            for (int k = 0; k < 2; k++)
+                if (tid + 128 * k < dv) second[tid + 128 * k] = lam * acc[k];
+        }
         __syncthreads();
-        ss = (red[0] + red[1]) + (red[2] + red[3]);
-        inv *= 1.0f / sqrtf(ss / (float)dv + a.rms_eps);
+        if (map == 0) {
+#pragma unroll
+            for (int k = 0; k < 2; k++)
+                if (tid + 128 * k < dv) acc[k] -= second[tid + 128 * k];
+            const float ss = warp_sum(acc[0] * acc[0] + acc[1] * acc[1]);
+            if (lane == 0) red[warp] = ss;
+        }
+        __syncthreads();
+        if (map == 1) return;
+        inv *= 1.0f / sqrtf(((red[0] + red[1]) + (red[2] + red[3])) / (float)dv + a.rms_eps);
     }
     const T* gate = (const T*)a.gate + t * a.gate_stride + (long)h * dv;
     T* out = (T*)a.out + t * a.out_stride + (long)h * dv;
@@ -718,6 +866,37 @@ extern "C" int ktb200_qkv_prep(const ktb200_qkv_prep_params* c, int n_tokens, in
     const QkvPrep a{c->proj, c->proj_stride, c->q_off, c->k_off, c->v_off, Hq, Gk, c->kv_heads, c->dim, c->vdim, c->rot_dims, c->rot_layout, c->inv_freq, c->qk_norm, c->q_weight,
                     c->k_weight, c->v_unit_rms, c->eps, c->v_other, c->v_other_stride, c->blend, c->conv_w, c->taps, c->seq_of, c->seqs, c->seqs_stride, c->state,
                     c->state_stride, c->conv_off, c->pos, c->slot, c->page_table, c->max_pages, c->page_size, c->cache, c->q_out, upc, vec_rows};
+    const size_t two = 2 * esz;
+    auto even = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (two - 1)) == 0; };
+    const bool pairs = c->conv_w && c->taps >= 2 && c->taps <= 4 && c->dim % 2 == 0 && c->vdim % 2 == 0 && c->vdim <= 32 * kPrepMaxPerLane && c->q_off % 2 == 0 && c->k_off % 2 == 0 &&
+                       c->v_off % 2 == 0 && c->proj_stride % 2 == 0 && even(c->proj) && even(c->q_out) && even(c->cache) && c->qk_norm != kQkNormRow && !c->v_other && !c->v_unit_rms &&
+                       (c->rot_dims == 0 || c->rot_layout == kRotInterleaved);
+    if (pairs) {      // tiles of 16 tokens once there are enough tokens to fill the SMs; unit blocks as above
+        const int tile = n_tokens >= 512 ? kPairTile : (n_tokens >= 64 ? 4 : 1), tiles = (n_tokens + tile - 1) / tile;
+        int y = (1184 + tiles - 1) / tiles;
+        y = y > max_y ? max_y : y;
+        QkvPrep b = a;
+        b.units_per_cta = ((units + y - 1) / y + 7) / 8 * 8;
+        const dim3 grid(tiles, (units + b.units_per_cta - 1) / b.units_per_cta);
+        const size_t smem = (size_t)tile * (c->rot_dims / 2) * sizeof(float2);
+        const int widest = c->dim > c->vdim ? c->dim : c->vdim;
+#define PAIR_LAUNCH(TAPS, PAIRS) conv_rope_cache_write_kernel<T, TAPS, PAIRS><<<grid, 256, smem, (cudaStream_t)stream>>>(b, n_tokens, tile)
+#define PAIR_SIZES(TAPS)                               \
+    do {                                               \
+        if (widest <= 64) PAIR_LAUNCH(TAPS, 1);        \
+        else if (widest <= 128) PAIR_LAUNCH(TAPS, 2);  \
+        else PAIR_LAUNCH(TAPS, 4);                     \
+    } while (0)
+        SEQ_DISPATCH(dtype, {
+            if (c->taps == 2) PAIR_SIZES(2);
+            else if (c->taps == 3) PAIR_SIZES(3);
+            else PAIR_SIZES(4);
+        });
+#undef PAIR_SIZES
+#undef PAIR_LAUNCH
+        KTB_LAUNCH_CHECK();
+        return KTB200_OK;
+    }
     SEQ_DISPATCH(dtype, {
         if (c->conv_w) rope_norm_cache_write_kernel<T, true><<<dim3(n_tokens, grid_y), 256, 0, (cudaStream_t)stream>>>(a);
         else rope_norm_cache_write_kernel<T, false><<<dim3(n_tokens, grid_y), 256, 0, (cudaStream_t)stream>>>(a);
@@ -805,7 +984,8 @@ extern "C" int ktb200_softmax_attn(const ktb200_softmax_attn_params* c, int n_to
 #undef MMA_LAUNCH
         KTB_LAUNCH_CHECK();
         if (merge) {
-            softmax_merge_kernel<B><<<(unsigned)rows, 128, 0, (cudaStream_t)stream>>>(a);
+            if (maps == 2) softmax_merge_kernel<B, 2><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(a);
+            else softmax_merge_kernel<B, 1><<<(unsigned)rows, 128, 0, (cudaStream_t)stream>>>(a);
             KTB_LAUNCH_CHECK();
         }
         return KTB200_OK;
@@ -818,7 +998,8 @@ extern "C" int ktb200_softmax_attn(const ktb200_softmax_attn_params* c, int n_to
         window_softmax_attn_kernel<T><<<dim3(n_tokens, kv_heads * maps * hblocks, splits), HB * 32, smem, (cudaStream_t)stream>>>(a);
         KTB_LAUNCH_CHECK();
         if (merge) {
-            softmax_merge_kernel<T><<<(unsigned)rows, 128, 0, (cudaStream_t)stream>>>(a);
+            if (maps == 2) softmax_merge_kernel<T, 2><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(a);
+            else softmax_merge_kernel<T, 1><<<(unsigned)rows, 128, 0, (cudaStream_t)stream>>>(a);
             KTB_LAUNCH_CHECK();
         }
     });

@@ -1,6 +1,6 @@
 """Throughput and per-kernel rooflines of a step-function model at layer sizes of real models, with random weights, beside
 the closest existing model's kernels at equal size (`bench.py --model lekapel`, `bench.py --model mabidra`,
-`bench.py --model zivulix`, `bench.py --model bilurax`).
+`bench.py --model zivulix`, `bench.py --model bilurax`, `bench.py --model rununex`).
 
 Two parts:
   * end to end through the Engine (scheduler, paged cache, step function): prompt tokens/s for a long prompt cut into portions,
@@ -107,6 +107,43 @@ def make_mabidra_attn_config(s):
             "loop": {"start": s["loop"][0], "stop": s["loop"][1], "times": s["loop"][2]}}
 
 
+RUNUNEX_SIZES = {
+    # the same widths, expert sizes and counts as BILURAX_SIZES with every feed-forward a mixture plus a shared expert; P: chunked attention over the
+    # grouped heads of Mabidra's attention layers side by side with a Mamba-2 state space of twice the width (heads of 64 channels, state 128),
+    # D: differential attention with as many query and key columns.  The chunk is as long as the benchmark's context, and `ctx` puts the decoded
+    # token at a chunk's last position.  The closest existing model at equal size is Mabidra: a sigmoid-attention layer without feed-forward
+    # followed by a gated-linear-attention layer (as many state values) for P, a sigmoid-attention layer for D, the same routed experts (of two
+    # matrices where these have three), no shared expert.
+    "2k-wide": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, chunk=2048, s_heads=64, s_vdim=64, state=128, groups=4, conv=4, norm_groups=4, d_dim=64, experts=32, top=4, ff=1024,
+                    shared_ff=2048, vocab=32768, order="PDPDP", ctx=2047, rank=64),
+    "v3-layer": dict(width=7168, heads=64, kv_heads=8, dim=128, vdim=128, chunk=4096, s_heads=224, s_vdim=64, state=128, groups=8, conv=4, norm_groups=8, d_dim=64, experts=32, top=8, ff=2048,
+                     shared_ff=2048, vocab=32768, order="PD", ctx=4095, rank=128),
+}
+
+
+def make_rununex_config(s):
+    left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5, "mask": {"size": s["chunk"]}}
+    right = {"heads": s["s_heads"], "vdim": s["s_vdim"], "state": s["state"], "groups": s["groups"], "conv": s["conv"], "norm_groups": s["norm_groups"]}
+    diff = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["d_dim"], "vdim": s["vdim"], "scale": s["d_dim"] ** -0.5, "mask": {"size": s["chunk"]}, "conv": s["conv"], "diff": 0.4,
+            "rot": {"base": 500000.0, "dims": s["d_dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    kinds = {"P": ("parallel", {"left": left, "right": right, "left_scale": 0.7, "right_scale": 1.2}), "D": ("attention", diff)}
+    moe = {"kind": "moe", "expert": {"ff": s["ff"]}, "router": {"experts": s["experts"], "top": s["top"]}, "shared": {"ff": s["shared_ff"]}}
+    return {"architecture": "Rununex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 4.0}, "residual_mult": 0.5, "logit_scale": 0.5,
+            "layers": [{"type": kinds[c][0], "mixer": kinds[c][1], "mlp": moe} for c in s["order"]]}
+
+
+def make_mabidra_mixed_config(s):
+    """Mabidra at the sizes of a Rununex size entry: per P a sigmoid-attention layer without feed-forward and a gated-linear-attention layer with as
+    many state values, per D a sigmoid-attention layer, the same routed expert sizes"""
+    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5, "bias_max": 1024, "q_temp": {"coef": 0.1, "every": 512}}
+    gla = {"heads": s["s_heads"] * s["s_vdim"] * s["state"] // (128 * 128), "dim": 128, "vdim": 128, "tau": 16.0}
+    moe = {"kind": "moe", "expert": {"ff": s["ff"]}, "router": {"experts": s["experts"], "top": s["top"]}}
+    layers = []
+    for c in s["order"]:
+        layers += [{"type": "attention", "mixer": attn, "mlp": None}, {"type": "gla", "mixer": gla, "mlp": moe}] if c == "P" else [{"type": "attention", "mixer": attn, "mlp": moe}]
+    return {"architecture": "Mabidra", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5, "groups": 4}, "embedding": {"scale": 1.0}, "layers": layers}
+
+
 def make_mabidra_dense_config(s):
     """Mabidra at the sizes of a Zivulix size entry: sigmoid attention for A and L, gated linear attention for D, dense feed-forwards"""
     attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5, "bias_max": 1024, "q_temp": {"coef": 0.1, "every": 512}}
@@ -116,7 +153,11 @@ def make_mabidra_dense_config(s):
 
 
 def random_model(cfg_dict, dtype=torch.bfloat16, device="cuda", size=None):
-    if cfg_dict["architecture"] == "Bilurax":
+    if cfg_dict["architecture"] == "Rununex":
+        from ..models.configuration_rununex import RununexConfig
+        from ..models.modeling_rununex import RununexForCausalLM
+        model = RununexForCausalLM(RununexConfig.from_dict(cfg_dict), dtype=dtype, device=device)
+    elif cfg_dict["architecture"] == "Bilurax":
         from ..models.configuration_bilurax import BiluraxConfig
         from ..models.modeling_bilurax import BiluraxForCausalLM
         model = BiluraxForCausalLM(BiluraxConfig.from_dict(cfg_dict), dtype=dtype, device=device)
@@ -181,7 +222,7 @@ def timed(fn, flush, iters=10, warmup=3):
 def engine_leg(name, size, flush, steps, warmup, family="lekapel"):
     from .engine import Engine
     cfg = {"lekapel": make_config, "mabidra": make_mabidra_config, "zivulix": make_zivulix_config, "mabidra-dense": make_mabidra_dense_config,
-           "bilurax": make_bilurax_config, "mabidra-attn": make_mabidra_attn_config}[family](size)
+           "bilurax": make_bilurax_config, "mabidra-attn": make_mabidra_attn_config, "rununex": make_rununex_config, "mabidra-mixed": make_mabidra_mixed_config}[family](size)
     model = random_model(cfg, size=size)
     if family == "zivulix":      # norm weights are zero-centred, decays and the value blend inside their usual ranges
         for pname, p in model.named_parameters():
@@ -189,6 +230,10 @@ def engine_leg(name, size, flush, steps, warmup, family="lekapel"):
                 p.data.sub_(1.0)
             if pname.endswith("a_log"):
                 p.data.sub_(3.0)
+    if family == "rununex":      # step logits and decays inside their usual ranges, small biases
+        for pname, p in model.named_parameters():
+            if pname.rsplit(".", 1)[-1] in ("dt_bias", "conv_b", "sink", "r2"):
+                p.data.sub_(1.0 if not pname.endswith("r2") else 0.9)
     prompt_len, chunk, ctx = 4096, 2048, min(4096, size["window"] * 2) if family == "lekapel" else size["ctx"]
     eng = Engine(model, max_tokens=8 * (ctx + 64) + prompt_len, max_slots=9, max_step_tokens=chunk)
     g = torch.Generator().manual_seed(0)
@@ -778,6 +823,190 @@ def bilurax_kernel_leg(flush, peak_gbs, peak_tflops):
     return rows
 
 
+def rununex_kernel_leg(flush, peak_gbs, peak_tflops):
+    """The kernels of the Rununex operators at real layer sizes (bf16), each beside the like kernel of the closest existing path."""
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    seq = native.seq_lib()
+    S = lambda: torch.cuda.current_stream().cuda_stream  # noqa: E731
+    rows = []
+    g = torch.Generator(device=dev).manual_seed(7)
+    rn = lambda *s, dt=bf: torch.randn(*s, generator=g, device=dev, dtype=torch.float32).to(dt)
+
+    def peer_of(kernel, ms, nbytes=None, flops=None):
+        r = {"kernel": kernel, "us": ms * 1e3}
+        if nbytes is not None:
+            r["frac_of_measured_hbm"] = nbytes / ms / 1e6 / peak_gbs
+        if flops is not None:
+            r.update(TFLOPs=flops / ms / 1e9, frac_of_measured_bf16=flops / ms / 1e9 / peak_tflops)
+        return r
+
+    def row(kernel, what, ms, nbytes=None, flops=None, peer=None, **more):
+        r = dict(peer_of(kernel, ms, nbytes, flops), case=what, **more)
+        if nbytes is not None:
+            r["GBps"] = nbytes / ms / 1e6
+        progress(f"{kernel} {what}: {ms * 1e3:.1f} us" + (f" (closest {peer['us']:.1f})" if peer else ""))
+        if peer:
+            r["closest"] = peer
+        rows.append(r)
+
+    class Batch:      # one sequence per entry of `lens`, each ending at position `ctx` - 1, on `pages` identity pages of 64 tokens
+        def __init__(self, lens, ctx):
+            T, B = sum(lens), len(lens)
+            i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+            starts = [sum(lens[:i]) for i in range(B)]
+            self.pos = torch.cat([torch.arange(ctx - n, ctx, dtype=torch.int32, device=dev) for n in lens])
+            self.slot = torch.arange(B, dtype=torch.int32, device=dev).repeat_interleave(i32(lens).long())
+            self.seq_of = self.slot
+            self.seqs = i32([starts, lens, [2 * i for i in range(B)], [2 * i + 1 for i in range(B)]])
+            self.n_seqs, self.n_tokens, self.max_kv = B, T, ctx
+            self.page_size, self.max_pages_per_seq = 64, (ctx + 63) // 64
+            self.page_table = torch.arange(B * self.max_pages_per_seq, dtype=torch.int32, device=dev).reshape(B, -1)
+
+        def cache(self, width):
+            return rn(self.n_seqs * self.max_pages_per_seq + 1, 64, width)
+
+    D = 7168
+    from ..operators.norm import KGroupRMSNormShift, KLayerNorm
+    for T in (1, 8, 2048):      # x + m (a + b), layer norm  vs  the same sum with an RMS norm
+        x, a, b = rn(T, D, dt=torch.float32), rn(T, D, dt=torch.float32), rn(T, D)
+        mine, theirs = KLayerNorm(D, 1e-6), KGroupRMSNormShift(D, 1, 1e-6, False)
+        nb = T * D * (4 + 4 + 2 + 4 + 2)
+        row("residual_layernorm_kernel", f"T={T} width={D}", timed(lambda: mine(x, a, b, 0.5), flush), nbytes=nb,
+            peer=peer_of("group_norm_shift_kernel (no shift)", timed(lambda: theirs(x, a, b, 0.5), flush), nb))
+
+    # ---- cache write: 64 / 8 heads.  Filter + rotation of two maps of 64  vs  rotation + unit rms + value blend of heads of 128 (as many columns)
+    from ..operators.attention import paged_softmax_attention, qkv_prep
+    from ..models.configuration_lekapel import RotarySpec
+    H, G, d, dv, taps = 64, 8, 128, 128, 4
+    n_q, n_k, n_v, cw = H * d, G * d, G * dv, G * (d + dv)
+    n_in = n_q + n_k + n_v
+    rot = RotarySpec(500000.0, 64, factor=8.0, low=1.0, high=4.0, original=8192)
+    inv, lam = rot.inv_freq(dev), torch.tensor([0.3], device=dev)
+    for T in (8, 2048):
+        bt = Batch([1] * 8 if T == 8 else [T], 4096)
+        proj, cwt, vo, kv = rn(T, n_in), rn(n_in, taps), rn(T, n_v), bt.cache(cw)
+        state = torch.zeros(2 * bt.n_seqs, (taps - 1) * n_in, device=dev)
+        qo = torch.empty(T, H, d, dtype=bf, device=dev)
+        nb = T * (n_in + n_q + cw) * 2
+        nb_conv = nb + (bt.n_seqs * (taps - 1) * n_in * 8)
+        theirs = lambda: native.check_seq(seq.ktb200_rope_norm_cache_write(proj.data_ptr(), n_in, 0, n_q, n_q + n_k, H, G, d, dv, d // 2, 0, inv.data_ptr(), 1, None, None, 0, 1e-6,
+                                                                           vo.data_ptr(), n_v, lam.data_ptr(), bt.pos.data_ptr(), bt.slot.data_ptr(), bt.page_table.data_ptr(),
+                                                                           bt.max_pages_per_seq, 64, kv.data_ptr(), qo.data_ptr(), T, 30, S()))
+        peer = peer_of("rope_norm_cache_write_kernel (rotation, per-head unit rms, value blend)", timed(theirs, flush), nb + T * n_v * 2)
+        row("rope_norm_cache_write_kernel<filter> (4 taps, two maps of 64, rotation)", f"T={T} heads={H}/{G}",
+            timed(lambda: qkv_prep(proj, bt, bt, kv, H, G, 64, dv, (0, n_q, n_q + n_k), maps=2, rot=rot, inv_freq=inv, conv_w=cwt, state=state), flush), nbytes=nb_conv, peer=peer)
+        row("rope_norm_cache_write_kernel (unit rms)", f"T={T} heads={H}/{G} dim={d}",
+            timed(lambda: qkv_prep(proj, bt, bt, kv, H, G, d, dv, (0, n_q, n_q + n_k), qk_norm=1, eps=1e-6), flush), nbytes=nb, peer=peer)
+
+    # ---- attention: distance bias + sink + gate, and differential maps  vs  the plain chunk mask of the same kernel over as many key columns
+    r1, r2, sink = 0.3 + torch.rand(H, device=dev), 0.02 + 0.1 * torch.rand(H, device=dev), torch.rand(H, device=dev)
+
+    def attn_rows(bt, chunk, what, nbytes=None, flops=None, iters=10, tcs=(True, False)):
+        T = bt.n_tokens
+        kv, q, gate, proj_gate = bt.cache(cw), rn(T, H, d), None, rn(T, n_in + H * dv)
+        gate = proj_gate[:, n_in:]
+        for tc in tcs:
+            plain = timed(lambda: paged_softmax_attention(q, kv, bt, bt, H, G, d, dv, d ** -0.5, chunk=chunk, tensor_cores=tc), flush, iters=iters)
+            nm = "window_softmax_attn_mma_kernel" if tc else "window_softmax_attn_kernel, CUDA cores"
+            peer = peer_of(nm + ", chunk mask", plain, nbytes, flops)
+            row(nm + ", distance bias, sink, gate", what,
+                timed(lambda: paged_softmax_attention(q, kv, bt, bt, H, G, d, dv, d ** -0.5, chunk=chunk, tensor_cores=tc, dist_bias=(r1, r2), sink=sink, gate=gate), flush, iters=iters),
+                nbytes, flops, peer)
+            # (two maps of 64: the same query and key columns, twice the value products)
+            row(nm + ", two maps of 64", what,
+                timed(lambda: paged_softmax_attention(q, kv, bt, bt, H, G, 64, dv, 0.125, chunk=chunk, tensor_cores=tc, maps=2, lam=lam, rms_eps=1e-6, out_scale=0.6), flush, iters=iters),
+                nbytes, flops * (d + 2 * dv) / (d + dv) if flops else None, peer)
+
+    for B, ctx in ((1, 4096), (8, 4096), (1, 32768)):
+        attn_rows(Batch([1] * B, ctx), ctx, f"decode B={B} last position of a chunk of {ctx} heads={H}/{G}", nbytes=B * ctx * cw * 2)
+    T, ctx = 2048, 4096
+    attn_rows(Batch([T], ctx), ctx, f"prompt portion T={T} positions {ctx - T}..{ctx - 1} heads={H}/{G}, one chunk of {ctx}", flops=float(sum(range(ctx - T + 1, ctx + 1))) * H * (d + dv) * 2,
+              iters=5, tcs=(True,))
+    attn_rows(Batch([T], ctx), 1024, "the same, chunks of 1024", flops=2 * float(sum(range(1, 1025))) * H * (d + dv) * 2, iters=5, tcs=(True,))
+
+    # ---- state space: 112 heads of 64 channels, state 128, 4 groups (as many state values as 56 heads of 128 x 128)  vs  gated linear attention
+    P, sv, N, J = 112, 64, 128, 4
+    inner, C_ = P * sv, P * sv + 2 * J * N
+    s_in = (inner + C_ + P + 7) // 8 * 8
+    sw = inner * N + (taps - 1) * C_
+    GH, gd = 56, 128
+    g_in = 4 * GH * gd
+    cwt, cb, dtb, al, ds = rn(C_, taps), rn(C_), rn(P, dt=torch.float32) - 2.0, rn(P, dt=torch.float32), rn(P, dt=torch.float32)
+    nw = rn(inner)
+    for B, T in ((1, 1), (8, 1), (1, 2048)):
+        bt = Batch([T] * B, max(T, 64))
+        n = B * T
+        proj, state = rn(n, s_in), torch.zeros(2 * B, sw, device=dev)
+        xbc, y, oo = torch.empty(n, C_, dtype=bf, device=dev), torch.empty(n, inner, device=dev), torch.empty(n, inner, dtype=bf, device=dev)
+        a = native.SsdParams(proj=proj.data_ptr(), proj_stride=s_in, xbc_off=inner, dt_off=inner + C_, conv_w=cwt.data_ptr(), conv_b=cb.data_ptr(), taps=taps, dt_bias=dtb.data_ptr(),
+                             a_log=al.data_ptr(), d_skip=ds.data_ptr(), heads=P, groups=J, state_size=N, vdim=sv, seq_of=bt.seq_of.data_ptr(), seqs=bt.seqs.data_ptr(), seqs_stride=B, n_seqs=B,
+                             state=state.data_ptr(), state_stride=sw)
+        gproj, z, zb = rn(n, g_in), rn(n, GH * gd), rn(GH * gd)
+        gstate, go = torch.zeros(2 * B, GH * gd * gd, device=dev), torch.empty(n, GH * gd, device=dev)
+        gla = lambda: native.check_seq(seq.ktb200_gla_scan(gproj.data_ptr(), g_in, 0, GH * gd, 2 * GH * gd, z.data_ptr(), GH * gd, zb.data_ptr(), 16.0, GH, gd, gd, bt.seqs.data_ptr(), B, B, n,
+                                                           gstate.data_ptr(), go.data_ptr(), 30, S()))
+        it = 5 if T > 1 else 10
+        ms_gla = timed(gla, flush, iters=it)
+        if T == 1:
+            nb = B * (inner * N * 8 + (taps - 1) * C_ * 8)
+            row("ssd_step_kernel (filter and recurrence)", f"decode B={B} heads={P} x {sv} state={N}", timed(lambda: native.check_seq(seq.ktb200_ssd_step(C.byref(a), y.data_ptr(), 30, S())), flush),
+                nbytes=nb, peer=peer_of("gla_scan_kernel", ms_gla, B * GH * gd * gd * 8))
+        else:
+            conv = lambda: native.check_seq(seq.ktb200_ssd_conv(C.byref(a), xbc.data_ptr(), n, 30, S()))
+            DH, DG = 56, 28
+            dC = 2 * DG * 128 + DH * 128
+            d_in = dC + DH * 128 + 2 * DH
+            dproj, dcw, dstate = rn(n, d_in), rn(dC, taps), torch.zeros(2, DH * 128 * 128 + (taps - 1) * dC, device=dev)
+            f32 = lambda *s: torch.empty(*s, device=dev)
+            qn, kn, vv, be, de = f32(n, DG * 128), f32(n, DG * 128), f32(n, DH * 128), f32(n, DH), f32(n, DH)
+            al2, db2 = rn(DH, dt=torch.float32) - 3.0, rn(DH, dt=torch.float32)
+            dprep = lambda: native.check_seq(seq.ktb200_delta_prep(dproj.data_ptr(), d_in, 0, dC + DH * 128, dC + DH * 128 + DH, dcw.data_ptr(), taps, al2.data_ptr(), db2.data_ptr(), DH, DG,
+                                                                   128, 128, 1e-6, bt.seq_of.data_ptr(), bt.seqs.data_ptr(), B, dstate.data_ptr(), dstate.shape[1], qn.data_ptr(), kn.data_ptr(),
+                                                                   vv.data_ptr(), be.data_ptr(), de.data_ptr(), n, 30, S()))
+            row("ssd_conv_kernel", f"T={T} channels={C_} taps={taps}", timed(conv, flush, iters=it), nbytes=n * C_ * 4,
+                peer=peer_of("delta_prep_kernel", timed(dprep, flush, iters=it), n * dC * 6))
+            conv()
+            ms = timed(lambda: native.check_seq(seq.ktb200_ssd_scan(C.byref(a), xbc.data_ptr(), y.data_ptr(), 30, S())), flush, iters=it)
+            row("ssd_scan_kernel", f"prompt portion T={T} heads={P} x {sv} state={N}", ms, flops=float(T) * P * sv * N * 5, us_per_token_step=ms * 1e3 / T,
+                peer=dict(peer_of("gla_scan_kernel", ms_gla, flops=float(T) * GH * gd * gd * 4), us_per_token_step=ms_gla * 1e3 / T))
+        gw = rn(gd)
+        ms = timed(lambda: native.check_seq(seq.ktb200_gla_out(go.data_ptr(), gw.data_ptr(), 1e-6, gproj.data_ptr(), g_in, oo.data_ptr(), n, GH, gd, 30, S())), flush)
+        row("gated_group_norm_kernel", f"T={n} width={inner} groups=8",
+            timed(lambda: native.check_seq(seq.ktb200_gated_group_norm(y.data_ptr(), proj.data_ptr(), s_in, nw.data_ptr(), 8, 1e-6, 0.9, oo.data_ptr(), inner, n, inner, 30, S())), flush),
+            nbytes=n * inner * 8, peer=peer_of("gla_out_kernel", ms, n * GH * gd * 8))
+
+    # ---- router: plain sigmoid top 8 of 256  vs  soft-max over all, 8 largest
+    from ..operators.gate import KSigmoidTopKGate, KSoftmaxTopKGate
+    E, top = 256, 8
+    mine, theirs = KSigmoidTopKGate(D, E, top), KSoftmaxTopKGate(D, E, top)
+    mine.weight.data.copy_(rn(E, D, dt=torch.float32) * D ** -0.5)
+    theirs.weight.data.copy_(mine.weight.data)
+    for T in (1, 8, 2048):
+        x = rn(T, D)
+        ours, ms = timed(lambda: mine(x), flush), timed(lambda: theirs(x), flush)
+        nb = E * D * 4 + T * D * 2
+        small = T < mine.gemm_min_tokens
+        row("gate_kernel (sigmoid, greedy)" if small else "fp32 GEMM + gate_select_kernel", f"T={T} experts={E} width={D} top={top}", ours, nbytes=nb,
+            peer=peer_of("gate_kernel (soft-max, greedy)" if small else "fp32 GEMM + torch soft-max and top-k", ms, nb))
+
+    # ---- experts: weights on the input beside weights on the output in the same kernels
+    E, top, ff = 32, 8, 2048
+    from ..operators.experts import KExpertsDense
+    ex = KExpertsDense(D, ff, E)
+    for p in ex.parameters():
+        p.data.copy_(rn(*p.shape) * p.shape[-1] ** -0.5)
+    for T in (1, 8, 2048):
+        x = rn(T, D)
+        ids = torch.stack([torch.randperm(E, generator=g, device=dev)[:top] for _ in range(T)])
+        w = torch.rand(T, top, generator=g, device=dev)
+        uniq = int(ids.unique().numel())
+        kw = dict(nbytes=uniq * 3 * ff * D * 2) if T < 48 else dict(flops=float(T) * top * 3 * ff * D * 2)
+        ms = timed(lambda: ex(x, ids, w), flush)
+        row("experts, weight on the input (whole call)", f"T={T} top={top} of {E} width={D} ff={ff}", timed(lambda: ex(x, ids, w, on_input=True), flush),
+            peer=peer_of("experts, weight on the output (whole call)", ms, **kw), **kw)
+    return rows
+
+
 def run_bilurax(args):
     torch.cuda.set_device(0)
     root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
@@ -795,6 +1024,28 @@ def run_bilurax(args):
         out["models"].append(engine_leg(name, BILURAX_SIZES[name], flush, args.steps, args.warmup, family="bilurax"))
         torch.cuda.empty_cache()
         out["closest_models"].append(engine_leg(name, BILURAX_SIZES[name], flush, args.steps, args.warmup, family="mabidra-attn"))      # Mabidra at the same sizes, in the same process
+        torch.cuda.empty_cache()
+    out["gpu_launches"] = int(native.seq_lib().ktb200_launch_count() - n0)
+    print(json.dumps(out))
+
+
+def run_rununex(args):
+    torch.cuda.set_device(0)
+    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    try:
+        m = json.load(open(os.path.join(root, "MEASURED_PEAKS.json")))
+        peak, tf, src = float(m["hbm_gbs"]), float(m["bf16_tflops"]), "measured (MEASURED_PEAKS.json hbm_gbs, bf16_tflops)"
+    except Exception:
+        peak, tf, src = 6650.0, 1590.0, "fallback"
+    flush = Flusher("cuda")
+    n0 = native.seq_lib().ktb200_launch_count()
+    out = {"bench": "rununex", "dtype": "bf16", "data": "synthetic (random weights and tokens)", "hbm_peak_GBps": peak, "bf16_peak_TFLOPs": tf, "peak_source": src,
+           "timing": "CUDA events, median, 256 MB L2 flush between timed calls", "kernels": [] if getattr(args, "no_kernels", False) else rununex_kernel_leg(flush, peak, tf),
+           "models": [], "closest_models": []}
+    for name in (args.sizes.split(",") if getattr(args, "sizes", None) else RUNUNEX_SIZES):
+        out["models"].append(engine_leg(name, RUNUNEX_SIZES[name], flush, args.steps, args.warmup, family="rununex"))
+        torch.cuda.empty_cache()
+        out["closest_models"].append(engine_leg(name, RUNUNEX_SIZES[name], flush, args.steps, args.warmup, family="mabidra-mixed"))      # Mabidra at the same sizes, in the same process
         torch.cuda.empty_cache()
     out["gpu_launches"] = int(native.seq_lib().ktb200_launch_count() - n0)
     print(json.dumps(out))
@@ -823,7 +1074,9 @@ def run_zivulix(args):
 
 
 def run(args):
-    """`bench.py --model lekapel | mabidra | zivulix | bilurax`: prints one JSON line."""
+    """`bench.py --model lekapel | mabidra | zivulix | bilurax | rununex`: prints one JSON line."""
+    if args.model == "rununex":
+        return run_rununex(args)
     if args.model == "mabidra":
         return run_mabidra(args)
     if args.model == "zivulix":
