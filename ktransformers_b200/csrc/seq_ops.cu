@@ -198,7 +198,7 @@ __global__ void __launch_bounds__(256) group_norm_shift_kernel(const float* __re
 // x_out[t] = x, h[t] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w * h_scale.  A thread keeps its NV float4 of the row in registers through
 // both sums (NV = 0: rows of any width, staged in shared memory).
 template <typename T, int NV>
-__global__ void __launch_bounds__(NV == 0 || NV > 4 ? 256 : (NV > 2 ? 512 : 1024)) residual_layernorm_kernel(const float* __restrict__ x_in, const void* __restrict__ da, int a_type, const void* __restrict__ db, int b_type,
+__global__ void __launch_bounds__(NV == 0 ? 256 : (NV > 4 ? 512 : 1024)) residual_layernorm_kernel(const float* __restrict__ x_in, const void* __restrict__ da, int a_type, const void* __restrict__ db, int b_type,
                                                                                  float mult, const int64_t* __restrict__ rows, float* __restrict__ x_out, const T* __restrict__ w, float eps,
                                                                                  float h_scale, T* __restrict__ h_out, int D) {
     extern __shared__ __align__(16) float sm[];
@@ -685,7 +685,7 @@ extern "C" int ktb200_residual_layernorm(const float* x_in, const void* delta_a,
     int threads = n_tokens >= 296 ? 256 : 1024;
     while (threads > 64 && threads * 2 > width) threads >>= 1;
     int nv = (width / 4 + threads - 1) / threads;
-    while ((nv > 2 && threads > 512) || (nv > 4 && threads > 256)) { threads >>= 1; nv = (width / 4 + threads - 1) / threads; }
+    if (nv > 4 || (nv > 2 && threads == 1024)) { threads = 512; nv = (width / 4 + threads - 1) / threads; }      // (eight float4 per thread need 128 registers)
 #define LN_LAUNCH(NV, TH, SM)                                                                                                                                             \
     residual_layernorm_kernel<T, NV><<<n_tokens, TH, SM, (cudaStream_t)stream>>>(x_in, delta_a, a_type, delta_b, b_type, mult, rows, x_out, (const T*)weight, eps, h_scale, \
                                                                                  (T*)h_out, width)
@@ -697,7 +697,7 @@ extern "C" int ktb200_residual_layernorm(const float* x_in, const void* delta_a,
         else {
             const size_t smem = (size_t)width * sizeof(float);
             if (smem > 200 * 1024) { set_error("residual_layernorm: row too wide"); return KTB200_EINVAL; }
-            static size_t granted = 48 * 1024;
+            static size_t granted = 46 * 1024;      // (less the kernel's static shared memory)
             if (smem > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(residual_layernorm_kernel<T, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
             LN_LAUNCH(0, 256, smem);
         }

@@ -840,7 +840,7 @@ using namespace ktb;
     } while (0)
 #define GRANT_SMEM(kernel, smem)                                                                                                       \
     do {                                                                                                                               \
-        static size_t granted = 48 * 1024;                                                                                             \
+        static size_t granted = 46 * 1024; /* less the kernels' static shared memory */                                               \
         if ((smem) > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(smem))); granted = (smem); } \
     } while (0)
 
