@@ -577,7 +577,9 @@ typedef struct {
     long state_stride;
 } ktb200_ssd_params;
 int ktb200_ssd_conv(const ktb200_ssd_params* params, void* xbc, int n_tokens, int dtype, void* stream);
-int ktb200_ssd_scan(const ktb200_ssd_params* params, const void* xbc, float* y, int dtype, void* stream);
+int ktb200_ssd_scan(const ktb200_ssd_params* params, const void* xbc, float* y, int dtype, int allow_tensor_cores, void* stream);
+/* whether that call may run chunks of 64 tokens on the tensor cores (bf16, state_size a multiple of 16 up to 256, vdim of 8) */
+int ktb200_ssd_scan_uses_tensor_cores(int heads, int groups, int state_size, int vdim, int dtype);
 int ktb200_ssd_step(const ktb200_ssd_params* params, float* y, int dtype, void* stream);
 int ktb200_gated_group_norm(const float* y, const void* z, long z_stride, const void* weight, int groups, float eps, float out_scale, void* out,
                             long out_stride, int n_tokens, int width, int dtype, void* stream);

@@ -176,7 +176,8 @@ SEQ_SYMBOLS = {
     "ktb200_softmax_attn_tiles": (_I, [_I, _I, _I, _I, _I]),
     # csrc/ssd.cu
     "ktb200_ssd_conv": (_I, [C.POINTER(SsdParams), _VP, _I, _I, _VP]),
-    "ktb200_ssd_scan": (_I, [C.POINTER(SsdParams), _VP, _VP, _I, _VP]),
+    "ktb200_ssd_scan": (_I, [C.POINTER(SsdParams), _VP, _VP, _I, _I, _VP]),
+    "ktb200_ssd_scan_uses_tensor_cores": (_I, [_I, _I, _I, _I, _I]),
     "ktb200_ssd_step": (_I, [C.POINTER(SsdParams), _VP, _I, _VP]),
     "ktb200_gated_group_norm": (_I, [_VP, _VP, _L, _VP, _I, _F, _F, _VP, _L, _I, _I, _I, _VP]),
 }

@@ -157,7 +157,14 @@ class KStateSpace(nn.Module):
     A sequence's state — the matrices and the last conv - 1 inputs of every filtered channel — lives in the cache manager's double-buffered
     fp32 state rows (models/custom_cache.PagedStateCache).  Alone (`forward`), or side by side with another mixer of the same input
     (operators/side_by_side.py) through `load_in` and `mix`, as KBiasedSinkAttention.  Sizes are constructor parameters
-    (models/configuration_rununex.StateSpaceSpec).  (The reference has no recurrent mixer.)"""
+    (models/configuration_rununex.StateSpaceSpec).
+
+    Two forms of the scan (csrc/ssd.cu): in bf16 with a state size that is a multiple of 16, chunks of 64 tokens on the tensor cores, operands
+    that carry fp32 factors as two bf16 terms, the state in fp32 accumulators; otherwise, in fp32 and for batches of mostly single tokens,
+    token by token with fp32 products.  (The reference has no recurrent mixer.)"""
+
+    use_tensor_cores = True
+    chunk_min_tokens = 32       # tokens beyond one per portion from which the chunked form runs
 
     def __init__(self, width: int, spec, eps: float, dtype=torch.bfloat16, device="cuda", stacked: bool = False):
         """`stacked`: the input and output matrices belong to whoever stacks this mixer with others."""
@@ -207,7 +214,8 @@ class KStateSpace(nn.Module):
         else:
             xbc = torch.empty((T, s.channels), dtype=dt, device=dev)
             native.check_seq(lib.ktb200_ssd_conv(C.byref(a), xbc.data_ptr(), T, code, st))
-            native.check_seq(lib.ktb200_ssd_scan(C.byref(a), xbc.data_ptr(), y.data_ptr(), code, st))
+            chunked = self.use_tensor_cores and T - batch.n_seqs >= self.chunk_min_tokens
+            native.check_seq(lib.ktb200_ssd_scan(C.byref(a), xbc.data_ptr(), y.data_ptr(), code, int(chunked), st))
         native.check_seq(lib.ktb200_gated_group_norm(y.data_ptr(), proj[:, off:].data_ptr(), proj.stride(0), self.norm.data_ptr(), s.norm_groups, float(self.eps), float(out_scale),
                                                      out.data_ptr(), out.stride(0), T, s.inner, code, st))
         return out

@@ -966,9 +966,10 @@ def rununex_kernel_leg(flush, peak_gbs, peak_tflops):
             row("ssd_conv_kernel", f"T={T} channels={C_} taps={taps}", timed(conv, flush, iters=it), nbytes=n * C_ * 4,
                 peer=peer_of("delta_prep_kernel", timed(dprep, flush, iters=it), n * dC * 6))
             conv()
-            ms = timed(lambda: native.check_seq(seq.ktb200_ssd_scan(C.byref(a), xbc.data_ptr(), y.data_ptr(), 30, S())), flush, iters=it)
-            row("ssd_scan_kernel", f"prompt portion T={T} heads={P} x {sv} state={N}", ms, flops=float(T) * P * sv * N * 5, us_per_token_step=ms * 1e3 / T,
-                peer=dict(peer_of("gla_scan_kernel", ms_gla, flops=float(T) * GH * gd * gd * 4), us_per_token_step=ms_gla * 1e3 / T))
+            for tc, name in ((1, "ssd_chunk_kernel"), (0, "ssd_scan_kernel, CUDA cores")):
+                ms = timed(lambda: native.check_seq(seq.ktb200_ssd_scan(C.byref(a), xbc.data_ptr(), y.data_ptr(), 30, tc, S())), flush, iters=it)
+                row(name, f"prompt portion T={T} heads={P} x {sv} state={N}", ms, flops=float(T) * P * sv * N * 4, us_per_token_step=ms * 1e3 / T,
+                    peer=dict(peer_of("gla_scan_kernel", ms_gla, flops=float(T) * GH * gd * gd * 4), us_per_token_step=ms_gla * 1e3 / T))
         gw = rn(gd)
         ms = timed(lambda: native.check_seq(seq.ktb200_gla_out(go.data_ptr(), gw.data_ptr(), 1e-6, gproj.data_ptr(), g_in, oo.data_ptr(), n, GH, gd, 30, S())), flush)
         row("gated_group_norm_kernel", f"T={n} width={inner} groups=8",
