@@ -207,48 +207,150 @@ __global__ void __launch_bounds__(256, 2) ssd_scan_kernel(const T* __restrict__ 
 }
 
 // ------------------------------------------------------------------------------------------------ the recurrence, chunked, tensor cores (bf16)
-// grid (portions, heads, column blocks of 32 value columns), 4 warps.  Tokens run in chunks of 64 with L the running sum of log decays inside
+// grid (portions, heads, column blocks of 32 value columns), 8 warps.  Tokens run in chunks of 64 with L the running sum of log decays inside
 // the chunk (fp32, L <= 0 and falling, so every factor below is at most one):
 //     y_i = exp(L_i) C_i S + sum_{j <= i} (C_i . B_j) exp(L_i - L_j) dt_j x_j + D x_i          S <- exp(L_last) S + sum_j B_j (exp(L_last - L_j) dt_j x_j)^T
 // as m16n8k16 bf16 MMAs with fp32 accumulators.  B, C and x are bf16 as they come; what the fp32 factors touch — the weighted scores, the weighted
-// x rows and S as an operand — enters as the sum of two bf16 terms (about 16 bits of mantissa).  S itself stays in fp32 accumulators from chunk
-// to chunk: warp w keeps the state rows of MT tiles of 16.
+// x rows and S as an operand — enters as the sum of two bf16 terms (about 16 bits of mantissa).  Warps 0..3 make the outputs of 16 tokens each;
+// warps 4..7 meanwhile take the chunk into S, whose fp32 accumulators they keep from chunk to chunk (MT tiles of 16 state rows each), and
+// publish it for the next chunk once the output warps have read the old one.  The next chunk's rows are on their way in the other stage.
 constexpr int kChunkQ = 64, kChunkCols = 32, kChunkLd = kChunkCols + 8;
 __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(a, b);
     lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
-static size_t ssd_chunk_smem(int N) { return ((size_t)2 * kChunkQ * (N + 8) + 3 * kChunkQ * kChunkLd + (size_t)2 * N * kChunkLd) * 2 + 4 * kChunkQ * sizeof(float); }
+static size_t ssd_chunk_smem(int N) { return ((size_t)4 * kChunkQ * (N + 8) + 4 * kChunkQ * kChunkLd + (size_t)2 * N * kChunkLd) * 2 + 8 * kChunkQ * sizeof(float); }
+
+// The outputs of the chunk's tokens 16 W .. 16 W + 15 by one warp: C S and the scores against the chunk's tokens up to its own in one pass over
+// the state rows, then the weighted scores times x.  W is a template parameter so that the tiles above the diagonal fall away at compile time
+// and the operand loads of a step are all issued ahead of its MMAs.
+template <int W>
+__device__ __forceinline__ void ssd_chunk_outputs(const __nv_bfloat16* Cs, const __nv_bfloat16* Bs, const __nv_bfloat16* Xs, const __nv_bfloat16* Sh, const float* Ls, const float* eL,
+                                                  const float* dts, int N, int nt, bool more, float Dh, float* __restrict__ y, long inner, int cols) {
+    constexpr int LD = kChunkLd;
+    const int ldn = N + 8, n16 = N >> 4, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
+    float Y[4][4], G[2 * W + 2][4];
+#pragma unroll
+    for (int n = 0; n < 4; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) Y[n][e] = 0.f;
+#pragma unroll
+    for (int n = 0; n < 2 * W + 2; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) G[n][e] = 0.f;
+    const __nv_bfloat16* ca = Cs + (W * 16 + (lane & 15)) * ldn + 8 * (lane >> 4);
+    const __nv_bfloat16* ba = Bs + ((lane & 7) + 8 * (lane >> 4)) * ldn + 8 * ((lane >> 3) & 1);
+    const __nv_bfloat16* sa = Sh + (lane & 15) * LD + 8 * (lane >> 4);
+#pragma unroll 2
+    for (int kk = 0; kk < n16; kk++) {
+        uint32_t a[4], b[W + 1][4], st[2][2][4];
+        ldmatrix_x4(a, ca + kk * 16);
+#pragma unroll
+        for (int np = 0; np <= W; np++) ldmatrix_x4(b[np], ba + np * 16 * ldn + kk * 16);
+#pragma unroll
+        for (int term = 0; term < 2; term++)
+#pragma unroll
+            for (int vp = 0; vp < 2; vp++) ldmatrix_x4_trans(st[term][vp], sa + (term * N + kk * 16) * LD + vp * 16);
+#pragma unroll
+        for (int np = 0; np <= W; np++) {
+            mma_bf16_16816(G[2 * np], a, b[np][0], b[np][1]);
+            mma_bf16_16816(G[2 * np + 1], a, b[np][2], b[np][3]);
+        }
+#pragma unroll
+        for (int term = 0; term < 2; term++)
+#pragma unroll
+            for (int vp = 0; vp < 2; vp++) {
+                mma_bf16_16816(Y[2 * vp], a, st[term][vp][0], st[term][vp][1]);
+                mma_bf16_16816(Y[2 * vp + 1], a, st[term][vp][2], st[term][vp][3]);
+            }
+    }
+    if (more) asm volatile("bar.arrive 2, 256;" ::: "memory");      // the old state is read
+    const int iA = W * 16 + gq, iB = iA + 8;
+    const float LA = Ls[iA], LB = Ls[iB], eA = eL[iA], eB = eL[iB];
+#pragma unroll
+    for (int n = 0; n < 4; n++) {
+        Y[n][0] *= eA;
+        Y[n][1] *= eA;
+        Y[n][2] *= eB;
+        Y[n][3] *= eB;
+    }
+#pragma unroll
+    for (int kk = 0; kk <= W; kk++) {
+        uint32_t b[2][4];
+#pragma unroll
+        for (int vp = 0; vp < 2; vp++) ldmatrix_x4_trans(b[vp], Xs + (kk * 16 + (lane & 15)) * LD + vp * 16 + 8 * (lane >> 4));
+#pragma unroll
+        for (int n = 2 * kk; n < 2 * kk + 2; n++) {
+            const int jj = n * 8 + 2 * tq;
+            const float2 Lj = *reinterpret_cast<const float2*>(Ls + jj), dj = *reinterpret_cast<const float2*>(dts + jj);
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const float f = __expf((e < 2 ? LA : LB) - ((e & 1) ? Lj.y : Lj.x)) * ((e & 1) ? dj.y : dj.x);
+                G[n][e] = kk < W || jj + (e & 1) <= (e < 2 ? iA : iB) ? G[n][e] * f : 0.f;      // (only the diagonal tile has anything to mask)
+            }
+        }
+        uint32_t hi[4], lo[4];
+        split_bf16(G[2 * kk][0], G[2 * kk][1], hi[0], lo[0]);
+        split_bf16(G[2 * kk][2], G[2 * kk][3], hi[1], lo[1]);
+        split_bf16(G[2 * kk + 1][0], G[2 * kk + 1][1], hi[2], lo[2]);
+        split_bf16(G[2 * kk + 1][2], G[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+        for (int vp = 0; vp < 2; vp++) {
+            mma_bf16_16816(Y[2 * vp], hi, b[vp][0], b[vp][1]);
+            mma_bf16_16816(Y[2 * vp + 1], hi, b[vp][2], b[vp][3]);
+        }
+#pragma unroll
+        for (int vp = 0; vp < 2; vp++) {
+            mma_bf16_16816(Y[2 * vp], lo, b[vp][0], b[vp][1]);
+            mma_bf16_16816(Y[2 * vp + 1], lo, b[vp][2], b[vp][3]);
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < 4; n++) {
+        const int c = n * 8 + 2 * tq;
+        if (c < cols) {
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+                const int i = e ? iB : iA;
+                if (i < nt) {
+                    const uint32_t u = *reinterpret_cast<const uint32_t*>(Xs + i * LD + c);
+                    *reinterpret_cast<float2*>(y + i * inner + c) = make_float2(fmaf(Dh, __uint_as_float(u << 16), Y[n][e]), fmaf(Dh, __uint_as_float(u & 0xffff0000u), Y[n][e + 1]));
+                }
+            }
+        }
+    }
+}
 
 template <int MT>
-__global__ void __launch_bounds__(128, MT <= 2 ? 3 : 1) ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, const __nv_bfloat16* __restrict__ dt_in, long dt_stride,
+__global__ void __launch_bounds__(256, MT <= 2 ? 2 : 1) ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, const __nv_bfloat16* __restrict__ dt_in, long dt_stride,
                                                                          const float* __restrict__ dt_bias, const float* __restrict__ a_log, const float* __restrict__ Dv, int P, int J, int N,
                                                                          int dv, const int* __restrict__ seqs, int seqs_stride, float* __restrict__ state, long state_stride,
                                                                          float* __restrict__ y_out) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     constexpr int Q = kChunkQ, LD = kChunkLd;
-    const int ldn = N + 8, n16 = N >> 4;
-    __nv_bfloat16* Cs = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [Q][ldn]
-    __nv_bfloat16* Bs = Cs + Q * ldn;                                    // [Q][ldn]
-    __nv_bfloat16* Xs = Bs + Q * ldn;                                    // [Q][LD]
-    __nv_bfloat16* Xh = Xs + Q * LD;                                     // [2][Q][LD]: the weighted rows, two terms
+    const int ldn = N + 8;
+    __nv_bfloat16* const ring = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // two stages of C [Q][ldn] | B [Q][ldn] | x [Q][LD]
+    const int stage_elems = 2 * Q * ldn + Q * LD;
+    __nv_bfloat16* Xh = ring + 2 * stage_elems;                          // [2][Q][LD]: the weighted rows, two terms
     __nv_bfloat16* Sh = Xh + 2 * Q * LD;                                 // [2][N][LD]: the state, two terms
-    float* Ls = reinterpret_cast<float*>(Sh + 2 * N * LD);               // [Q] each: L, exp(L), dt, exp(L_last - L) dt
-    float *eL = Ls + Q, *dts = eL + Q, *wts = dts + Q;
+    float* const factors = reinterpret_cast<float*>(Sh + 2 * N * LD);    // two sets of L, exp(L), dt, exp(L_last - L) dt, [Q] each
     const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kChunkCols, j = h / (P / J), inner = P * dv, C = inner + 2 * J * N;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, tq = lane & 3;
+    const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, warp = wid & 3, gq = lane >> 2, tq = lane & 3;
     const int start = seqs[s], len = seqs[seqs_stride + s], rd = seqs[2 * seqs_stride + s], wr = seqs[3 * seqs_stride + s];
+    const bool reads_out = wid < 4;      // warps 0..3 make the outputs, warps 4..7 carry the state
     const float rate = expf(a_log[h]), bias = dt_bias[h], Dh = Dv[h];
-    float S[MT][4][4];      // [tile of 16 state rows][8 columns]
+    float S[MT][4][4];      // state warps: [tile of 16 state rows][8 columns]
+    if (!reads_out) {
 #pragma unroll
-    for (int m = 0; m < MT; m++)
+        for (int m = 0; m < MT; m++)
 #pragma unroll
-        for (int n = 0; n < 4; n++)
+            for (int n = 0; n < 4; n++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int r = (warp * MT + m) * 16 + gq + 8 * (e >> 1), c = c0 + n * 8 + 2 * tq + (e & 1);
-                S[m][n][e] = rd >= 0 && r < N && c < dv ? state[(long)rd * state_stride + ((long)h * N + r) * dv + c] : 0.f;
-            }
+                for (int e = 0; e < 4; e++) {
+                    const int r = (warp * MT + m) * 16 + gq + 8 * (e >> 1), c = c0 + n * 8 + 2 * tq + (e & 1);
+                    S[m][n][e] = rd >= 0 && r < N && c < dv ? state[(long)rd * state_stride + ((long)h * N + r) * dv + c] : 0.f;
+                }
+    }
     auto publish = [&]() {      // S as two bf16 terms for the next chunk
 #pragma unroll
         for (int m = 0; m < MT; m++)
@@ -265,169 +367,133 @@ __global__ void __launch_bounds__(128, MT <= 2 ? 3 : 1) ssd_chunk_kernel(const _
                     }
                 }
     };
-    publish();
+    if (!reads_out) publish();
     const int nc = N >> 3;      // 16-byte pieces per B or C row
-    for (int t0 = 0; t0 < len; t0 += Q) {
+    auto fetch = [&](int t0, int stage) {
         const int nt = min(Q, len - t0);
-        __syncthreads();      // the previous chunk's rows are consumed
-        for (int i = tid; i < Q * nc; i += 128) {
+        __nv_bfloat16 *Cd = ring + stage * stage_elems, *Bd = Cd + Q * ldn, *Xd = Bd + Q * ldn;
+        for (int i = tid; i < Q * nc; i += 256) {
             const int r = i / nc, c = i - r * nc;
             const __nv_bfloat16* src = xbc + (long)(start + t0 + (r < nt ? r : 0)) * C + inner + j * N + c * 8;
-            cp_async16(Bs + r * ldn + c * 8, src, r < nt);
-            cp_async16(Cs + r * ldn + c * 8, src + J * N, r < nt);
+            cp_async16(Bd + r * ldn + c * 8, src, r < nt);
+            cp_async16(Cd + r * ldn + c * 8, src + J * N, r < nt);
         }
-        for (int i = tid; i < Q * (kChunkCols / 8); i += 128) {
+        for (int i = tid; i < Q * (kChunkCols / 8); i += 256) {
             const int r = i >> 2, c = (i & 3) * 8;
             const bool ok = r < nt && c0 + c < dv;
-            cp_async16(Xs + r * LD + c, ok ? xbc + (long)(start + t0 + r) * C + h * dv + c0 + c : xbc, ok);
+            cp_async16(Xd + r * LD + c, ok ? xbc + (long)(start + t0 + r) * C + h * dv + c0 + c : xbc, ok);
         }
-        if (warp == 0) {      // tokens 2 lane and 2 lane + 1
-            float dt[2], la[2];
+    };
+    // the factors of the chunk at t0 by one warp, tokens 2 lane and 2 lane + 1 per lane; the step logits are asked for ahead of time
+    float dt_next[2];
+    auto fetch_dt = [&](int t0) {
 #pragma unroll
-            for (int e = 0; e < 2; e++) {
-                const int t = 2 * lane + e;
-                dt[e] = t < nt ? ssd_softplus(__bfloat162float(dt_in[(long)(start + t0 + t) * dt_stride + h]) + bias) : 0.f;
-                la[e] = -rate * dt[e];
-            }
-            float run = la[0] + la[1];
+        for (int e = 0; e < 2; e++) dt_next[e] = t0 + 2 * lane + e < len ? __bfloat162float(dt_in[(long)(start + t0 + 2 * lane + e) * dt_stride + h]) : 0.f;
+    };
+    auto make_factors = [&](int t0, int set) {
+        float *Ls = factors + set * 4 * Q, *eL = Ls + Q, *dts = eL + Q, *wts = dts + Q;
+        float dt[2], la[2];
 #pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float up = __shfl_up_sync(0xffffffffu, run, o);
-                if (lane >= o) run += up;
-            }
-            const float last = __shfl_sync(0xffffffffu, run, 31);
-            const float L0 = run - la[1];
-            Ls[2 * lane] = L0;
-            Ls[2 * lane + 1] = run;
-            eL[2 * lane] = expf(L0);
-            eL[2 * lane + 1] = expf(run);
-            dts[2 * lane] = dt[0];
-            dts[2 * lane + 1] = dt[1];
-            wts[2 * lane] = expf(last - L0) * dt[0];
-            wts[2 * lane + 1] = expf(last - run) * dt[1];
+        for (int e = 0; e < 2; e++) {
+            dt[e] = t0 + 2 * lane + e < len ? ssd_softplus(dt_next[e] + bias) : 0.f;
+            la[e] = -rate * dt[e];
         }
+        float run = la[0] + la[1];
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float up = __shfl_up_sync(0xffffffffu, run, o);
+            if (lane >= o) run += up;
+        }
+        const float last = __shfl_sync(0xffffffffu, run, 31);
+        const float L0 = run - la[1];
+        Ls[2 * lane] = L0;
+        Ls[2 * lane + 1] = run;
+        eL[2 * lane] = expf(L0);
+        eL[2 * lane + 1] = expf(run);
+        dts[2 * lane] = dt[0];
+        dts[2 * lane + 1] = dt[1];
+        wts[2 * lane] = expf(last - L0) * dt[0];
+        wts[2 * lane + 1] = expf(last - run) * dt[1];
+    };
+    const int factor_warp = 7;
+    if (len > 0) {
+        fetch(0, 0);
+        if (wid == factor_warp) {
+            fetch_dt(0);
+            make_factors(0, 0);
+        }
+    }
+    int stage = 0;
+    for (int t0 = 0; t0 < len; t0 += Q, stage ^= 1) {
+        const int nt = min(Q, len - t0);
+        const __nv_bfloat16 *Cs = ring + stage * stage_elems, *Bs = Cs + Q * ldn, *Xs = Bs + Q * ldn;
+        const float *Ls = factors + stage * 4 * Q, *eL = Ls + Q, *dts = eL + Q, *wts = dts + Q;
         cp_async_wait_all();
-        __syncthreads();
-        for (int i = tid; i < Q * kChunkCols / 2; i += 128) {
-            const int r = i / (kChunkCols / 2), c = (i % (kChunkCols / 2)) * 2;
-            const uint32_t u = *reinterpret_cast<const uint32_t*>(Xs + r * LD + c);
-            uint32_t hi, lo;
-            split_bf16(__uint_as_float(u << 16) * wts[r], __uint_as_float(u & 0xffff0000u) * wts[r], hi, lo);
-            *reinterpret_cast<uint32_t*>(Xh + r * LD + c) = hi;
-            *reinterpret_cast<uint32_t*>(Xh + (Q + r) * LD + c) = lo;
+        __syncthreads();      // this chunk, its factors and the state ahead of it are there; the other stage is free
+        if (t0 + Q < len) {
+            fetch(t0 + Q, stage ^ 1);
+            if (wid == factor_warp) fetch_dt(t0 + Q);
         }
-        const bool live = warp * 16 < nt;
-        if (live) {      // this warp's 16 tokens: C S and the scores against the chunk's tokens up to its own, one pass over the state rows
-            float Y[4][4], G[8][4];
-#pragma unroll
-            for (int n = 0; n < 4; n++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) Y[n][e] = 0.f;
-#pragma unroll
-            for (int n = 0; n < 8; n++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) G[n][e] = 0.f;
-            for (int kk = 0; kk < n16; kk++) {
-                uint32_t a[4], b[4];
-                ldmatrix_x4(a, Cs + (warp * 16 + (lane & 15)) * ldn + kk * 16 + 8 * (lane >> 4));
-#pragma unroll
-                for (int np = 0; np < 4; np++)
-                    if (np <= warp) {
-                        ldmatrix_x4(b, Bs + (np * 16 + (lane & 7) + 8 * (lane >> 4)) * ldn + kk * 16 + 8 * ((lane >> 3) & 1));
-                        mma_bf16_16816(G[2 * np], a, b[0], b[1]);
-                        mma_bf16_16816(G[2 * np + 1], a, b[2], b[3]);
-                    }
-#pragma unroll
-                for (int term = 0; term < 2; term++)
-#pragma unroll
-                    for (int vp = 0; vp < 2; vp++) {
-                        ldmatrix_x4_trans(b, Sh + (term * N + kk * 16 + (lane & 15)) * LD + vp * 16 + 8 * (lane >> 4));
-                        mma_bf16_16816(Y[2 * vp], a, b[0], b[1]);
-                        mma_bf16_16816(Y[2 * vp + 1], a, b[2], b[3]);
-                    }
+        if (!reads_out) {
+            for (int i = tid - 128; i < Q * kChunkCols / 2; i += 128) {      // the weighted x rows
+                const int r = i / (kChunkCols / 2), c = (i % (kChunkCols / 2)) * 2;
+                const uint32_t u = *reinterpret_cast<const uint32_t*>(Xs + r * LD + c);
+                uint32_t hi, lo;
+                split_bf16(__uint_as_float(u << 16) * wts[r], __uint_as_float(u & 0xffff0000u) * wts[r], hi, lo);
+                *reinterpret_cast<uint32_t*>(Xh + r * LD + c) = hi;
+                *reinterpret_cast<uint32_t*>(Xh + (Q + r) * LD + c) = lo;
             }
-            const int iA = warp * 16 + gq, iB = iA + 8;
-            const float LA = Ls[iA], LB = Ls[iB], eA = eL[iA], eB = eL[iB];
+            asm volatile("bar.sync 1, 128;" ::: "memory");      // among the state warps
+            const float keep = eL[Q - 1];
+            const int k16 = (nt + 15) >> 4;
 #pragma unroll
-            for (int n = 0; n < 4; n++) {
-                Y[n][0] *= eA;
-                Y[n][1] *= eA;
-                Y[n][2] *= eB;
-                Y[n][3] *= eB;
-            }
-#pragma unroll
-            for (int n = 0; n < 8; n++) {
-                if (n < 2 * (warp + 1)) {
-#pragma unroll
-                    for (int e = 0; e < 4; e++) {
-                        const int jj = n * 8 + 2 * tq + (e & 1), ii = e < 2 ? iA : iB;
-                        G[n][e] = jj <= ii ? G[n][e] * __expf((e < 2 ? LA : LB) - Ls[jj]) * dts[jj] : 0.f;
-                    }
-                }
-            }
-#pragma unroll
-            for (int kk = 0; kk < 4; kk++) {
-                if (kk <= warp) {
-                    uint32_t hi[4], lo[4];
-                    split_bf16(G[2 * kk][0], G[2 * kk][1], hi[0], lo[0]);
-                    split_bf16(G[2 * kk][2], G[2 * kk][3], hi[1], lo[1]);
-                    split_bf16(G[2 * kk + 1][0], G[2 * kk + 1][1], hi[2], lo[2]);
-                    split_bf16(G[2 * kk + 1][2], G[2 * kk + 1][3], hi[3], lo[3]);
-#pragma unroll
-                    for (int vp = 0; vp < 2; vp++) {
-                        uint32_t b[4];
-                        ldmatrix_x4_trans(b, Xs + (kk * 16 + (lane & 15)) * LD + vp * 16 + 8 * (lane >> 4));
-                        mma_bf16_16816(Y[2 * vp], hi, b[0], b[1]);
-                        mma_bf16_16816(Y[2 * vp + 1], hi, b[2], b[3]);
-                        mma_bf16_16816(Y[2 * vp], lo, b[0], b[1]);
-                        mma_bf16_16816(Y[2 * vp + 1], lo, b[2], b[3]);
-                    }
-                }
-            }
-#pragma unroll
-            for (int n = 0; n < 4; n++) {
-                const int c = c0 + n * 8 + 2 * tq;
-                if (c < dv) {
-#pragma unroll
-                    for (int e = 0; e < 4; e += 2) {
-                        const int i = e ? iB : iA;
-                        if (i < nt) {
-                            const uint32_t u = *reinterpret_cast<const uint32_t*>(Xs + i * LD + n * 8 + 2 * tq);
-                            *reinterpret_cast<float2*>(y_out + (long)(start + t0 + i) * inner + h * dv + c) =
-                                make_float2(fmaf(Dh, __uint_as_float(u << 16), Y[n][e]), fmaf(Dh, __uint_as_float(u & 0xffff0000u), Y[n][e + 1]));
-                        }
-                    }
-                }
-            }
-        }
-        __syncthreads();      // every warp has read the old state, and the weighted rows are there
-        const float keep = eL[Q - 1];
-        const int k16 = (nt + 15) >> 4;
-#pragma unroll
-        for (int m = 0; m < MT; m++) {
-            const int r0 = (warp * MT + m) * 16;
-            if (r0 < N) {
+            for (int m = 0; m < MT; m++)
 #pragma unroll
                 for (int n = 0; n < 4; n++)
 #pragma unroll
                     for (int e = 0; e < 4; e++) S[m][n][e] *= keep;
+            if (warp * MT * 16 < N) {
+#pragma unroll 2
                 for (int kk = 0; kk < k16; kk++) {
-                    uint32_t a[4], b[4];
-                    ldmatrix_x4_trans(a, Bs + (kk * 16 + (lane & 7) + 8 * (lane >> 4)) * ldn + r0 + 8 * ((lane >> 3) & 1));
+                    uint32_t x[2][2][4];
 #pragma unroll
                     for (int term = 0; term < 2; term++)
 #pragma unroll
-                        for (int vp = 0; vp < 2; vp++) {
-                            ldmatrix_x4_trans(b, Xh + (term * Q + kk * 16 + (lane & 15)) * LD + vp * 16 + 8 * (lane >> 4));
-                            mma_bf16_16816(S[m][2 * vp], a, b[0], b[1]);
-                            mma_bf16_16816(S[m][2 * vp + 1], a, b[2], b[3]);
+                        for (int vp = 0; vp < 2; vp++) ldmatrix_x4_trans(x[term][vp], Xh + (term * Q + kk * 16 + (lane & 15)) * LD + vp * 16 + 8 * (lane >> 4));
+#pragma unroll
+                    for (int m = 0; m < MT; m++) {
+                        const int r0 = (warp * MT + m) * 16;
+                        if (r0 < N) {
+                            uint32_t a[4];
+                            ldmatrix_x4_trans(a, Bs + (kk * 16 + (lane & 7) + 8 * (lane >> 4)) * ldn + r0 + 8 * ((lane >> 3) & 1));
+#pragma unroll
+                            for (int term = 0; term < 2; term++)
+#pragma unroll
+                                for (int vp = 0; vp < 2; vp++) {
+                                    mma_bf16_16816(S[m][2 * vp], a, x[term][vp][0], x[term][vp][1]);
+                                    mma_bf16_16816(S[m][2 * vp + 1], a, x[term][vp][2], x[term][vp][3]);
+                                }
                         }
+                    }
                 }
             }
+            if (t0 + Q < len) {
+                if (wid == factor_warp) make_factors(t0 + Q, stage ^ 1);
+                asm volatile("bar.sync 2, 256;" ::: "memory");      // the output warps have read the old state
+                publish();
+            }
+            continue;
         }
-        if (t0 + Q < len) publish();
+        if (warp * 16 < nt) {
+            float* y = y_out + (long)(start + t0) * inner + h * dv + c0;
+            const bool more = t0 + Q < len;
+            if (warp == 0) ssd_chunk_outputs<0>(Cs, Bs, Xs, Sh, Ls, eL, dts, N, nt, more, Dh, y, inner, dv - c0);
+            else if (warp == 1) ssd_chunk_outputs<1>(Cs, Bs, Xs, Sh, Ls, eL, dts, N, nt, more, Dh, y, inner, dv - c0);
+            else if (warp == 2) ssd_chunk_outputs<2>(Cs, Bs, Xs, Sh, Ls, eL, dts, N, nt, more, Dh, y, inner, dv - c0);
+            else ssd_chunk_outputs<3>(Cs, Bs, Xs, Sh, Ls, eL, dts, N, nt, more, Dh, y, inner, dv - c0);
+        }
     }
-    if (wr >= 0) {
+    if (!reads_out && wr >= 0) {
 #pragma unroll
         for (int m = 0; m < MT; m++)
 #pragma unroll
@@ -622,7 +688,7 @@ extern "C" int ktb200_ssd_scan(const ktb200_ssd_params* c, const void* xbc, floa
 #define CHUNK_LAUNCH(MT)                                                                                                                                                       \
     do {                                                                                                                                                                       \
         GRANT_SMEM(ssd_chunk_kernel<MT>, smem);                                                                                                                                \
-        ssd_chunk_kernel<MT><<<grid, 128, smem, (cudaStream_t)stream>>>((const B*)xbc, (const B*)c->proj + c->dt_off, c->proj_stride, c->dt_bias, c->a_log, c->d_skip, c->heads, \
+        ssd_chunk_kernel<MT><<<grid, 256, smem, (cudaStream_t)stream>>>((const B*)xbc, (const B*)c->proj + c->dt_off, c->proj_stride, c->dt_bias, c->a_log, c->d_skip, c->heads, \
                                                                         c->groups, c->state_size, c->vdim, c->seqs, c->seqs_stride, c->state, c->state_stride, y);            \
     } while (0)
         if (c->state_size <= 64) CHUNK_LAUNCH(1);
