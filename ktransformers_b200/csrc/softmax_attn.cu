@@ -193,7 +193,7 @@ __global__ void __launch_bounds__(256) rope_norm_cache_write_kernel(const QkvPre
 // The same behind a filter, by column pairs: grid (tiles of `tile` consecutive tokens, unit blocks), a warp per unit walks over the tile's tokens with
 // the filter's last TAPS - 1 inputs in registers, a lane owning the column pairs 2 lane + 64 e: every input is read once per tile instead of TAPS
 // times, a rotated pair (interleaved layout) lies in one lane, loads and stores take two columns.  Loads of kPairBatch tokens are in flight
-// together.  Even head sizes and offsets; no row-wide norm, value blend or value norm (those take the kernel above).
+// together.  Without norms the maps of a head are one unit (a column turns by its place among turn_width).  Even head sizes and offsets; no row-wide norm, value blend or value norm (those take the kernel above).
 constexpr int kPairTile = 16, kPairBatch = 4;
 __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
 __device__ __forceinline__ float2 load2(const __nv_bfloat16* p) {
@@ -204,7 +204,7 @@ __device__ __forceinline__ void store2(float* p, float x, float y) { *reinterpre
 __device__ __forceinline__ void store2(__nv_bfloat16* p, float x, float y) { *reinterpret_cast<uint32_t*>(p) = pack_bf16(x, y); }
 
 template <typename T, int TAPS, int PAIRS>
-__global__ void __launch_bounds__(256, PAIRS > 2 ? 1 : 2) conv_rope_cache_write_kernel(const QkvPrep a, int n_tokens, int tile) {
+__global__ void __launch_bounds__(256, PAIRS > 2 ? 1 : 2) conv_rope_cache_write_kernel(const QkvPrep a, int n_tokens, int tile, int turn_width) {
     extern __shared__ __align__(16) float2 turn_s[];      // [tile][rot_dims / 2] (cos, sin)
     __shared__ int info[kPairTile][5];                    // per token: first row, tokens, row to read, row to write of its portion; cache row
     constexpr int BACK = TAPS - 1;
@@ -244,6 +244,9 @@ __global__ void __launch_bounds__(256, PAIRS > 2 ? 1 : 2) conv_rope_cache_write_
                 w[j][e][1] = i < n ? to_f(cw[(long)(ch0 + i + 1) * TAPS + j]) : 0.f;
             }
         }
+        int at_turn[PAIRS];      // which pair of its map a lane's column pair is
+#pragma unroll
+        for (int e = 0; e < PAIRS; e++) at_turn[e] = ((2 * lane + 64 * e) % turn_width) >> 1;
         int cur = -1;
         for (int b = 0; b < nt; b += kPairBatch) {
             float2 in[kPairBatch][PAIRS];
@@ -297,8 +300,8 @@ __global__ void __launch_bounds__(256, PAIRS > 2 ? 1 : 2) conv_rope_cache_write_
                     }
                     win[BACK - 1][e][0] = in[k][e].x;
                     win[BACK - 1][e][1] = in[k][e].y;
-                    if (!is_v && i < a.rot_dims) {
-                        const float2 cs = turn_s[tt * half + (i >> 1)];
+                    if (!is_v && at_turn[e] < half) {
+                        const float2 cs = turn_s[tt * half + at_turn[e]];
                         const float z = x0;
                         x0 = z * cs.x - x1 * cs.y;
                         x1 = x1 * cs.x + z * cs.y;
@@ -876,11 +879,16 @@ extern "C" int ktb200_qkv_prep(const ktb200_qkv_prep_params* c, int n_tokens, in
         int y = (1184 + tiles - 1) / tiles;
         y = y > max_y ? max_y : y;
         QkvPrep b = a;
-        b.units_per_cta = ((units + y - 1) / y + 7) / 8 * 8;
-        const dim3 grid(tiles, (units + b.units_per_cta - 1) / b.units_per_cta);
+        int n_units = units;
+        if (c->maps > 1 && c->qk_norm == kQkNormNone && c->dim * c->maps <= 32 * kPrepMaxPerLane) {
+            b.Hq = c->heads; b.Gk = c->kv_heads; b.d = c->dim * c->maps;
+            n_units = c->heads + 2 * c->kv_heads;
+        }
+        b.units_per_cta = ((n_units + y - 1) / y + 7) / 8 * 8;
+        const dim3 grid(tiles, (n_units + b.units_per_cta - 1) / b.units_per_cta);
         const size_t smem = (size_t)tile * (c->rot_dims / 2) * sizeof(float2);
-        const int widest = c->dim > c->vdim ? c->dim : c->vdim;
-#define PAIR_LAUNCH(TAPS, PAIRS) conv_rope_cache_write_kernel<T, TAPS, PAIRS><<<grid, 256, smem, (cudaStream_t)stream>>>(b, n_tokens, tile)
+        const int widest = b.d > c->vdim ? b.d : c->vdim;
+#define PAIR_LAUNCH(TAPS, PAIRS) conv_rope_cache_write_kernel<T, TAPS, PAIRS><<<grid, 256, smem, (cudaStream_t)stream>>>(b, n_tokens, tile, c->dim)
 #define PAIR_SIZES(TAPS)                               \
     do {                                               \
         if (widest <= 64) PAIR_LAUNCH(TAPS, 1);        \
