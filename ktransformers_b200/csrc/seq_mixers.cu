@@ -592,14 +592,23 @@ __global__ void xielu_kernel(const T* __restrict__ z, T* __restrict__ out, const
 // ------------------------------------------------------------------------------------------------ gated activation
 // out[t][i] = gated_act(r gate[t * stride + i], r up[t * stride + i]) (seq_common.cuh), r = row_scale ? row_scale[t] : 1; rows [gate F | up F]:
 // up = gate + F, stride = 2 F
-template <typename T>
-__global__ void gated_act_mul_kernel(const T* __restrict__ gate, const T* __restrict__ up, long stride, T* __restrict__ out, long n_rows, int F, int act, float limit, const float* __restrict__ row_scale) {
-    const long n = n_rows * F;
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) gated_act_mul_kernel(const T* __restrict__ gate, const T* __restrict__ up, long stride, T* __restrict__ out, long n_rows, int F, int act, float limit,
+                                                            const float* __restrict__ row_scale) {
+    const int per_row = F / VEC;      // VEC = 4: rows of whole groups of four, 16- / 8-byte accesses
+    const long n = n_rows * per_row;
     for (long i = blockIdx.x * (long)blockDim.x + threadIdx.x; i < n; i += (long)gridDim.x * blockDim.x) {
-        const long t = i / F;
-        const int c = (int)(i - t * F);
+        const long t = n <= 0x7fffffffL ? (long)((unsigned)i / (unsigned)per_row) : i / per_row;
+        const int c = (int)(i - t * per_row) * VEC;
         const float r = row_scale ? row_scale[t] : 1.0f;
-        out[i] = from_f<T>(gated_act(r * to_f(gate[t * stride + c]), r * to_f(up[t * stride + c]), act, limit));
+        const T *gp = gate + t * stride + c, *upp = up + t * stride + c;
+        if (VEC == 4) {
+            const float4 g = load4(gp), u = load4(upp);
+            store4(out + t * F + c, make_float4(gated_act(r * g.x, r * u.x, act, limit), gated_act(r * g.y, r * u.y, act, limit), gated_act(r * g.z, r * u.z, act, limit),
+                                                gated_act(r * g.w, r * u.w, act, limit)));
+        } else {
+            out[t * F + c] = from_f<T>(gated_act(r * to_f(gp[0]), r * to_f(upp[0]), act, limit));
+        }
     }
 }
 // out = relu(z)^2, element by element
@@ -781,8 +790,13 @@ extern "C" int ktb200_xielu(const void* z, void* out, const float* pq, long n, i
 extern "C" int ktb200_gated_act_mul(const void* gate, const void* up, long in_stride, void* out, int n_tokens, int ff, int act, float limit, const float* row_scale, int dtype, void* stream) {
     if (!gate || !up || !out || ff <= 0 || in_stride < ff || act < kActSilu || act > kActClampedGlu) { set_error("gated_act_mul: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
-    SEQ_DISPATCH(dtype, (gated_act_mul_kernel<T><<<grid_for((long)n_tokens * ff, 256 * 4), 256, 0, (cudaStream_t)stream>>>((const T*)gate, (const T*)up, in_stride, (T*)out,
-                                                                                                                         n_tokens, ff, act, limit, row_scale)));
+    const size_t four = dtype == KTB200_TYPE_BF16 ? 8 : 16;
+    auto al = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (four - 1)) == 0; };
+    const bool vec = ff % 4 == 0 && in_stride % 4 == 0 && al(gate) && al(up) && al(out);
+    SEQ_DISPATCH(dtype, {
+        if (vec) gated_act_mul_kernel<T, 4><<<grid_for((long)n_tokens * ff / 4, 256), 256, 0, (cudaStream_t)stream>>>((const T*)gate, (const T*)up, in_stride, (T*)out, n_tokens, ff, act, limit, row_scale);
+        else gated_act_mul_kernel<T, 1><<<grid_for((long)n_tokens * ff, 256 * 4), 256, 0, (cudaStream_t)stream>>>((const T*)gate, (const T*)up, in_stride, (T*)out, n_tokens, ff, act, limit, row_scale);
+    });
     KTB_LAUNCH_CHECK();
     return KTB200_OK;
 }
