@@ -147,11 +147,11 @@ class KStateSpace(nn.Module):
         [z | x | B | C | dt] = W_in h                          x: heads x vdim; B, C: groups x state_size, shared by heads / groups heads each
         x, B, C = silu(filter(x, B, C) + b)                     a causal filter of `conv` taps along time on every channel
         dt      = softplus(dt + dt_bias) ;  S <- exp(-exp(A_log) dt) S + dt B x^T ;  y = S^T C + D x      per head, S in fp32
-        out     = W_o (norm(y silu(z)) w)                       norm: `norm_groups` equal parts, each divided by its own rms
+        out     = W_o (norm(y silu(z)) w)                       norm: `norm_groups` equal parts, each to unit rms
 
         P     = W_in h                                          one GEMM
         y     = prompt portions: ktb200_ssd_conv + ktb200_ssd_scan; decode steps (one token per sequence): ktb200_ssd_step
-        o     = ktb200_gated_group_norm                         (the gate comes before the norm)
+        o     = ktb200_gated_group_norm                         (gated first, then normed)
         out   = W_o o                                           GEMM
 
     A sequence's state — the matrices and the last conv - 1 inputs of every filtered channel — lives in the cache manager's double-buffered

@@ -134,7 +134,7 @@ def state_space_scan(x, B, Cm, dt, a_log, D, S):
 
 
 def gated_group_norm(y, z, w, groups, eps):
-    """y silu(z), then every one of `groups` equal parts divided by its own root mean square, then times w"""
+    """u = y silu(z) is cut into `groups` equal parts, each part scaled to unit rms, and the row multiplied by w"""
     T, n = y.shape
     u = (y * silu(z)).reshape(T, groups, n // groups)
     return rms(u, eps).reshape(T, n) * w
