@@ -200,7 +200,8 @@ typedef struct ktb200_gate_config {
     int n_group;               /* 1 = no grouping */
     int topk_group;
     int scoring;               /* 0 sigmoid (V3), 1 softmax (V2), 2 softmax over the chosen logits only, `bias` added to the logits */
-    int topk_method;           /* 0 noaux_tc (V3), 1 greedy, 2 group_limited_greedy (V2) */
+    int topk_method;           /* 0 noaux_tc (V3), 1 greedy, 2 group_limited_greedy (V2), 3 biased_group_max: as 0 with a group's largest biased
+                                  score as its score (ktb200_moe_gate_forward and _select only) */
     int norm_topk_prob;
     float routed_scaling_factor;
     const float* weight;       /* DEVICE fp32 [n_experts][hidden] */
@@ -401,9 +402,9 @@ int ktb200_rope_rows(const void* q, int num_heads, int dim, int rot_dim, int rot
 int ktb200_sigmoid_gate_mul(const void* heads, const void* gate, long gate_stride, void* out, int n_tokens, int num_heads, int vdim,
                             int dtype, void* stream);
 int ktb200_poly_norm(const void* z, void* out, const float* coef, float eps, int n_tokens, int ff, int dtype, void* stream);
-int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top, const void* w_gate, const void* w_up, void* act, int n_tokens,
+int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top, int n_experts, const void* w_gate, const void* w_up, void* act, int n_tokens,
                            int width, int ff, int act_kind, float limit, const float* in_weights, int dtype, void* stream);
-int ktb200_experts_down(const void* act, const int64_t* ids, const float* weights, int top, const void* w_down, float* out, int n_tokens,
+int ktb200_experts_down(const void* act, const int64_t* ids, const float* weights, int top, int n_experts, const void* w_down, float* out, int n_tokens,
                         int width, int ff, int dtype, void* stream);
 /* the same for batches of a few tokens, by expert: each expert's rows are streamed once per `staged` (2 or 4; 0: chosen from the
  *   batch) pairs routed to it instead of once per pair; pair_rows [T*top][width] fp32 is scratch for the per-pair down rows
@@ -413,6 +414,10 @@ int ktb200_experts_gate_up_by_expert(const void* x, const int64_t* ids, int top,
                                      void* stream);
 int ktb200_experts_down_by_expert(const void* act, const int64_t* ids, const float* weights, int top, int n_experts, const void* w_down,
                                   float* pair_rows, float* out, int n_tokens, int width, int ff, int staged, int dtype, void* stream);
+/* ktb200_experts_combine: out[t] = sum_j weights[t][j] rows[place[t * top + j]] (place NULL: row t * top + j), rows of dtype, fp32 sums in slot
+ *   order: the last step of a grouped run.  In all of these calls an id at or beyond n_experts names no expert: its pair adds nothing. */
+int ktb200_experts_combine(const void* rows, const int64_t* place, const int64_t* ids, int n_experts, const float* weights, int top, float* out,
+                           int n_tokens, int width, int dtype, void* stream);
 /* w_gate == NULL in the four calls above: experts of two matrices, act = relu(W_up x)^2.  Otherwise act_kind picks what becomes of
  * g = W_gate x and u = W_up x: 0 silu(g) u; 1 gelu(g) u (tanh form); 2 g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit),
  * u' = clamp(u, -limit, limit).  in_weights [T*top] (NULL: none): an expert sees in_weights[pair] * x; the down calls take weights == NULL
@@ -430,7 +435,7 @@ int ktb200_experts_down_by_expert(const void* act, const int64_t* ids, const flo
  *   ktb200_gla_scan                 per sequence portion seqs[0..3][s] = (first row, rows, state row to read or -1, state row to write or -1):
  *                                   S <- diag(a_t) S + k_t v_t^T, o_t = S^T q_t / sqrt(dim), a = sigmoid(z + z_bias)^(1 / tau); state rows
  *                                   [heads][dim][vdim] fp32; q / k / v at column offsets of proj; dim <= 256
- *   ktb200_gla_out                  out = o / sqrt(mean_vdim(o^2) + eps) * norm_w * silu(gate)
+ *   ktb200_gla_out                  out = o / sqrt(mean_vdim(o^2) + eps) * norm_w * silu(gate) (norm_w NULL: ones)
  *   ktb200_xielu                    z > 0: softplus(pq[0]) z^2 + z/2 ; else (1/2 + softplus(pq[1])) (exp(z) - 1 - z) + z/2 */
 int ktb200_group_rmsnorm_sandwich(const float* x_in, const void* y, int y_type, const void* w_post, const float* row_add, float* x_out,
                                   const void* w_pre, void* h_out, int groups, float eps, float weight_offset, int n_tokens, int width, int dtype,
@@ -464,7 +469,8 @@ int ktb200_softcap(const void* z, float* out, long n, float cap, int dtype, void
 /* Soft-max attention over grouped key/value heads (csrc/softmax_attn.cu) and the gated delta rule (csrc/delta_rule.cu):
  *   ktb200_rope_norm_cache_write   proj rows hold q [H*d] at q_off, k [G*d] at k_off, v [G*dv] at v_off: q and k turn over their first rot_dims
  *                                  columns (rot_layout as above), are divided by sqrt(mean(x^2) + eps) per head (qk_norm 1), or over the whole
- *                                  q (k) row and then multiplied by q_weight [H*d] (k_weight [G*d]) (qk_norm 2; 0: neither), v becomes
+ *                                  q (k) row and then multiplied by q_weight [H*d] (k_weight [G*d]) (qk_norm 2; 0: neither; 3: per head times a weight [d], ahead of
+ *                                  the rotation), v becomes
  *                                  (1 - blend[0]) v + blend[0] v_other[token] when v_other is given and is then divided by sqrt(mean(v^2) + eps)
  *                                  per value head when v_unit_rms; [k | v] into the paged cache, q into q_out
  *   ktb200_window_softmax_attn     out[t][h] = sum_j softmax_j(cap(scale head_scale[h] q.k_j)) v_j over the keys j <= pos with pos - j < window
@@ -583,6 +589,84 @@ int ktb200_ssd_scan_uses_tensor_cores(int heads, int groups, int state_size, int
 int ktb200_ssd_step(const ktb200_ssd_params* params, float* y, int dtype, void* stream);
 int ktb200_gated_group_norm(const float* y, const void* z, long z_stride, const void* weight, int groups, float eps, float out_scale, void* out,
                             long out_stride, int n_tokens, int width, int dtype, void* stream);
+
+/* A norm that follows the residual sum and whose row is the new stream (csrc/seq_ops.cu): with row r = rows ? rows[t] : t of x, a, b, b_scale, ids
+ * and id_weights,
+ *     s = (x_scale + sum of id_weights[r][j] over the j with ids[r][j] >= first_identity) x + a + b_scale[r] b ;  y = s / sqrt(mean(s^2) + eps) * weight
+ * (every term but x may be NULL; x, a, b fp32 or bf16 by their types).  y to x_out (fp32) and h_out (dtype), at least one of them; with dot_weight
+ * also dot_out[t] = sigmoid(y . dot_weight). */
+typedef struct {
+    const void* x;
+    int x_type;
+    float x_scale;
+    const void* a;
+    int a_type;
+    const void* b;
+    int b_type;
+    const float* b_scale;
+    const int64_t* ids;
+    const float* id_weights;
+    int top, first_identity;
+    const int64_t* rows;
+    const void* weight;
+    float eps;
+    float* x_out;
+    void* h_out;
+    const void* dot_weight;
+    float* dot_out;
+} ktb200_sum_rmsnorm_params;
+int ktb200_sum_rmsnorm(const ktb200_sum_rmsnorm_params* params, int n_tokens, int width, int dtype, void* stream);
+
+/* Retention (csrc/retention.cu): proj rows hold q and k [heads*dim] and v [heads*vdim] at their offsets and an output gate [heads*vdim] at g_off;
+ * q and k turn over their first rot_dims columns by the (cos, sin) pairs turn [n_tokens][rot_dims / 2], k is multiplied by k_scale; per portion
+ * (seqs as for ktb200_gla_scan) and head, fp32:
+ *     S <- decay[h] S + k v^T ;  o = S^T q ;  out = o / sqrt(mean_vdim(o^2) + eps) * silu(g)
+ * log2_decay[h] = log2(decay[h]).  State rows [heads][dim][vdim] fp32, row stride state_stride; dim <= 256.
+ *   ktb200_turn_table        turn[t][i] = (cos, sin) of pos[t] * inv_freq[i], angles in fp64
+ *   ktb200_retention_chunk   chunks of 64 tokens on the tensor cores (bf16; dim and vdim multiples of 16 up to 128): the states ahead of every chunk, then
+ *                            all chunks at once; workspace: ktb200_retention_chunk_workspace bytes
+ *   ktb200_retention_scan    token by token; o [n_tokens][heads*vdim] fp32 is left for ktb200_gla_out
+ *   ktb200_retention_step    decode steps (one token per portion), norm and gate included; vdim <= ktb200_retention_step_max_vdim() */
+typedef struct {
+    const void* proj;
+    long proj_stride;
+    int q_off, k_off, v_off, g_off, heads, dim, vdim, rot_dims, rot_layout;
+    const float* turn;
+    float k_scale;
+    const float *decay, *log2_decay;
+    float eps;
+    const int* seqs;
+    int seqs_stride, n_seqs;
+    float* state;
+    long state_stride;
+} ktb200_retention_params;
+int ktb200_turn_table(const int* pos, const double* inv_freq, int pairs, float* turn, int n_tokens, void* stream);
+int ktb200_retention_chunk_supported(int dim, int vdim, int dtype);
+size_t ktb200_retention_chunk_workspace(int heads, int dim, int vdim, int n_tokens, int n_seqs);
+int ktb200_retention_chunk(const ktb200_retention_params* params, void* out, int n_tokens, void* workspace, size_t workspace_bytes, int dtype, void* stream);
+int ktb200_retention_scan(const ktb200_retention_params* params, float* o, int dtype, void* stream);
+int ktb200_retention_step_max_vdim(void);
+int ktb200_retention_step(const ktb200_retention_params* params, void* out, int dtype, void* stream);
+
+/* Mamba, the selective scan (csrc/selective_scan.cu): per channel c and state n, fp32,
+ *     dt = softplus(dt_logit + dt_bias[c]) ;  S[c][n] <- exp(dt a[c][n]) S[c][n] + dt x B[n] ;  y = sum_n S[c][n] C[n] + d_skip[c] x ;  out = y silu(z)
+ * x [n_tokens][inner] (ktb200_conv_silu's output), dt_logit, z rows of their strides, B and C runs of `state_size` values at b and c (row stride
+ * bc_stride); a [inner][state_size] negative.  State rows [S inner*state_size | filter inputs (taps - 1)*inner], row stride state_stride;
+ * portions seqs as for ktb200_gla_scan; state_size <= 256.
+ *   ktb200_conv_silu   out = silu(filter(in) + bias) on `channels` channels, the portions' last taps - 1 inputs at conv_off of their state rows */
+typedef struct {
+    const void *x, *dt_logit, *b, *c, *z;
+    long dt_stride, bc_stride, z_stride;
+    const float *dt_bias, *a, *d_skip;
+    int inner, state_size;
+    const int* seqs;
+    int seqs_stride, n_seqs;
+    float* state;
+    long state_stride;
+} ktb200_selective_scan_params;
+int ktb200_conv_silu(const void* in, long in_stride, const void* conv_w, const void* conv_b, int taps, int channels, const int* seq_of, const int* seqs,
+                     int seqs_stride, float* state, long state_stride, long conv_off, void* out, int n_tokens, int n_seqs, int dtype, void* stream);
+int ktb200_selective_scan(const ktb200_selective_scan_params* params, void* out, int dtype, void* stream);
 
 /* Diagnostics (bench.py --probe): time a plain read-only stream over `bytes` of device memory.
  * mode 0 = grid-stride coalesced 16-byte loads; mode 1 = every warp reads chunk_bytes pieces at hashed offsets

@@ -91,7 +91,7 @@ __device__ void gate_select_token(const GateParams& pin, int t, float* sm, int64
 #pragma unroll
     for (int i = 0; i < kGateEPT; i++) {
         const int e = tid + kGateThreads * i;
-        bv[i] = (p.topk_method == 0 && p.bias && e < E) ? __ldg(p.bias + e) : 0.f;
+        bv[i] = ((p.topk_method == 0 || p.topk_method == 3) && p.bias && e < E) ? __ldg(p.bias + e) : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < kGateEPT; i++) {
@@ -154,7 +154,8 @@ __device__ void gate_select_token(const GateParams& pin, int t, float* sm, int64
     }
     gate_sync<BAR>();
 
-    // group selection (noaux_tc: sum of the group's top-2 biased scores; group_limited_greedy: group max)
+    // group selection (noaux_tc: sum of the group's top-2 biased scores; group_limited_greedy: group max; 3, biased_group_max: the
+    // group's largest biased score)
     if (p.n_group > 1 && p.topk_method != 1) {
         const int gs = E / p.n_group;
         for (int g = warp; g < p.n_group; g += kGateWarps) {   // one warp per group
@@ -171,7 +172,7 @@ __device__ void gate_select_token(const GateParams& pin, int t, float* sm, int64
             if (lane == 0) gsc[g] = (p.topk_method == 0 && gs > 1) ? (fkey_inv(mx1) + fkey_inv(mx2)) : fkey_inv(mx1);
         }
         gate_sync<BAR>();
-        const float fill = (p.topk_method == 0) ? -INFINITY : 0.0f;  // V3 masks with -inf, V2 with 0.0
+        const float fill = (p.topk_method == 2) ? 0.0f : -INFINITY;  // V3 and biased_group_max mask with -inf, V2 with 0.0
 #pragma unroll
         for (int i = 0; i < kGateEPT; i++) {
             const int e = tid + kGateThreads * i;

@@ -1,0 +1,766 @@
+// Retention: linear attention whose matrix state per head decays by one fixed number per head, with rotated queries and keys, a unit-rms head
+// output and an output gate (libktb200_seq.so).
+//
+//   S <- decay_h S + k v^T ;  o = S^T q ;  out = o / sqrt(mean_c(o_c^2) + eps) * silu(g)          per head; q, k turned, k times k_scale
+//
+//   ktb200_turn_table        the (cos, sin) pairs of a step's tokens, once for all layers of the same rotation
+//   ktb200_retention_chunk   prompt portions in chunks of 64 tokens on the tensor cores, chunks in parallel (bf16)
+//   ktb200_retention_scan    token by token on CUDA cores (fp32, sizes outside the tiles, short portions), o left for ktb200_gla_out
+//   ktb200_retention_step    decode steps: rotation, recurrence, norm and gate in one launch, a head's column blocks as a thread-block cluster
+//
+// State row of a sequence and layer (fp32): S [heads][dim][vdim], read from the row seqs[2][s] (or zeros when -1) and written to the row seqs[3][s].
+// Storage type T (bf16 or float) for projections and outputs; turned queries and keys, decays, the state and everything read from it are fp32 (on
+// the tensor cores: two bf16 terms per operand).
+#include <cooperative_groups.h>
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+#include "seq_common.cuh"
+#include "mma_tile.cuh"
+
+namespace ktb {
+
+struct Retention {
+    const void* proj;
+    long stride;
+    int q_off, k_off, v_off, g_off, H, d, dv, rot_dims, layout;
+    const float2* turn;      // [T][rot_dims / 2]
+    float k_scale;
+    const float *decay, *log2_decay;
+    float eps;
+    const int* seqs;
+    int seqs_stride, n_seqs;
+    float* state;
+    long state_stride;
+};
+
+__global__ void turn_table_kernel(const int* __restrict__ pos, const double* __restrict__ inv_freq, int pairs, float2* __restrict__ turn, long n) {
+    for (long i = blockIdx.x * (long)blockDim.x + threadIdx.x; i < n; i += (long)gridDim.x * blockDim.x) {
+        const long t = i / pairs;
+        double sn, cs;
+        sincos((double)pos[t] * inv_freq[i - t * pairs], &sn, &cs);
+        turn[i] = make_float2((float)cs, (float)sn);
+    }
+}
+
+// column c of a head's row after the rotation; tr: the token's pairs
+template <typename T>
+__device__ __forceinline__ float turned(const T* __restrict__ row, int c, int rot_dims, int layout, const float2* __restrict__ tr) {
+    const float v = to_f(row[c]);
+    if (c >= rot_dims) return v;
+    const float other = to_f(row[rot_partner(c, rot_dims, layout)]);
+    const int half = rot_dims >> 1;
+    const bool second = layout == kRotHalves ? c >= half : (c & 1);
+    const float2 cs = tr[layout == kRotHalves ? (second ? c - half : c) : (c >> 1)];
+    return second ? v * cs.x + other * cs.y : v * cs.x - other * cs.y;
+}
+
+// ------------------------------------------------------------------------------------------------ token by token
+// grid (portions, heads, column blocks of 32 value columns); 8 warps; thread (warp w, lane) keeps S[i][col] for a contiguous run of key rows i in
+// registers.  Tokens run in order in chunks of kRetChunk staged in shared memory, the next chunk's inputs fetched (and turned) while the current one
+// runs; per token every warp leaves its part of o in shared memory, summed in warp order once per chunk.
+constexpr int kRetChunk = 16, kRetWarps = 8, kRetRows = 32;      // dim <= 256
+template <typename T, int ROWS>
+__global__ void __launch_bounds__(256, 2) retention_scan_kernel(const Retention a, float* __restrict__ o_out) {
+    extern __shared__ __align__(16) float sm[];
+    const int d = a.d, dv = a.dv, H = a.H, half = a.rot_dims >> 1;
+    const int rpt = (((d + kRetWarps - 1) / kRetWarps) + 3) & ~3, dp = rpt * kRetWarps;
+    float* qs = sm;                             // [chunk][dp]
+    float* ks = qs + kRetChunk * dp;            // [chunk][dp]
+    float* vs = ks + kRetChunk * dp;            // [chunk][32]
+    float* part = vs + kRetChunk * 32;          // [chunk][warps][32]
+    const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * 32;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, col = c0 + lane;
+    const int start = a.seqs[s], len = a.seqs[a.seqs_stride + s], rd = a.seqs[2 * a.seqs_stride + s], wr = a.seqs[3 * a.seqs_stride + s];
+    const T* proj = (const T*)a.proj;
+    const float keep = a.decay[h];
+    float S[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; r++) {
+        const int i = warp * rpt + r;
+        S[r] = (rd >= 0 && r < rpt && i < d && col < dv) ? a.state[(long)rd * a.state_stride + ((long)h * d + i) * dv + col] : 0.f;
+    }
+    constexpr int E = kRetChunk * ROWS * kRetWarps / 256;      // staged values per thread and array, at most
+    float rq[E], rk[E], rv[2];
+    auto fetch = [&](int t0) {
+        const int nt = min(kRetChunk, len - t0);
+#pragma unroll
+        for (int e = 0; e < E; e++) {
+            const int i = threadIdx.x + e * 256;
+            rq[e] = rk[e] = 0.f;
+            if (i < nt * dp) {
+                const int tt = i / dp, c = i - tt * dp;
+                const long t = (long)(start + t0 + tt);
+                if (c < d) {
+                    rq[e] = turned(proj + t * a.stride + a.q_off + (long)h * d, c, a.rot_dims, a.layout, a.turn + t * half);
+                    rk[e] = turned(proj + t * a.stride + a.k_off + (long)h * d, c, a.rot_dims, a.layout, a.turn + t * half) * a.k_scale;
+                }
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int i = threadIdx.x + e * 256, c = c0 + (i & 31);
+            rv[e] = (i < nt * 32 && c < dv) ? to_f(proj[(long)(start + t0 + (i >> 5)) * a.stride + a.v_off + (long)h * dv + c]) : 0.f;
+        }
+    };
+    if (len > 0) fetch(0);
+    for (int t0 = 0; t0 < len; t0 += kRetChunk) {
+        const int nt = min(kRetChunk, len - t0);
+        __syncthreads();      // the previous chunk is consumed
+#pragma unroll
+        for (int e = 0; e < E; e++) {
+            const int i = threadIdx.x + e * 256;
+            if (i < nt * dp) { qs[i] = rq[e]; ks[i] = rk[e]; }
+        }
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int i = threadIdx.x + e * 256;
+            if (i < nt * 32) vs[i] = rv[e];
+        }
+        __syncthreads();
+        if (t0 + kRetChunk < len) fetch(t0 + kRetChunk);
+#pragma unroll 2
+        for (int tt = 0; tt < nt; tt++) {
+            const float v = vs[tt * 32 + lane];
+            const float4* qr = reinterpret_cast<const float4*>(qs + tt * dp + warp * rpt);
+            const float4* kr = reinterpret_cast<const float4*>(ks + tt * dp + warp * rpt);
+            float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+            for (int r4 = 0; r4 < ROWS / 4; r4++) {
+                if (4 * r4 < rpt) {
+                    const float4 k = kr[r4], q = qr[r4];
+                    S[4 * r4] = fmaf(keep, S[4 * r4], k.x * v);
+                    o0 = fmaf(S[4 * r4], q.x, o0);
+                    S[4 * r4 + 1] = fmaf(keep, S[4 * r4 + 1], k.y * v);
+                    o1 = fmaf(S[4 * r4 + 1], q.y, o1);
+                    S[4 * r4 + 2] = fmaf(keep, S[4 * r4 + 2], k.z * v);
+                    o0 = fmaf(S[4 * r4 + 2], q.z, o0);
+                    S[4 * r4 + 3] = fmaf(keep, S[4 * r4 + 3], k.w * v);
+                    o1 = fmaf(S[4 * r4 + 3], q.w, o1);
+                }
+            }
+            part[(tt * kRetWarps + warp) * 32 + lane] = o0 + o1;
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < nt * 32; i += blockDim.x) {
+            const int tt = i >> 5, c = c0 + (i & 31);
+            float o = 0.f;
+#pragma unroll
+            for (int w = 0; w < kRetWarps; w++) o += part[(tt * kRetWarps + w) * 32 + (i & 31)];
+            if (c < dv) o_out[((long)(start + t0 + tt) * H + h) * dv + c] = o;
+        }
+    }
+    if (wr >= 0) {
+#pragma unroll
+        for (int r = 0; r < ROWS; r++) {
+            const int i = warp * rpt + r;
+            if (r < rpt && i < d && col < dv) a.state[(long)wr * a.state_stride + ((long)h * d + i) * dv + col] = S[r];
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ chunks of 64 tokens on the tensor cores (bf16)
+// With fixed decays the states ahead of all chunks follow from one pass over per-chunk sums, so every chunk of every portion and head is a CTA:
+//   1. chunk_state   U_c = sum_j decay^(n - 1 - j) k_j v_j^T                        (n tokens in the chunk)
+//   2. carry         S_c = the state ahead of chunk c: S_(c+1) = decay^n S_c + U_c, elementwise along the portion's chunks; S_c replaces U_c
+//   3. chunk_out     o_i = decay^(i + 1) S_c^T q_i + sum_{j <= i} decay^(i - j) (q_i . k_j) v_j, then norm and gate
+// m16n8k16 bf16 MMAs with fp32 accumulators; v is bf16 as it comes, every other operand (turned q and k, weighted k and scores, S) enters as the
+// sum of two bf16 terms hi + lo (about 16 bits of mantissa), products of two such operands as hi hi + hi lo + lo hi.
+// Workspace per (chunk tile, head): dim * vdim fp32 of U, then in the same bytes S as groups of 8 columns [8 hi | 8 lo].
+constexpr int kRetQ = 64;
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    hi = pack_bf16(a, b);
+    lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
+}
+// which portion and which of its chunks tile b is: {portion or -1, first token's offset in the portion, tokens}
+__device__ __forceinline__ void find_chunk(const int* __restrict__ seqs, int stride, int n_seqs, int b, int (&info)[3]) {
+    info[0] = -1;
+    for (int s = 0; s < n_seqs; s++) {
+        const int len = seqs[stride + s], nt = (len + kRetQ - 1) / kRetQ;
+        if (b < nt) {
+            info[0] = s;
+            info[1] = b * kRetQ;
+            info[2] = min(kRetQ, len - b * kRetQ);
+            return;
+        }
+        b -= nt;
+    }
+}
+// Stage nt rows of a head (first row `src`, rows `stride` apart; the rest of the 64 rows zeros), turned and times scale * row_w[row], as two bf16 planes
+// [64][ld].  Four pairs at a time where the pair halves are four neighbouring columns each.
+__device__ __forceinline__ void stage_turned(__nv_bfloat16* hi, __nv_bfloat16* lo, int ld, const __nv_bfloat16* __restrict__ src, long stride, int nt, int d, int rot_dims, int layout,
+                                             const float2* __restrict__ turn, float scale, const float* row_w) {
+    const int half = rot_dims >> 1;
+    const bool wide = layout == kRotHalves && half % 4 == 0 && rot_dims > 0;
+    auto put = [&](int at, float4 v, float w) {
+        uint32_t h0, l0, h1, l1;
+        split2(v.x * w, v.y * w, h0, l0);
+        split2(v.z * w, v.w * w, h1, l1);
+        *reinterpret_cast<uint2*>(hi + at) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2*>(lo + at) = make_uint2(l0, l1);
+    };
+    if (wide) {
+        const int per = half / 4 + (d - rot_dims) / 4;      // units of a row: four pairs, or four columns that pass (d - rot_dims is a multiple of 4 here)
+        for (int i = threadIdx.x; i < kRetQ * per; i += blockDim.x) {
+            const int r = i / per, u = i - r * per;
+            const float w = r < nt ? (row_w ? scale * row_w[r] : scale) : 0.f;
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (u < half / 4) {
+                const int c = u * 4;
+                float4 x = zero, y = zero;
+                if (r < nt) {
+                    const float4 p = load4(src + (long)r * stride + c), q = load4(src + (long)r * stride + half + c);
+                    const float4 t0 = *reinterpret_cast<const float4*>(turn + (long)r * half + c), t1 = *reinterpret_cast<const float4*>(turn + (long)r * half + c + 2);
+                    x = make_float4(p.x * t0.x - q.x * t0.y, p.y * t0.z - q.y * t0.w, p.z * t1.x - q.z * t1.y, p.w * t1.z - q.w * t1.w);
+                    y = make_float4(q.x * t0.x + p.x * t0.y, q.y * t0.z + p.y * t0.w, q.z * t1.x + p.z * t1.y, q.w * t1.z + p.w * t1.w);
+                }
+                put(r * ld + c, x, w);
+                put(r * ld + half + c, y, w);
+            } else {
+                const int c = rot_dims + (u - half / 4) * 4;
+                put(r * ld + c, r < nt ? load4(src + (long)r * stride + c) : zero, w);
+            }
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < kRetQ * (d / 2); i += blockDim.x) {
+        const int r = i / (d / 2), c = (i - r * (d / 2)) * 2;
+        uint32_t h = 0, l = 0;
+        if (r < nt) {
+            const float w = row_w ? scale * row_w[r] : scale;
+            const __nv_bfloat16* row = src + (long)r * stride;
+            split2(turned(row, c, rot_dims, layout, turn + (long)r * half) * w, turned(row, c + 1, rot_dims, layout, turn + (long)r * half) * w, h, l);
+        }
+        *reinterpret_cast<uint32_t*>(hi + r * ld + c) = h;
+        *reinterpret_cast<uint32_t*>(lo + r * ld + c) = l;
+    }
+}
+
+// grid (tiles, heads), 8 warps; a unit of work is 16 key rows x up to 64 value columns of U
+__global__ void __launch_bounds__(256) retention_chunk_state_kernel(const Retention a, float* __restrict__ ws) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __shared__ int info[3];
+    __shared__ float row_w[kRetQ];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, tq = lane & 3, h = blockIdx.y;
+    const int d = a.d, dv = a.dv, ldk = d + 8, ldv = dv + 8;
+    if (tid == 0) find_chunk(a.seqs, a.seqs_stride, a.n_seqs, blockIdx.x, info);
+    __syncthreads();
+    if (info[0] < 0) return;
+    const int nt = info[2];
+    const long t0 = a.seqs[info[0]] + info[1];
+    __nv_bfloat16* Kh = reinterpret_cast<__nv_bfloat16*>(smem_raw);
+    __nv_bfloat16* Kl = Kh + kRetQ * ldk;
+    __nv_bfloat16* Vs = Kl + kRetQ * ldk;
+    const __nv_bfloat16* proj = (const __nv_bfloat16*)a.proj;
+    const int vc = dv >> 3;
+    for (int i = tid; i < kRetQ * vc; i += 256) {
+        const int r = i / vc, c = (i - r * vc) * 8;
+        cp_async16(Vs + r * ldv + c, proj + (t0 + (r < nt ? r : 0)) * a.stride + a.v_off + (long)h * dv + c, r < nt);
+    }
+    if (tid < kRetQ) row_w[tid] = tid < nt ? exp2f((float)(nt - 1 - tid) * a.log2_decay[h]) : 0.f;
+    __syncthreads();
+    stage_turned(Kh, Kl, ldk, proj + t0 * a.stride + a.k_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, a.turn + t0 * (a.rot_dims >> 1), a.k_scale, row_w);
+    cp_async_wait_all();
+    __syncthreads();
+    float* U = ws + ((long)blockIdx.x * a.H + h) * d * dv;
+    const int d16 = d >> 4, dv16 = dv >> 4, cgroups = (dv16 + 3) >> 2, k16 = (nt + 15) >> 4;
+    for (int unit = warp; unit < d16 * cgroups; unit += 8) {
+        const int r0 = (unit / cgroups) * 16, v0 = (unit % cgroups) * 4;
+        float acc[8][4];
+#pragma unroll
+        for (int n = 0; n < 8; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) acc[n][e] = 0.f;
+        for (int kk = 0; kk < k16; kk++) {
+            uint32_t ah[4], al[4];
+            const int at = (kk * 16 + (lane & 7) + 8 * (lane >> 4)) * ldk + r0 + 8 * ((lane >> 3) & 1);
+            ldmatrix_x4_trans(ah, Kh + at);
+            ldmatrix_x4_trans(al, Kl + at);
+#pragma unroll
+            for (int vp = 0; vp < 4; vp++) {
+                if (v0 + vp < dv16) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, Vs + (kk * 16 + (lane & 15)) * ldv + (v0 + vp) * 16 + 8 * (lane >> 4));
+                    mma_bf16_16816(acc[2 * vp], ah, b[0], b[1]);
+                    mma_bf16_16816(acc[2 * vp + 1], ah, b[2], b[3]);
+                    mma_bf16_16816(acc[2 * vp], al, b[0], b[1]);
+                    mma_bf16_16816(acc[2 * vp + 1], al, b[2], b[3]);
+                }
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < 8; n++) {
+            const int c = v0 * 16 + n * 8 + 2 * tq;
+            if (c < dv) {
+                *reinterpret_cast<float2*>(U + (long)(r0 + gq) * dv + c) = make_float2(acc[n][0], acc[n][1]);
+                *reinterpret_cast<float2*>(U + (long)(r0 + gq + 8) * dv + c) = make_float2(acc[n][2], acc[n][3]);
+            }
+        }
+    }
+}
+
+// grid (blocks of 256 x 8 elements, heads, portions); a thread carries eight neighbouring columns along the portion's chunks, kCarryAhead of whose sums
+// are in flight
+constexpr int kCarryAhead = 4;
+__global__ void __launch_bounds__(256) retention_carry_kernel(const Retention a, float* __restrict__ ws) {
+    const int s = blockIdx.z, h = blockIdx.y;
+    const long n = (long)a.d * a.dv, i = (blockIdx.x * 256L + threadIdx.x) * 8;
+    if (i >= n) return;
+    long tile = 0;
+    for (int k = 0; k < s; k++) tile += (a.seqs[a.seqs_stride + k] + kRetQ - 1) / kRetQ;
+    const int len = a.seqs[a.seqs_stride + s], rd = a.seqs[2 * a.seqs_stride + s], wr = a.seqs[3 * a.seqs_stride + s], chunks = (len + kRetQ - 1) / kRetQ;
+    const float l2 = a.log2_decay[h], full = exp2f((float)kRetQ * l2);
+    float4 S0 = make_float4(0.f, 0.f, 0.f, 0.f), S1 = S0;
+    if (rd >= 0) {
+        const float* p = a.state + (long)rd * a.state_stride + (long)h * n + i;
+        S0 = load4(p);
+        S1 = load4(p + 4);
+    }
+    const long step = (long)a.H * n;
+    float* U = ws + (tile * a.H + h) * n + i;
+    for (int c0 = 0; c0 < chunks; c0 += kCarryAhead) {
+        float4 u[kCarryAhead][2];
+#pragma unroll
+        for (int k = 0; k < kCarryAhead; k++)
+            if (c0 + k < chunks) {
+                u[k][0] = load4(U + (c0 + k) * step);
+                u[k][1] = load4(U + (c0 + k) * step + 4);
+            }
+#pragma unroll
+        for (int k = 0; k < kCarryAhead; k++) {
+            const int c = c0 + k;
+            if (c >= chunks) break;
+            uint4 hi, lo;
+            split2(S0.x, S0.y, hi.x, lo.x);
+            split2(S0.z, S0.w, hi.y, lo.y);
+            split2(S1.x, S1.y, hi.z, lo.z);
+            split2(S1.z, S1.w, hi.w, lo.w);
+            uint4* o = reinterpret_cast<uint4*>(U + c * step);
+            o[0] = hi;
+            o[1] = lo;
+            const float f = c + 1 < chunks ? full : exp2f((float)(len - c * kRetQ) * l2);
+            S0 = make_float4(fmaf(f, S0.x, u[k][0].x), fmaf(f, S0.y, u[k][0].y), fmaf(f, S0.z, u[k][0].z), fmaf(f, S0.w, u[k][0].w));
+            S1 = make_float4(fmaf(f, S1.x, u[k][1].x), fmaf(f, S1.y, u[k][1].y), fmaf(f, S1.z, u[k][1].z), fmaf(f, S1.w, u[k][1].w));
+        }
+    }
+    if (wr >= 0) {
+        float* p = a.state + (long)wr * a.state_stride + (long)h * n + i;
+        store4(p, S0);
+        store4(p + 4, S1);
+    }
+}
+
+// grid (tiles, heads), 4 warps of 16 tokens each.  Shared memory: Q hi, lo | V | the state in pieces of 64 value columns, then K hi, lo
+constexpr int kRetPiece = 64, kRetLdS = kRetPiece + 8;
+static size_t ret_out_smem(int d, int dv) {
+    const size_t k = (size_t)2 * kRetQ * (d + 8), s = (size_t)2 * d * kRetLdS;
+    return ((size_t)2 * kRetQ * (d + 8) + (size_t)kRetQ * (dv + 8) + (k > s ? k : s)) * sizeof(__nv_bfloat16);
+}
+template <int D16MAX, int DV16MAX>
+__global__ void __launch_bounds__(128, DV16MAX > 4 ? 2 : 3) retention_chunk_out_kernel(const Retention a, const float* __restrict__ ws, __nv_bfloat16* __restrict__ out) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __shared__ int info[3];
+    __shared__ float pw[kRetQ + 1];      // powers of the decay
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, tq = lane & 3, h = blockIdx.y;
+    const int d = a.d, dv = a.dv, d16 = d >> 4, dv16 = dv >> 4, ldk = d + 8, ldv = dv + 8;
+    if (tid == 0) find_chunk(a.seqs, a.seqs_stride, a.n_seqs, blockIdx.x, info);
+    if (tid <= kRetQ) pw[tid] = exp2f((float)tid * a.log2_decay[h]);
+    __syncthreads();
+    if (info[0] < 0) return;
+    const int nt = info[2];
+    const long t0 = a.seqs[info[0]] + info[1];
+    const bool has_state = info[1] > 0 || a.seqs[2 * a.seqs_stride + info[0]] >= 0;
+    __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(smem_raw);
+    __nv_bfloat16* Ql = Qh + kRetQ * ldk;
+    __nv_bfloat16* Vs = Ql + kRetQ * ldk;
+    __nv_bfloat16* Kh = Vs + kRetQ * ldv;
+    __nv_bfloat16* Kl = Kh + kRetQ * ldk;
+    __nv_bfloat16 *Sh = Kh, *Sl = Kh + d * kRetLdS;
+    const __nv_bfloat16* proj = (const __nv_bfloat16*)a.proj;
+    const __nv_bfloat16* Sg = reinterpret_cast<const __nv_bfloat16*>(ws + ((long)blockIdx.x * a.H + h) * d * dv);
+    auto fetch_state = [&](int c0) {      // columns c0 .. c0 + 63: groups of 8 columns [8 hi | 8 lo]
+        const int groups = min(kRetPiece, dv - c0) >> 3;
+        for (int i = tid; i < d * groups; i += 128) {
+            const int r = i / groups, g = i - r * groups;
+            const __nv_bfloat16* src = Sg + ((long)r * dv + c0 + g * 8) * 2;
+            cp_async16(Sh + r * kRetLdS + g * 8, src, true);
+            cp_async16(Sl + r * kRetLdS + g * 8, src + 8, true);
+        }
+    };
+    if (has_state) fetch_state(0);
+    const int vc = dv >> 3;
+    for (int i = tid; i < kRetQ * vc; i += 128) {
+        const int r = i / vc, c = (i - r * vc) * 8;
+        cp_async16(Vs + r * ldv + c, proj + (t0 + (r < nt ? r : 0)) * a.stride + a.v_off + (long)h * dv + c, r < nt);
+    }
+    const float2* turn = a.turn + t0 * (a.rot_dims >> 1);
+    stage_turned(Qh, Ql, ldk, proj + t0 * a.stride + a.q_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, turn, 1.0f, nullptr);
+    const bool live = warp * 16 < nt;
+    float Y[2 * DV16MAX][4];
+#pragma unroll
+    for (int n = 0; n < 2 * DV16MAX; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) Y[n][e] = 0.f;
+    const int qat = (warp * 16 + (lane & 15)) * ldk + 8 * (lane >> 4);
+    if (has_state) {
+#pragma unroll
+        for (int piece = 0; piece < (DV16MAX + 3) / 4; piece++) {
+            if (piece * kRetPiece < dv) {
+                if (piece) {
+                    __syncthreads();      // the previous piece is consumed
+                    fetch_state(piece * kRetPiece);
+                }
+                cp_async_wait_all();
+                __syncthreads();
+                if (live) {
+#pragma unroll 2
+                    for (int kk = 0; kk < d16; kk++) {
+                        uint32_t qh[4], ql[4];
+                        ldmatrix_x4(qh, Qh + qat + kk * 16);
+                        ldmatrix_x4(ql, Ql + qat + kk * 16);
+#pragma unroll
+                        for (int vp = 0; vp < 4; vp++) {
+                            const int n = piece * 4 + vp;
+                            if (n < DV16MAX && n < dv16) {
+                                uint32_t bh[4], bl[4];
+                                const int at = (kk * 16 + (lane & 15)) * kRetLdS + vp * 16 + 8 * (lane >> 4);
+                                ldmatrix_x4_trans(bh, Sh + at);
+                                ldmatrix_x4_trans(bl, Sl + at);
+                                mma_bf16_16816(Y[2 * n], qh, bh[0], bh[1]);
+                                mma_bf16_16816(Y[2 * n + 1], qh, bh[2], bh[3]);
+                                mma_bf16_16816(Y[2 * n], ql, bh[0], bh[1]);
+                                mma_bf16_16816(Y[2 * n + 1], ql, bh[2], bh[3]);
+                                mma_bf16_16816(Y[2 * n], qh, bl[0], bl[1]);
+                                mma_bf16_16816(Y[2 * n + 1], qh, bl[2], bl[3]);
+                            }
+                        }
+                    }
+                }
+            }
+        }
+        __syncthreads();      // the last piece is consumed: K goes there
+    }
+    const int iA = warp * 16 + gq, iB = iA + 8;
+    {
+        const float fA = pw[iA + 1], fB = pw[iB + 1];
+#pragma unroll
+        for (int n = 0; n < 2 * DV16MAX; n++) {
+            Y[n][0] *= fA;
+            Y[n][1] *= fA;
+            Y[n][2] *= fB;
+            Y[n][3] *= fB;
+        }
+    }
+    stage_turned(Kh, Kl, ldk, proj + t0 * a.stride + a.k_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, turn, a.k_scale, nullptr);
+    cp_async_wait_all();
+    __syncthreads();
+    if (!live) return;
+    for (int np = 0; np <= warp; np++) {      // 16 keys per step, up to the warp's own tokens
+        float G[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) G[n][e] = 0.f;
+        const int kat = (np * 16 + (lane & 7) + 8 * (lane >> 4)) * ldk + 8 * ((lane >> 3) & 1);
+#pragma unroll
+        for (int kk = 0; kk < D16MAX; kk++) {
+            if (kk < d16) {
+                uint32_t qh[4], ql[4], kh[4], kl[4];
+                ldmatrix_x4(qh, Qh + qat + kk * 16);
+                ldmatrix_x4(ql, Ql + qat + kk * 16);
+                ldmatrix_x4(kh, Kh + kat + kk * 16);
+                ldmatrix_x4(kl, Kl + kat + kk * 16);
+                mma_bf16_16816(G[0], qh, kh[0], kh[1]);
+                mma_bf16_16816(G[1], qh, kh[2], kh[3]);
+                mma_bf16_16816(G[0], ql, kh[0], kh[1]);
+                mma_bf16_16816(G[1], ql, kh[2], kh[3]);
+                mma_bf16_16816(G[0], qh, kl[0], kl[1]);
+                mma_bf16_16816(G[1], qh, kl[2], kl[3]);
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < 2; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int back = (e < 2 ? iA : iB) - (np * 16 + n * 8 + 2 * tq + (e & 1));
+                G[n][e] = back >= 0 ? G[n][e] * pw[back] : 0.f;
+            }
+        uint32_t gh[4], gl[4];
+        split2(G[0][0], G[0][1], gh[0], gl[0]);
+        split2(G[0][2], G[0][3], gh[1], gl[1]);
+        split2(G[1][0], G[1][1], gh[2], gl[2]);
+        split2(G[1][2], G[1][3], gh[3], gl[3]);
+#pragma unroll
+        for (int vp = 0; vp < DV16MAX; vp++) {
+            if (vp < dv16) {
+                uint32_t b[4];
+                ldmatrix_x4_trans(b, Vs + (np * 16 + (lane & 15)) * ldv + vp * 16 + 8 * (lane >> 4));
+                mma_bf16_16816(Y[2 * vp], gh, b[0], b[1]);
+                mma_bf16_16816(Y[2 * vp + 1], gh, b[2], b[3]);
+                mma_bf16_16816(Y[2 * vp], gl, b[0], b[1]);
+                mma_bf16_16816(Y[2 * vp + 1], gl, b[2], b[3]);
+            }
+        }
+    }
+    float sA = 0.f, sB = 0.f;      // (columns at or beyond dv hold zeros)
+#pragma unroll
+    for (int n = 0; n < 2 * DV16MAX; n++) {
+        sA += Y[n][0] * Y[n][0] + Y[n][1] * Y[n][1];
+        sB += Y[n][2] * Y[n][2] + Y[n][3] * Y[n][3];
+    }
+    sA += __shfl_xor_sync(0xffffffffu, sA, 1);
+    sA += __shfl_xor_sync(0xffffffffu, sA, 2);
+    sB += __shfl_xor_sync(0xffffffffu, sB, 1);
+    sB += __shfl_xor_sync(0xffffffffu, sB, 2);
+    const float inv[2] = {1.0f / sqrtf(sA / (float)dv + a.eps), 1.0f / sqrtf(sB / (float)dv + a.eps)};
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        const int i = r ? iB : iA;
+        if (i >= nt) continue;
+        const __nv_bfloat16* g = proj + (t0 + i) * a.stride + a.g_off + (long)h * dv;
+        __nv_bfloat16* o = out + ((t0 + i) * a.H + h) * (long)dv;
+#pragma unroll
+        for (int n = 0; n < 2 * DV16MAX; n++) {
+            const int c = n * 8 + 2 * tq;
+            if (c < dv) {
+                const uint32_t u = *reinterpret_cast<const uint32_t*>(g + c);
+                *reinterpret_cast<uint32_t*>(o + c) = pack_bf16(Y[n][2 * r] * inv[r] * act_silu(__uint_as_float(u << 16)), Y[n][2 * r + 1] * inv[r] * act_silu(__uint_as_float(u & 0xffff0000u)));
+            }
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ one token per portion
+// grid (portions, heads, column blocks of `cpb` columns); the column blocks of a head are a thread-block cluster, which adds up the squares of the
+// head's output over distributed shared memory.  A thread owns VEC columns of every `rows_par`-th state row, kRetStepRows of which it requests
+// before q and k are turned.
+constexpr int kRetStepRows = 8, kRetMaxBlocks = 8;
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) retention_step_kernel(const Retention a, T* __restrict__ out, int cpb) {
+    namespace cg = cooperative_groups;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[32], squares;
+    const int d = a.d, dv = a.dv, half = a.rot_dims >> 1;
+    float* qs = sm;                        // [d]
+    float* ks = qs + ((d + 3) & ~3);       // [d]
+    float* os = ks + ((d + 3) & ~3);       // [cpb]
+    float* part = os + ((cpb + 3) & ~3);   // [rows_par][cpb]
+    const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * cpb, ncol = min(cpb, dv - c0);
+    const int tcol = cpb / VEC, rows_par = blockDim.x / tcol, tc = threadIdx.x % tcol, tr = threadIdx.x / tcol, cc = tc * VEC;
+    const bool mine = tr < rows_par && cc < ncol;
+    const long t = a.seqs[s];
+    const int rd = a.seqs[2 * a.seqs_stride + s], wr = a.seqs[3 * a.seqs_stride + s];
+    const float* Sr = a.state + (long)rd * a.state_stride + (long)h * d * dv + c0 + cc;
+    float* Sw = a.state + (long)wr * a.state_stride + (long)h * d * dv + c0 + cc;
+    float v[kRetStepRows][VEC];
+    auto request = [&](int base) {
+#pragma unroll
+        for (int k = 0; k < kRetStepRows; k++) {
+            const int n = base + k * rows_par + tr;
+            if (mine && rd >= 0 && n < d) {
+                if (VEC == 4) {
+                    const float4 u = load4(Sr + (long)n * dv);
+                    v[k][0] = u.x; v[k][VEC > 1 ? 1 : 0] = u.y; v[k][VEC > 2 ? 2 : 0] = u.z; v[k][VEC > 3 ? 3 : 0] = u.w;
+                } else {
+                    v[k][0] = Sr[(long)n * dv];
+                }
+            } else {
+#pragma unroll
+                for (int e = 0; e < VEC; e++) v[k][e] = 0.f;
+            }
+        }
+    };
+    request(0);
+    const T* row = (const T*)a.proj + t * a.stride;
+    float x[VEC], y[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) {
+        x[e] = mine && cc + e < ncol ? to_f(row[a.v_off + (long)h * dv + c0 + cc + e]) : 0.f;
+        y[e] = 0.f;
+    }
+    for (int i = threadIdx.x; i < 2 * d; i += blockDim.x) {
+        const bool is_k = i >= d;
+        const int c = is_k ? i - d : i;
+        const float u = turned(row + (is_k ? a.k_off : a.q_off) + (long)h * d, c, a.rot_dims, a.layout, a.turn + t * half);
+        if (is_k) ks[c] = u * a.k_scale;
+        else qs[c] = u;
+    }
+    const float keep = a.decay[h];
+    __syncthreads();
+    for (int base = 0; base < d; base += kRetStepRows * rows_par) {
+        if (base) request(base);
+#pragma unroll
+        for (int k = 0; k < kRetStepRows; k++) {
+            const int n = base + k * rows_par + tr;
+            if (mine && n < d) {
+                const float kn = ks[n], qn = qs[n];
+#pragma unroll
+                for (int e = 0; e < VEC; e++) {
+                    v[k][e] = fmaf(keep, v[k][e], kn * x[e]);
+                    y[e] = fmaf(v[k][e], qn, y[e]);
+                }
+                if (wr >= 0) {
+                    if (VEC == 4) store4(Sw + (long)n * dv, make_float4(v[k][0], v[k][VEC > 1 ? 1 : 0], v[k][VEC > 2 ? 2 : 0], v[k][VEC > 3 ? 3 : 0]));
+                    else Sw[(long)n * dv] = v[k][0];
+                }
+            }
+        }
+    }
+    if (mine) {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) part[tr * cpb + cc + e] = y[e];
+    }
+    __syncthreads();
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < ncol; i += blockDim.x) {
+        float o = 0.f;
+        for (int r = 0; r < rows_par; r++) o += part[r * cpb + i];
+        os[i] = o;      // read back by the same thread only
+        sq += o * o;
+    }
+    sq = block_sum(sq, red);
+    if (gridDim.z > 1) {
+        cg::cluster_group cluster = cg::this_cluster();
+        if (threadIdx.x == 0) squares = sq;
+        cluster.sync();
+        sq = 0.f;
+        for (unsigned r = 0; r < cluster.num_blocks(); r++) sq += *cluster.map_shared_rank(&squares, r);
+        cluster.sync();      // no CTA leaves while its sum may still be read
+    }
+    const float inv = 1.0f / sqrtf(sq / (float)dv + a.eps);
+    for (int i = threadIdx.x; i < ncol; i += blockDim.x) {
+        const long c = (long)h * dv + c0 + i;
+        out[t * (long)a.H * dv + c] = from_f<T>(os[i] * inv * act_silu(to_f(row[a.g_off + c])));
+    }
+}
+
+}  // namespace ktb
+
+using namespace ktb;
+
+#define SEQ_DISPATCH(dtype, ...)                                                           \
+    do {                                                                                   \
+        if ((dtype) == KTB200_TYPE_BF16) { using T = __nv_bfloat16; __VA_ARGS__; }         \
+        else if ((dtype) == KTB200_TYPE_F32) { using T = float; __VA_ARGS__; }             \
+        else { set_error("dtype must be bf16 or f32"); return KTB200_EINVAL; }             \
+    } while (0)
+#define GRANT_SMEM(kernel, smem)                                                                                                       \
+    do {                                                                                                                               \
+        static size_t granted = 46 * 1024; /* less the kernels' static shared memory */                                               \
+        if ((smem) > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(smem))); granted = (smem); } \
+    } while (0)
+
+static bool ret_aligned(const void* p, size_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
+static bool ret_bad(const ktb200_retention_params* c) {
+    return !c || !c->proj || !c->decay || !c->log2_decay || !c->seqs || !c->state || c->heads <= 0 || c->dim <= 0 || c->vdim <= 0 || c->rot_dims < 0 || c->rot_dims > c->dim ||
+           (c->rot_dims & 1) || (c->rot_dims && !c->turn) || (c->rot_layout != kRotInterleaved && c->rot_layout != kRotHalves);
+}
+static Retention ret_args(const ktb200_retention_params* c) {
+    return Retention{c->proj, c->proj_stride, c->q_off, c->k_off, c->v_off, c->g_off, c->heads, c->dim, c->vdim, c->rot_dims, c->rot_layout, reinterpret_cast<const float2*>(c->turn),
+                     c->k_scale, c->decay, c->log2_decay, c->eps, c->seqs, c->seqs_stride, c->n_seqs, c->state, c->state_stride};
+}
+
+extern "C" int ktb200_turn_table(const int* pos, const double* inv_freq, int pairs, float* turn, int n_tokens, void* stream) {
+    if (!pos || !inv_freq || !turn || pairs <= 0 || !ret_aligned(turn, 8)) { set_error("turn_table: bad argument"); return KTB200_EINVAL; }
+    if (n_tokens <= 0) return KTB200_OK;
+    const long n = (long)n_tokens * pairs;
+    turn_table_kernel<<<(unsigned)((n + 127) / 128 < 148 * 16 ? (n + 127) / 128 : 148 * 16), 128, 0, (cudaStream_t)stream>>>(pos, inv_freq, pairs, reinterpret_cast<float2*>(turn), n);
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
+extern "C" int ktb200_retention_scan(const ktb200_retention_params* c, float* o, int dtype, void* stream) {
+    if (ret_bad(c) || !o || c->dim > kRetWarps * kRetRows) { set_error("retention_scan: bad argument (head size <= %d)", kRetWarps * kRetRows); return KTB200_EINVAL; }
+    if (c->n_seqs <= 0) return KTB200_OK;
+    const Retention a = ret_args(c);
+    const int rpt = (((c->dim + kRetWarps - 1) / kRetWarps) + 3) & ~3, dp = rpt * kRetWarps;
+    const size_t smem = ((size_t)2 * kRetChunk * dp + kRetChunk * 32 + (size_t)kRetChunk * kRetWarps * 32) * sizeof(float);
+    const dim3 grid(c->n_seqs, c->heads, (c->vdim + 31) / 32);
+#define SCAN_LAUNCH(ROWS)                                                                                        \
+    SEQ_DISPATCH(dtype, {                                                                                        \
+        GRANT_SMEM((retention_scan_kernel<T, ROWS>), smem);                                                      \
+        retention_scan_kernel<T, ROWS><<<grid, kRetWarps * 32, smem, (cudaStream_t)stream>>>(a, o);              \
+    })
+    if (rpt <= 8) SCAN_LAUNCH(8);
+    else if (rpt <= 16) SCAN_LAUNCH(16);
+    else SCAN_LAUNCH(32);
+#undef SCAN_LAUNCH
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
+extern "C" int ktb200_retention_chunk_supported(int dim, int vdim, int dtype) {
+    return dtype == KTB200_TYPE_BF16 && dim > 0 && vdim > 0 && dim % 16 == 0 && vdim % 16 == 0 && dim <= 128 && vdim <= 128;
+}
+static long ret_tiles(int n_tokens, int n_seqs) { return n_tokens / kRetQ + n_seqs; }      // (an upper bound: whole chunks and one partial per portion)
+extern "C" size_t ktb200_retention_chunk_workspace(int heads, int dim, int vdim, int n_tokens, int n_seqs) {
+    return (size_t)ret_tiles(n_tokens, n_seqs) * heads * dim * vdim * sizeof(float);
+}
+
+extern "C" int ktb200_retention_chunk(const ktb200_retention_params* c, void* out, int n_tokens, void* workspace, size_t workspace_bytes, int dtype, void* stream) {
+    if (ret_bad(c) || !out || !ktb200_retention_chunk_supported(c->dim, c->vdim, dtype) || !workspace || !ret_aligned(workspace, 32) || !ret_aligned(c->proj, 16) || !ret_aligned(out, 4) ||
+        !ret_aligned(c->state, 16) || !ret_aligned(c->turn, 16) || c->proj_stride % 8 || c->state_stride % 4 || c->q_off % 8 || c->k_off % 8 || c->v_off % 8 || c->g_off % 2 ||
+        workspace_bytes < ktb200_retention_chunk_workspace(c->heads, c->dim, c->vdim, n_tokens, c->n_seqs)) {
+        set_error("retention_chunk: bad argument (bf16, head sizes multiples of 16 up to 128, rows aligned to 16 bytes)");
+        return KTB200_EINVAL;
+    }
+    if (n_tokens <= 0 || c->n_seqs <= 0) return KTB200_OK;
+    const Retention a = ret_args(c);
+    float* ws = (float*)workspace;
+    cudaStream_t st = (cudaStream_t)stream;
+    const dim3 grid((unsigned)ret_tiles(n_tokens, c->n_seqs), c->heads);
+    const size_t s1 = ((size_t)2 * kRetQ * (c->dim + 8) + (size_t)kRetQ * (c->vdim + 8)) * sizeof(__nv_bfloat16);
+    GRANT_SMEM(retention_chunk_state_kernel, s1);
+    retention_chunk_state_kernel<<<grid, 256, s1, st>>>(a, ws);
+    KTB_LAUNCH_CHECK();
+    retention_carry_kernel<<<dim3((c->dim * c->vdim / 8 + 255) / 256, c->heads, c->n_seqs), 256, 0, st>>>(a, ws);
+    KTB_LAUNCH_CHECK();
+    const size_t s3 = ret_out_smem(c->dim, c->vdim);
+#define OUT_LAUNCH(DK, DV)                                                                                      \
+    do {                                                                                                        \
+        GRANT_SMEM((retention_chunk_out_kernel<DK, DV>), s3);                                                   \
+        retention_chunk_out_kernel<DK, DV><<<grid, 128, s3, st>>>(a, ws, (__nv_bfloat16*)out);                  \
+    } while (0)
+    if (c->dim <= 64 && c->vdim <= 64) OUT_LAUNCH(4, 4);
+    else if (c->vdim <= 64) OUT_LAUNCH(8, 4);
+    else OUT_LAUNCH(8, 8);
+#undef OUT_LAUNCH
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
+extern "C" int ktb200_retention_step_max_vdim(void) { return kRetMaxBlocks * 256; }
+
+extern "C" int ktb200_retention_step(const ktb200_retention_params* c, void* out, int dtype, void* stream) {
+    if (ret_bad(c) || !out || c->vdim > ktb200_retention_step_max_vdim() || c->dim > 4096) { set_error("retention_step: bad argument"); return KTB200_EINVAL; }
+    if (c->n_seqs <= 0) return KTB200_OK;
+    const Retention a = ret_args(c);
+    const int dv = c->vdim;
+    const bool vec = dv % 4 == 0 && c->state_stride % 4 == 0 && ret_aligned(c->state, 16);
+    // columns per CTA: up to 128, or 32 while that leaves SMs idle; at most kRetMaxBlocks column blocks per head
+    int cpb = (long)c->n_seqs * c->heads < 2 * 148 ? 32 : 128;
+    const int least = (dv + kRetMaxBlocks - 1) / kRetMaxBlocks;
+    if (cpb < least) cpb = least;
+    if (cpb > dv) cpb = dv;
+    if (vec) cpb = (cpb + 3) & ~3;
+    const int blocks = (dv + cpb - 1) / cpb, rows_par = 256 / (vec ? cpb / 4 : cpb);
+    const size_t smem = ((size_t)2 * ((c->dim + 3) & ~3) + ((cpb + 3) & ~3) + (size_t)rows_par * cpb) * sizeof(float);
+    cudaLaunchConfig_t cfg{};
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeClusterDimension;
+    attr.val.clusterDim.x = 1;
+    attr.val.clusterDim.y = 1;
+    attr.val.clusterDim.z = blocks;
+    cfg.gridDim = dim3(c->n_seqs, c->heads, blocks);
+    cfg.blockDim = dim3(256);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = (cudaStream_t)stream;
+    cfg.attrs = &attr;
+    cfg.numAttrs = 1;
+    SEQ_DISPATCH(dtype, {
+        if (vec) KTB_CUDA_CHECK(cudaLaunchKernelEx(&cfg, retention_step_kernel<T, 4>, a, (T*)out, cpb));
+        else KTB_CUDA_CHECK(cudaLaunchKernelEx(&cfg, retention_step_kernel<T, 1>, a, (T*)out, cpb));
+    });
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}

@@ -562,7 +562,7 @@ __global__ void __launch_bounds__(256, AHEAD ? 2 : 3) gla_scan_kernel(const T* _
     }
 }
 
-// out[t][h][c] = o[t][h][c] / sqrt(mean_c o^2 + eps) * w[c] * silu(gate[t][h][c]); a warp per (token, head)
+// out[t][h][c] = o[t][h][c] / sqrt(mean_c o^2 + eps) * w[c] * silu(gate[t][h][c]) (w == nullptr: ones); a warp per (token, head)
 template <typename T>
 __global__ void __launch_bounds__(256) gla_out_kernel(const float* __restrict__ o, const T* __restrict__ w, float eps, const T* __restrict__ gate, long gate_stride,
                                                       T* __restrict__ out, long n_rows, int H, int dv) {
@@ -575,7 +575,7 @@ __global__ void __launch_bounds__(256) gla_out_kernel(const float* __restrict__ 
         const float inv = 1.0f / sqrtf(s / (float)dv + eps);
         const long t = row / H;
         const int h = (int)(row - t * H);
-        for (int c = lane; c < dv; c += 32) out[row * dv + c] = from_f<T>(src[c] * inv * to_f(w[c]) * act_silu(to_f(gate[t * gate_stride + (long)h * dv + c])));
+        for (int c = lane; c < dv; c += 32) out[row * dv + c] = from_f<T>(src[c] * inv * (w ? to_f(w[c]) : 1.0f) * act_silu(to_f(gate[t * gate_stride + (long)h * dv + c])));
     }
 }
 
@@ -771,7 +771,7 @@ extern "C" int ktb200_gla_scan(const void* proj, long proj_stride, int q_off, in
 
 extern "C" int ktb200_gla_out(const float* o, const void* norm_w, float eps, const void* gate, long gate_stride, void* out, int n_tokens, int heads, int vdim, int dtype,
                               void* stream) {
-    if (!o || !norm_w || !gate || !out || heads <= 0 || vdim <= 0) { set_error("gla_out: bad argument"); return KTB200_EINVAL; }
+    if (!o || !gate || !out || heads <= 0 || vdim <= 0) { set_error("gla_out: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
     const long rows = (long)n_tokens * heads;
     SEQ_DISPATCH(dtype, (gla_out_kernel<T><<<grid_for(rows, 8), 256, 0, (cudaStream_t)stream>>>(o, (const T*)norm_w, eps, (const T*)gate, gate_stride, (T*)out, rows, heads, vdim)));

@@ -4,6 +4,7 @@
 //                                optional token shift  hs_t = h_t + (h_{t-1} - h_t) * mu  whose h_{t-1} comes from the same
 //                                step (recomputed from the previous row) or from the per-sequence state rows
 //   ktb200_residual_layernorm    x_out = x_in + mult * (a + b), then layer norm (mean taken off, weight without bias); rows picked by an index
+//   ktb200_sum_rmsnorm           s = x_scale x + a + b_scale b, x and h <- s / sqrt(mean(s^2) + eps) * w: the norm AFTER a residual sum, whose row is the new stream
 //   ktb200_latent_prep           what follows the fused down-projections of latent attention: RMS norm of the query latent,
 //                                RMS norm of the key/value latent, rotation of the shared rotated key part, paged cache write
 //   ktb200_sigmoid_gate_mul      heads [H][T][dv] * sigmoid(gate [T][H*dv]) -> [T][H*dv]
@@ -259,6 +260,102 @@ __global__ void __launch_bounds__(NV == 0 ? 256 : (NV > 4 ? 512 : 1024)) residua
     for (int i = tid; i < D; i += blockDim.x) h_out[t * D + i] = from_f<T>((sm[i] - mean) * inv * to_f(w[i]));
 }
 
+// ------------------------------------------------------------------------------------------------ residual sum, then the norm that becomes the stream
+// One CTA per token.  Row r = rows ? rows[t] : t of x, a, b, b_scale, ids and id_w:
+//     s = (x_scale + sum_{j: ids[r][j] >= first_identity} id_w[r][j]) x + a + b_scale[r] b ;  y = s / sqrt(mean(s^2) + eps) * w
+// every term but x optional (choices at or beyond first_identity are experts whose output is their input, x).  y goes to x_out (fp32, the new
+// residual stream) and h_out (T), and with dot_w also as sigmoid(y . dot_w) to dot_out[t].  NV as in residual_layernorm_kernel.
+struct SumNorm {
+    const void* x;
+    int x_type;
+    float x_scale;
+    const void* a;
+    int a_type;
+    const void* b;
+    int b_type;
+    const float* b_scale;
+    const int64_t* ids;
+    const float* id_w;
+    int top, first_identity;
+    const int64_t* rows;
+    const void* w;
+    float eps;
+    float* x_out;
+    void* h_out;
+    const void* dot_w;
+    float* dot_out;
+};
+template <typename T, int NV>
+__global__ void __launch_bounds__(NV == 0 ? 256 : (NV > 4 ? 512 : 1024)) sum_rmsnorm_kernel(const SumNorm p, int D) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[32];
+    const long t = blockIdx.x, row = p.rows ? (long)p.rows[t] : t, r = row * D;
+    const int tid = threadIdx.x;
+    const T *w = (const T*)p.w, *dw = (const T*)p.dot_w;
+    T* h_out = (T*)p.h_out;
+    float xs = p.x_scale;
+    if (p.ids)
+        for (int j = 0; j < p.top; j++) {      // (the same few numbers for every thread)
+            const float iw = p.id_w[row * p.top + j];
+            if (p.ids[row * p.top + j] >= p.first_identity) xs += iw;
+        }
+    const float bs = p.b && p.b_scale ? p.b_scale[row] : 1.0f;
+    float dot = 0.f;
+    if (NV > 0) {
+        float4 v[NV > 0 ? NV : 1], wv[NV > 0 ? NV : 1];
+        float s = 0.f;
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (k * blockDim.x + tid) * 4;
+            v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < D) {
+                float4 u = make_float4(0.f, 0.f, 0.f, 0.f), z = u;
+                const float4 x = load4_hidden(p.x, r + i, p.x_type);
+                if (p.a) u = load4_hidden(p.a, r + i, p.a_type);
+                if (p.b) z = load4_hidden(p.b, r + i, p.b_type);
+                wv[k] = load4(w + i);
+                v[k] = make_float4(fmaf(xs, x.x, fmaf(bs, z.x, u.x)), fmaf(xs, x.y, fmaf(bs, z.y, u.y)), fmaf(xs, x.z, fmaf(bs, z.z, u.z)), fmaf(xs, x.w, fmaf(bs, z.w, u.w)));
+            }
+            s += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+        }
+        const float inv = 1.0f / sqrtf(block_sum(s, red) / (float)D + p.eps);
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (k * blockDim.x + tid) * 4;
+            if (i < D) {
+                const float4 y = make_float4(v[k].x * inv * wv[k].x, v[k].y * inv * wv[k].y, v[k].z * inv * wv[k].z, v[k].w * inv * wv[k].w);
+                if (p.x_out) store4(p.x_out + t * D + i, y);
+                if (h_out) store4(h_out + t * D + i, y);
+                if (dw) {
+                    const float4 g = load4(dw + i);
+                    dot += (y.x * g.x + y.y * g.y) + (y.z * g.z + y.w * g.w);
+                }
+            }
+        }
+    } else {
+        float s = 0.f;
+        for (int i = tid; i < D; i += blockDim.x) {
+            float u = 0.f;
+            if (p.a) u = load_hidden(p.a, r + i, p.a_type);
+            if (p.b) u = fmaf(bs, load_hidden(p.b, r + i, p.b_type), u);
+            const float v = fmaf(xs, load_hidden(p.x, r + i, p.x_type), u);
+            sm[i] = v;      // read back by the same thread only
+            s += v * v;
+        }
+        const float inv = 1.0f / sqrtf(block_sum(s, red) / (float)D + p.eps);
+        for (int i = tid; i < D; i += blockDim.x) {
+            const float y = sm[i] * inv * to_f(w[i]);
+            if (p.x_out) p.x_out[t * D + i] = y;
+            if (h_out) h_out[t * D + i] = from_f<T>(y);
+            if (dw) dot = fmaf(y, to_f(dw[i]), dot);
+        }
+    }
+    if (dw) {
+        dot = block_sum(dot, red);
+        if (tid == 0) p.dot_out[t] = __fdiv_rn(1.0f, 1.0f + expf(-dot));
+    }
+}
+
 // ------------------------------------------------------------------------------------------------ latent prep
 // One CTA per token.  proj row = [ q latent (q_rank) | kv latent (kv_rank) | rotated key part (rot_dim) | ... ].
 template <typename T>
@@ -343,17 +440,19 @@ __global__ void __launch_bounds__(256) poly_norm_kernel(const T* __restrict__ z,
 // in_wts (optional, one per pair): the expert sees in_wts[p] * x, i.e. both pre-activations are multiplied by it (fp32); the down kernels
 // then take no weights.
 __device__ __forceinline__ float act_relu_sq(float x) { const float r = fmaxf(x, 0.f); return r * r; }
+// An id at or beyond n_experts names no expert with weights (an identity expert, a padding choice): its pair adds nothing here.
 // grid (pairs, row blocks); a warp owns ff rows r = blockIdx.y * nw + warp (+ stride); the token's row sits in shared memory.
 template <typename T>
-__global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restrict__ x, const int64_t* __restrict__ ids, int top, const T* __restrict__ Wg, const T* __restrict__ Wu,
+__global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restrict__ x, const int64_t* __restrict__ ids, int top, int n_experts, const T* __restrict__ Wg, const T* __restrict__ Wu,
                                                               T* __restrict__ act, int D, int F, int act_kind, float limit, const float* __restrict__ in_wts) {
     extern __shared__ __align__(16) float xs[];
     const long p = blockIdx.x;
     const long t = p / top;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    const long e = ids[p];
+    if (e >= n_experts) return;
     for (int i = threadIdx.x; i < D; i += blockDim.x) xs[i] = to_f(x[t * D + i]);
     __syncthreads();
-    const long e = ids[p];
     const T* u = Wu + e * (long)F * D;
     if (!Wg) {      // experts without a gate matrix: relu(up)^2
         const bool vec = rows_vectorise(Wu, D);
@@ -378,16 +477,17 @@ __global__ void __launch_bounds__(256) experts_gate_up_kernel(const T* __restric
 // grid (tokens, row blocks); out[t][d] = sum_j w[t][j] * Wd[ids[t][j]][d] . act[t*top + j]   (fp32, slot order)
 template <typename T>
 __global__ void __launch_bounds__(256) experts_down_kernel(const T* __restrict__ act, const int64_t* __restrict__ ids, const float* __restrict__ wts, int top,
-                                                           const T* __restrict__ Wd, float* __restrict__ out, int D, int F) {
+                                                           int n_experts, const T* __restrict__ Wd, float* __restrict__ out, int D, int F) {
     extern __shared__ __align__(16) float as[];   // [top][F]
     const long t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    for (int i = threadIdx.x; i < top * F; i += blockDim.x) as[i] = to_f(act[t * top * F + i]);
+    for (int i = threadIdx.x; i < top * F; i += blockDim.x) as[i] = ids[t * top + i / F] < n_experts ? to_f(act[t * top * F + i]) : 0.f;
     __syncthreads();
     const bool vec = rows_vectorise(Wd, F);
     for (int d = blockIdx.y * nw + warp; d < D; d += gridDim.y * nw) {
         float acc = 0.f;      // this lane's share of sum_j w_j * (row . act_j): ONE warp reduction per output row, and the
         for (int j = 0; j < top; j++) {   // next expert's loads are not held up behind a shuffle chain
+            if (ids[t * top + j] >= n_experts) continue;
             const T* wd = Wd + (ids[t * top + j] * (long)D + d) * F;
             acc = fmaf(wts ? wts[t * top + j] : 1.0f, lane_dot(wd, as + j * F, F, lane, vec), acc);
         }
@@ -630,14 +730,34 @@ __global__ void __launch_bounds__(256) experts_down_by_expert_kernel(const T* __
     }
 }
 
-// out[t][d] = sum_j w[t][j] * y[t * top + j][d], fp32, slot order
-__global__ void __launch_bounds__(256) experts_combine_kernel(const float* __restrict__ y, const float* __restrict__ wts, int top, float* __restrict__ out, long n, int D) {
+// out[t][d] = sum_j w[t][j] * y[row(t, j)][d], fp32, slot order; row = place[t * top + j] (place == nullptr: t * top + j); ids at or beyond n_experts
+// have no row.  VEC columns per thread.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) experts_combine_kernel(const T* __restrict__ y, const int64_t* __restrict__ place, const int64_t* __restrict__ ids, int n_experts,
+                                                              const float* __restrict__ wts, int top, float* __restrict__ out, long n, int D) {
     for (long i = blockIdx.x * (long)blockDim.x + threadIdx.x; i < n; i += (long)gridDim.x * blockDim.x) {
-        const long t = i / D;
-        const int d = (int)(i - t * D);
-        float acc = 0.f;
-        for (int j = 0; j < top; j++) acc = fmaf(wts ? wts[t * top + j] : 1.0f, y[(t * top + j) * D + d], acc);
-        out[i] = acc;
+        const long t = i * VEC / D;
+        const int d = (int)(i * VEC - t * D);
+        float acc[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; e++) acc[e] = 0.f;
+        for (int j = 0; j < top; j++) {
+            const long p = t * top + j;
+            if (ids[p] >= n_experts) continue;
+            const float w = wts ? wts[p] : 1.0f;
+            const T* row = y + (place ? place[p] : p) * D + d;
+            if (VEC == 4) {
+                const float4 v = load4(row);
+                acc[0] = fmaf(w, v.x, acc[0]);
+                acc[VEC > 1 ? 1 : 0] = fmaf(w, v.y, acc[VEC > 1 ? 1 : 0]);
+                acc[VEC > 2 ? 2 : 0] = fmaf(w, v.z, acc[VEC > 2 ? 2 : 0]);
+                acc[VEC > 3 ? 3 : 0] = fmaf(w, v.w, acc[VEC > 3 ? 3 : 0]);
+            } else {
+                acc[0] = fmaf(w, to_f(row[0]), acc[0]);
+            }
+        }
+        if (VEC == 4) store4(out + i * 4, make_float4(acc[0], acc[VEC > 1 ? 1 : 0], acc[VEC > 2 ? 2 : 0], acc[VEC > 3 ? 3 : 0]));
+        else out[i] = acc[0];
     }
 }
 
@@ -707,6 +827,40 @@ extern "C" int ktb200_residual_layernorm(const float* x_in, const void* delta_a,
     return KTB200_OK;
 }
 
+extern "C" int ktb200_sum_rmsnorm(const ktb200_sum_rmsnorm_params* c, int n_tokens, int width, int dtype, void* stream) {
+    if (!c || !c->x || !c->weight || (!c->x_out && !c->h_out) || width <= 0 || (c->ids && (!c->id_weights || c->top <= 0)) || (c->dot_weight && !c->dot_out) ||
+        (c->x_out && (const void*)c->x_out == c->x)) {
+        set_error("sum_rmsnorm: bad argument");
+        return KTB200_EINVAL;
+    }
+    if (n_tokens <= 0) return KTB200_OK;
+    auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const bool vec = width % 8 == 0 && al(c->x) && al(c->a) && al(c->b) && al(c->x_out) && al(c->weight) && al(c->h_out) && al(c->dot_weight);
+    const SumNorm p{c->x, c->x_type, c->x_scale, c->a, c->a_type, c->b, c->b_type, c->b_scale, c->ids, c->id_weights, c->top, c->first_identity, c->rows, c->weight, c->eps,
+                    c->x_out, c->h_out, c->dot_weight, c->dot_out};
+    int threads = n_tokens >= 296 ? 256 : 1024;      // as for residual_layernorm
+    while (threads > 64 && threads * 2 > width) threads >>= 1;
+    int nv = (width / 4 + threads - 1) / threads;
+    if (nv > 4 || (nv > 2 && threads == 1024)) { threads = 512; nv = (width / 4 + threads - 1) / threads; }
+#define SN_LAUNCH(NV, TH, SM) sum_rmsnorm_kernel<T, NV><<<n_tokens, TH, SM, (cudaStream_t)stream>>>(p, width)
+    SEQ_DISPATCH(dtype, {
+        if (vec && nv <= 1) SN_LAUNCH(1, threads, 0);
+        else if (vec && nv <= 2) SN_LAUNCH(2, threads, 0);
+        else if (vec && nv <= 4) SN_LAUNCH(4, threads, 0);
+        else if (vec && nv <= 8) SN_LAUNCH(8, threads, 0);
+        else {
+            const size_t smem = (size_t)width * sizeof(float);
+            if (smem > 200 * 1024) { set_error("sum_rmsnorm: row too wide"); return KTB200_EINVAL; }
+            static size_t granted = 46 * 1024;      // (less the kernel's static shared memory)
+            if (smem > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(sum_rmsnorm_kernel<T, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
+            SN_LAUNCH(0, 256, smem);
+        }
+    });
+#undef SN_LAUNCH
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
 extern "C" int ktb200_latent_prep(const void* proj, long proj_stride, int q_rank, int kv_rank, int rot_dim, int rot_dims, int rot_layout, const double* inv_freq, const void* q_norm_w,
                                   const void* kv_norm_w, float eps, const int* pos, const int* slot, const int* page_table, int max_pages, int page_size, void* cache,
                                   void* cq_out, int n_tokens, int dtype, void* stream) {
@@ -756,9 +910,9 @@ extern "C" int ktb200_poly_norm(const void* z, void* out, const float* coef, flo
     return KTB200_OK;
 }
 
-extern "C" int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top, const void* w_gate, const void* w_up, void* act, int n_tokens, int width, int ff, int act_kind,
+extern "C" int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top, int n_experts, const void* w_gate, const void* w_up, void* act, int n_tokens, int width, int ff, int act_kind,
                                       float limit, const float* in_weights, int dtype, void* stream) {
-    if (!x || !ids || !w_up || !act || top <= 0 || width <= 0 || ff <= 0 || width * sizeof(float) > 200 * 1024 || act_kind < kActSilu || act_kind > kActClampedGlu) { set_error("experts_gate_up: bad argument"); return KTB200_EINVAL; }
+    if (!x || !ids || !w_up || !act || top <= 0 || n_experts <= 0 || width <= 0 || ff <= 0 || width * sizeof(float) > 200 * 1024 || act_kind < kActSilu || act_kind > kActClampedGlu) { set_error("experts_gate_up: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
     const size_t smem = (size_t)width * sizeof(float);
     int ry = (ff + 7) / 8;   // row blocks: enough CTAs to fill 148 SMs several times over when there are few pairs
@@ -766,15 +920,15 @@ extern "C" int ktb200_experts_gate_up(const void* x, const int64_t* ids, int top
     SEQ_DISPATCH(dtype, {
         static size_t granted = 48 * 1024;
         if (smem > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(experts_gate_up_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
-        experts_gate_up_kernel<T><<<dim3(n_tokens * top, ry), 256, smem, (cudaStream_t)stream>>>((const T*)x, ids, top, (const T*)w_gate, (const T*)w_up, (T*)act, width, ff, act_kind, limit, in_weights);
+        experts_gate_up_kernel<T><<<dim3(n_tokens * top, ry), 256, smem, (cudaStream_t)stream>>>((const T*)x, ids, top, n_experts, (const T*)w_gate, (const T*)w_up, (T*)act, width, ff, act_kind, limit, in_weights);
     });
     KTB_LAUNCH_CHECK();
     return KTB200_OK;
 }
 
-extern "C" int ktb200_experts_down(const void* act, const int64_t* ids, const float* weights, int top, const void* w_down, float* out, int n_tokens, int width, int ff, int dtype,
+extern "C" int ktb200_experts_down(const void* act, const int64_t* ids, const float* weights, int top, int n_experts, const void* w_down, float* out, int n_tokens, int width, int ff, int dtype,
                                    void* stream) {
-    if (!act || !ids || !w_down || !out || top <= 0 || width <= 0 || ff <= 0 || (size_t)top * ff * sizeof(float) > 200 * 1024) { set_error("experts_down: bad argument"); return KTB200_EINVAL; }
+    if (!act || !ids || !w_down || !out || top <= 0 || n_experts <= 0 || width <= 0 || ff <= 0 || (size_t)top * ff * sizeof(float) > 200 * 1024) { set_error("experts_down: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
     const size_t smem = (size_t)top * ff * sizeof(float);
     int ry = (width + 7) / 8;
@@ -782,7 +936,7 @@ extern "C" int ktb200_experts_down(const void* act, const int64_t* ids, const fl
     SEQ_DISPATCH(dtype, {
         static size_t granted = 48 * 1024;
         if (smem > granted) { KTB_CUDA_CHECK(cudaFuncSetAttribute(experts_down_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
-        experts_down_kernel<T><<<dim3(n_tokens, ry), 256, smem, (cudaStream_t)stream>>>((const T*)act, ids, weights, top, (const T*)w_down, out, width, ff);
+        experts_down_kernel<T><<<dim3(n_tokens, ry), 256, smem, (cudaStream_t)stream>>>((const T*)act, ids, weights, top, n_experts, (const T*)w_down, out, width, ff);
     });
     KTB_LAUNCH_CHECK();
     return KTB200_OK;
@@ -824,6 +978,18 @@ extern "C" int ktb200_experts_gate_up_by_expert(const void* x, const int64_t* id
     return KTB200_OK;
 }
 
+template <typename T>
+static int combine_launch(const T* rows, const int64_t* place, const int64_t* ids, int n_experts, const float* weights, int top, float* out, int n_tokens, int width, void* stream) {
+    auto al = [](const void* p, size_t b) { return (reinterpret_cast<uintptr_t>(p) & (b - 1)) == 0; };
+    const bool vec = width % 4 == 0 && al(rows, 4 * sizeof(T)) && al(out, 16);
+    const long n = (long)n_tokens * width / (vec ? 4 : 1);
+    const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
+    if (vec) experts_combine_kernel<T, 4><<<blocks, 256, 0, (cudaStream_t)stream>>>(rows, place, ids, n_experts, weights, top, out, n, width);
+    else experts_combine_kernel<T, 1><<<blocks, 256, 0, (cudaStream_t)stream>>>(rows, place, ids, n_experts, weights, top, out, n, width);
+    KTB_LAUNCH_CHECK();
+    return KTB200_OK;
+}
+
 extern "C" int ktb200_experts_down_by_expert(const void* act, const int64_t* ids, const float* weights, int top, int n_experts, const void* w_down, float* pair_rows, float* out,
                                              int n_tokens, int width, int ff, int staged, int dtype, void* stream) {
     if (!act || !ids || !w_down || !pair_rows || !out || top <= 0 || n_experts <= 0 || width <= 0 || ff <= 0) {
@@ -840,9 +1006,13 @@ extern "C" int ktb200_experts_down_by_expert(const void* act, const int64_t* ids
         BY_EXPERT_LAUNCH(experts_down_by_expert_kernel, width, 4, (size_t)ff, (const T*)act, ids, P, (const T*)w_down, pair_rows, width, ff);
     }
     KTB_LAUNCH_CHECK();
-    const long n = (long)n_tokens * width;
-    const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
-    experts_combine_kernel<<<blocks, 256, 0, (cudaStream_t)stream>>>(pair_rows, weights, top, out, n, width);
-    KTB_LAUNCH_CHECK();
+    return combine_launch<float>(pair_rows, nullptr, ids, n_experts, weights, top, out, n_tokens, width, stream);
+}
+
+extern "C" int ktb200_experts_combine(const void* rows, const int64_t* place, const int64_t* ids, int n_experts, const float* weights, int top, float* out, int n_tokens, int width,
+                                      int dtype, void* stream) {
+    if (!rows || !ids || !out || top <= 0 || n_experts <= 0 || width <= 0) { set_error("experts_combine: bad argument"); return KTB200_EINVAL; }
+    if (n_tokens <= 0) return KTB200_OK;
+    SEQ_DISPATCH(dtype, { return combine_launch<T>((const T*)rows, place, ids, n_experts, weights, top, out, n_tokens, width, stream); });
     return KTB200_OK;
 }

@@ -5,7 +5,8 @@
 //   ktb200_qkv_prep       proj rows [... q ... k ... v ...], q and k with `maps` rows of d columns per head: a causal filter of `taps` taps along time
 //                         on every channel (optional); q and k turn over their first rot_dims columns (pairs of either layout, angle
 //                         pos * inv_freq[i]), then (qk_norm 1) are scaled to unit rms row by row, or (qk_norm 2) divided by the rms of the WHOLE
-//                         q (k) row and multiplied by a weight per column; v <- (1 - t) v + t v_other with one learned t (optional), then each
+//                         q (k) row and multiplied by a weight per column, or (qk_norm 3) scaled to unit rms row by row and multiplied by one weight row of d numbers
+//                         AHEAD of the rotation; v <- (1 - t) v + t v_other with one learned t (optional), then each
 //                         value head to unit rms (optional); [k | v] into the paged cache, q into q_out.
 //                         ktb200_rope_norm_cache_write: the same with one map and no filter, arguments spelled out
 //   ktb200_softmax_attn   o_i = sum_j softmax_j(s_ij) v_j over the keys j <= i with i - j < window (window > 0) and floor(j / chunk) ==
@@ -36,7 +37,7 @@ namespace ktb {
 // CONV: every channel of q, k and v first passes a causal filter along time; a unit's filtered columns sit in shared memory so that a rotated
 // column finds its partner, and the CTAs of a portion's last token move the last taps - 1 inputs into the portion's state row.
 constexpr int kPrepMaxPerLane = 8;      // head size <= 256
-constexpr int kQkNormNone = 0, kQkNormHead = 1, kQkNormRow = 2;
+constexpr int kQkNormNone = 0, kQkNormHead = 1, kQkNormRow = 2, kQkNormHeadFirst = 3;
 struct QkvPrep {
     const void* proj;
     long proj_stride;
@@ -122,6 +123,7 @@ __global__ void __launch_bounds__(256) rope_norm_cache_write_kernel(const QkvPre
             for (int i = lane; i < d; i += 32) filtered[warp][i] = cv.value(col0 + i, ch0 + i);
             __syncwarp();
         }
+        const T* first_w = a.qk_norm == kQkNormHeadFirst ? (is_q ? (const T*)a.q_w : (const T*)a.k_w) : nullptr;
         auto column = [&](int i) -> float { return CONV ? filtered[warp][i] : to_f(src[i]); };
         float r[kPrepMaxPerLane];
         float s = 0.f;
@@ -131,18 +133,22 @@ __global__ void __launch_bounds__(256) rope_norm_cache_write_kernel(const QkvPre
             r[e] = 0.f;
             if (i < d) {
                 float v = column(i);
+                const float raw = v;
+                if (first_w) v *= to_f(first_w[i]);      // (the unit-rms factor is one number per row: it follows the rotation)
                 if (i < a.rot_dims) {
-                    const float other = column(rot_partner(i, a.rot_dims, a.rot_layout));
+                    const int pi = rot_partner(i, a.rot_dims, a.rot_layout);
+                    float other = column(pi);
+                    if (first_w) other *= to_f(first_w[pi]);
                     const bool second = a.rot_layout == kRotHalves ? i >= half : (i & 1);
                     const float2 cs = turn[a.rot_layout == kRotHalves ? (second ? i - half : i) : (i >> 1)];
                     v = second ? v * cs.x + other * cs.y : v * cs.x - other * cs.y;
                 }
                 r[e] = v;
-                s += v * v;
+                s += first_w ? raw * raw : v * v;
             }
         }
         float inv = 1.f;
-        if (a.qk_norm == kQkNormHead) {
+        if (a.qk_norm == kQkNormHead || first_w) {
             s = warp_sum(s);
             inv = 1.0f / sqrtf(s / (float)d + a.eps);
         } else if (a.qk_norm == kQkNormRow) {
@@ -850,7 +856,7 @@ using namespace ktb;
 extern "C" int ktb200_qkv_prep(const ktb200_qkv_prep_params* c, int n_tokens, int dtype, void* stream) {
     if (!c || !c->proj || !c->pos || !c->slot || !c->page_table || !c->cache || !c->q_out || c->heads <= 0 || c->kv_heads <= 0 || c->heads % c->kv_heads || c->maps < 1 ||
         c->dim <= 0 || c->dim > 32 * kPrepMaxPerLane || c->vdim <= 0 || c->rot_dims < 0 || c->rot_dims > c->dim || (c->rot_dims & 1) || (c->rot_dims && !c->inv_freq) ||
-        (c->rot_layout != kRotInterleaved && c->rot_layout != kRotHalves) || (c->v_other && !c->blend) || c->qk_norm < kQkNormNone || c->qk_norm > kQkNormRow ||
+        (c->rot_layout != kRotInterleaved && c->rot_layout != kRotHalves) || (c->v_other && !c->blend) || c->qk_norm < kQkNormNone || c->qk_norm > kQkNormHeadFirst || (c->qk_norm == kQkNormHeadFirst && (!c->q_weight || !c->k_weight)) ||
         (c->qk_norm == kQkNormRow && (!c->q_weight || !c->k_weight || c->conv_w)) || c->page_size <= 0 || c->max_pages <= 0) {
         set_error("qkv_prep: bad argument (head size <= %d; no row-wide norm behind a filter)", 32 * kPrepMaxPerLane);
         return KTB200_EINVAL;
@@ -872,7 +878,7 @@ extern "C" int ktb200_qkv_prep(const ktb200_qkv_prep_params* c, int n_tokens, in
     const size_t two = 2 * esz;
     auto even = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (two - 1)) == 0; };
     const bool pairs = c->conv_w && c->taps >= 2 && c->taps <= 4 && c->dim % 2 == 0 && c->vdim % 2 == 0 && c->vdim <= 32 * kPrepMaxPerLane && c->q_off % 2 == 0 && c->k_off % 2 == 0 &&
-                       c->v_off % 2 == 0 && c->proj_stride % 2 == 0 && even(c->proj) && even(c->q_out) && even(c->cache) && c->qk_norm != kQkNormRow && !c->v_other && !c->v_unit_rms &&
+                       c->v_off % 2 == 0 && c->proj_stride % 2 == 0 && even(c->proj) && even(c->q_out) && even(c->cache) && c->qk_norm != kQkNormRow && c->qk_norm != kQkNormHeadFirst && !c->v_other && !c->v_unit_rms &&
                        (c->rot_dims == 0 || c->rot_layout == kRotInterleaved);
     if (pairs) {      // tiles of 16 tokens once there are enough tokens to fill the SMs; unit blocks as above
         const int tile = n_tokens >= 512 ? kPairTile : (n_tokens >= 64 ? 4 : 1), tiles = (n_tokens + tile - 1) / tile;

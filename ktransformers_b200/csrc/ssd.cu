@@ -1,6 +1,7 @@
 // Mamba-2 (state-space duality): a recurrent mixer whose matrix state per head decays by one number per token and head
 // (libktb200_seq.so).
 //
+//   ktb200_conv_silu  causal filter of `taps` taps along time with bias on a run of channels, then SiLU, over prompt portions and decode steps alike
 //   ktb200_ssd_conv   prompt portions: causal filter of `taps` taps along time with bias on the [x | B | C] channels, then SiLU; the last taps - 1
 //                     inputs of every portion go to its state row
 //   ktb200_ssd_scan   per portion and head p (group j = p / (P / J)), tokens in order, fp32:
@@ -23,7 +24,7 @@ namespace ktb {
 __device__ __forceinline__ float ssd_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
 // ------------------------------------------------------------------------------------------------ filter + SiLU over prompt portions
-// grid (token blocks, channel blocks); a thread owns VEC consecutive channels and runs over kConvTokens tokens with the last TAPS - 1 inputs
+// grid (token blocks, channel blocks); a thread owns VEC consecutive channels and runs over `tile` tokens (kConvTokens; 1 when every portion is one token) with the last TAPS - 1 inputs
 // in registers (TAPS = 0: any number of taps, one channel, inputs read again per token).
 constexpr int kConvTokens = 16, kConvThreads = 128;
 template <typename T, int VEC> __device__ __forceinline__ void load_vec(float (&v)[VEC], const T* p) {
@@ -35,12 +36,12 @@ template <typename T, int VEC> __device__ __forceinline__ void load_vec(float (&
     }
 }
 template <typename T, int VEC, int TAPS>
-__global__ void __launch_bounds__(kConvThreads) ssd_conv_kernel(const T* __restrict__ in, long stride, const T* __restrict__ w, const T* __restrict__ bias, int taps_rt, int C,
+__global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const T* __restrict__ in, long stride, const T* __restrict__ w, const T* __restrict__ bias, int taps_rt, int C,
                                                                 const int* __restrict__ seq_of, const int* __restrict__ seqs, int seqs_stride, float* __restrict__ state,
-                                                                long state_stride, long conv_off, T* __restrict__ out, int n_tokens) {
+                                                                long state_stride, long conv_off, T* __restrict__ out, int n_tokens, int tile) {
     const int c = (blockIdx.y * kConvThreads + threadIdx.x) * VEC;
     if (c >= C) return;
-    const int t0 = blockIdx.x * kConvTokens, t1 = min(n_tokens, t0 + kConvTokens);
+    const int t0 = blockIdx.x * tile, t1 = min(n_tokens, t0 + tile);
     constexpr int BACK = TAPS > 1 ? TAPS - 1 : 1;
     float win[BACK][VEC], wv[TAPS > 0 ? TAPS : 1][VEC], bv[VEC];
 #pragma unroll
@@ -651,26 +652,33 @@ static bool ssd_bad(const ktb200_ssd_params* c) {
            c->state_size <= 0 || c->vdim <= 0 || c->taps < 1;
 }
 
-extern "C" int ktb200_ssd_conv(const ktb200_ssd_params* c, void* xbc, int n_tokens, int dtype, void* stream) {
-    if (ssd_bad(c) || !c->seq_of || !xbc) { set_error("ssd_conv: bad argument"); return KTB200_EINVAL; }
+extern "C" int ktb200_conv_silu(const void* in, long in_stride, const void* conv_w, const void* conv_b, int taps, int channels, const int* seq_of, const int* seqs, int seqs_stride,
+                                float* state, long state_stride, long conv_off, void* out, int n_tokens, int n_seqs, int dtype, void* stream) {
+    if (!in || !conv_w || !out || !seq_of || !seqs || taps < 1 || (taps > 1 && !state) || channels <= 0) { set_error("conv_silu: bad argument"); return KTB200_EINVAL; }
     if (n_tokens <= 0) return KTB200_OK;
-    const int C = c->heads * c->vdim + 2 * c->groups * c->state_size;
-    const long conv_off = (long)c->heads * c->state_size * c->vdim;
+    const int C = channels, tile = n_tokens == n_seqs ? 1 : kConvTokens;
     const size_t esz = dtype == KTB200_TYPE_BF16 ? 2 : 4;
-    const bool vec = C % 4 == 0 && c->xbc_off % 4 == 0 && c->proj_stride % 4 == 0 && ssd_aligned(c->proj, 4 * esz) && ssd_aligned(xbc, 4 * esz);
-#define CONV_LAUNCH(VEC, TAPS)                                                                                                                                        \
-    ssd_conv_kernel<T, VEC, TAPS><<<dim3((n_tokens + kConvTokens - 1) / kConvTokens, (C + kConvThreads * VEC - 1) / (kConvThreads * VEC)), kConvThreads, 0,           \
-                                    (cudaStream_t)stream>>>((const T*)c->proj + c->xbc_off, c->proj_stride, (const T*)c->conv_w, (const T*)c->conv_b, c->taps, C,      \
-                                                            c->seq_of, c->seqs, c->seqs_stride, c->state, c->state_stride, conv_off, (T*)xbc, n_tokens)
+    const bool vec = C % 4 == 0 && in_stride % 4 == 0 && ssd_aligned(in, 4 * esz) && ssd_aligned(out, 4 * esz);
+#define CONV_LAUNCH(VEC, TAPS)                                                                                                                                \
+    conv_silu_kernel<T, VEC, TAPS><<<dim3((n_tokens + tile - 1) / tile, (C + kConvThreads * VEC - 1) / (kConvThreads * VEC)), kConvThreads, 0,                \
+                                     (cudaStream_t)stream>>>((const T*)in, in_stride, (const T*)conv_w, (const T*)conv_b, taps, C, seq_of, seqs, seqs_stride, \
+                                                             state, state_stride, conv_off, (T*)out, n_tokens, tile)
     SEQ_DISPATCH(dtype, {
-        if (vec && c->taps == 4) CONV_LAUNCH(4, 4);
-        else if (vec && c->taps == 3) CONV_LAUNCH(4, 3);
-        else if (vec && c->taps == 2) CONV_LAUNCH(4, 2);
+        if (vec && taps == 4) CONV_LAUNCH(4, 4);
+        else if (vec && taps == 3) CONV_LAUNCH(4, 3);
+        else if (vec && taps == 2) CONV_LAUNCH(4, 2);
         else CONV_LAUNCH(1, 0);
     });
 #undef CONV_LAUNCH
     KTB_LAUNCH_CHECK();
     return KTB200_OK;
+}
+
+extern "C" int ktb200_ssd_conv(const ktb200_ssd_params* c, void* xbc, int n_tokens, int dtype, void* stream) {
+    if (ssd_bad(c) || !c->seq_of || !xbc) { set_error("ssd_conv: bad argument"); return KTB200_EINVAL; }
+    const size_t esz = dtype == KTB200_TYPE_BF16 ? 2 : 4;
+    return ktb200_conv_silu((const char*)c->proj + (size_t)c->xbc_off * esz, c->proj_stride, c->conv_w, c->conv_b, c->taps, c->heads * c->vdim + 2 * c->groups * c->state_size, c->seq_of,
+                            c->seqs, c->seqs_stride, c->state, c->state_stride, (long)c->heads * c->state_size * c->vdim, xbc, n_tokens, c->n_seqs, dtype, stream);
 }
 
 /* whether ktb200_ssd_scan may run the chunked tensor-core form: bf16, a state size that is a multiple of 16 up to 256, 16-byte aligned rows */

@@ -11,6 +11,7 @@ MODEL_REGISTRY = {
     "Mabidra": ("ktransformers_b200.models.modeling_mabidra", "MabidraForCausalLM"),
     "Zivulix": ("ktransformers_b200.models.modeling_zivulix", "ZivulixForCausalLM"),
     "Bilurax": ("ktransformers_b200.models.modeling_bilurax", "BiluraxForCausalLM"),
+    "Lipadra": ("ktransformers_b200.models.modeling_lipadra", "LipadraForCausalLM"),
     "Rununex": ("ktransformers_b200.models.modeling_rununex", "RununexForCausalLM"),
     "DeepseekV3ForCausalLM": ("ktransformers_b200.models.modeling_deepseek_v3", "DeepseekV3MoEOnlyForCausalLM"),
     "DeepseekV2ForCausalLM": ("ktransformers_b200.models.modeling_deepseek", "DeepseekV2MoE"),

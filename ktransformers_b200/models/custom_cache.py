@@ -76,11 +76,12 @@ class ForwardBatch:
     step or -1), `rd_row` / `wr_row` (state rows to read when the previous token came in an earlier step / to write for the
     last token of a sequence's portion; -1: none).  `seqs` [4, >= n_seqs]: the same per sequence portion, for layers whose
     state is a recurrence over the portion's tokens, and `seq_of` [T]: the portion a token belongs to (column of `seqs`), for
-    layers that look further back than one token.  `want` [W]: rows whose logits the caller asked for."""
+    layers that look further back than one token.  `want` [W]: rows whose logits the caller asked for.  `turns`: the (cos, sin) tables that
+    this step's layers have made so far, by rotation (`turn_table`)."""
 
     N_META = 10      # index rows per token: pos, slot, prev_idx, rd_row, wr_row, the four rows of `seqs`, seq_of
 
-    __slots__ = ("tokens", "pos", "slot", "prev_idx", "rd_row", "wr_row", "want", "n_tokens", "max_kv", "seqs", "n_seqs", "seq_of")
+    __slots__ = ("tokens", "pos", "slot", "prev_idx", "rd_row", "wr_row", "want", "n_tokens", "max_kv", "seqs", "n_seqs", "seq_of", "turns")
 
     def __init__(self, meta: torch.Tensor, tokens: torch.Tensor, want: torch.Tensor, max_kv: int, n_seqs: int = 0):
         self.pos, self.slot, self.prev_idx, self.rd_row, self.wr_row = meta[0], meta[1], meta[2], meta[3], meta[4]
@@ -89,6 +90,18 @@ class ForwardBatch:
         # read or -1, state row to write) in the first n_seqs columns
         self.seqs, self.n_seqs = (meta[5:9] if meta.shape[0] >= 9 else None), n_seqs
         self.seq_of = meta[9] if meta.shape[0] >= 10 else None
+        self.turns: Dict[Any, torch.Tensor] = {}
+
+    def turn_table(self, rot, inv_freq: torch.Tensor) -> torch.Tensor:
+        """(cos, sin) of position * frequency for every token, [T, rot.dims / 2, 2] fp32 (angles fp64): one `ktb200_turn_table` launch per
+        step for all layers of the same rotation `rot`; `inv_freq`: its fp64 frequencies on the device"""
+        key = (rot.base, rot.dims, rot.factor, rot.low, rot.high, rot.original)
+        if key not in self.turns:
+            t = torch.empty((self.n_tokens, rot.dims // 2, 2), dtype=torch.float32, device=self.pos.device)
+            native.check_seq(native.seq_lib().ktb200_turn_table(self.pos.data_ptr(), inv_freq.data_ptr(), rot.dims // 2, t.data_ptr(), self.n_tokens,
+                                                                torch.cuda.current_stream(t.device).cuda_stream))
+            self.turns[key] = t
+        return self.turns[key]
 
 
 class PagedStateCache:

@@ -127,6 +127,22 @@ class SsdParams(C.Structure):
                        "l:state_stride")
 
 
+class SumRmsnormParams(C.Structure):
+    """ktb200_sum_rmsnorm_params (include/ktb200.h)"""
+    _fields_ = _fields("p:x i:x_type f:x_scale p:a i:a_type p:b i:b_type p:b_scale,ids,id_weights i:top,first_identity p:rows,weight f:eps p:x_out,h_out,dot_weight,dot_out")
+
+
+class RetentionParams(C.Structure):
+    """ktb200_retention_params (include/ktb200.h)"""
+    _fields_ = _fields("p:proj l:proj_stride i:q_off,k_off,v_off,g_off,heads,dim,vdim,rot_dims,rot_layout p:turn f:k_scale p:decay,log2_decay f:eps p:seqs i:seqs_stride,n_seqs "
+                       "p:state l:state_stride")
+
+
+class SelectiveScanParams(C.Structure):
+    """ktb200_selective_scan_params (include/ktb200.h)"""
+    _fields_ = _fields("p:x,dt_logit,b,c,z l:dt_stride,bc_stride,z_stride p:dt_bias,a,d_skip i:inner,state_size p:seqs i:seqs_stride,n_seqs p:state l:state_stride")
+
+
 # libktb200_seq.so: the token-major operators (csrc/seq_ops.cu, csrc/window_attn.cu) + the router (csrc/gate.cu)
 _F, _D = C.c_float, C.POINTER(C.c_double)
 SEQ_SYMBOLS = {
@@ -144,10 +160,12 @@ SEQ_SYMBOLS = {
     "ktb200_rope_rows": (_I, [_VP, _I, _I, _I, _I, _I, _VP, _VP, _VP, _I, _I, _VP]),
     "ktb200_sigmoid_gate_mul": (_I, [_VP, _VP, _L, _VP, _I, _I, _I, _I, _VP]),
     "ktb200_poly_norm": (_I, [_VP, _VP, _VP, _F, _I, _I, _I, _VP]),
-    "ktb200_experts_gate_up": (_I, [_VP, _VP, _I, _VP, _VP, _VP, _I, _I, _I, _I, _F, _VP, _I, _VP]),
-    "ktb200_experts_down": (_I, [_VP, _VP, _VP, _I, _VP, _VP, _I, _I, _I, _I, _VP]),
+    "ktb200_experts_gate_up": (_I, [_VP, _VP, _I, _I, _VP, _VP, _VP, _I, _I, _I, _I, _F, _VP, _I, _VP]),
+    "ktb200_experts_down": (_I, [_VP, _VP, _VP, _I, _I, _VP, _VP, _I, _I, _I, _I, _VP]),
     "ktb200_experts_gate_up_by_expert": (_I, [_VP, _VP, _I, _I, _VP, _VP, _VP, _I, _I, _I, _I, _I, _F, _VP, _I, _VP]),
     "ktb200_experts_down_by_expert": (_I, [_VP, _VP, _VP, _I, _I, _VP, _VP, _VP, _I, _I, _I, _I, _I, _VP]),
+    "ktb200_experts_combine": (_I, [_VP, _VP, _VP, _I, _VP, _I, _VP, _I, _I, _I, _VP]),
+    "ktb200_sum_rmsnorm": (_I, [C.POINTER(SumRmsnormParams), _I, _I, _I, _VP]),
     # csrc/seq_mixers.cu
     "ktb200_group_rmsnorm_sandwich": (_I, [_VP, _VP, _I, _VP, _VP, _VP, _VP, _VP, _I, _F, _F, _I, _I, _I, _VP]),
     "ktb200_qk_norm_cache_write": (_I, [_VP, _L, _I, _I, _I, _I, _VP, _VP, _F, _F, _I, _VP, _VP, _VP, _I, _I, _VP, _VP, _I, _I, _VP]),
@@ -174,7 +192,17 @@ SEQ_SYMBOLS = {
     "ktb200_softmax_attn_workspace": (C.c_size_t, [_I, _I, _I, _I, _I, _I]),
     "ktb200_softmax_attn_uses_tensor_cores": (_I, [_I, _I, _I, _I, _I, _I]),
     "ktb200_softmax_attn_tiles": (_I, [_I, _I, _I, _I, _I]),
+    # csrc/retention.cu, csrc/selective_scan.cu
+    "ktb200_turn_table": (_I, [_VP, _VP, _I, _VP, _I, _VP]),
+    "ktb200_retention_chunk_supported": (_I, [_I, _I, _I]),
+    "ktb200_retention_chunk_workspace": (C.c_size_t, [_I, _I, _I, _I, _I]),
+    "ktb200_retention_chunk": (_I, [C.POINTER(RetentionParams), _VP, _I, _VP, C.c_size_t, _I, _VP]),
+    "ktb200_retention_scan": (_I, [C.POINTER(RetentionParams), _VP, _I, _VP]),
+    "ktb200_retention_step_max_vdim": (_I, []),
+    "ktb200_retention_step": (_I, [C.POINTER(RetentionParams), _VP, _I, _VP]),
+    "ktb200_selective_scan": (_I, [C.POINTER(SelectiveScanParams), _VP, _I, _VP]),
     # csrc/ssd.cu
+    "ktb200_conv_silu": (_I, [_VP, _L, _VP, _VP, _I, _I, _VP, _VP, _I, _VP, _L, _L, _VP, _I, _I, _I, _VP]),
     "ktb200_ssd_conv": (_I, [C.POINTER(SsdParams), _VP, _I, _I, _VP]),
     "ktb200_ssd_scan": (_I, [C.POINTER(SsdParams), _VP, _VP, _I, _I, _VP]),
     "ktb200_ssd_scan_uses_tensor_cores": (_I, [_I, _I, _I, _I, _I]),

@@ -357,16 +357,18 @@ def paged_softmax_attention(q: torch.Tensor, kv: torch.Tensor, batch, cache, hea
 
 
 def qkv_prep(proj: torch.Tensor, batch, cache, kv: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, offsets, maps: int = 1, rot=None, inv_freq: Optional[torch.Tensor] = None,
-             qk_norm: int = 0, eps: float = 0.0, conv_w: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None) -> torch.Tensor:
+             qk_norm: int = 0, eps: float = 0.0, q_weight: Optional[torch.Tensor] = None, k_weight: Optional[torch.Tensor] = None, conv_w: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None) -> torch.Tensor:
     """From a projection's q, k and v columns (`offsets`) to the queries [T, heads, maps * dim] and the [k | v] rows of cache layer `kv`, one
     `ktb200_qkv_prep` launch (csrc/softmax_attn.cu): a short causal filter on every channel (conv_w [channels, taps]; its last inputs per
-    sequence live at the front of the `state` rows), the rotation, unit rms per row (qk_norm = 1)."""
+    sequence live at the front of the `state` rows), the rotation, unit rms per row (qk_norm = 1; qk_norm = 3: per row, times q_weight / k_weight
+    [dim], ahead of the rotation)."""
     T, dt = proj.shape[0], proj.dtype
     q = torch.empty((T, heads, maps * dim), dtype=dt, device=proj.device)
     ptr = lambda t: t.data_ptr() if t is not None else None
     rot_dims = rot.dims if rot is not None else 0
     a = native.QkvPrepParams(proj=proj.data_ptr(), proj_stride=proj.stride(0), q_off=offsets[0], k_off=offsets[1], v_off=offsets[2], heads=heads, kv_heads=kv_heads, maps=maps, dim=dim,
-                             vdim=vdim, rot_dims=rot_dims, rot_layout=rot.layout_code if rot_dims else 0, inv_freq=ptr(inv_freq) if rot_dims else None, qk_norm=qk_norm, eps=float(eps),
+                             vdim=vdim, rot_dims=rot_dims, rot_layout=rot.layout_code if rot_dims else 0, inv_freq=ptr(inv_freq) if rot_dims else None, qk_norm=qk_norm, q_weight=ptr(q_weight),
+                             k_weight=ptr(k_weight), eps=float(eps),
                              conv_w=ptr(conv_w), taps=conv_w.shape[1] if conv_w is not None else 0, seq_of=batch.seq_of.data_ptr(), seqs=batch.seqs.data_ptr(),
                              seqs_stride=batch.seqs.stride(0), state=ptr(state), state_stride=state.stride(0) if state is not None else 0, conv_off=0, pos=batch.pos.data_ptr(),
                              slot=batch.slot.data_ptr(), page_table=cache.page_table.data_ptr(), max_pages=cache.max_pages_per_seq, page_size=cache.page_size, cache=kv.data_ptr(),
@@ -616,4 +618,55 @@ class KDifferentialAttention(torch.nn.Module):
                      conv_w=self.conv_w, state=cache.state[cache_idx])
         o = paged_softmax_attention(q, kv, batch, cache, s.heads, s.kv_heads, s.dim, s.vdim, s.scale, chunk=s.chunk, tensor_cores=self.use_tensor_cores, maps=2, lam=self.lam,
                                     rms_eps=self.eps, out_scale=1.0 - s.diff)
+        return torch.nn.functional.linear(o, self.o)
+
+
+class KPlusOneAttention(torch.nn.Module):
+    """Causal soft-max attention over grouped key/value heads inside chunks of the sequence, with biased projections, weighted query and key
+    norms per head ahead of a partial rotation, and one added to the soft-max denominator (a sink of score 0 without a value):
+
+        P       = [W_q ; W_k ; W_v] h + b                       one GEMM over the matrices that read the mixer input
+        q, k    = rot(x / sqrt(mean(x^2) + eps) * w)  per head of P[q], P[k] (one w for all query heads, one for all key heads)
+        [k | v] -> paged cache                                  ktb200_qkv_prep, the above in one launch
+        o_i     = sum_j exp(s_ij) v_j / (1 + sum_j exp(s_ij)) , s_ij = scale q_i . k_j               ktb200_softmax_attn, its sink at 0
+                  over j <= i with floor(j / C) == floor(i / C), C = chunk
+        out     = W_o o                                         GEMM
+
+    Sizes, scale, chunk length and the rotation's constants and layout are constructor parameters
+    (models/configuration_lipadra.PlusOneAttentionSpec); `cache_idx` picks the cache layer, so one set of weights can run several times per
+    step with separate caches.  (The reference's attention operators: archive/ktransformers/operators/attention.py.)"""
+
+    use_tensor_cores = True
+
+    def __init__(self, width: int, spec, eps: float, dtype=torch.bfloat16, device="cuda"):
+        super().__init__()
+        P = lambda *shape, dt=dtype: torch.nn.Parameter(torch.zeros(shape, dtype=dt, device=device), requires_grad=False)
+        s = self.spec = spec
+        if s.heads % s.kv_heads:
+            raise ValueError("query heads must divide into the key/value heads")
+        self.width, self.eps = width, eps
+        self.n_q, self.n_k, self.n_v = s.heads * s.dim, s.kv_heads * s.dim, s.kv_heads * s.vdim
+        self.n_in = (self.n_q + self.n_k + self.n_v + 7) // 8 * 8       # rows padded so that every row of P starts 16-byte aligned
+        self.w_in, self.b_in = P(self.n_in, width), P(self.n_in)
+        self.q_norm, self.k_norm = P(s.dim), P(s.dim)
+        self.o = P(width, s.heads * s.vdim)
+        self.register_buffer("sink", torch.zeros(s.heads, dtype=torch.float32, device=device), persistent=False)      # exp(0): the one in the denominator
+        self.register_buffer("inv_freq", s.rot.inv_freq(device) if s.rot is not None else torch.zeros(1, dtype=torch.float64, device=device), persistent=False)
+
+    def load(self, loader, prefix: str):
+        t = lambda n: loader.load_tensor(prefix + n, "cpu")
+        rows = self.n_q + self.n_k + self.n_v
+        self.w_in.data[:rows].copy_(torch.cat([t("q"), t("k"), t("v")], 0))
+        self.b_in.data[:rows].copy_(torch.cat([t("q.b"), t("k.b"), t("v.b")], 0))
+        self.q_norm.data.copy_(t("q.norm"))
+        self.k_norm.data.copy_(t("k.norm"))
+        self.o.data.copy_(t("o"))
+
+    def forward(self, h: torch.Tensor, batch, cache, cache_idx: int) -> torch.Tensor:
+        s = self.spec
+        kv = cache.key_cache[cache_idx]
+        proj = torch.nn.functional.linear(h, self.w_in, self.b_in)
+        q = qkv_prep(proj, batch, cache, kv, s.heads, s.kv_heads, s.dim, s.vdim, offsets=(0, self.n_q, self.n_q + self.n_k), rot=s.rot, inv_freq=self.inv_freq, qk_norm=3, eps=self.eps,
+                     q_weight=self.q_norm, k_weight=self.k_norm)
+        o = paged_softmax_attention(q, kv, batch, cache, s.heads, s.kv_heads, s.dim, s.vdim, s.scale, chunk=s.chunk, tensor_cores=self.use_tensor_cores, sink=self.sink)
         return torch.nn.functional.linear(o, self.o)

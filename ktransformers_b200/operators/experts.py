@@ -535,6 +535,7 @@ class KExpertsDense(nn.Module):
     and each matrix runs as ONE library grouped GEMM over the per-expert token segments (bf16; fp32 and odd sizes: one GEMM
     per expert), so an expert's weights are read once per step instead of once per pair; the weighted sum over a token's
     slots stays fp32 in slot order.
+    A choice at or beyond `experts` names no expert with weights (an identity expert): it adds nothing on any path.
     The counterpart of KExpertsB200 for checkpoints that ship dense experts (the reference's KExpertsTorch, experts.py:562-678,
     loops over experts in torch)."""
 
@@ -607,9 +608,9 @@ class KExpertsDense(nn.Module):
             native.check_seq(lib.ktb200_experts_down_by_expert(act.data_ptr(), ids.data_ptr(), out_w, top, self.experts, self.down.data_ptr(),
                                                                pair_rows.data_ptr(), out.data_ptr(), T, self.width, self.ff, self.by_expert_staged, dt, st))
             return out
-        native.check_seq(lib.ktb200_experts_gate_up(x.data_ptr(), ids.data_ptr(), top, gate_ptr, self.up.data_ptr(), act.data_ptr(), T, self.width,
+        native.check_seq(lib.ktb200_experts_gate_up(x.data_ptr(), ids.data_ptr(), top, self.experts, gate_ptr, self.up.data_ptr(), act.data_ptr(), T, self.width,
                                                     self.ff, self.act, self.limit, in_w, dt, st))
-        native.check_seq(lib.ktb200_experts_down(act.data_ptr(), ids.data_ptr(), out_w, top, self.down.data_ptr(), out.data_ptr(), T, self.width,
+        native.check_seq(lib.ktb200_experts_down(act.data_ptr(), ids.data_ptr(), out_w, top, self.experts, self.down.data_ptr(), out.data_ptr(), T, self.width,
                                                  self.ff, dt, st))
         return out
 
@@ -632,7 +633,8 @@ class KExpertsDense(nn.Module):
         F = nn.functional
         flat = ids.reshape(-1)
         order = torch.argsort(flat, stable=True)
-        counts = torch.bincount(flat, minlength=self.experts)
+        # (choices beyond the experts sort behind every segment and are left out of the counts)
+        counts = torch.zeros(self.experts + 1, dtype=torch.int64, device=x.device).scatter_add_(0, flat.clamp(max=self.experts), torch.ones_like(flat))[:self.experts]
         xs = x.index_select(0, torch.div(order, top, rounding_mode="floor"))
         rs = weights.reshape(-1).index_select(0, order) if on_input else None            # the weights in the order of the sorted pairs
         if x.dtype == torch.bfloat16 and self.width % 8 == 0 and self.ff % 8 == 0 and hasattr(F, "grouped_mm"):
@@ -650,10 +652,12 @@ class KExpertsDense(nn.Module):
                     a = self._activate(F.linear(seg, self.gate[e]) if self.gated else None, F.linear(seg, self.up[e]), rs[lo:lo + n] if on_input else None)
                     y[lo:lo + n] = F.linear(a, self.down[e])
                     lo += n
-        pairs = torch.empty_like(y)
-        pairs[order] = y
-        pairs = pairs.view(T, top, self.width).float()
-        return pairs.sum(1) if on_input else (pairs * weights.unsqueeze(-1)).sum(1)
+        place = torch.empty_like(order)      # where each pair's row is among the sorted rows
+        place[order] = torch.arange(T * top, device=x.device)
+        out = torch.empty((T, self.width), dtype=torch.float32, device=x.device)
+        native.check_seq(native.seq_lib().ktb200_experts_combine(y.data_ptr(), place.data_ptr(), ids.data_ptr(), self.experts, None if on_input else weights.data_ptr(), top,
+                                                                 out.data_ptr(), T, self.width, TORCH_TO_GGML_HIDDEN[y.dtype], _stream(x.device)))
+        return out
 
 
 class KSoftmaxTopKMoE(nn.Module):
@@ -735,3 +739,32 @@ class KSharedSigmoidMoE(nn.Module):
     def forward(self, h: torch.Tensor):
         ids, w = self.router(h)
         return self.experts(h, ids, w, on_input=True), self.shared(h) if self.shared is not None else None
+
+
+class KIdentityMoE(nn.Module):
+    """router (operators/gate.KGroupedSoftmaxGate) -> dense gated-SiLU experts, the last `identity` router outputs being experts whose output
+    is their input, plus a shared gated expert (operators/mlp.KGatedMLP) times sigmoid(w_sg . h).  `forward` runs what has matrices; the
+    identity experts' share of the sum and the shared expert's factor belong to the norms on both sides (operators/norm.KSumRMSNorm), which
+    hold the fp32 row: `shared_gate` is w_sg, and `forward` returns (routed sum fp32, ids, weights, shared output or None)."""
+
+    def __init__(self, width: int, ff: int, experts: int, identity: int, top: int, groups: int, keep_groups: int, out_scale: float, shared_ff: Optional[int], dtype=torch.bfloat16,
+                 device="cuda"):
+        super().__init__()
+        from .gate import KGroupedSoftmaxGate
+        from .mlp import KGatedMLP
+        self.identity = identity
+        self.router = KGroupedSoftmaxGate(width, experts + identity, top, groups, keep_groups, out_scale, device=device)
+        self.experts = KExpertsDense(width, ff, experts, dtype=dtype, device=device)
+        self.shared = KGatedMLP(width, shared_ff, dtype=dtype, device=device) if shared_ff else None
+        self.shared_gate = nn.Parameter(torch.empty(width, dtype=dtype, device=device), requires_grad=False) if shared_ff else None
+
+    def load(self, loader, prefix: str):
+        self.router.load(loader, prefix + "router", prefix + "correction")
+        self.experts.load(loader, prefix)
+        if self.shared is not None:
+            self.shared.load(loader, prefix + "shared.")
+            self.shared_gate.data.copy_(loader.load_tensor(prefix + "shared.sg", "cpu").reshape(-1))
+
+    def forward(self, h: torch.Tensor):
+        ids, w = self.router(h)
+        return self.experts(h, ids, w), ids, w, self.shared(h) if self.shared is not None else None

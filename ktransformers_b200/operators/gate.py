@@ -17,7 +17,7 @@ from ..util.custom_gguf import TORCH_TO_GGML_HIDDEN
 from .base_operator import BaseInjectedModule
 
 _SCORING = {"sigmoid": 0, "softmax": 1, "topk_softmax": 2}
-_TOPK = {"noaux_tc": 0, "greedy": 1, "group_limited_greedy": 2}
+_TOPK = {"noaux_tc": 0, "greedy": 1, "group_limited_greedy": 2, "biased_group_max": 3}
 
 
 class KMoEGateBase:
@@ -225,6 +225,44 @@ class KSigmoidTopKGate(nn.Module):
         idx = torch.empty((n, self.top), dtype=torch.int64, device=x.device)
         wt = torch.empty((n, self.top), dtype=torch.float32, device=x.device)
         cfg = native.GateConfig(self.experts, self.width, self.top, 1, 1, _SCORING["sigmoid"], _TOPK["greedy"], 0, 1.0, self.weight.data_ptr(), None, TORCH_TO_GGML_HIDDEN[x.dtype])
+        st = torch.cuda.current_stream(x.device).cuda_stream
+        if n >= self.gemm_min_tokens or self.width % 4:
+            logits = nn.functional.linear(x.float(), self.weight)
+            native.check_seq(native.seq_lib().ktb200_moe_gate_select(C.byref(cfg), n, logits.data_ptr(), idx.data_ptr(), wt.data_ptr(), st))
+        else:
+            native.check_seq(native.seq_lib().ktb200_moe_gate_forward(C.byref(cfg), n, x.data_ptr(), idx.data_ptr(), wt.data_ptr(), None, None, st))
+        return idx, wt
+
+
+class KGroupedSoftmaxGate(nn.Module):
+    """Soft-max scores s = softmax(W x) in fp32 over every output; outputs are CHOSEN by s + correction among those of the `keep_groups` groups
+    (of neighbours) whose largest choice score is largest, every other one counting as minus infinity; the WEIGHTS are the chosen outputs' s
+    times `out_scale`, not normalised: the router kernel's `scoring = softmax, topk_method = biased_group_max` case.  As for
+    KGroupedSigmoidGate, decode-sized batches run the one-launch kernel, and batches from `gemm_min_tokens` tokens an fp32 library GEMM (TF32
+    off) and `ktb200_moe_gate_select`."""
+
+    gemm_min_tokens = 48
+
+    def __init__(self, width: int, outputs: int, top: int, groups: int, keep_groups: int, out_scale: float, device="cuda"):
+        super().__init__()
+        if outputs % groups or not (1 <= keep_groups <= groups) or top > keep_groups * (outputs // groups):
+            raise ValueError(f"router: {outputs} outputs do not divide into {groups} groups of which {keep_groups} hold {top} choices")
+        if outputs > 512 or top > 32 or groups > 32:
+            raise ValueError("router: at most 512 outputs, 32 groups and 32 choices per token")
+        self.width, self.outputs, self.top, self.groups, self.keep_groups, self.out_scale = width, outputs, top, groups, keep_groups, float(out_scale)
+        self.weight = nn.Parameter(torch.empty((outputs, width), dtype=torch.float32, device=device), requires_grad=False)
+        self.correction = nn.Parameter(torch.zeros(outputs, dtype=torch.float32, device=device), requires_grad=False)
+
+    def load(self, loader, key: str, correction_key: str):
+        self.weight.data.copy_(loader.load_tensor(key, "cpu").float())
+        self.correction.data.copy_(loader.load_tensor(correction_key, "cpu").float())
+
+    def forward(self, x: torch.Tensor):
+        n = x.shape[0]
+        idx = torch.empty((n, self.top), dtype=torch.int64, device=x.device)
+        wt = torch.empty((n, self.top), dtype=torch.float32, device=x.device)
+        cfg = native.GateConfig(self.outputs, self.width, self.top, self.groups, self.keep_groups, _SCORING["softmax"], _TOPK["biased_group_max"], 0, self.out_scale,
+                                self.weight.data_ptr(), self.correction.data_ptr(), TORCH_TO_GGML_HIDDEN[x.dtype])
         st = torch.cuda.current_stream(x.device).cuda_stream
         if n >= self.gemm_min_tokens or self.width % 4:
             logits = nn.functional.linear(x.float(), self.weight)

@@ -1,5 +1,6 @@
 """Recurrent mixers with a matrix state per head.  KGatedDeltaRule (below) — the gated delta rule behind short convolutions.
 KStateSpace (below) — Mamba-2 (state-space duality): one decay per token and head.
+KRetention (below) — a fixed decay per head.  KSelectiveScan (below) — Mamba: a state per channel, one decay per token, channel and state.
 KGatedLinearAttention — linear attention with a decay per key channel and a recurrent matrix state per head:
 
     q = W_q h / sqrt(dim) ,  k = W_k h ,  v = W_v h ,  a = sigmoid(W_a2 (W_a1 h) + b) ** (1 / tau)        (a per head and key channel)
@@ -20,6 +21,7 @@ archive/ktransformers/models/custom_cache.py:26-200.)"""
 from __future__ import annotations
 
 import ctypes as C
+import math
 
 import torch
 from torch import nn
@@ -224,3 +226,133 @@ class KStateSpace(nn.Module):
         proj = nn.functional.linear(h, self.w_in)
         o = torch.empty((h.shape[0], self.n_out), dtype=h.dtype, device=h.device)
         return nn.functional.linear(self.mix(proj, 0, batch, cache, cache_idx, o), self.o)
+
+
+class KRetention(nn.Module):
+    """Retention — linear attention whose matrix state per head decays by one fixed number, with rotated queries and keys, unit-rms head outputs and an
+    output gate:
+
+        S <- decay_h S + k v^T ,  o = S^T q                     per head, q = rot(W_q h), k = rot(W_k h) / sqrt(dim), v = W_v h; S in fp32
+        out = W_o (o / sqrt(mean_vdim(o^2) + eps) * silu(W_g h))
+
+        P     = [W_q ; W_k ; W_v ; W_g] h                       one GEMM over the matrices that read the mixer input
+        turns                                                    ktb200_turn_table, once per step for all layers of one rotation
+        o     = prompt portions: ktb200_retention_chunk (bf16: chunks of 64 tokens in parallel, norm and gate included), or
+                ktb200_retention_scan + ktb200_gla_out (fp32, other sizes, short portions); decode steps: ktb200_retention_step
+        out   = W_o o                                           GEMM
+
+    The state starts at zero and lives in the cache manager's double-buffered fp32 state rows (models/custom_cache.PagedStateCache); there are no
+    per-token cache rows.  Sizes, decays and the rotation are constructor parameters (models/configuration_lipadra.RetentionSpec); `cache_idx`
+    picks the cache layer.  (The reference has no recurrent mixer.)"""
+
+    use_tensor_cores = True
+    chunk_min_tokens = 32       # tokens beyond one per portion from which the chunked form runs
+
+    def __init__(self, width: int, spec, eps: float, dtype=torch.bfloat16, device="cuda"):
+        super().__init__()
+        P = lambda *shape: nn.Parameter(torch.zeros(shape, dtype=dtype, device=device), requires_grad=False)
+        s = self.spec = spec
+        self.width, self.eps = width, eps
+        up = lambda n: (n + 7) // 8 * 8       # q, k, v and g start 16-byte aligned in every row of P
+        self.n_qk, self.n_v = s.heads * s.dim, s.heads * s.vdim
+        self.offsets = [0, up(self.n_qk), 2 * up(self.n_qk), 2 * up(self.n_qk) + up(self.n_v)]
+        self.n_in = self.offsets[3] + up(self.n_v)
+        self.w_in, self.o = P(self.n_in, width), P(width, self.n_v)
+        self.register_buffer("decay", torch.tensor(s.decay, dtype=torch.float32, device=device), persistent=False)
+        self.register_buffer("log2_decay", torch.tensor([math.log2(x) for x in s.decay], dtype=torch.float32, device=device), persistent=False)
+        self.register_buffer("inv_freq", s.rot.inv_freq(device) if s.rot is not None else torch.zeros(1, dtype=torch.float64, device=device), persistent=False)
+
+    def load(self, loader, prefix: str):
+        for name, at in zip(("q", "k", "v", "g"), self.offsets):
+            w = loader.load_tensor(prefix + name, "cpu")
+            self.w_in.data[at:at + w.shape[0]].copy_(w)
+        self.o.data.copy_(loader.load_tensor(prefix + "o", "cpu"))
+
+    def forward(self, h: torch.Tensor, batch, cache, cache_idx: int) -> torch.Tensor:
+        s, T, dev, dt = self.spec, h.shape[0], h.device, h.dtype
+        lib, code, st = native.seq_lib(), native.GGML_BF16 if dt == torch.bfloat16 else native.GGML_F32, torch.cuda.current_stream(h.device).cuda_stream
+        state = cache.state[cache_idx]
+        proj = nn.functional.linear(h, self.w_in)
+        turn = batch.turn_table(s.rot, self.inv_freq) if s.rot is not None else None
+        q, k, v, g = self.offsets
+        a = native.RetentionParams(proj=proj.data_ptr(), proj_stride=self.n_in, q_off=q, k_off=k, v_off=v, g_off=g, heads=s.heads, dim=s.dim, vdim=s.vdim,
+                                   rot_dims=s.rot.dims if s.rot is not None else 0, rot_layout=s.rot.layout_code if s.rot is not None else 0,
+                                   turn=turn.data_ptr() if turn is not None else None, k_scale=s.dim ** -0.5, decay=self.decay.data_ptr(), log2_decay=self.log2_decay.data_ptr(),
+                                   eps=float(self.eps), seqs=batch.seqs.data_ptr(), seqs_stride=batch.seqs.stride(0), n_seqs=batch.n_seqs, state=state.data_ptr(),
+                                   state_stride=state.stride(0))
+        out = torch.empty((T, self.n_v), dtype=dt, device=dev)
+        if T == batch.n_seqs and s.vdim <= lib.ktb200_retention_step_max_vdim():
+            native.check_seq(lib.ktb200_retention_step(C.byref(a), out.data_ptr(), code, st))
+        elif self.use_tensor_cores and T - batch.n_seqs >= self.chunk_min_tokens and lib.ktb200_retention_chunk_supported(s.dim, s.vdim, code):
+            ws = torch.empty(lib.ktb200_retention_chunk_workspace(s.heads, s.dim, s.vdim, T, batch.n_seqs), dtype=torch.uint8, device=dev)
+            native.check_seq(lib.ktb200_retention_chunk(C.byref(a), out.data_ptr(), T, ws.data_ptr(), ws.numel(), code, st))
+        else:
+            o = torch.empty((T, self.n_v), dtype=torch.float32, device=dev)
+            native.check_seq(lib.ktb200_retention_scan(C.byref(a), o.data_ptr(), code, st))
+            native.check_seq(lib.ktb200_gla_out(o.data_ptr(), None, float(self.eps), proj[:, g:].data_ptr(), self.n_in, out.data_ptr(), T, s.heads, s.vdim, code, st))
+        return nn.functional.linear(out, self.o)
+
+
+class KSelectiveScan(nn.Module):
+    """Mamba, the selective scan — a recurrent mixer whose channels keep `state_size` numbers each, every one with a decay of its own per token:
+
+        [x | z] = W_in h ;  x = silu(filter(x) + b)             a causal filter of `conv` taps along time on every channel
+        [r | B | C] = W_x x ;  dt = softplus(W_dt r + dt_b)     one dt per channel
+        S_cn <- exp(-exp(A_log_cn) dt_c) S_cn + dt_c x_c B_n ;  y_c = sum_n S_cn C_n + D_c x_c             S in fp32
+        out = W_o (y silu(z))
+
+        P     = W_in h                                          GEMM
+        x     = ktb200_conv_silu ;  p = W_x x ,  W_dt p[r]       two GEMMs
+        y     = ktb200_selective_scan                           softplus, recurrence, skip and gate in one launch, prompts and decode steps alike
+        out   = W_o y                                           GEMM
+
+    A sequence's state — S and the last conv - 1 inputs of every channel — lives in the cache manager's double-buffered fp32 state rows
+    (models/custom_cache.PagedStateCache).  Tokens of a portion run in order.  Sizes are constructor parameters
+    (models/configuration_lipadra.SelectiveScanSpec); `cache_idx` picks the cache layer.  (The reference has no recurrent mixer.)"""
+
+    def __init__(self, width: int, spec, eps: float, dtype=torch.bfloat16, device="cuda"):
+        super().__init__()
+        P = lambda *shape, dt=dtype: nn.Parameter(torch.zeros(shape, dtype=dt, device=device), requires_grad=False)
+        s = self.spec = spec
+        self.width = width
+        up = lambda n: (n + 7) // 8 * 8       # x and z, and the step's, B's and C's columns, start 16-byte aligned in their rows
+        self.z_off, self.b_off = up(s.inner), up(s.dt_rank)
+        self.c_off = self.b_off + up(s.state_size)
+        self.w_in, self.w_x = P(self.z_off + up(s.inner), width), P(self.c_off + up(s.state_size), s.inner)
+        self.w_dt, self.o = P(s.inner, s.dt_rank), P(width, s.inner)
+        self.conv_w, self.conv_b = P(s.inner, s.conv), P(s.inner)
+        self.dt_bias, self.a, self.d_skip = P(s.inner, dt=torch.float32), P(s.inner, s.state_size, dt=torch.float32), P(s.inner, dt=torch.float32)
+
+    def load(self, loader, prefix: str):
+        s, t = self.spec, lambda n: loader.load_tensor(prefix + n, "cpu")
+        w = t("in")
+        self.w_in.data[:s.inner].copy_(w[:s.inner])
+        self.w_in.data[self.z_off:self.z_off + s.inner].copy_(w[s.inner:])
+        w = t("x")
+        for at, lo, n in ((0, 0, s.dt_rank), (self.b_off, s.dt_rank, s.state_size), (self.c_off, s.dt_rank + s.state_size, s.state_size)):
+            self.w_x.data[at:at + n].copy_(w[lo:lo + n])
+        self.w_dt.data.copy_(t("dt"))
+        self.conv_w.data.copy_(t("conv"))
+        self.conv_b.data.copy_(t("conv.b"))
+        self.dt_bias.data.copy_(t("dt.b").float())
+        self.a.data.copy_(-torch.exp(t("A_log").float()))
+        self.d_skip.data.copy_(t("D").float())
+        self.o.data.copy_(t("o"))
+
+    def forward(self, h: torch.Tensor, batch, cache, cache_idx: int) -> torch.Tensor:
+        s, T, dev, dt = self.spec, h.shape[0], h.device, h.dtype
+        lib, code, st = native.seq_lib(), native.GGML_BF16 if dt == torch.bfloat16 else native.GGML_F32, torch.cuda.current_stream(h.device).cuda_stream
+        state = cache.state[cache_idx]
+        proj = nn.functional.linear(h, self.w_in)
+        x = torch.empty((T, s.inner), dtype=dt, device=dev)
+        native.check_seq(lib.ktb200_conv_silu(proj.data_ptr(), proj.stride(0), self.conv_w.data_ptr(), self.conv_b.data_ptr(), s.conv, s.inner, batch.seq_of.data_ptr(),
+                                              batch.seqs.data_ptr(), batch.seqs.stride(0), state.data_ptr(), state.stride(0), s.inner * s.state_size, x.data_ptr(), T, batch.n_seqs, code, st))
+        p = nn.functional.linear(x, self.w_x)
+        step = nn.functional.linear(p[:, :s.dt_rank], self.w_dt)
+        a = native.SelectiveScanParams(x=x.data_ptr(), dt_logit=step.data_ptr(), b=p[:, self.b_off:].data_ptr(), c=p[:, self.c_off:].data_ptr(), z=proj[:, self.z_off:].data_ptr(),
+                                       dt_stride=step.stride(0), bc_stride=p.stride(0), z_stride=proj.stride(0), dt_bias=self.dt_bias.data_ptr(), a=self.a.data_ptr(),
+                                       d_skip=self.d_skip.data_ptr(), inner=s.inner, state_size=s.state_size, seqs=batch.seqs.data_ptr(), seqs_stride=batch.seqs.stride(0),
+                                       n_seqs=batch.n_seqs, state=state.data_ptr(), state_stride=state.stride(0))
+        y = torch.empty((T, s.inner), dtype=dt, device=dev)
+        native.check_seq(lib.ktb200_selective_scan(C.byref(a), y.data_ptr(), code, st))
+        return nn.functional.linear(y, self.o)

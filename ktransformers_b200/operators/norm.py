@@ -13,7 +13,8 @@ kernel recomputes when the previous token is part of the same launch, so results
 (The reference's norms are plain torch modules, archive/ktransformers/models/modeling_deepseek_v3.py:65-80.)"""
 from __future__ import annotations
 
-from typing import Optional
+import ctypes as C
+from typing import Optional, Tuple
 
 import torch
 from torch import nn
@@ -136,3 +137,39 @@ class KLayerNorm(nn.Module):
             _ptr(x), _ptr(a), GGML_OF[a.dtype] if a is not None else 0, _ptr(b), GGML_OF[b.dtype] if b is not None else 0, float(mult), _ptr(rows), _ptr(x_out), self.weight.data_ptr(),
             self.eps, float(h_scale), _ptr(h), T, self.width, GGML_OF[dt], torch.cuda.current_stream(dev).cuda_stream))
         return (x if plain else x_out), h
+
+
+class KSumRMSNorm(nn.Module):
+    """An RMS norm that follows the residual sum, so that the normed row is the new stream: one `ktb200_sum_rmsnorm` launch (csrc/seq_ops.cu) for
+
+        s = (x_scale + w_id) x + a + b_scale b ;  y = s / sqrt(mean(s^2) + eps) * weight           (every term but x optional)
+
+    with w_id the summed weights of the token's choices that are identity experts (whose output is x itself) and b_scale one number per token.
+    y is kept in fp32 (the stream) and rounded once to the compute dtype (what the next sublayer reads).  `rows` [T] int64 picks the rows of every
+    input; `dot` [width]: also sigmoid(y . dot) per token, from the fp32 row."""
+
+    def __init__(self, width: int, eps: float, dtype=torch.bfloat16, device="cuda"):
+        super().__init__()
+        self.width, self.eps = width, float(eps)
+        self.weight = nn.Parameter(torch.ones(width, dtype=dtype, device=device), requires_grad=False)
+
+    def load(self, loader, key: str):
+        self.weight.data.copy_(loader.load_tensor(key, "cpu"))
+
+    def forward(self, x: torch.Tensor, x_scale: float = 1.0, a: Optional[torch.Tensor] = None, b: Optional[torch.Tensor] = None, b_scale: Optional[torch.Tensor] = None,
+                identity: Optional[Tuple[torch.Tensor, torch.Tensor, int]] = None, rows: Optional[torch.Tensor] = None, dot: Optional[torch.Tensor] = None, keep_x: bool = True):
+        """x, a, b [T, width], each fp32 or the compute dtype; b_scale [T] fp32; identity: (ids [T, top] int64, weights [T, top] fp32, first
+        identity expert).  Returns (y in fp32 or None, y in the compute dtype, the sigmoids [T] fp32 or None)."""
+        T, dt, dev = (x.shape[0] if rows is None else rows.shape[0]), self.weight.dtype, x.device
+        for d in (x, a, b):
+            assert d is None or (d.is_contiguous() and d.shape[-1] == self.width)
+        assert rows is None or (rows.dtype == torch.int64 and rows.is_contiguous())
+        ids, id_w, first = identity if identity is not None else (None, None, 0)
+        y = torch.empty((T, self.width), dtype=torch.float32, device=dev) if keep_x or dt == torch.float32 else None
+        h = torch.empty((T, self.width), dtype=dt, device=dev) if dt != torch.float32 else None
+        gate = torch.empty(T, dtype=torch.float32, device=dev) if dot is not None else None
+        p = native.SumRmsnormParams(x=x.data_ptr(), x_type=GGML_OF[x.dtype], x_scale=float(x_scale), a=_ptr(a), a_type=GGML_OF[a.dtype] if a is not None else 0, b=_ptr(b),
+                                    b_type=GGML_OF[b.dtype] if b is not None else 0, b_scale=_ptr(b_scale), ids=_ptr(ids), id_weights=_ptr(id_w), top=ids.shape[1] if ids is not None else 0,
+                                    first_identity=first, rows=_ptr(rows), weight=self.weight.data_ptr(), eps=self.eps, x_out=_ptr(y), h_out=_ptr(h), dot_weight=_ptr(dot), dot_out=_ptr(gate))
+        native.check_seq(native.seq_lib().ktb200_sum_rmsnorm(C.byref(p), T, self.width, GGML_OF[dt], torch.cuda.current_stream(dev).cuda_stream))
+        return y, h if h is not None else y, gate

@@ -359,8 +359,8 @@ def kernel_leg(flush, peak_gbs, have_main_lib):
         ids = torch.stack([torch.randperm(E, generator=g, device=dev)[:top] for _ in range(T)]).to(torch.int64)
         wts = torch.rand(T, top, generator=g, device=dev)
         act, out = torch.empty(T * top, ff, dtype=bf, device=dev), torch.empty(T, D, device=dev)
-        f1 = lambda: native.check_seq(seq.ktb200_experts_gate_up(x.data_ptr(), ids.data_ptr(), top, Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0.0, None, 30, S()))
-        f2 = lambda: native.check_seq(seq.ktb200_experts_down(act.data_ptr(), ids.data_ptr(), wts.data_ptr(), top, Wd.data_ptr(), out.data_ptr(), T, D, ff, 30, S()))
+        f1 = lambda: native.check_seq(seq.ktb200_experts_gate_up(x.data_ptr(), ids.data_ptr(), top, Wg.shape[0], Wg.data_ptr(), Wu.data_ptr(), act.data_ptr(), T, D, ff, 0, 0.0, None, 30, S()))
+        f2 = lambda: native.check_seq(seq.ktb200_experts_down(act.data_ptr(), ids.data_ptr(), wts.data_ptr(), top, Wd.shape[0], Wd.data_ptr(), out.data_ptr(), T, D, ff, 30, S()))
         uniq = len(set(ids.flatten().tolist()))                            # every chosen expert is read from HBM at least once
         row("experts_gate_up_kernel", f"T={T} top={top} width={D} ff={ff} bf16", timed(f1, flush), uniq * 2 * ff * D * 2,
             {"kernel": "moe_block_kernel (Q4_K/Q6_K, whole block)", "frac_of_measured_hbm": 0.55, "note": "committed measurement of the DeepSeek path, one token"})
