@@ -621,7 +621,7 @@ int ktb200_sum_rmsnorm(const ktb200_sum_rmsnorm_params* params, int n_tokens, in
  * q and k turn over their first rot_dims columns by the (cos, sin) pairs turn [n_tokens][rot_dims / 2], k is multiplied by k_scale; per portion
  * (seqs as for ktb200_gla_scan) and head, fp32:
  *     S <- decay[h] S + k v^T ;  o = S^T q ;  out = o / sqrt(mean_vdim(o^2) + eps) * silu(g)
- * log2_decay[h] = log2(decay[h]).  State rows [heads][dim][vdim] fp32, row stride state_stride; dim <= 256.
+ * decay[h] + decay_low[h]: the decay as two floats (decay_low is read in 32-bit runs); log2_decay[h] = log2 of it.  State rows [heads][dim][vdim] fp32, row stride state_stride; dim <= 256.
  *   ktb200_turn_table        turn[t][i] = (cos, sin) of pos[t] * inv_freq[i], angles in fp64
  *   ktb200_retention_chunk   chunks of 64 tokens on the tensor cores (bf16; dim and vdim multiples of 16 up to 128): the states ahead of every chunk, then
  *                            all chunks at once; workspace: ktb200_retention_chunk_workspace bytes
@@ -633,7 +633,7 @@ typedef struct {
     int q_off, k_off, v_off, g_off, heads, dim, vdim, rot_dims, rot_layout;
     const float* turn;
     float k_scale;
-    const float *decay, *log2_decay;
+    const float *decay, *decay_low, *log2_decay;
     float eps;
     const int* seqs;
     int seqs_stride, n_seqs;

@@ -26,13 +26,16 @@ struct Retention {
     int q_off, k_off, v_off, g_off, H, d, dv, rot_dims, layout;
     const float2* turn;      // [T][rot_dims / 2]
     float k_scale;
-    const float *decay, *log2_decay;
+    const float *decay, *decay_low, *log2_decay;
     float eps;
     const int* seqs;
     int seqs_stride, n_seqs;
     float* state;
     long state_stride;
 };
+
+// S decay + u with the decay as the sum of two floats in 32-bit runs: what its rounding leaves out would add up along the tokens
+template <typename T> __device__ __forceinline__ float kept(float S, float decay, float low, float u) { return fmaf(decay, S, sizeof(T) == 4 ? fmaf(low, S, u) : u); }
 
 __global__ void turn_table_kernel(const int* __restrict__ pos, const double* __restrict__ inv_freq, int pairs, float2* __restrict__ turn, long n) {
     for (long i = blockIdx.x * (long)blockDim.x + threadIdx.x; i < n; i += (long)gridDim.x * blockDim.x) {
@@ -73,7 +76,7 @@ __global__ void __launch_bounds__(256, 2) retention_scan_kernel(const Retention 
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, col = c0 + lane;
     const int start = a.seqs[s], len = a.seqs[a.seqs_stride + s], rd = a.seqs[2 * a.seqs_stride + s], wr = a.seqs[3 * a.seqs_stride + s];
     const T* proj = (const T*)a.proj;
-    const float keep = a.decay[h];
+    const float keep = a.decay[h], low = a.decay_low[h];
     float S[ROWS];
 #pragma unroll
     for (int r = 0; r < ROWS; r++) {
@@ -129,13 +132,13 @@ __global__ void __launch_bounds__(256, 2) retention_scan_kernel(const Retention 
             for (int r4 = 0; r4 < ROWS / 4; r4++) {
                 if (4 * r4 < rpt) {
                     const float4 k = kr[r4], q = qr[r4];
-                    S[4 * r4] = fmaf(keep, S[4 * r4], k.x * v);
+                    S[4 * r4] = kept<T>(S[4 * r4], keep, low, k.x * v);
                     o0 = fmaf(S[4 * r4], q.x, o0);
-                    S[4 * r4 + 1] = fmaf(keep, S[4 * r4 + 1], k.y * v);
+                    S[4 * r4 + 1] = kept<T>(S[4 * r4 + 1], keep, low, k.y * v);
                     o1 = fmaf(S[4 * r4 + 1], q.y, o1);
-                    S[4 * r4 + 2] = fmaf(keep, S[4 * r4 + 2], k.z * v);
+                    S[4 * r4 + 2] = kept<T>(S[4 * r4 + 2], keep, low, k.z * v);
                     o0 = fmaf(S[4 * r4 + 2], q.z, o0);
-                    S[4 * r4 + 3] = fmaf(keep, S[4 * r4 + 3], k.w * v);
+                    S[4 * r4 + 3] = kept<T>(S[4 * r4 + 3], keep, low, k.w * v);
                     o1 = fmaf(S[4 * r4 + 3], q.w, o1);
                 }
             }
@@ -585,7 +588,7 @@ __global__ void __launch_bounds__(256) retention_step_kernel(const Retention a, 
         if (is_k) ks[c] = u * a.k_scale;
         else qs[c] = u;
     }
-    const float keep = a.decay[h];
+    const float keep = a.decay[h], low = a.decay_low[h];
     __syncthreads();
     for (int base = 0; base < d; base += kRetStepRows * rows_par) {
         if (base) request(base);
@@ -596,7 +599,7 @@ __global__ void __launch_bounds__(256) retention_step_kernel(const Retention a, 
                 const float kn = ks[n], qn = qs[n];
 #pragma unroll
                 for (int e = 0; e < VEC; e++) {
-                    v[k][e] = fmaf(keep, v[k][e], kn * x[e]);
+                    v[k][e] = kept<T>(v[k][e], keep, low, kn * x[e]);
                     y[e] = fmaf(v[k][e], qn, y[e]);
                 }
                 if (wr >= 0) {
@@ -652,12 +655,12 @@ using namespace ktb;
 
 static bool ret_aligned(const void* p, size_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
 static bool ret_bad(const ktb200_retention_params* c) {
-    return !c || !c->proj || !c->decay || !c->log2_decay || !c->seqs || !c->state || c->heads <= 0 || c->dim <= 0 || c->vdim <= 0 || c->rot_dims < 0 || c->rot_dims > c->dim ||
+    return !c || !c->proj || !c->decay || !c->decay_low || !c->log2_decay || !c->seqs || !c->state || c->heads <= 0 || c->dim <= 0 || c->vdim <= 0 || c->rot_dims < 0 || c->rot_dims > c->dim ||
            (c->rot_dims & 1) || (c->rot_dims && !c->turn) || (c->rot_layout != kRotInterleaved && c->rot_layout != kRotHalves);
 }
 static Retention ret_args(const ktb200_retention_params* c) {
     return Retention{c->proj, c->proj_stride, c->q_off, c->k_off, c->v_off, c->g_off, c->heads, c->dim, c->vdim, c->rot_dims, c->rot_layout, reinterpret_cast<const float2*>(c->turn),
-                     c->k_scale, c->decay, c->log2_decay, c->eps, c->seqs, c->seqs_stride, c->n_seqs, c->state, c->state_stride};
+                     c->k_scale, c->decay, c->decay_low, c->log2_decay, c->eps, c->seqs, c->seqs_stride, c->n_seqs, c->state, c->state_stride};
 }
 
 extern "C" int ktb200_turn_table(const int* pos, const double* inv_freq, int pairs, float* turn, int n_tokens, void* stream) {

@@ -26,16 +26,17 @@ struct SelScan {
     int vec_state;
 };
 
-// exp(dt a): one base-2 exponential of a factor scaled once per thread where activations are bf16; expf in 32-bit runs
+// S exp(dt a) + u.  Where activations are bf16: one base-2 exponential of a factor scaled once per thread.  In 32-bit runs the factor is taken as
+// 1 + expm1(dt a): slow channels (factors just below one) would otherwise lose the same part of an ulp with every token.
 template <typename T> __device__ __forceinline__ float decay_factor(float a);
 template <> __device__ __forceinline__ float decay_factor<float>(float a) { return a; }
 template <> __device__ __forceinline__ float decay_factor<__nv_bfloat16>(float a) { return a * 1.4426950408889634f; }
-template <typename T> __device__ __forceinline__ float decay_of(float dt, float f);
-template <> __device__ __forceinline__ float decay_of<float>(float dt, float f) { return expf(dt * f); }
-template <> __device__ __forceinline__ float decay_of<__nv_bfloat16>(float dt, float f) {
+template <typename T> __device__ __forceinline__ float decayed(float S, float dt, float f, float u);
+template <> __device__ __forceinline__ float decayed<float>(float S, float dt, float f, float u) { return fmaf(expm1f(dt * f), S, S) + u; }
+template <> __device__ __forceinline__ float decayed<__nv_bfloat16>(float S, float dt, float f, float u) {
     float r;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(dt * f));
-    return r;
+    return fmaf(r, S, u);
 }
 
 // grid (channel blocks, portions), 128 threads: L neighbouring lanes share a channel, SPT states each, in registers.  Tokens run in order in chunks of
@@ -140,13 +141,13 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const SelScan a, T*
 #pragma unroll
                 for (int k = 0; k < SPT; k += 4) {
                     const float4 b = load4(Bs + tt * NP + l * SPT + k), c = load4(Cs + tt * NP + l * SPT + k);
-                    S[k] = fmaf(decay_of<T>(dt, f[k]), S[k], dx * b.x);
+                    S[k] = decayed<T>(S[k], dt, f[k], dx * b.x);
                     y[q] = fmaf(S[k], c.x, y[q]);
-                    S[k + 1] = fmaf(decay_of<T>(dt, f[k + 1]), S[k + 1], dx * b.y);
+                    S[k + 1] = decayed<T>(S[k + 1], dt, f[k + 1], dx * b.y);
                     y[q] = fmaf(S[k + 1], c.y, y[q]);
-                    S[k + 2] = fmaf(decay_of<T>(dt, f[k + 2]), S[k + 2], dx * b.z);
+                    S[k + 2] = decayed<T>(S[k + 2], dt, f[k + 2], dx * b.z);
                     y[q] = fmaf(S[k + 2], c.z, y[q]);
-                    S[k + 3] = fmaf(decay_of<T>(dt, f[k + 3]), S[k + 3], dx * b.w);
+                    S[k + 3] = decayed<T>(S[k + 3], dt, f[k + 3], dx * b.w);
                     y[q] = fmaf(S[k + 3], c.w, y[q]);
                 }
             }

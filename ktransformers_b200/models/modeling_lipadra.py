@@ -90,7 +90,7 @@ class LipadraForCausalLM(nn.Module):
             last = i + 1 == len(layers)
             y = layer.mix(h, batch, cache, i)
             if last and want.shape[0] == 0 and residual_trace is None:      # a portion whose logits nobody asked for: caches and states are written
-                return torch.empty((0, c.vocab), dtype=torch.float32, device=h.device)
+                break
             rows = want if last and residual_trace is None else None      # behind the last mixer only the rows asked for go on
             mlp = layer.mlp
             x, h, gate = layer.norm1(x, c.alpha, a=y, rows=rows, dot=mlp.shared_gate if mlp is not None else None)
@@ -99,5 +99,7 @@ class LipadraForCausalLM(nn.Module):
                 x, h, _ = layer.norm2(x, c.alpha, a=routed, b=shared, b_scale=gate, identity=(ids, weights, mlp.experts.experts) if mlp.identity else None)
             if residual_trace is not None:
                 residual_trace.append(x)
+        if want.shape[0] == 0:
+            return torch.empty((0, c.vocab), dtype=torch.float32, device=h.device)
         _, h, _ = self.final_norm(x, rows=want if residual_trace is not None or not layers else None, keep_x=False)
         return F.linear(h, self.embed).float()

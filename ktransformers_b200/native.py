@@ -134,7 +134,7 @@ class SumRmsnormParams(C.Structure):
 
 class RetentionParams(C.Structure):
     """ktb200_retention_params (include/ktb200.h)"""
-    _fields_ = _fields("p:proj l:proj_stride i:q_off,k_off,v_off,g_off,heads,dim,vdim,rot_dims,rot_layout p:turn f:k_scale p:decay,log2_decay f:eps p:seqs i:seqs_stride,n_seqs "
+    _fields_ = _fields("p:proj l:proj_stride i:q_off,k_off,v_off,g_off,heads,dim,vdim,rot_dims,rot_layout p:turn f:k_scale p:decay,decay_low,log2_decay f:eps p:seqs i:seqs_stride,n_seqs "
                        "p:state l:state_stride")
 
 

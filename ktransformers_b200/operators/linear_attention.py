@@ -259,6 +259,7 @@ class KRetention(nn.Module):
         self.n_in = self.offsets[3] + up(self.n_v)
         self.w_in, self.o = P(self.n_in, width), P(width, self.n_v)
         self.register_buffer("decay", torch.tensor(s.decay, dtype=torch.float32, device=device), persistent=False)
+        self.register_buffer("decay_low", torch.tensor([x - float(y) for x, y in zip(s.decay, self.decay.tolist())], dtype=torch.float32, device=device), persistent=False)
         self.register_buffer("log2_decay", torch.tensor([math.log2(x) for x in s.decay], dtype=torch.float32, device=device), persistent=False)
         self.register_buffer("inv_freq", s.rot.inv_freq(device) if s.rot is not None else torch.zeros(1, dtype=torch.float64, device=device), persistent=False)
 
@@ -277,7 +278,7 @@ class KRetention(nn.Module):
         q, k, v, g = self.offsets
         a = native.RetentionParams(proj=proj.data_ptr(), proj_stride=self.n_in, q_off=q, k_off=k, v_off=v, g_off=g, heads=s.heads, dim=s.dim, vdim=s.vdim,
                                    rot_dims=s.rot.dims if s.rot is not None else 0, rot_layout=s.rot.layout_code if s.rot is not None else 0,
-                                   turn=turn.data_ptr() if turn is not None else None, k_scale=s.dim ** -0.5, decay=self.decay.data_ptr(), log2_decay=self.log2_decay.data_ptr(),
+                                   turn=turn.data_ptr() if turn is not None else None, k_scale=s.dim ** -0.5, decay=self.decay.data_ptr(), decay_low=self.decay_low.data_ptr(), log2_decay=self.log2_decay.data_ptr(),
                                    eps=float(self.eps), seqs=batch.seqs.data_ptr(), seqs_stride=batch.seqs.stride(0), n_seqs=batch.n_seqs, state=state.data_ptr(),
                                    state_stride=state.stride(0))
         out = torch.empty((T, self.n_v), dtype=dt, device=dev)
