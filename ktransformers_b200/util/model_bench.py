@@ -1,6 +1,6 @@
 """Throughput and per-kernel rooflines of a step-function model at layer sizes of real models, with random weights, beside
 the closest existing model's kernels at equal size (`bench.py --model lekapel`, `bench.py --model mabidra`,
-`bench.py --model zivulix`, `bench.py --model bilurax`, `bench.py --model rununex`).
+`bench.py --model zivulix`, `bench.py --model bilurax`, `bench.py --model rununex`, `bench.py --model lipadra`).
 
 Two parts:
   * end to end through the Engine (scheduler, paged cache, step function): prompt tokens/s for a long prompt cut into portions,
@@ -132,6 +132,56 @@ def make_rununex_config(s):
             "layers": [{"type": kinds[c][0], "mixer": kinds[c][1], "mlp": moe} for c in s["order"]]}
 
 
+LIPADRA_SIZES = {
+    # the same widths and expert sizes as RUNUNEX_SIZES; R: retention, M: the selective scan with twice the width in channels and 16 states each, A:
+    # chunked attention over the grouped heads of Mabidra's attention layers; every feed-forward a mixture with a quarter as many identity experts
+    # as experts, plus a shared expert.  The chunk is as long as the benchmark's context, and `ctx` puts the decoded token at a chunk's last
+    # position.  The closest existing model at equal size is Mabidra: gated linear attention of the same heads for R and of as many channels for M,
+    # sigmoid attention for A, the same routed experts (of two matrices where these have three), no shared expert, no identity experts.
+    "2k-wide": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, chunk=2048, r_heads=16, r_dim=128, r_vdim=128, inner=4096, state=16, dt_rank=128, conv=4, experts=32, identity=8, top=4, groups=4,
+                    keep=2, ff=1024, shared_ff=2048, vocab=32768, order="RMARM", ctx=2047, rank=64),
+    "v3-layer": dict(width=7168, heads=64, kv_heads=8, dim=128, vdim=128, chunk=4096, r_heads=56, r_dim=128, r_vdim=128, inner=14336, state=16, dt_rank=448, conv=4, experts=32, identity=8, top=8,
+                     groups=4, keep=2, ff=2048, shared_ff=2048, vocab=32768, order="RMA", ctx=4095, rank=128),
+}
+
+
+def make_lipadra_config(s):
+    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5, "mask": {"size": s["chunk"]},
+            "rot": {"base": 10000.0, "dims": s["dim"] // 2}}
+    ret = {"heads": s["r_heads"], "dim": s["r_dim"], "vdim": s["r_vdim"], "decay": [1.0 - 2.0 ** (-4.0 - 6.0 * h / s["r_heads"]) for h in range(s["r_heads"])],
+           "rot": {"base": 10000.0, "dims": s["r_dim"]}}
+    scan = {"inner": s["inner"], "state": s["state"], "dt_rank": s["dt_rank"], "conv": s["conv"]}
+    kinds = {"A": ("attention", attn), "R": ("retention", ret), "M": ("mamba1", scan)}
+    moe = {"kind": "moe", "expert": {"ff": s["ff"]}, "shared": {"ff": s["shared_ff"]},
+           "router": {"experts": s["experts"], "identity": s["identity"], "top": s["top"], "groups": {"count": s["groups"], "keep": s["keep"]}, "scale": 2.0}}
+    return {"architecture": "Lipadra", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "postln_alpha": 3.0,
+            "layers": [{"type": kinds[c][0], "mixer": kinds[c][1], "mlp": moe} for c in s["order"]]}
+
+
+def settle_lipadra(model):
+    """the parameters whose usual range is not that of a projection or of a norm weight: small biases and corrections, negative state rates"""
+    for pname, p in model.named_parameters():
+        last = pname.rsplit(".", 1)[-1]
+        if last in ("b_in", "conv_b", "correction"):
+            p.data.sub_(1.0)
+        elif last == "dt_bias":
+            p.data.sub_(3.0)
+        elif last == "a":
+            p.data.copy_(-torch.arange(1, p.shape[1] + 1, device=p.device, dtype=torch.float32).expand_as(p))
+    return model
+
+
+def make_mabidra_recurrent_config(s):
+    """Mabidra at the sizes of a Lipadra size entry: gated linear attention of the same heads for R and of as many channels for M, sigmoid attention
+    for A, the same routed expert sizes"""
+    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5, "bias_max": 1024, "q_temp": {"coef": 0.1, "every": 512}}
+    gla = lambda heads: {"heads": heads, "dim": s["r_dim"], "vdim": s["r_vdim"], "tau": 16.0}
+    moe = {"kind": "moe", "expert": {"ff": s["ff"]}, "router": {"experts": s["experts"], "top": s["top"]}}
+    kinds = {"A": ("attention", attn), "R": ("gla", gla(s["r_heads"])), "M": ("gla", gla(s["inner"] // s["r_vdim"]))}
+    return {"architecture": "Mabidra", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5, "groups": 4}, "embedding": {"scale": 1.0},
+            "layers": [{"type": kinds[c][0], "mixer": kinds[c][1], "mlp": moe} for c in s["order"]]}
+
+
 def make_mabidra_mixed_config(s):
     """Mabidra at the sizes of a Rununex size entry: per P a sigmoid-attention layer without feed-forward and a gated-linear-attention layer with as
     many state values, per D a sigmoid-attention layer, the same routed expert sizes"""
@@ -153,7 +203,11 @@ def make_mabidra_dense_config(s):
 
 
 def random_model(cfg_dict, dtype=torch.bfloat16, device="cuda", size=None):
-    if cfg_dict["architecture"] == "Rununex":
+    if cfg_dict["architecture"] == "Lipadra":
+        from ..models.configuration_lipadra import LipadraConfig
+        from ..models.modeling_lipadra import LipadraForCausalLM
+        model = LipadraForCausalLM(LipadraConfig.from_dict(cfg_dict), dtype=dtype, device=device)
+    elif cfg_dict["architecture"] == "Rununex":
         from ..models.configuration_rununex import RununexConfig
         from ..models.modeling_rununex import RununexForCausalLM
         model = RununexForCausalLM(RununexConfig.from_dict(cfg_dict), dtype=dtype, device=device)
@@ -185,6 +239,8 @@ def random_model(cfg_dict, dtype=torch.bfloat16, device="cuda", size=None):
             p.data.copy_(1 + 0.1 * torch.randn(p.shape, generator=g, device=device))
         else:
             p.data.copy_(torch.randn(p.shape, generator=g, device=device, dtype=torch.float32) * p.shape[-1] ** -0.5)
+    if cfg_dict["architecture"] == "Lipadra":
+        settle_lipadra(model)
     return model.eval()
 
 
@@ -222,7 +278,8 @@ def timed(fn, flush, iters=10, warmup=3):
 def engine_leg(name, size, flush, steps, warmup, family="lekapel"):
     from .engine import Engine
     cfg = {"lekapel": make_config, "mabidra": make_mabidra_config, "zivulix": make_zivulix_config, "mabidra-dense": make_mabidra_dense_config,
-           "bilurax": make_bilurax_config, "mabidra-attn": make_mabidra_attn_config, "rununex": make_rununex_config, "mabidra-mixed": make_mabidra_mixed_config}[family](size)
+           "bilurax": make_bilurax_config, "mabidra-attn": make_mabidra_attn_config, "rununex": make_rununex_config, "mabidra-mixed": make_mabidra_mixed_config,
+           "lipadra": make_lipadra_config, "mabidra-recurrent": make_mabidra_recurrent_config}[family](size)
     model = random_model(cfg, size=size)
     if family == "zivulix":      # norm weights are zero-centred, decays and the value blend inside their usual ranges
         for pname, p in model.named_parameters():
@@ -965,7 +1022,7 @@ def rununex_kernel_leg(flush, peak_gbs, peak_tflops):
             dprep = lambda: native.check_seq(seq.ktb200_delta_prep(dproj.data_ptr(), d_in, 0, dC + DH * 128, dC + DH * 128 + DH, dcw.data_ptr(), taps, al2.data_ptr(), db2.data_ptr(), DH, DG,
                                                                    128, 128, 1e-6, bt.seq_of.data_ptr(), bt.seqs.data_ptr(), B, dstate.data_ptr(), dstate.shape[1], qn.data_ptr(), kn.data_ptr(),
                                                                    vv.data_ptr(), be.data_ptr(), de.data_ptr(), n, 30, S()))
-            row("ssd_conv_kernel", f"T={T} channels={C_} taps={taps}", timed(conv, flush, iters=it), nbytes=n * C_ * 4,
+            row("conv_silu_kernel", f"T={T} channels={C_} taps={taps}", timed(conv, flush, iters=it), nbytes=n * C_ * 4,
                 peer=peer_of("delta_prep_kernel", timed(dprep, flush, iters=it), n * dC * 6))
             conv()
             for tc, name in ((1, "ssd_chunk_kernel"), (0, "ssd_scan_kernel, CUDA cores")):
@@ -1010,7 +1067,209 @@ def rununex_kernel_leg(flush, peak_gbs, peak_tflops):
     return rows
 
 
-def run_bilurax(args):
+class KernelRows:
+    """rows of a kernel leg: times beside the like kernel of the closest path, as fractions of the measured peaks"""
+
+    def __init__(self, peak_gbs, peak_tf):
+        self.peak_gbs, self.peak_tf, self.rows = peak_gbs, peak_tf, []
+
+    def measure(self, kernel, ms, nbytes=None, flops=None):
+        r = {"kernel": kernel, "us": ms * 1e3}
+        if nbytes is not None:
+            r["GBps"], r["frac_of_measured_hbm"] = nbytes / ms / 1e6, nbytes / ms / 1e6 / self.peak_gbs
+        if flops is not None:
+            r["TFLOPs"], r["frac_of_measured_bf16"] = flops / ms / 1e9, flops / ms / 1e9 / self.peak_tf
+        return r
+
+    def add(self, kernel, case, ms, nbytes=None, flops=None, peer=None, **extra):
+        r = dict(self.measure(kernel, ms, nbytes, flops), case=case, **extra)
+        progress(f"{kernel} {case}: {ms * 1e3:.1f} us" + (f" (closest {peer['us']:.1f})" if peer else ""))
+        if peer:
+            r["closest"] = peer
+        self.rows.append(r)
+
+
+class KernelBatch:
+    """one sequence per entry of `lens`, each ending at position `ctx` - 1, on identity pages of 64 tokens"""
+
+    def __init__(self, lens, ctx, dev):
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        B, starts = len(lens), [sum(lens[:i]) for i in range(len(lens))]
+        self.pos = torch.cat([torch.arange(ctx - n, ctx, dtype=torch.int32, device=dev) for n in lens])
+        self.slot = torch.arange(B, dtype=torch.int32, device=dev).repeat_interleave(i32(lens).long())
+        self.seq_of = self.slot
+        self.seqs = i32([starts, lens, [2 * i for i in range(B)], [2 * i + 1 for i in range(B)]])
+        self.n_seqs, self.n_tokens, self.max_kv = B, sum(lens), ctx
+        self.page_size, self.max_pages_per_seq = 64, (ctx + 63) // 64
+        self.page_table = torch.arange(B * self.max_pages_per_seq, dtype=torch.int32, device=dev).reshape(B, -1)
+
+    def cache(self, width, fill):
+        return fill(self.n_seqs * self.max_pages_per_seq + 1, 64, width)
+
+
+def lipadra_kernel_leg(flush, peak_gbs, peak_tf):
+    """Lipadra's kernels beside their like kernels at DeepSeek-V3 widths (bf16)"""
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    seq, S = native.seq_lib(), lambda: torch.cuda.current_stream().cuda_stream
+    K = KernelRows(peak_gbs, peak_tf)
+    g = torch.Generator(device=dev).manual_seed(7)
+    rn = lambda *s, dt=bf: torch.randn(*s, generator=g, device=dev, dtype=torch.float32).to(dt)
+    f32, ok = torch.float32, native.check_seq
+    from ..operators.attention import paged_softmax_attention, qkv_prep
+    from ..operators.experts import KExpertsDense
+    from ..operators.gate import KGroupedSigmoidGate, KGroupedSoftmaxGate
+    from ..operators.norm import KLayerNorm, KSumRMSNorm
+    from ..models.configuration_lekapel import RotarySpec
+    D, top = 7168, 8
+    for _ in range(50):         # the first launches of a process also pay for what the host sets up
+        KLayerNorm(D, 1e-6)(rn(1, D, dt=f32))
+    for T in (1, 8, 2048):      # the sum with identity experts and a gated addend, RMS norm  vs  the sum of two addends, layer norm
+        x, a, b, bs, dot = rn(T, D, dt=f32), rn(T, D, dt=f32), rn(T, D), torch.rand(T, device=dev), rn(D)
+        ids, iw = torch.randint(0, 40, (T, top), device=dev), torch.rand(T, top, device=dev)
+        mine, theirs, nb = KSumRMSNorm(D, 1e-6), KLayerNorm(D, 1e-6), T * D * (4 + 4 + 2 + 4 + 2)
+        peer = K.measure("residual_layernorm_kernel", timed(lambda: theirs(x, a, b, 0.5), flush), nb)
+        K.add("sum_rmsnorm_kernel (identity experts, gated addend)", f"T={T} width={D}", timed(lambda: mine(x, 3.0, a, b, bs, (ids, iw, 32)), flush), nb, peer=peer)
+        K.add("sum_rmsnorm_kernel (one addend, gate dot)", f"T={T} width={D}", timed(lambda: mine(x, 3.0, a=b, dot=dot), flush), T * D * (4 + 2 + 4 + 2),
+              peer=K.measure("residual_layernorm_kernel (one addend)", timed(lambda: theirs(x, b, None, 0.5), flush), T * D * (4 + 2 + 4 + 2)))
+
+    # ---- attention: 64 / 8 heads of 128; weighted norms ahead of half a rotation; one added to the denominator
+    H, G, d, dv = 64, 8, 128, 128
+    n_q, n_k, n_v, cw = H * d, G * d, G * dv, G * (d + dv)
+    n_in = n_q + n_k + n_v
+    rot = RotarySpec(10000.0, 64, layout="halves")
+    inv, qw, kw, zero = rot.inv_freq(dev), rn(d), rn(d), torch.zeros(H, device=dev)
+    for T in (8, 2048):
+        bt = KernelBatch([1] * 8 if T == 8 else [T], 4096, dev)
+        proj, kv, nb = rn(T, n_in), bt.cache(cw, rn), T * (n_in + n_q + cw) * 2
+        prep = lambda **o: timed(lambda: qkv_prep(proj, bt, bt, kv, H, G, d, dv, (0, n_q, n_q + n_k), eps=1e-6, rot=rot, inv_freq=inv, **o), flush)
+        K.add("rope_norm_cache_write_kernel (weighted norm, then rotation)", f"T={T} heads={H}/{G} dim={d}", prep(qk_norm=3, q_weight=qw, k_weight=kw), nb,
+              peer=K.measure("rope_norm_cache_write_kernel (rotation, then unit rms)", prep(qk_norm=1), nb))
+    cases = [(KernelBatch([1] * B, ctx, dev), ctx, f"decode B={B} last position of a chunk of {ctx} heads={H}/{G}", B * ctx * cw * 2, None) for B, ctx in ((1, 4096), (8, 4096), (1, 32768))]
+    T, ctx = 2048, 4096
+    cases += [(KernelBatch([T], ctx, dev), ctx, f"prompt portion T={T} positions {ctx - T}..{ctx - 1} heads={H}/{G}, one chunk of {ctx}", None, float(sum(range(ctx - T + 1, ctx + 1))) * H * (d + dv) * 2),
+              (KernelBatch([T], ctx, dev), 1024, "the same, chunks of 1024", None, 2 * float(sum(range(1, 1025))) * H * (d + dv) * 2)]
+    for bt, chunk, case, nb, fl in cases:
+        kv, q = bt.cache(cw, rn), rn(bt.n_tokens, H, d)
+        run_ = lambda **o: timed(lambda: paged_softmax_attention(q, kv, bt, bt, H, G, d, dv, d ** -0.5, chunk=chunk, **o), flush, iters=5 if fl else 10)
+        K.add("window_softmax_attn_mma_kernel (+merge), one in the denominator", case, run_(sink=zero), nb, fl, peer=K.measure("the same kernel, plain soft-max", run_(), nb, fl))
+
+    # ---- retention: 56 heads of 128 x 128  vs  Mamba-2 (112 heads of 64, state 128: as many state values) and gated linear attention of the same heads
+    RH, P, sv, N, J, taps = 56, 112, 64, 128, 4, 4
+    r_in, inner2 = 4 * RH * d, P * sv
+    C_ = inner2 + 2 * J * N
+    s_in, sw = (inner2 + C_ + P + 7) // 8 * 8, inner2 * N + (taps - 1) * C_
+    rrot = RotarySpec(10000.0, 128, layout="halves")
+    rinv, decays = rrot.inv_freq(dev), [1.0 - 2.0 ** (-4.0 - 6.0 * h / RH) for h in range(RH)]
+    dec, low, l2 = torch.tensor(decays, device=dev), torch.zeros(RH, device=dev), torch.tensor(decays, device=dev).log2()
+    scw, scb, dtb, al, ds = rn(C_, taps), rn(C_), rn(P, dt=f32) - 2.0, rn(P, dt=f32), rn(P, dt=f32)
+    for B, T in ((1, 1), (8, 1), (1, 2048), (1, 8192)):
+        bt = KernelBatch([T] * B, max(T, 64), dev)
+        n, it = B * T, 5 if T > 1 else 10
+        proj, state, out, o = rn(n, r_in), torch.zeros(2 * B, RH * d * dv, device=dev), torch.empty(n, RH * dv, dtype=bf, device=dev), torch.empty(n, RH * dv, device=dev)
+        turn = torch.empty(n, 64, 2, device=dev)
+        table = lambda: ok(seq.ktb200_turn_table(bt.pos.data_ptr(), rinv.data_ptr(), 64, turn.data_ptr(), n, S()))
+        K.add("turn_table_kernel (once per step)", f"T={n} pairs=64", timed(table, flush), n * 64 * 8)
+        a = native.RetentionParams(proj=proj.data_ptr(), proj_stride=r_in, q_off=0, k_off=RH * d, v_off=2 * RH * d, g_off=3 * RH * d, heads=RH, dim=d, vdim=dv, rot_dims=128, rot_layout=1,
+                                   turn=turn.data_ptr(), k_scale=d ** -0.5, decay=dec.data_ptr(), decay_low=low.data_ptr(), log2_decay=l2.data_ptr(), eps=1e-6, seqs=bt.seqs.data_ptr(),
+                                   seqs_stride=B, n_seqs=B, state=state.data_ptr(), state_stride=state.stride(0))
+        z, zb, gw = rn(n, RH * d), rn(RH * d), rn(d)
+        gla = lambda: ok(seq.ktb200_gla_scan(proj.data_ptr(), r_in, 0, RH * d, 2 * RH * d, z.data_ptr(), RH * d, zb.data_ptr(), 16.0, RH, d, dv, bt.seqs.data_ptr(), B, B, n, state.data_ptr(),
+                                             o.data_ptr(), 30, S()))
+        gout = lambda: ok(seq.ktb200_gla_out(o.data_ptr(), gw.data_ptr(), 1e-6, proj[:, 3 * RH * d:].data_ptr(), r_in, out.data_ptr(), n, RH, dv, 30, S()))
+        sproj, sstate = rn(n, s_in), torch.zeros(2 * B, sw, device=dev)
+        xbc, y = torch.empty(n, C_, dtype=bf, device=dev), torch.empty(n, inner2, device=dev)
+        sa = native.SsdParams(proj=sproj.data_ptr(), proj_stride=s_in, xbc_off=inner2, dt_off=inner2 + C_, conv_w=scw.data_ptr(), conv_b=scb.data_ptr(), taps=taps, dt_bias=dtb.data_ptr(),
+                              a_log=al.data_ptr(), d_skip=ds.data_ptr(), heads=P, groups=J, state_size=N, vdim=sv, seq_of=bt.seq_of.data_ptr(), seqs=bt.seqs.data_ptr(), seqs_stride=B, n_seqs=B,
+                              state=sstate.data_ptr(), state_stride=sw)
+        if T == 1:
+            nb = B * RH * d * dv * 8
+            both = lambda: (gla(), gout())
+            K.add("retention_step_kernel (rotation, recurrence, norm, gate)", f"decode B={B} heads={RH} of {d} x {dv}", timed(lambda: ok(seq.ktb200_retention_step(C.byref(a), out.data_ptr(), 30, S())), flush),
+                  nb, peer=K.measure("gla_scan_kernel + gla_out_kernel", timed(both, flush), nb),
+                  like=K.measure("ssd_step_kernel", timed(lambda: ok(seq.ktb200_ssd_step(C.byref(sa), y.data_ptr(), 30, S())), flush), B * (inner2 * N + (taps - 1) * C_) * 8))
+        else:
+            fl = float(T) * RH * d * dv * 4
+            ws = torch.empty(seq.ktb200_retention_chunk_workspace(RH, d, dv, n, B), dtype=torch.uint8, device=dev)
+            ok(seq.ktb200_ssd_conv(C.byref(sa), xbc.data_ptr(), n, 30, S()))
+            ssd = timed(lambda: ok(seq.ktb200_ssd_scan(C.byref(sa), xbc.data_ptr(), y.data_ptr(), 30, 1, S())), flush, iters=it)
+            ms = timed(lambda: ok(seq.ktb200_retention_chunk(C.byref(a), out.data_ptr(), n, ws.data_ptr(), ws.numel(), 30, S())), flush, iters=it)
+            K.add("retention_chunk_state + carry + chunk_out kernels", f"prompt portion T={T} heads={RH} of {d} x {dv}", ms, flops=fl, peer=K.measure("ssd_chunk_kernel", ssd, flops=float(T) * inner2 * N * 4),
+                  frac_of_hbm_floor=n * RH * (3 * d + 2 * dv) * 2 / ms / 1e6 / peak_gbs)
+            if T == 2048:
+                K.add("retention_scan_kernel, CUDA cores", f"prompt portion T={T} heads={RH} of {d} x {dv}", timed(lambda: ok(seq.ktb200_retention_scan(C.byref(a), o.data_ptr(), 30, S())), flush, iters=it),
+                      flops=fl, peer=K.measure("gla_scan_kernel", timed(gla, flush, iters=it), flops=fl))
+
+    # ---- selective scan: 14336 channels of 16 states; its floor is the exponentials (one per channel, state and token: 16 a clock and SM)
+    I, N1 = 14336, 16
+    R_ = 448
+    bcw = R_ + 2 * N1
+    cwt, cb = rn(I, taps), rn(I)
+    bias, A, Dk = rn(I, dt=f32) - 3.0, -torch.arange(1, N1 + 1, device=dev, dtype=f32).repeat(I, 1).contiguous(), rn(I, dt=f32)
+    props = torch.cuda.get_device_properties(0)
+    ex_per_s = props.multi_processor_count * 16 * 1.965e9
+    for B, T in ((1, 1), (8, 1), (1, 2048), (8, 256)):
+        bt = KernelBatch([T] * B, max(T, 64), dev)
+        n, it = B * T, 5 if T > 1 else 10
+        proj, p, step, x, y = rn(n, 2 * I), rn(n, bcw), rn(n, I), torch.empty(n, I, dtype=bf, device=dev), torch.empty(n, I, dtype=bf, device=dev)
+        state = torch.zeros(2 * B, I * (N1 + taps - 1), device=dev)
+        conv = lambda: ok(seq.ktb200_conv_silu(proj.data_ptr(), 2 * I, cwt.data_ptr(), cb.data_ptr(), taps, I, bt.seq_of.data_ptr(), bt.seqs.data_ptr(), B, state.data_ptr(), state.stride(0), I * N1,
+                                               x.data_ptr(), n, B, 30, S()))
+        nbc = n * I * 4 + B * (taps - 1) * I * 8
+        K.add("conv_silu_kernel", f"T={n} ({B} portions) channels={I} taps={taps}", timed(conv, flush, iters=it), nbc)
+        conv()
+        a = native.SelectiveScanParams(x=x.data_ptr(), dt_logit=step.data_ptr(), b=p[:, R_:].data_ptr(), c=p[:, R_ + N1:].data_ptr(), z=proj[:, I:].data_ptr(), dt_stride=I, bc_stride=bcw, z_stride=2 * I,
+                                       dt_bias=bias.data_ptr(), a=A.data_ptr(), d_skip=Dk.data_ptr(), inner=I, state_size=N1, seqs=bt.seqs.data_ptr(), seqs_stride=B, n_seqs=B, state=state.data_ptr(),
+                                       state_stride=state.stride(0))
+        ms = timed(lambda: ok(seq.ktb200_selective_scan(C.byref(a), y.data_ptr(), 30, S())), flush, iters=it)
+        sproj, sstate = rn(n, s_in), torch.zeros(2 * B, sw, device=dev)
+        xbc, sy = torch.empty(n, C_, dtype=bf, device=dev), torch.empty(n, inner2, device=dev)
+        sa = native.SsdParams(proj=sproj.data_ptr(), proj_stride=s_in, xbc_off=inner2, dt_off=inner2 + C_, conv_w=scw.data_ptr(), conv_b=scb.data_ptr(), taps=taps, dt_bias=dtb.data_ptr(),
+                              a_log=al.data_ptr(), d_skip=ds.data_ptr(), heads=P, groups=J, state_size=N, vdim=sv, seq_of=bt.seq_of.data_ptr(), seqs=bt.seqs.data_ptr(), seqs_stride=B, n_seqs=B,
+                              state=sstate.data_ptr(), state_stride=sw)
+        nb = n * (I * 8 + 4 * N1) + B * I * N1 * 8
+        if T == 1:
+            peer = K.measure("ssd_step_kernel", timed(lambda: ok(seq.ktb200_ssd_step(C.byref(sa), sy.data_ptr(), 30, S())), flush), B * (inner2 * N + (taps - 1) * C_) * 8)
+        else:
+            ok(seq.ktb200_ssd_conv(C.byref(sa), xbc.data_ptr(), n, 30, S()))
+            peer = K.measure("ssd_chunk_kernel", timed(lambda: ok(seq.ktb200_ssd_scan(C.byref(sa), xbc.data_ptr(), sy.data_ptr(), 30, 1, S())), flush, iters=it),
+                             n * (C_ * 2 + inner2 * 4) + B * inner2 * N * 8)
+        K.add("selective_scan_kernel", f"{B} x {T} tokens, {I} channels of {N1}", ms, nb, peer=peer, frac_of_exponentials=n * I * N1 / ms * 1e3 / ex_per_s)
+
+    # ---- router: grouped soft-max top 8 of 256 + 64  vs  grouped sigmoid
+    E = 320
+    mine, theirs = KGroupedSoftmaxGate(D, E, top, 8, 4, 2.0), KGroupedSigmoidGate(D, E, top, 8, 4, 2.0)
+    mine.weight.data.copy_(rn(E, D, dt=f32) * D ** -0.5)
+    theirs.weight.data.copy_(mine.weight.data)
+    for T in (1, 8, 2048):
+        x, nb = rn(T, D), E * D * 4 + T * D * 2
+        small = T < mine.gemm_min_tokens
+        K.add("gate_kernel (soft-max, biased group max)" if small else "fp32 GEMM + gate_select_kernel", f"T={T} outputs={E} width={D} top={top}", timed(lambda: mine(x), flush), nb,
+              peer=K.measure("the same, grouped sigmoid", timed(lambda: theirs(x), flush), nb))
+
+    # ---- experts: a fifth of the choices identity experts  vs  every choice an expert
+    E, ff = 32, 2048
+    ex = KExpertsDense(D, ff, E)
+    for p_ in ex.parameters():
+        p_.data.copy_(rn(*p_.shape) * p_.shape[-1] ** -0.5)
+    for T in (1, 8, 2048):
+        x, w = rn(T, D), torch.rand(T, top, generator=g, device=dev)
+        draw = lambda n: torch.stack([torch.randperm(n, generator=g, device=dev)[:top] for _ in range(T)])
+        ids, all_ids = draw(40), draw(E)
+        cost = lambda i: dict(nbytes=int(i[i < E].unique().numel()) * 3 * ff * D * 2) if T < 48 else dict(flops=float((i < E).sum()) * 3 * ff * D * 2)
+        K.add("experts, a fifth of the choices identities (whole call)", f"T={T} top={top} of 32 + 8 width={D} ff={ff}", timed(lambda: ex(x, ids, w), flush), **cost(ids),
+              peer=K.measure("experts, every choice an expert (whole call)", timed(lambda: ex(x, all_ids, w), flush), **cost(all_ids)))
+    return K.rows
+
+
+# family -> (sizes, kernel leg, the closest existing model: its family name in engine_leg and its sizes)
+FAMILIES = {"mabidra": (MABIDRA_SIZES, mabidra_kernel_leg, "lekapel", SIZES), "zivulix": (ZIVULIX_SIZES, zivulix_kernel_leg, "mabidra-dense", ZIVULIX_SIZES),
+            "bilurax": (BILURAX_SIZES, bilurax_kernel_leg, "mabidra-attn", BILURAX_SIZES), "rununex": (RUNUNEX_SIZES, rununex_kernel_leg, "mabidra-mixed", RUNUNEX_SIZES),
+            "lipadra": (LIPADRA_SIZES, lipadra_kernel_leg, "mabidra-recurrent", LIPADRA_SIZES)}
+
+
+def run_family(args, family):
+    """one JSON line: the family's kernels, then per size the model and the closest existing model, in one process"""
+    sizes, leg, closest, closest_sizes = FAMILIES[family]
     torch.cuda.set_device(0)
     root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
     try:
@@ -1020,72 +1279,22 @@ def run_bilurax(args):
         peak, tf, src = 6650.0, 1590.0, "fallback"
     flush = Flusher("cuda")
     n0 = native.seq_lib().ktb200_launch_count()
-    out = {"bench": "bilurax", "dtype": "bf16", "data": "synthetic (random weights and tokens)", "hbm_peak_GBps": peak, "bf16_peak_TFLOPs": tf, "peak_source": src,
-           "timing": "CUDA events, median, 256 MB L2 flush between timed calls", "kernels": [] if getattr(args, "no_kernels", False) else bilurax_kernel_leg(flush, peak, tf),
+    out = {"bench": family, "dtype": "bf16", "data": "synthetic (random weights and tokens)", "hbm_peak_GBps": peak, "bf16_peak_TFLOPs": tf, "peak_source": src,
+           "timing": "CUDA events, median, 256 MB L2 flush between timed calls", "kernels": [] if getattr(args, "no_kernels", False) else leg(flush, peak, tf),
            "models": [], "closest_models": []}
-    for name in (args.sizes.split(",") if getattr(args, "sizes", None) else BILURAX_SIZES):
-        out["models"].append(engine_leg(name, BILURAX_SIZES[name], flush, args.steps, args.warmup, family="bilurax"))
+    for name in (args.sizes.split(",") if getattr(args, "sizes", None) else sizes):
+        out["models"].append(engine_leg(name, sizes[name], flush, args.steps, args.warmup, family=family))
         torch.cuda.empty_cache()
-        out["closest_models"].append(engine_leg(name, BILURAX_SIZES[name], flush, args.steps, args.warmup, family="mabidra-attn"))      # Mabidra at the same sizes, in the same process
-        torch.cuda.empty_cache()
-    out["gpu_launches"] = int(native.seq_lib().ktb200_launch_count() - n0)
-    print(json.dumps(out))
-
-
-def run_rununex(args):
-    torch.cuda.set_device(0)
-    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
-    try:
-        m = json.load(open(os.path.join(root, "MEASURED_PEAKS.json")))
-        peak, tf, src = float(m["hbm_gbs"]), float(m["bf16_tflops"]), "measured (MEASURED_PEAKS.json hbm_gbs, bf16_tflops)"
-    except Exception:
-        peak, tf, src = 6650.0, 1590.0, "fallback"
-    flush = Flusher("cuda")
-    n0 = native.seq_lib().ktb200_launch_count()
-    out = {"bench": "rununex", "dtype": "bf16", "data": "synthetic (random weights and tokens)", "hbm_peak_GBps": peak, "bf16_peak_TFLOPs": tf, "peak_source": src,
-           "timing": "CUDA events, median, 256 MB L2 flush between timed calls", "kernels": [] if getattr(args, "no_kernels", False) else rununex_kernel_leg(flush, peak, tf),
-           "models": [], "closest_models": []}
-    for name in (args.sizes.split(",") if getattr(args, "sizes", None) else RUNUNEX_SIZES):
-        out["models"].append(engine_leg(name, RUNUNEX_SIZES[name], flush, args.steps, args.warmup, family="rununex"))
-        torch.cuda.empty_cache()
-        out["closest_models"].append(engine_leg(name, RUNUNEX_SIZES[name], flush, args.steps, args.warmup, family="mabidra-mixed"))      # Mabidra at the same sizes, in the same process
-        torch.cuda.empty_cache()
-    out["gpu_launches"] = int(native.seq_lib().ktb200_launch_count() - n0)
-    print(json.dumps(out))
-
-
-def run_zivulix(args):
-    torch.cuda.set_device(0)
-    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
-    try:
-        m = json.load(open(os.path.join(root, "MEASURED_PEAKS.json")))
-        peak, tf, src = float(m["hbm_gbs"]), float(m["bf16_tflops"]), "measured (MEASURED_PEAKS.json hbm_gbs, bf16_tflops)"
-    except Exception:
-        peak, tf, src = 6650.0, 1590.0, "fallback"
-    flush = Flusher("cuda")
-    n0 = native.seq_lib().ktb200_launch_count()
-    out = {"bench": "zivulix", "dtype": "bf16", "data": "synthetic (random weights and tokens)", "hbm_peak_GBps": peak, "bf16_peak_TFLOPs": tf, "peak_source": src,
-           "timing": "CUDA events, median, 256 MB L2 flush between timed calls", "kernels": [] if getattr(args, "no_kernels", False) else zivulix_kernel_leg(flush, peak, tf),
-           "models": [], "closest_models": []}
-    for name in (args.sizes.split(",") if getattr(args, "sizes", None) else ZIVULIX_SIZES):
-        out["models"].append(engine_leg(name, ZIVULIX_SIZES[name], flush, args.steps, args.warmup, family="zivulix"))
-        torch.cuda.empty_cache()
-        out["closest_models"].append(engine_leg(name, ZIVULIX_SIZES[name], flush, args.steps, args.warmup, family="mabidra-dense"))      # Mabidra at the same sizes, in the same process
+        out["closest_models"].append(engine_leg(name, closest_sizes[name], flush, args.steps, args.warmup, family=closest))
         torch.cuda.empty_cache()
     out["gpu_launches"] = int(native.seq_lib().ktb200_launch_count() - n0)
     print(json.dumps(out))
 
 
 def run(args):
-    """`bench.py --model lekapel | mabidra | zivulix | bilurax | rununex`: prints one JSON line."""
-    if args.model == "rununex":
-        return run_rununex(args)
-    if args.model == "mabidra":
-        return run_mabidra(args)
-    if args.model == "zivulix":
-        return run_zivulix(args)
-    if args.model == "bilurax":
-        return run_bilurax(args)
+    """`bench.py --model lekapel | mabidra | zivulix | bilurax | rununex | lipadra`: prints one JSON line."""
+    if args.model in FAMILIES:
+        return run_family(args, args.model)
     torch.cuda.set_device(0)
     root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
     try:
@@ -1099,28 +1308,6 @@ def run(args):
            "timing": "CUDA events, median, 256 MB L2 flush between timed calls", "kernels": kernel_leg(flush, peak, have_main), "models": []}
     for name in (args.sizes.split(",") if getattr(args, "sizes", None) else SIZES):
         out["models"].append(engine_leg(name, SIZES[name], flush, args.steps, args.warmup))
-        torch.cuda.empty_cache()
-    out["gpu_launches"] = int(native.seq_lib().ktb200_launch_count() - n0)
-    print(json.dumps(out))
-
-
-def run_mabidra(args):
-    torch.cuda.set_device(0)
-    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
-    try:
-        m = json.load(open(os.path.join(root, "MEASURED_PEAKS.json")))
-        peak, tf, src = float(m["hbm_gbs"]), float(m["bf16_tflops"]), "measured (MEASURED_PEAKS.json hbm_gbs, bf16_tflops)"
-    except Exception:
-        peak, tf, src = 6650.0, 1590.0, "fallback"
-    flush = Flusher("cuda")
-    n0 = native.seq_lib().ktb200_launch_count()
-    out = {"bench": "mabidra", "dtype": "bf16", "data": "synthetic (random weights and tokens)", "hbm_peak_GBps": peak, "bf16_peak_TFLOPs": tf, "peak_source": src,
-           "timing": "CUDA events, median, 256 MB L2 flush between timed calls", "kernels": [] if getattr(args, "no_kernels", False) else mabidra_kernel_leg(flush, peak, tf),
-           "models": [], "closest_models": []}
-    for name in (args.sizes.split(",") if getattr(args, "sizes", None) else MABIDRA_SIZES):
-        out["models"].append(engine_leg(name, MABIDRA_SIZES[name], flush, args.steps, args.warmup, family="mabidra"))
-        torch.cuda.empty_cache()
-        out["closest_models"].append(engine_leg(name, SIZES[name], flush, args.steps, args.warmup))      # Lekapel at the same widths, in the same process
         torch.cuda.empty_cache()
     out["gpu_launches"] = int(native.seq_lib().ktb200_launch_count() - n0)
     print(json.dumps(out))
