@@ -623,8 +623,8 @@ int ktb200_sum_rmsnorm(const ktb200_sum_rmsnorm_params* params, int n_tokens, in
  *     S <- decay[h] S + k v^T ;  o = S^T q ;  out = o / sqrt(mean_vdim(o^2) + eps) * silu(g)
  * decay[h] + decay_low[h]: the decay as two floats (decay_low is read in 32-bit runs); log2_decay[h] = log2 of it.  State rows [heads][dim][vdim] fp32, row stride state_stride; dim <= 256.
  *   ktb200_turn_table        turn[t][i] = (cos, sin) of pos[t] * inv_freq[i], angles in fp64
- *   ktb200_retention_chunk   chunks of 64 tokens on the tensor cores (bf16; dim and vdim multiples of 16 up to 128): the states ahead of every chunk, then
- *                            all chunks at once; workspace: ktb200_retention_chunk_workspace bytes
+ *   ktb200_retention_chunk   on the tensor cores (bf16; dim and vdim multiples of 16 up to 128): the states ahead of every span of 128 tokens, then all
+ *                            chunks of 64 at once; workspace: ktb200_retention_chunk_workspace bytes
  *   ktb200_retention_scan    token by token; o [n_tokens][heads*vdim] fp32 is left for ktb200_gla_out
  *   ktb200_retention_step    decode steps (one token per portion), norm and gate included; vdim <= ktb200_retention_step_max_vdim() */
 typedef struct {

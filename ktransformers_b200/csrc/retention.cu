@@ -4,7 +4,7 @@
 //   S <- decay_h S + k v^T ;  o = S^T q ;  out = o / sqrt(mean_c(o_c^2) + eps) * silu(g)          per head; q, k turned, k times k_scale
 //
 //   ktb200_turn_table        the (cos, sin) pairs of a step's tokens, once for all layers of the same rotation
-//   ktb200_retention_chunk   prompt portions in chunks of 64 tokens on the tensor cores, chunks in parallel (bf16)
+//   ktb200_retention_chunk   prompt portions in chunks on the tensor cores, all chunks in parallel (bf16)
 //   ktb200_retention_scan    token by token on CUDA cores (fp32, sizes outside the tiles, short portions), o left for ktb200_gla_out
 //   ktb200_retention_step    decode steps: rotation, recurrence, norm and gate in one launch, a head's column blocks as a thread-block cluster
 //
@@ -162,35 +162,39 @@ __global__ void __launch_bounds__(256, 2) retention_scan_kernel(const Retention 
     }
 }
 
-// ------------------------------------------------------------------------------------------------ chunks of 64 tokens on the tensor cores (bf16)
-// With fixed decays the states ahead of all chunks follow from one pass over per-chunk sums, so every chunk of every portion and head is a CTA:
-//   1. chunk_state   U_c = sum_j decay^(n - 1 - j) k_j v_j^T                        (n tokens in the chunk)
-//   2. carry         S_c = the state ahead of chunk c: S_(c+1) = decay^n S_c + U_c, elementwise along the portion's chunks; S_c replaces U_c
-//   3. chunk_out     o_i = decay^(i + 1) S_c^T q_i + sum_{j <= i} decay^(i - j) (q_i . k_j) v_j, then norm and gate
+// ------------------------------------------------------------------------------------------------ chunks on the tensor cores (bf16)
+// With fixed decays the states along a portion follow from one pass over the sums of its parts, so all parts of all portions and heads run at once:
+//   1. chunk_state   spans of 128 tokens:  U_s = sum_j decay^(n - 1 - j) k_j v_j^T                        (n tokens in the span)
+//   2. carry         S_s = the state ahead of span s: S_(s+1) = decay^n S_s + U_s, elementwise along the portion's spans; S_s replaces U_s
+//   3. chunk_out     chunks of 64 tokens, c tokens behind their span's start (0 or 64):
+//                    o_i = decay^(c + i + 1) S_s^T q_i + sum over the span's keys j up to i of decay^(i - j) (q_i . k_j) v_j, then norm and gate
 // m16n8k16 bf16 MMAs with fp32 accumulators; v is bf16 as it comes, every other operand (turned q and k, weighted k and scores, S) enters as the
 // sum of two bf16 terms hi + lo (about 16 bits of mantissa), products of two such operands as hi hi + hi lo + lo hi.
-// Workspace per (chunk tile, head): dim * vdim fp32 of U, then in the same bytes S as groups of 8 columns [8 hi | 8 lo].
-constexpr int kRetQ = 64;
+// Workspace per (span, head): dim * vdim fp32 of U, then in the same bytes S as groups of 8 columns [8 hi | 8 lo].
+constexpr int kRetQ = 64, kRetSpan = 2 * kRetQ;
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(a, b);
     lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
-// which portion and which of its chunks tile b is: {portion or -1, first token's offset in the portion, tokens}
-__device__ __forceinline__ void find_chunk(const int* __restrict__ seqs, int stride, int n_seqs, int b, int (&info)[3]) {
+// which portion tile b of `per` tokens belongs to: {portion or -1, first token's offset in the portion, tokens, the portion's first span}
+__device__ __forceinline__ void find_chunk(const int* __restrict__ seqs, int stride, int n_seqs, int b, int per, int (&info)[4]) {
     info[0] = -1;
+    int spans = 0;
     for (int s = 0; s < n_seqs; s++) {
-        const int len = seqs[stride + s], nt = (len + kRetQ - 1) / kRetQ;
+        const int len = seqs[stride + s], nt = (len + per - 1) / per;
         if (b < nt) {
             info[0] = s;
-            info[1] = b * kRetQ;
-            info[2] = min(kRetQ, len - b * kRetQ);
+            info[1] = b * per;
+            info[2] = min(per, len - b * per);
+            info[3] = spans;
             return;
         }
         b -= nt;
+        spans += (len + kRetSpan - 1) / kRetSpan;
     }
 }
 // Stage nt rows of a head (first row `src`, rows `stride` apart; the rest of the 64 rows zeros), turned and times scale * row_w[row], as two bf16 planes
-// [64][ld].  Four pairs at a time where the pair halves are four neighbouring columns each.
+// [64][ld].  Where the pair halves are runs of four columns: four pairs at a time, the loads of four such units in flight together.
 __device__ __forceinline__ void stage_turned(__nv_bfloat16* hi, __nv_bfloat16* lo, int ld, const __nv_bfloat16* __restrict__ src, long stride, int nt, int d, int rot_dims, int layout,
                                              const float2* __restrict__ turn, float scale, const float* row_w) {
     const int half = rot_dims >> 1;
@@ -203,25 +207,46 @@ __device__ __forceinline__ void stage_turned(__nv_bfloat16* hi, __nv_bfloat16* l
         *reinterpret_cast<uint2*>(lo + at) = make_uint2(l0, l1);
     };
     if (wide) {
-        const int per = half / 4 + (d - rot_dims) / 4;      // units of a row: four pairs, or four columns that pass (d - rot_dims is a multiple of 4 here)
-        for (int i = threadIdx.x; i < kRetQ * per; i += blockDim.x) {
-            const int r = i / per, u = i - r * per;
-            const float w = r < nt ? (row_w ? scale * row_w[r] : scale) : 0.f;
-            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (u < half / 4) {
-                const int c = u * 4;
-                float4 x = zero, y = zero;
-                if (r < nt) {
-                    const float4 p = load4(src + (long)r * stride + c), q = load4(src + (long)r * stride + half + c);
-                    const float4 t0 = *reinterpret_cast<const float4*>(turn + (long)r * half + c), t1 = *reinterpret_cast<const float4*>(turn + (long)r * half + c + 2);
-                    x = make_float4(p.x * t0.x - q.x * t0.y, p.y * t0.z - q.y * t0.w, p.z * t1.x - q.z * t1.y, p.w * t1.z - q.w * t1.w);
-                    y = make_float4(q.x * t0.x + p.x * t0.y, q.y * t0.z + p.y * t0.w, q.z * t1.x + p.z * t1.y, q.w * t1.z + p.w * t1.w);
+        const int pairs = half / 4, per = pairs + (d - rot_dims) / 4;      // units of a row: four pairs, or four columns that pass (d - rot_dims is a multiple of 4 here)
+        constexpr int AHEAD = 4;
+        for (int i0 = threadIdx.x; i0 < kRetQ * per; i0 += AHEAD * blockDim.x) {
+            uint2 p[AHEAD], q[AHEAD];
+            float4 c0[AHEAD], c1[AHEAD];
+#pragma unroll
+            for (int k = 0; k < AHEAD; k++) {
+                const int i = i0 + k * blockDim.x, r = i / per, u = i - r * per;
+                p[k] = q[k] = make_uint2(0, 0);
+                if (r < nt && i < kRetQ * per) {
+                    const __nv_bfloat16* row = src + (long)r * stride;
+                    if (u < pairs) {
+                        p[k] = *reinterpret_cast<const uint2*>(row + u * 4);
+                        q[k] = *reinterpret_cast<const uint2*>(row + half + u * 4);
+                        c0[k] = *reinterpret_cast<const float4*>(turn + (long)r * half + u * 4);
+                        c1[k] = *reinterpret_cast<const float4*>(turn + (long)r * half + u * 4 + 2);
+                    } else {
+                        p[k] = *reinterpret_cast<const uint2*>(row + rot_dims + (u - pairs) * 4);
+                    }
                 }
-                put(r * ld + c, x, w);
-                put(r * ld + half + c, y, w);
-            } else {
-                const int c = rot_dims + (u - half / 4) * 4;
-                put(r * ld + c, r < nt ? load4(src + (long)r * stride + c) : zero, w);
+            }
+#pragma unroll
+            for (int k = 0; k < AHEAD; k++) {
+                const int i = i0 + k * blockDim.x, r = i / per, u = i - r * per;
+                if (i >= kRetQ * per) break;
+                const bool in = r < nt;
+                const float w = in ? (row_w ? scale * row_w[r] : scale) : 0.f;
+                const float4 a = make_float4(__uint_as_float(p[k].x << 16), __uint_as_float(p[k].x & 0xffff0000u), __uint_as_float(p[k].y << 16), __uint_as_float(p[k].y & 0xffff0000u));
+                if (u < pairs) {
+                    const float4 b = make_float4(__uint_as_float(q[k].x << 16), __uint_as_float(q[k].x & 0xffff0000u), __uint_as_float(q[k].y << 16), __uint_as_float(q[k].y & 0xffff0000u));
+                    float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
+                    if (in) {
+                        x = make_float4(a.x * c0[k].x - b.x * c0[k].y, a.y * c0[k].z - b.y * c0[k].w, a.z * c1[k].x - b.z * c1[k].y, a.w * c1[k].z - b.w * c1[k].w);
+                        y = make_float4(b.x * c0[k].x + a.x * c0[k].y, b.y * c0[k].z + a.y * c0[k].w, b.z * c1[k].x + a.z * c1[k].y, b.w * c1[k].z + a.w * c1[k].w);
+                    }
+                    put(r * ld + u * 4, x, w);
+                    put(r * ld + half + u * 4, y, w);
+                } else {
+                    put(r * ld + rot_dims + (u - pairs) * 4, a, w);
+                }
             }
         }
         return;
@@ -238,81 +263,101 @@ __device__ __forceinline__ void stage_turned(__nv_bfloat16* hi, __nv_bfloat16* l
         *reinterpret_cast<uint32_t*>(lo + r * ld + c) = l;
     }
 }
+__device__ __forceinline__ void fetch_rows(__nv_bfloat16* dst, int ld, const __nv_bfloat16* __restrict__ src, long stride, int nt, int n) {      // nt of 64 rows of n columns, the rest zeros
+    const int pieces = n >> 3;
+    for (int i = threadIdx.x; i < kRetQ * pieces; i += blockDim.x) {
+        const int r = i / pieces, c = (i - r * pieces) * 8;
+        cp_async16(dst + r * ld + c, src + (long)(r < nt ? r : 0) * stride + c, r < nt);
+    }
+}
 
-// grid (tiles, heads), 8 warps; a unit of work is 16 key rows x up to 64 value columns of U
-__global__ void __launch_bounds__(256) retention_chunk_state_kernel(const Retention a, float* __restrict__ ws) {
+// grid (spans, heads), 8 warps; a unit of work is 16 key rows x up to 64 value columns of U, at most two per warp
+__global__ void __launch_bounds__(256, 2) retention_chunk_state_kernel(const Retention a, float* __restrict__ ws) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    __shared__ int info[3];
-    __shared__ float row_w[kRetQ];
+    __shared__ int info[4];
+    __shared__ float row_w[kRetSpan];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, tq = lane & 3, h = blockIdx.y;
     const int d = a.d, dv = a.dv, ldk = d + 8, ldv = dv + 8;
-    if (tid == 0) find_chunk(a.seqs, a.seqs_stride, a.n_seqs, blockIdx.x, info);
+    if (tid == 0) find_chunk(a.seqs, a.seqs_stride, a.n_seqs, blockIdx.x, kRetSpan, info);
     __syncthreads();
     if (info[0] < 0) return;
-    const int nt = info[2];
+    const int n = info[2];
     const long t0 = a.seqs[info[0]] + info[1];
     __nv_bfloat16* Kh = reinterpret_cast<__nv_bfloat16*>(smem_raw);
     __nv_bfloat16* Kl = Kh + kRetQ * ldk;
     __nv_bfloat16* Vs = Kl + kRetQ * ldk;
     const __nv_bfloat16* proj = (const __nv_bfloat16*)a.proj;
-    const int vc = dv >> 3;
-    for (int i = tid; i < kRetQ * vc; i += 256) {
-        const int r = i / vc, c = (i - r * vc) * 8;
-        cp_async16(Vs + r * ldv + c, proj + (t0 + (r < nt ? r : 0)) * a.stride + a.v_off + (long)h * dv + c, r < nt);
-    }
-    if (tid < kRetQ) row_w[tid] = tid < nt ? exp2f((float)(nt - 1 - tid) * a.log2_decay[h]) : 0.f;
-    __syncthreads();
-    stage_turned(Kh, Kl, ldk, proj + t0 * a.stride + a.k_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, a.turn + t0 * (a.rot_dims >> 1), a.k_scale, row_w);
-    cp_async_wait_all();
-    __syncthreads();
-    float* U = ws + ((long)blockIdx.x * a.H + h) * d * dv;
-    const int d16 = d >> 4, dv16 = dv >> 4, cgroups = (dv16 + 3) >> 2, k16 = (nt + 15) >> 4;
-    for (int unit = warp; unit < d16 * cgroups; unit += 8) {
-        const int r0 = (unit / cgroups) * 16, v0 = (unit % cgroups) * 4;
-        float acc[8][4];
+    if (tid < kRetSpan) row_w[tid] = tid < n ? exp2f((float)(n - 1 - tid) * a.log2_decay[h]) : 0.f;
+    const int d16 = d >> 4, dv16 = dv >> 4, cgroups = (dv16 + 3) >> 2;
+    float acc[2][8][4];
 #pragma unroll
-        for (int n = 0; n < 8; n++)
+    for (int k = 0; k < 2; k++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) acc[n][e] = 0.f;
-        for (int kk = 0; kk < k16; kk++) {
-            uint32_t ah[4], al[4];
-            const int at = (kk * 16 + (lane & 7) + 8 * (lane >> 4)) * ldk + r0 + 8 * ((lane >> 3) & 1);
-            ldmatrix_x4_trans(ah, Kh + at);
-            ldmatrix_x4_trans(al, Kl + at);
+        for (int m = 0; m < 8; m++)
 #pragma unroll
-            for (int vp = 0; vp < 4; vp++) {
-                if (v0 + vp < dv16) {
-                    uint32_t b[4];
-                    ldmatrix_x4_trans(b, Vs + (kk * 16 + (lane & 15)) * ldv + (v0 + vp) * 16 + 8 * (lane >> 4));
-                    mma_bf16_16816(acc[2 * vp], ah, b[0], b[1]);
-                    mma_bf16_16816(acc[2 * vp + 1], ah, b[2], b[3]);
-                    mma_bf16_16816(acc[2 * vp], al, b[0], b[1]);
-                    mma_bf16_16816(acc[2 * vp + 1], al, b[2], b[3]);
+            for (int e = 0; e < 4; e++) acc[k][m][e] = 0.f;
+    for (int part = 0; part * kRetQ < n; part++) {
+        const long t1 = t0 + part * kRetQ;
+        const int nt = min(kRetQ, n - part * kRetQ), k16 = (nt + 15) >> 4;
+        __syncthreads();      // row_w is there; the first half is consumed
+        fetch_rows(Vs, ldv, proj + t1 * a.stride + a.v_off + (long)h * dv, a.stride, nt, dv);
+        stage_turned(Kh, Kl, ldk, proj + t1 * a.stride + a.k_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, a.turn + t1 * (a.rot_dims >> 1), a.k_scale, row_w + part * kRetQ);
+        cp_async_wait_all();
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < 2; k++) {
+            const int unit = warp + 8 * k;
+            if (unit < d16 * cgroups) {
+                const int r0 = (unit / cgroups) * 16, v0 = (unit % cgroups) * 4;
+                for (int kk = 0; kk < k16; kk++) {
+                    uint32_t ah[4], al[4];
+                    const int at = (kk * 16 + (lane & 7) + 8 * (lane >> 4)) * ldk + r0 + 8 * ((lane >> 3) & 1);
+                    ldmatrix_x4_trans(ah, Kh + at);
+                    ldmatrix_x4_trans(al, Kl + at);
+#pragma unroll
+                    for (int vp = 0; vp < 4; vp++) {
+                        if (v0 + vp < dv16) {
+                            uint32_t b[4];
+                            ldmatrix_x4_trans(b, Vs + (kk * 16 + (lane & 15)) * ldv + (v0 + vp) * 16 + 8 * (lane >> 4));
+                            mma_bf16_16816(acc[k][2 * vp], ah, b[0], b[1]);
+                            mma_bf16_16816(acc[k][2 * vp + 1], ah, b[2], b[3]);
+                            mma_bf16_16816(acc[k][2 * vp], al, b[0], b[1]);
+                            mma_bf16_16816(acc[k][2 * vp + 1], al, b[2], b[3]);
+                        }
+                    }
                 }
             }
         }
+    }
+    float* U = ws + ((long)blockIdx.x * a.H + h) * d * dv;
 #pragma unroll
-        for (int n = 0; n < 8; n++) {
-            const int c = v0 * 16 + n * 8 + 2 * tq;
-            if (c < dv) {
-                *reinterpret_cast<float2*>(U + (long)(r0 + gq) * dv + c) = make_float2(acc[n][0], acc[n][1]);
-                *reinterpret_cast<float2*>(U + (long)(r0 + gq + 8) * dv + c) = make_float2(acc[n][2], acc[n][3]);
+    for (int k = 0; k < 2; k++) {
+        const int unit = warp + 8 * k;
+        if (unit < d16 * cgroups) {
+            const int r0 = (unit / cgroups) * 16, v0 = (unit % cgroups) * 4;
+#pragma unroll
+            for (int m = 0; m < 8; m++) {
+                const int c = v0 * 16 + m * 8 + 2 * tq;
+                if (c < dv) {
+                    *reinterpret_cast<float2*>(U + (long)(r0 + gq) * dv + c) = make_float2(acc[k][m][0], acc[k][m][1]);
+                    *reinterpret_cast<float2*>(U + (long)(r0 + gq + 8) * dv + c) = make_float2(acc[k][m][2], acc[k][m][3]);
+                }
             }
         }
     }
 }
 
-// grid (blocks of 256 x 8 elements, heads, portions); a thread carries eight neighbouring columns along the portion's chunks, kCarryAhead of whose sums
+// grid (blocks of 128 x 8 elements, heads, portions); a thread carries eight neighbouring columns along the portion's spans, kCarryAhead of whose sums
 // are in flight
 constexpr int kCarryAhead = 4;
-__global__ void __launch_bounds__(256) retention_carry_kernel(const Retention a, float* __restrict__ ws) {
+__global__ void __launch_bounds__(128) retention_carry_kernel(const Retention a, float* __restrict__ ws) {
     const int s = blockIdx.z, h = blockIdx.y;
-    const long n = (long)a.d * a.dv, i = (blockIdx.x * 256L + threadIdx.x) * 8;
+    const long n = (long)a.d * a.dv, i = (blockIdx.x * 128L + threadIdx.x) * 8;
     if (i >= n) return;
-    long tile = 0;
-    for (int k = 0; k < s; k++) tile += (a.seqs[a.seqs_stride + k] + kRetQ - 1) / kRetQ;
-    const int len = a.seqs[a.seqs_stride + s], rd = a.seqs[2 * a.seqs_stride + s], wr = a.seqs[3 * a.seqs_stride + s], chunks = (len + kRetQ - 1) / kRetQ;
-    const float l2 = a.log2_decay[h], full = exp2f((float)kRetQ * l2);
+    long first = 0;
+    for (int k = 0; k < s; k++) first += (a.seqs[a.seqs_stride + k] + kRetSpan - 1) / kRetSpan;
+    const int len = a.seqs[a.seqs_stride + s], rd = a.seqs[2 * a.seqs_stride + s], wr = a.seqs[3 * a.seqs_stride + s], spans = (len + kRetSpan - 1) / kRetSpan;
+    const float l2 = a.log2_decay[h], full = exp2f((float)kRetSpan * l2);
     float4 S0 = make_float4(0.f, 0.f, 0.f, 0.f), S1 = S0;
     if (rd >= 0) {
         const float* p = a.state + (long)rd * a.state_stride + (long)h * n + i;
@@ -320,19 +365,19 @@ __global__ void __launch_bounds__(256) retention_carry_kernel(const Retention a,
         S1 = load4(p + 4);
     }
     const long step = (long)a.H * n;
-    float* U = ws + (tile * a.H + h) * n + i;
-    for (int c0 = 0; c0 < chunks; c0 += kCarryAhead) {
+    float* U = ws + (first * a.H + h) * n + i;
+    for (int c0 = 0; c0 < spans; c0 += kCarryAhead) {
         float4 u[kCarryAhead][2];
 #pragma unroll
         for (int k = 0; k < kCarryAhead; k++)
-            if (c0 + k < chunks) {
+            if (c0 + k < spans) {
                 u[k][0] = load4(U + (c0 + k) * step);
                 u[k][1] = load4(U + (c0 + k) * step + 4);
             }
 #pragma unroll
         for (int k = 0; k < kCarryAhead; k++) {
             const int c = c0 + k;
-            if (c >= chunks) break;
+            if (c >= spans) break;
             uint4 hi, lo;
             split2(S0.x, S0.y, hi.x, lo.x);
             split2(S0.z, S0.w, hi.y, lo.y);
@@ -341,7 +386,7 @@ __global__ void __launch_bounds__(256) retention_carry_kernel(const Retention a,
             uint4* o = reinterpret_cast<uint4*>(U + c * step);
             o[0] = hi;
             o[1] = lo;
-            const float f = c + 1 < chunks ? full : exp2f((float)(len - c * kRetQ) * l2);
+            const float f = c + 1 < spans ? full : exp2f((float)(len - c * kRetSpan) * l2);
             S0 = make_float4(fmaf(f, S0.x, u[k][0].x), fmaf(f, S0.y, u[k][0].y), fmaf(f, S0.z, u[k][0].z), fmaf(f, S0.w, u[k][0].w));
             S1 = make_float4(fmaf(f, S1.x, u[k][1].x), fmaf(f, S1.y, u[k][1].y), fmaf(f, S1.z, u[k][1].z), fmaf(f, S1.w, u[k][1].w));
         }
@@ -353,161 +398,175 @@ __global__ void __launch_bounds__(256) retention_carry_kernel(const Retention a,
     }
 }
 
-// grid (tiles, heads), 4 warps of 16 tokens each.  Shared memory: Q hi, lo | V | the state in pieces of 64 value columns, then K hi, lo
-constexpr int kRetPiece = 64, kRetLdS = kRetPiece + 8;
+// grid (chunks, heads), 8 warps: warp w has the chunk's tokens 16 (w & 3) .. + 15 and one half of the value columns.  Shared memory: Q hi, lo | V |
+// K hi, lo, and before that the state in pieces of 64 key rows | weighted scores hi, lo.  The score tiles of 16 tokens are shared out between their two
+// warps and pass through shared memory.
+constexpr int kRetLdA = kRetQ + 8;
 static size_t ret_out_smem(int d, int dv) {
-    const size_t k = (size_t)2 * kRetQ * (d + 8), s = (size_t)2 * d * kRetLdS;
-    return ((size_t)2 * kRetQ * (d + 8) + (size_t)kRetQ * (dv + 8) + (k > s ? k : s)) * sizeof(__nv_bfloat16);
+    const int wide = d > dv ? d : dv;      // (K rows are d columns, state rows dv)
+    return ((size_t)2 * kRetQ * (d + 8) + (size_t)kRetQ * (dv + 8) + (size_t)2 * kRetQ * (wide + 8) + (size_t)2 * kRetQ * kRetLdA) * sizeof(__nv_bfloat16);
 }
 template <int D16MAX, int DV16MAX>
-__global__ void __launch_bounds__(128, DV16MAX > 4 ? 2 : 3) retention_chunk_out_kernel(const Retention a, const float* __restrict__ ws, __nv_bfloat16* __restrict__ out) {
+__global__ void __launch_bounds__(256, 2) retention_chunk_out_kernel(const Retention a, const float* __restrict__ ws, __nv_bfloat16* __restrict__ out) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    __shared__ int info[3];
-    __shared__ float pw[kRetQ + 1];      // powers of the decay
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gq = lane >> 2, tq = lane & 3, h = blockIdx.y;
+    constexpr int VT = (DV16MAX + 1) / 2;      // 16-column tiles per warp
+    __shared__ int info[4];
+    __shared__ float pw[kRetSpan + 1], row_sq[2][kRetQ];      // powers of the decay; squares of the two column halves
+    const int tid = threadIdx.x, lane = tid & 31, rg = (tid >> 5) & 3, side = tid >> 7, gq = lane >> 2, tq = lane & 3, h = blockIdx.y;
     const int d = a.d, dv = a.dv, d16 = d >> 4, dv16 = dv >> 4, ldk = d + 8, ldv = dv + 8;
-    if (tid == 0) find_chunk(a.seqs, a.seqs_stride, a.n_seqs, blockIdx.x, info);
-    if (tid <= kRetQ) pw[tid] = exp2f((float)tid * a.log2_decay[h]);
+    if (tid == 0) find_chunk(a.seqs, a.seqs_stride, a.n_seqs, blockIdx.x, kRetQ, info);
+    if (tid <= kRetSpan) pw[tid] = exp2f((float)tid * a.log2_decay[h]);
     __syncthreads();
     if (info[0] < 0) return;
-    const int nt = info[2];
+    const int nt = info[2], behind = info[1] % kRetSpan;      // tokens of the span ahead of this chunk
     const long t0 = a.seqs[info[0]] + info[1];
-    const bool has_state = info[1] > 0 || a.seqs[2 * a.seqs_stride + info[0]] >= 0;
+    const bool has_state = info[1] >= kRetSpan || a.seqs[2 * a.seqs_stride + info[0]] >= 0;
     __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(smem_raw);
     __nv_bfloat16* Ql = Qh + kRetQ * ldk;
     __nv_bfloat16* Vs = Ql + kRetQ * ldk;
     __nv_bfloat16* Kh = Vs + kRetQ * ldv;
     __nv_bfloat16* Kl = Kh + kRetQ * ldk;
-    __nv_bfloat16 *Sh = Kh, *Sl = Kh + d * kRetLdS;
+    __nv_bfloat16 *Sh = Kh, *Sl = Kh + kRetQ * ldv;
+    __nv_bfloat16* Ah = Kh + 2 * kRetQ * ((d > dv ? d : dv) + 8);
+    __nv_bfloat16* Al = Ah + kRetQ * kRetLdA;
     const __nv_bfloat16* proj = (const __nv_bfloat16*)a.proj;
-    const __nv_bfloat16* Sg = reinterpret_cast<const __nv_bfloat16*>(ws + ((long)blockIdx.x * a.H + h) * d * dv);
-    auto fetch_state = [&](int c0) {      // columns c0 .. c0 + 63: groups of 8 columns [8 hi | 8 lo]
-        const int groups = min(kRetPiece, dv - c0) >> 3;
-        for (int i = tid; i < d * groups; i += 128) {
+    const __nv_bfloat16* Sg = reinterpret_cast<const __nv_bfloat16*>(ws + (((long)info[3] + info[1] / kRetSpan) * a.H + h) * d * dv);
+    const int groups = dv >> 3;
+    auto fetch_state = [&](int r0) {      // key rows r0 .. r0 + 63, groups of 8 columns [8 hi | 8 lo]
+        const int rows = min(kRetQ, d - r0);
+        for (int i = tid; i < rows * groups; i += 256) {
             const int r = i / groups, g = i - r * groups;
-            const __nv_bfloat16* src = Sg + ((long)r * dv + c0 + g * 8) * 2;
-            cp_async16(Sh + r * kRetLdS + g * 8, src, true);
-            cp_async16(Sl + r * kRetLdS + g * 8, src + 8, true);
+            const __nv_bfloat16* src = Sg + ((long)(r0 + r) * dv + g * 8) * 2;
+            cp_async16(Sh + r * ldv + g * 8, src, true);
+            cp_async16(Sl + r * ldv + g * 8, src + 8, true);
         }
     };
     if (has_state) fetch_state(0);
-    const int vc = dv >> 3;
-    for (int i = tid; i < kRetQ * vc; i += 128) {
-        const int r = i / vc, c = (i - r * vc) * 8;
-        cp_async16(Vs + r * ldv + c, proj + (t0 + (r < nt ? r : 0)) * a.stride + a.v_off + (long)h * dv + c, r < nt);
-    }
     const float2* turn = a.turn + t0 * (a.rot_dims >> 1);
     stage_turned(Qh, Ql, ldk, proj + t0 * a.stride + a.q_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, turn, 1.0f, nullptr);
-    const bool live = warp * 16 < nt;
-    float Y[2 * DV16MAX][4];
+    const bool live = rg * 16 < nt;
+    const int v0 = side * ((dv16 + 1) >> 1), v1 = side ? dv16 : (dv16 + 1) >> 1;      // this warp's column tiles
+    float Y[2 * VT][4];
 #pragma unroll
-    for (int n = 0; n < 2 * DV16MAX; n++)
+    for (int n = 0; n < 2 * VT; n++)
 #pragma unroll
         for (int e = 0; e < 4; e++) Y[n][e] = 0.f;
-    const int qat = (warp * 16 + (lane & 15)) * ldk + 8 * (lane >> 4);
+    const int qat = (rg * 16 + (lane & 15)) * ldk + 8 * (lane >> 4);
+    const int iA = rg * 16 + gq, iB = iA + 8;
     if (has_state) {
-#pragma unroll
-        for (int piece = 0; piece < (DV16MAX + 3) / 4; piece++) {
-            if (piece * kRetPiece < dv) {
-                if (piece) {
-                    __syncthreads();      // the previous piece is consumed
-                    fetch_state(piece * kRetPiece);
-                }
-                cp_async_wait_all();
-                __syncthreads();
-                if (live) {
+        for (int r0 = 0; r0 < d; r0 += kRetQ) {
+            if (r0) {
+                __syncthreads();      // the previous piece is consumed
+                fetch_state(r0);
+            }
+            cp_async_wait_all();
+            __syncthreads();
+            if (live) {
+                const int k16 = min(4, (d - r0) >> 4);
 #pragma unroll 2
-                    for (int kk = 0; kk < d16; kk++) {
-                        uint32_t qh[4], ql[4];
-                        ldmatrix_x4(qh, Qh + qat + kk * 16);
-                        ldmatrix_x4(ql, Ql + qat + kk * 16);
+                for (int kk = 0; kk < k16; kk++) {
+                    uint32_t qh[4], ql[4];
+                    ldmatrix_x4(qh, Qh + qat + r0 + kk * 16);
+                    ldmatrix_x4(ql, Ql + qat + r0 + kk * 16);
 #pragma unroll
-                        for (int vp = 0; vp < 4; vp++) {
-                            const int n = piece * 4 + vp;
-                            if (n < DV16MAX && n < dv16) {
-                                uint32_t bh[4], bl[4];
-                                const int at = (kk * 16 + (lane & 15)) * kRetLdS + vp * 16 + 8 * (lane >> 4);
-                                ldmatrix_x4_trans(bh, Sh + at);
-                                ldmatrix_x4_trans(bl, Sl + at);
-                                mma_bf16_16816(Y[2 * n], qh, bh[0], bh[1]);
-                                mma_bf16_16816(Y[2 * n + 1], qh, bh[2], bh[3]);
-                                mma_bf16_16816(Y[2 * n], ql, bh[0], bh[1]);
-                                mma_bf16_16816(Y[2 * n + 1], ql, bh[2], bh[3]);
-                                mma_bf16_16816(Y[2 * n], qh, bl[0], bl[1]);
-                                mma_bf16_16816(Y[2 * n + 1], qh, bl[2], bl[3]);
-                            }
+                    for (int vp = 0; vp < VT; vp++) {
+                        if (v0 + vp < v1) {
+                            uint32_t bh[4], bl[4];
+                            const int at = (kk * 16 + (lane & 15)) * ldv + (v0 + vp) * 16 + 8 * (lane >> 4);
+                            ldmatrix_x4_trans(bh, Sh + at);
+                            ldmatrix_x4_trans(bl, Sl + at);
+                            mma_bf16_16816(Y[2 * vp], qh, bh[0], bh[1]);
+                            mma_bf16_16816(Y[2 * vp + 1], qh, bh[2], bh[3]);
+                            mma_bf16_16816(Y[2 * vp], ql, bh[0], bh[1]);
+                            mma_bf16_16816(Y[2 * vp + 1], ql, bh[2], bh[3]);
+                            mma_bf16_16816(Y[2 * vp], qh, bl[0], bl[1]);
+                            mma_bf16_16816(Y[2 * vp + 1], qh, bl[2], bl[3]);
                         }
                     }
                 }
             }
         }
-        __syncthreads();      // the last piece is consumed: K goes there
-    }
-    const int iA = warp * 16 + gq, iB = iA + 8;
-    {
-        const float fA = pw[iA + 1], fB = pw[iB + 1];
+        const float fA = pw[min(kRetSpan, behind + iA + 1)], fB = pw[min(kRetSpan, behind + iB + 1)];
 #pragma unroll
-        for (int n = 0; n < 2 * DV16MAX; n++) {
+        for (int n = 0; n < 2 * VT; n++) {
             Y[n][0] *= fA;
             Y[n][1] *= fA;
             Y[n][2] *= fB;
             Y[n][3] *= fB;
         }
     }
-    stage_turned(Kh, Kl, ldk, proj + t0 * a.stride + a.k_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, turn, a.k_scale, nullptr);
-    cp_async_wait_all();
-    __syncthreads();
-    if (!live) return;
-    for (int np = 0; np <= warp; np++) {      // 16 keys per step, up to the warp's own tokens
-        float G[2][4];
+    // the span's keys: the 64 tokens ahead of this chunk when it is the second of its span, then the chunk's own
+    for (int back = behind; back >= 0; back -= kRetQ) {
+        const long t1 = t0 - back;
+        const int kt = back ? kRetQ : nt;
+        __syncthreads();      // the state's last piece, or the keys and scores ahead, are consumed
+        fetch_rows(Vs, ldv, proj + t1 * a.stride + a.v_off + (long)h * dv, a.stride, kt, dv);
+        stage_turned(Kh, Kl, ldk, proj + t1 * a.stride + a.k_off + (long)h * d, a.stride, kt, d, a.rot_dims, a.layout, a.turn + t1 * (a.rot_dims >> 1), a.k_scale, nullptr);
+        cp_async_wait_all();
+        __syncthreads();
+        const int tiles = back ? kRetQ / 16 : rg + 1;      // key tiles of 16 that the warp's tokens see
+        if (live) {
+            for (int np = side; np < tiles; np += 2) {
+                float G[2][4];
 #pragma unroll
-        for (int n = 0; n < 2; n++)
+                for (int n = 0; n < 2; n++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) G[n][e] = 0.f;
-        const int kat = (np * 16 + (lane & 7) + 8 * (lane >> 4)) * ldk + 8 * ((lane >> 3) & 1);
+                    for (int e = 0; e < 4; e++) G[n][e] = 0.f;
+                const int kat = (np * 16 + (lane & 7) + 8 * (lane >> 4)) * ldk + 8 * ((lane >> 3) & 1);
 #pragma unroll
-        for (int kk = 0; kk < D16MAX; kk++) {
-            if (kk < d16) {
-                uint32_t qh[4], ql[4], kh[4], kl[4];
-                ldmatrix_x4(qh, Qh + qat + kk * 16);
-                ldmatrix_x4(ql, Ql + qat + kk * 16);
-                ldmatrix_x4(kh, Kh + kat + kk * 16);
-                ldmatrix_x4(kl, Kl + kat + kk * 16);
-                mma_bf16_16816(G[0], qh, kh[0], kh[1]);
-                mma_bf16_16816(G[1], qh, kh[2], kh[3]);
-                mma_bf16_16816(G[0], ql, kh[0], kh[1]);
-                mma_bf16_16816(G[1], ql, kh[2], kh[3]);
-                mma_bf16_16816(G[0], qh, kl[0], kl[1]);
-                mma_bf16_16816(G[1], qh, kl[2], kl[3]);
+                for (int kk = 0; kk < D16MAX; kk++) {
+                    if (kk < d16) {
+                        uint32_t qh[4], ql[4], kh[4], kl[4];
+                        ldmatrix_x4(qh, Qh + qat + kk * 16);
+                        ldmatrix_x4(ql, Ql + qat + kk * 16);
+                        ldmatrix_x4(kh, Kh + kat + kk * 16);
+                        ldmatrix_x4(kl, Kl + kat + kk * 16);
+                        mma_bf16_16816(G[0], qh, kh[0], kh[1]);
+                        mma_bf16_16816(G[1], qh, kh[2], kh[3]);
+                        mma_bf16_16816(G[0], ql, kh[0], kh[1]);
+                        mma_bf16_16816(G[1], ql, kh[2], kh[3]);
+                        mma_bf16_16816(G[0], qh, kl[0], kl[1]);
+                        mma_bf16_16816(G[1], qh, kl[2], kl[3]);
+                    }
+                }
+#pragma unroll
+                for (int n = 0; n < 2; n++) {
+                    const int j = np * 16 + n * 8 + 2 * tq;
+#pragma unroll
+                    for (int e = 0; e < 4; e += 2) {
+                        const int i = back + (e ? iB : iA);
+                        uint32_t hi, lo;
+                        split2(i >= j ? G[n][e] * pw[i - j] : 0.f, i > j ? G[n][e + 1] * pw[max(0, i - j - 1)] : 0.f, hi, lo);
+                        *reinterpret_cast<uint32_t*>(Ah + (e ? iB : iA) * kRetLdA + j) = hi;
+                        *reinterpret_cast<uint32_t*>(Al + (e ? iB : iA) * kRetLdA + j) = lo;
+                    }
+                }
             }
         }
+        __syncthreads();
+        if (live) {
+            for (int np = 0; np < tiles; np++) {
+                uint32_t gh[4], gl[4];
+                const int at = (rg * 16 + (lane & 15)) * kRetLdA + np * 16 + 8 * (lane >> 4);
+                ldmatrix_x4(gh, Ah + at);
+                ldmatrix_x4(gl, Al + at);
 #pragma unroll
-        for (int n = 0; n < 2; n++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int back = (e < 2 ? iA : iB) - (np * 16 + n * 8 + 2 * tq + (e & 1));
-                G[n][e] = back >= 0 ? G[n][e] * pw[back] : 0.f;
-            }
-        uint32_t gh[4], gl[4];
-        split2(G[0][0], G[0][1], gh[0], gl[0]);
-        split2(G[0][2], G[0][3], gh[1], gl[1]);
-        split2(G[1][0], G[1][1], gh[2], gl[2]);
-        split2(G[1][2], G[1][3], gh[3], gl[3]);
-#pragma unroll
-        for (int vp = 0; vp < DV16MAX; vp++) {
-            if (vp < dv16) {
-                uint32_t b[4];
-                ldmatrix_x4_trans(b, Vs + (np * 16 + (lane & 15)) * ldv + vp * 16 + 8 * (lane >> 4));
-                mma_bf16_16816(Y[2 * vp], gh, b[0], b[1]);
-                mma_bf16_16816(Y[2 * vp + 1], gh, b[2], b[3]);
-                mma_bf16_16816(Y[2 * vp], gl, b[0], b[1]);
-                mma_bf16_16816(Y[2 * vp + 1], gl, b[2], b[3]);
+                for (int vp = 0; vp < VT; vp++) {
+                    if (v0 + vp < v1) {
+                        uint32_t b[4];
+                        ldmatrix_x4_trans(b, Vs + (np * 16 + (lane & 15)) * ldv + (v0 + vp) * 16 + 8 * (lane >> 4));
+                        mma_bf16_16816(Y[2 * vp], gh, b[0], b[1]);
+                        mma_bf16_16816(Y[2 * vp + 1], gh, b[2], b[3]);
+                        mma_bf16_16816(Y[2 * vp], gl, b[0], b[1]);
+                        mma_bf16_16816(Y[2 * vp + 1], gl, b[2], b[3]);
+                    }
+                }
             }
         }
     }
-    float sA = 0.f, sB = 0.f;      // (columns at or beyond dv hold zeros)
+    float sA = 0.f, sB = 0.f;      // (tiles beyond the warp's own hold zeros)
 #pragma unroll
-    for (int n = 0; n < 2 * DV16MAX; n++) {
+    for (int n = 0; n < 2 * VT; n++) {
         sA += Y[n][0] * Y[n][0] + Y[n][1] * Y[n][1];
         sB += Y[n][2] * Y[n][2] + Y[n][3] * Y[n][3];
     }
@@ -515,19 +574,25 @@ __global__ void __launch_bounds__(128, DV16MAX > 4 ? 2 : 3) retention_chunk_out_
     sA += __shfl_xor_sync(0xffffffffu, sA, 2);
     sB += __shfl_xor_sync(0xffffffffu, sB, 1);
     sB += __shfl_xor_sync(0xffffffffu, sB, 2);
-    const float inv[2] = {1.0f / sqrtf(sA / (float)dv + a.eps), 1.0f / sqrtf(sB / (float)dv + a.eps)};
+    if (tq == 0) {
+        row_sq[side][iA] = sA;
+        row_sq[side][iB] = sB;
+    }
+    __syncthreads();
 #pragma unroll
     for (int r = 0; r < 2; r++) {
         const int i = r ? iB : iA;
         if (i >= nt) continue;
+        const float inv = 1.0f / sqrtf((row_sq[0][i] + row_sq[1][i]) / (float)dv + a.eps);
         const __nv_bfloat16* g = proj + (t0 + i) * a.stride + a.g_off + (long)h * dv;
         __nv_bfloat16* o = out + ((t0 + i) * a.H + h) * (long)dv;
 #pragma unroll
-        for (int n = 0; n < 2 * DV16MAX; n++) {
-            const int c = n * 8 + 2 * tq;
-            if (c < dv) {
+        for (int n = 0; n < 2 * VT; n++) {
+            const int c = v0 * 16 + n * 8 + 2 * tq;
+            if (c < v1 * 16) {
                 const uint32_t u = *reinterpret_cast<const uint32_t*>(g + c);
-                *reinterpret_cast<uint32_t*>(o + c) = pack_bf16(Y[n][2 * r] * inv[r] * act_silu(__uint_as_float(u << 16)), Y[n][2 * r + 1] * inv[r] * act_silu(__uint_as_float(u & 0xffff0000u)));
+                *reinterpret_cast<uint32_t*>(o + c) =
+                    pack_bf16(Y[n][2 * r] * inv * silu_for<__nv_bfloat16>(__uint_as_float(u << 16)), Y[n][2 * r + 1] * inv * silu_for<__nv_bfloat16>(__uint_as_float(u & 0xffff0000u)));
             }
         }
     }
@@ -695,9 +760,9 @@ extern "C" int ktb200_retention_scan(const ktb200_retention_params* c, float* o,
 extern "C" int ktb200_retention_chunk_supported(int dim, int vdim, int dtype) {
     return dtype == KTB200_TYPE_BF16 && dim > 0 && vdim > 0 && dim % 16 == 0 && vdim % 16 == 0 && dim <= 128 && vdim <= 128;
 }
-static long ret_tiles(int n_tokens, int n_seqs) { return n_tokens / kRetQ + n_seqs; }      // (an upper bound: whole chunks and one partial per portion)
+static long ret_tiles(int n_tokens, int n_seqs, int per) { return n_tokens / per + n_seqs; }      // (an upper bound: whole tiles and one partial per portion)
 extern "C" size_t ktb200_retention_chunk_workspace(int heads, int dim, int vdim, int n_tokens, int n_seqs) {
-    return (size_t)ret_tiles(n_tokens, n_seqs) * heads * dim * vdim * sizeof(float);
+    return (size_t)ret_tiles(n_tokens, n_seqs, kRetSpan) * heads * dim * vdim * sizeof(float);
 }
 
 extern "C" int ktb200_retention_chunk(const ktb200_retention_params* c, void* out, int n_tokens, void* workspace, size_t workspace_bytes, int dtype, void* stream) {
@@ -711,18 +776,18 @@ extern "C" int ktb200_retention_chunk(const ktb200_retention_params* c, void* ou
     const Retention a = ret_args(c);
     float* ws = (float*)workspace;
     cudaStream_t st = (cudaStream_t)stream;
-    const dim3 grid((unsigned)ret_tiles(n_tokens, c->n_seqs), c->heads);
+    const dim3 spans((unsigned)ret_tiles(n_tokens, c->n_seqs, kRetSpan), c->heads), chunks((unsigned)ret_tiles(n_tokens, c->n_seqs, kRetQ), c->heads);
     const size_t s1 = ((size_t)2 * kRetQ * (c->dim + 8) + (size_t)kRetQ * (c->vdim + 8)) * sizeof(__nv_bfloat16);
     GRANT_SMEM(retention_chunk_state_kernel, s1);
-    retention_chunk_state_kernel<<<grid, 256, s1, st>>>(a, ws);
+    retention_chunk_state_kernel<<<spans, 256, s1, st>>>(a, ws);
     KTB_LAUNCH_CHECK();
-    retention_carry_kernel<<<dim3((c->dim * c->vdim / 8 + 255) / 256, c->heads, c->n_seqs), 256, 0, st>>>(a, ws);
+    retention_carry_kernel<<<dim3((c->dim * c->vdim / 8 + 127) / 128, c->heads, c->n_seqs), 128, 0, st>>>(a, ws);
     KTB_LAUNCH_CHECK();
     const size_t s3 = ret_out_smem(c->dim, c->vdim);
 #define OUT_LAUNCH(DK, DV)                                                                                      \
     do {                                                                                                        \
         GRANT_SMEM((retention_chunk_out_kernel<DK, DV>), s3);                                                   \
-        retention_chunk_out_kernel<DK, DV><<<grid, 128, s3, st>>>(a, ws, (__nv_bfloat16*)out);                  \
+        retention_chunk_out_kernel<DK, DV><<<chunks, 256, s3, st>>>(a, ws, (__nv_bfloat16*)out);                  \
     } while (0)
     if (c->dim <= 64 && c->vdim <= 64) OUT_LAUNCH(4, 4);
     else if (c->vdim <= 64) OUT_LAUNCH(8, 4);

@@ -125,6 +125,15 @@ template <typename T> struct ConvRows {
     }
 };
 
+// 2^x, and SiLU to the precision that storage type T keeps: bf16 results take the base-2 exponential and the fast quotient
+__device__ __forceinline__ float exp2_approx(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+template <typename T> __device__ __forceinline__ float silu_for(float z) { return act_silu(z); }
+template <> __device__ __forceinline__ float silu_for<__nv_bfloat16>(float z) { return __fdividef(z, 1.0f + exp2_approx(-1.4426950408889634f * z)); }
+
 // Gated feed-forward activations, fp32: what becomes of a (gate, up) pair of pre-activations.
 //   kActSilu        silu(g) * u
 //   kActGeluTanh    gelu(g) * u, gelu in its tanh form

@@ -26,7 +26,7 @@ __device__ __forceinline__ float ssd_softplus(float x) { return x > 20.f ? x : l
 // ------------------------------------------------------------------------------------------------ filter + SiLU over prompt portions
 // grid (token blocks, channel blocks); a thread owns VEC consecutive channels and runs over `tile` tokens (kConvTokens; 1 when every portion is one token) with the last TAPS - 1 inputs
 // in registers (TAPS = 0: any number of taps, one channel, inputs read again per token).
-constexpr int kConvTokens = 16, kConvThreads = 128;
+constexpr int kConvTokens = 16, kConvThreads = 128, kConvAhead = 4;
 template <typename T, int VEC> __device__ __forceinline__ void load_vec(float (&v)[VEC], const T* p) {
     if (VEC == 4) {
         const float4 u = load4(p);
@@ -52,46 +52,56 @@ __global__ void __launch_bounds__(kConvThreads) conv_silu_kernel(const T* __rest
             for (int j = 0; j < TAPS; j++) wv[j][e] = to_f(w[(long)(c + e) * TAPS + j]);
     }
     int cur = -1, start = 0, len = 0, rd = -1, wr = -1;
-    for (int t = t0; t < t1; t++) {
-        const int s = seq_of[t];
-        const bool fresh = s != cur;      // another portion, or this thread's first token: fetch the inputs ahead of it
-        if (fresh) {
-            cur = s;
-            start = seqs[s]; len = seqs[seqs_stride + s]; rd = seqs[2 * seqs_stride + s]; wr = seqs[3 * seqs_stride + s];
+    for (int tb = t0; tb < t1; tb += kConvAhead) {
+        float in_rows[kConvAhead][VEC];      // the next tokens' inputs, asked for together
+        if (TAPS > 0) {
+#pragma unroll
+            for (int q = 0; q < kConvAhead; q++)
+                if (tb + q < t1) load_vec<T, VEC>(in_rows[q], in + (long)(tb + q) * stride + c);
         }
-        const int off = t - start;
-        const ConvRows<T> cv{in + (long)start * stride, stride, w, TAPS > 0 ? TAPS : taps_rt, C, rd >= 0 ? state + (long)rd * state_stride + conv_off : nullptr,
-                             wr >= 0 ? state + (long)wr * state_stride + conv_off : nullptr, off};
-        if (TAPS == 0) {
-            out[(long)t * C + c] = from_f<T>(act_silu(cv.value(c, c) + bv[0]));
-            if (off == len - 1 && wr >= 0) cv.store_tail(c, c);
-            continue;
-        }
-        if (fresh && TAPS > 1) {
 #pragma unroll
-            for (int j = 0; j < TAPS - 1; j++)
+        for (int q = 0; q < kConvAhead; q++) {
+            const int t = tb + q;
+            if (t >= t1) break;
+            const int s = seq_of[t];
+            const bool fresh = s != cur;      // another portion, or this thread's first token: fetch the inputs ahead of it
+            if (fresh) {
+                cur = s;
+                start = seqs[s]; len = seqs[seqs_stride + s]; rd = seqs[2 * seqs_stride + s]; wr = seqs[3 * seqs_stride + s];
+            }
+            const int off = t - start;
+            const ConvRows<T> cv{in + (long)start * stride, stride, w, TAPS > 0 ? TAPS : taps_rt, C, rd >= 0 ? state + (long)rd * state_stride + conv_off : nullptr,
+                                 wr >= 0 ? state + (long)wr * state_stride + conv_off : nullptr, off};
+            if (TAPS == 0) {
+                out[(long)t * C + c] = from_f<T>(silu_for<T>(cv.value(c, c) + bv[0]));
+                if (off == len - 1 && wr >= 0) cv.store_tail(c, c);
+                continue;
+            }
+            if (fresh && TAPS > 1) {
 #pragma unroll
-                for (int e = 0; e < VEC; e++) win[j][e] = cv.input(off - (TAPS - 1) + j, c + e, c + e);
-        }
-        float u[VEC], y[VEC];
-        load_vec<T, VEC>(u, in + (long)t * stride + c);
+                for (int j = 0; j < TAPS - 1; j++)
 #pragma unroll
-        for (int e = 0; e < VEC; e++) {
-            float a = 0.f;
+                    for (int e = 0; e < VEC; e++) win[j][e] = cv.input(off - (TAPS - 1) + j, c + e, c + e);
+            }
+            float y[VEC];
 #pragma unroll
-            for (int j = 0; j < TAPS - 1; j++) a = fmaf(wv[j][e], win[j][e], a);
-            y[e] = act_silu(fmaf(wv[TAPS - 1 > 0 ? TAPS - 1 : 0][e], u[e], a) + bv[e]);
+            for (int e = 0; e < VEC; e++) {
+                float a = 0.f;
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS - 1; j++) win[j][e] = win[j + 1][e];
-            if (TAPS > 1) win[BACK - 1][e] = u[e];
-        }
-        if (VEC == 4) store4(out + (long)t * C + c, make_float4(y[0], y[VEC > 1 ? 1 : 0], y[VEC > 2 ? 2 : 0], y[VEC > 3 ? 3 : 0]));
-        else out[(long)t * C + c] = from_f<T>(y[0]);
-        if (TAPS > 1 && off == len - 1 && wr >= 0) {
+                for (int j = 0; j < TAPS - 1; j++) a = fmaf(wv[j][e], win[j][e], a);
+                y[e] = silu_for<T>(fmaf(wv[TAPS - 1 > 0 ? TAPS - 1 : 0][e], in_rows[q][e], a) + bv[e]);
 #pragma unroll
-            for (int j = 0; j < TAPS - 1; j++)
+                for (int j = 0; j + 1 < TAPS - 1; j++) win[j][e] = win[j + 1][e];
+                if (TAPS > 1) win[BACK - 1][e] = in_rows[q][e];
+            }
+            if (VEC == 4) store4(out + (long)t * C + c, make_float4(y[0], y[VEC > 1 ? 1 : 0], y[VEC > 2 ? 2 : 0], y[VEC > 3 ? 3 : 0]));
+            else out[(long)t * C + c] = from_f<T>(y[0]);
+            if (TAPS > 1 && off == len - 1 && wr >= 0) {
 #pragma unroll
-                for (int e = 0; e < VEC; e++) cv.after[(long)j * C + c + e] = win[j][e];
+                for (int j = 0; j < TAPS - 1; j++)
+#pragma unroll
+                    for (int e = 0; e < VEC; e++) cv.after[(long)j * C + c + e] = win[j][e];
+            }
         }
     }
 }

@@ -237,9 +237,12 @@ class KSigmoidTopKGate(nn.Module):
 class KGroupedSoftmaxGate(nn.Module):
     """Soft-max scores s = softmax(W x) in fp32 over every output; outputs are CHOSEN by s + correction among those of the `keep_groups` groups
     (of neighbours) whose largest choice score is largest, every other one counting as minus infinity; the WEIGHTS are the chosen outputs' s
-    times `out_scale`, not normalised: the router kernel's `scoring = softmax, topk_method = biased_group_max` case.  As for
-    KGroupedSigmoidGate, decode-sized batches run the one-launch kernel, and batches from `gemm_min_tokens` tokens an fp32 library GEMM (TF32
-    off) and `ktb200_moe_gate_select`."""
+    times `out_scale`, not normalised: the router kernel's `scoring = softmax, topk_method = biased_group_max` case.
+
+    Logits: for bf16 activations and router weights that are bf16 numbers (as checkpoints ship them) every product is exact in fp32, and the
+    library's tensor-core GEMM with fp32 accumulation and fp32 output makes the fp32 logits at any batch size.  Otherwise, as for
+    KGroupedSigmoidGate: decode-sized batches run the one-launch kernel, batches from `gemm_min_tokens` tokens an fp32 library GEMM (TF32 off).
+    The selection behind a GEMM is `ktb200_moe_gate_select`."""
 
     gemm_min_tokens = 48
 
@@ -252,10 +255,16 @@ class KGroupedSoftmaxGate(nn.Module):
         self.width, self.outputs, self.top, self.groups, self.keep_groups, self.out_scale = width, outputs, top, groups, keep_groups, float(out_scale)
         self.weight = nn.Parameter(torch.empty((outputs, width), dtype=torch.float32, device=device), requires_grad=False)
         self.correction = nn.Parameter(torch.zeros(outputs, dtype=torch.float32, device=device), requires_grad=False)
+        self.weight_bf16 = None      # the same numbers in bf16, when they are bf16 numbers
 
     def load(self, loader, key: str, correction_key: str):
         self.weight.data.copy_(loader.load_tensor(key, "cpu").float())
         self.correction.data.copy_(loader.load_tensor(correction_key, "cpu").float())
+        self.find_bf16()
+
+    def find_bf16(self):
+        b = self.weight.data.bfloat16()
+        self.weight_bf16 = b if self.width % 8 == 0 and bool((b.float() == self.weight.data).all()) else None
 
     def forward(self, x: torch.Tensor):
         n = x.shape[0]
@@ -264,7 +273,10 @@ class KGroupedSoftmaxGate(nn.Module):
         cfg = native.GateConfig(self.outputs, self.width, self.top, self.groups, self.keep_groups, _SCORING["softmax"], _TOPK["biased_group_max"], 0, self.out_scale,
                                 self.weight.data_ptr(), self.correction.data_ptr(), TORCH_TO_GGML_HIDDEN[x.dtype])
         st = torch.cuda.current_stream(x.device).cuda_stream
-        if n >= self.gemm_min_tokens or self.width % 4:
+        if x.dtype == torch.bfloat16 and self.weight_bf16 is not None:
+            logits = torch.mm(x, self.weight_bf16.t(), out_dtype=torch.float32)
+            native.check_seq(native.seq_lib().ktb200_moe_gate_select(C.byref(cfg), n, logits.data_ptr(), idx.data_ptr(), wt.data_ptr(), st))
+        elif n >= self.gemm_min_tokens or self.width % 4:
             logits = nn.functional.linear(x.float(), self.weight)
             native.check_seq(native.seq_lib().ktb200_moe_gate_select(C.byref(cfg), n, logits.data_ptr(), idx.data_ptr(), wt.data_ptr(), st))
         else:

@@ -168,6 +168,11 @@ def settle_lipadra(model):
             p.data.sub_(3.0)
         elif last == "a":
             p.data.copy_(-torch.arange(1, p.shape[1] + 1, device=p.device, dtype=torch.float32).expand_as(p))
+        elif pname.endswith("router.weight"):      # as a bf16 checkpoint ships it
+            p.data.copy_(p.data.bfloat16().float())
+    for layer in model.owned.values():
+        if layer.mlp is not None:
+            layer.mlp.router.find_bf16()
     return model
 
 
@@ -1238,13 +1243,16 @@ def lipadra_kernel_leg(flush, peak_gbs, peak_tf):
     # ---- router: grouped soft-max top 8 of 256 + 64  vs  grouped sigmoid
     E = 320
     mine, theirs = KGroupedSoftmaxGate(D, E, top, 8, 4, 2.0), KGroupedSigmoidGate(D, E, top, 8, 4, 2.0)
-    mine.weight.data.copy_(rn(E, D, dt=f32) * D ** -0.5)
+    mine.weight.data.copy_((rn(E, D, dt=f32) * D ** -0.5).bfloat16().float())
     theirs.weight.data.copy_(mine.weight.data)
     for T in (1, 8, 2048):
         x, nb = rn(T, D), E * D * 4 + T * D * 2
-        small = T < mine.gemm_min_tokens
-        K.add("gate_kernel (soft-max, biased group max)" if small else "fp32 GEMM + gate_select_kernel", f"T={T} outputs={E} width={D} top={top}", timed(lambda: mine(x), flush), nb,
-              peer=K.measure("the same, grouped sigmoid", timed(lambda: theirs(x), flush), nb))
+        peer = K.measure("grouped sigmoid: " + ("gate_kernel" if T < mine.gemm_min_tokens else "fp32 GEMM + gate_select_kernel"), timed(lambda: theirs(x), flush), nb)
+        mine.weight_bf16 = None
+        K.add("gate_kernel (soft-max, biased group max)" if T < mine.gemm_min_tokens else "fp32 GEMM + gate_select_kernel", f"T={T} outputs={E} width={D} top={top}", timed(lambda: mine(x), flush),
+              nb, peer=peer)
+        mine.find_bf16()
+        K.add("bf16 GEMM with fp32 sums + gate_select_kernel", f"T={T} outputs={E} width={D} top={top}", timed(lambda: mine(x), flush), E * D * 2 + T * D * 2, peer=peer)
 
     # ---- experts: a fifth of the choices identity experts  vs  every choice an expert
     E, ff = 32, 2048
