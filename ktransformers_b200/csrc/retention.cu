@@ -164,13 +164,14 @@ __global__ void __launch_bounds__(256, 2) retention_scan_kernel(const Retention 
 
 // ------------------------------------------------------------------------------------------------ chunks on the tensor cores (bf16)
 // With fixed decays the states along a portion follow from one pass over the sums of its parts, so all parts of all portions and heads run at once:
-//   1. chunk_state   spans of 128 tokens:  U_s = sum_j decay^(n - 1 - j) k_j v_j^T                        (n tokens in the span)
+//   1. chunk_state   turns q and k, and per span of 128 tokens:  U_s = sum_j decay^(n - 1 - j) k_j v_j^T                        (n tokens in the span)
 //   2. carry         S_s = the state ahead of span s: S_(s+1) = decay^n S_s + U_s, elementwise along the portion's spans; S_s replaces U_s
 //   3. chunk_out     chunks of 64 tokens, c tokens behind their span's start (0 or 64):
 //                    o_i = decay^(c + i + 1) S_s^T q_i + sum over the span's keys j up to i of decay^(i - j) (q_i . k_j) v_j, then norm and gate
 // m16n8k16 bf16 MMAs with fp32 accumulators; v is bf16 as it comes, every other operand (turned q and k, weighted k and scores, S) enters as the
 // sum of two bf16 terms hi + lo (about 16 bits of mantissa), products of two such operands as hi hi + hi lo + lo hi.
-// Workspace per (span, head): dim * vdim fp32 of U, then in the same bytes S as groups of 8 columns [8 hi | 8 lo].
+// Workspace: per (span, head) dim * vdim fp32 of U, then in the same bytes S as groups of 8 columns [8 hi | 8 lo]; per (token, head) the turned q
+// and the turned and scaled k as rows [dim hi | dim lo].
 constexpr int kRetQ = 64, kRetSpan = 2 * kRetQ;
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(a, b);
@@ -193,22 +194,14 @@ __device__ __forceinline__ void find_chunk(const int* __restrict__ seqs, int str
         spans += (len + kRetSpan - 1) / kRetSpan;
     }
 }
-// Stage nt rows of a head (first row `src`, rows `stride` apart; the rest of the 64 rows zeros), turned and times scale * row_w[row], as two bf16 planes
-// [64][ld].  Where the pair halves are runs of four columns: four pairs at a time, the loads of four such units in flight together.
-__device__ __forceinline__ void stage_turned(__nv_bfloat16* hi, __nv_bfloat16* lo, int ld, const __nv_bfloat16* __restrict__ src, long stride, int nt, int d, int rot_dims, int layout,
-                                             const float2* __restrict__ turn, float scale, const float* row_w) {
+// The nt rows of a head (first row `src`, rows `stride` apart; up to 64 rows as zeros behind them), turned: sink(row, column, four neighbouring columns).
+// Where the pair halves are runs of four columns: four pairs at a time, the loads of AHEAD such units in flight together.
+template <int AHEAD, class Sink>
+__device__ __forceinline__ void turned_rows(const __nv_bfloat16* __restrict__ src, long stride, int nt, int d, int rot_dims, int layout, const float2* __restrict__ turn, Sink sink) {
     const int half = rot_dims >> 1;
-    const bool wide = layout == kRotHalves && half % 4 == 0 && rot_dims > 0;
-    auto put = [&](int at, float4 v, float w) {
-        uint32_t h0, l0, h1, l1;
-        split2(v.x * w, v.y * w, h0, l0);
-        split2(v.z * w, v.w * w, h1, l1);
-        *reinterpret_cast<uint2*>(hi + at) = make_uint2(h0, h1);
-        *reinterpret_cast<uint2*>(lo + at) = make_uint2(l0, l1);
-    };
-    if (wide) {
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (layout == kRotHalves && half % 4 == 0 && rot_dims > 0) {
         const int pairs = half / 4, per = pairs + (d - rot_dims) / 4;      // units of a row: four pairs, or four columns that pass (d - rot_dims is a multiple of 4 here)
-        constexpr int AHEAD = 4;
         for (int i0 = threadIdx.x; i0 < kRetQ * per; i0 += AHEAD * blockDim.x) {
             uint2 p[AHEAD], q[AHEAD];
             float4 c0[AHEAD], c1[AHEAD];
@@ -216,6 +209,7 @@ __device__ __forceinline__ void stage_turned(__nv_bfloat16* hi, __nv_bfloat16* l
             for (int k = 0; k < AHEAD; k++) {
                 const int i = i0 + k * blockDim.x, r = i / per, u = i - r * per;
                 p[k] = q[k] = make_uint2(0, 0);
+                c0[k] = c1[k] = zero;
                 if (r < nt && i < kRetQ * per) {
                     const __nv_bfloat16* row = src + (long)r * stride;
                     if (u < pairs) {
@@ -232,36 +226,32 @@ __device__ __forceinline__ void stage_turned(__nv_bfloat16* hi, __nv_bfloat16* l
             for (int k = 0; k < AHEAD; k++) {
                 const int i = i0 + k * blockDim.x, r = i / per, u = i - r * per;
                 if (i >= kRetQ * per) break;
-                const bool in = r < nt;
-                const float w = in ? (row_w ? scale * row_w[r] : scale) : 0.f;
                 const float4 a = make_float4(__uint_as_float(p[k].x << 16), __uint_as_float(p[k].x & 0xffff0000u), __uint_as_float(p[k].y << 16), __uint_as_float(p[k].y & 0xffff0000u));
                 if (u < pairs) {
                     const float4 b = make_float4(__uint_as_float(q[k].x << 16), __uint_as_float(q[k].x & 0xffff0000u), __uint_as_float(q[k].y << 16), __uint_as_float(q[k].y & 0xffff0000u));
-                    float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
-                    if (in) {
-                        x = make_float4(a.x * c0[k].x - b.x * c0[k].y, a.y * c0[k].z - b.y * c0[k].w, a.z * c1[k].x - b.z * c1[k].y, a.w * c1[k].z - b.w * c1[k].w);
-                        y = make_float4(b.x * c0[k].x + a.x * c0[k].y, b.y * c0[k].z + a.y * c0[k].w, b.z * c1[k].x + a.z * c1[k].y, b.w * c1[k].z + a.w * c1[k].w);
-                    }
-                    put(r * ld + u * 4, x, w);
-                    put(r * ld + half + u * 4, y, w);
+                    sink(r, u * 4, make_float4(a.x * c0[k].x - b.x * c0[k].y, a.y * c0[k].z - b.y * c0[k].w, a.z * c1[k].x - b.z * c1[k].y, a.w * c1[k].z - b.w * c1[k].w));
+                    sink(r, half + u * 4, make_float4(b.x * c0[k].x + a.x * c0[k].y, b.y * c0[k].z + a.y * c0[k].w, b.z * c1[k].x + a.z * c1[k].y, b.w * c1[k].z + a.w * c1[k].w));
                 } else {
-                    put(r * ld + rot_dims + (u - pairs) * 4, a, w);
+                    sink(r, rot_dims + (u - pairs) * 4, a);
                 }
             }
         }
         return;
     }
-    for (int i = threadIdx.x; i < kRetQ * (d / 2); i += blockDim.x) {
-        const int r = i / (d / 2), c = (i - r * (d / 2)) * 2;
-        uint32_t h = 0, l = 0;
-        if (r < nt) {
-            const float w = row_w ? scale * row_w[r] : scale;
-            const __nv_bfloat16* row = src + (long)r * stride;
-            split2(turned(row, c, rot_dims, layout, turn + (long)r * half) * w, turned(row, c + 1, rot_dims, layout, turn + (long)r * half) * w, h, l);
-        }
-        *reinterpret_cast<uint32_t*>(hi + r * ld + c) = h;
-        *reinterpret_cast<uint32_t*>(lo + r * ld + c) = l;
+    for (int i = threadIdx.x; i < kRetQ * (d / 4); i += blockDim.x) {
+        const int r = i / (d / 4), c = (i - r * (d / 4)) * 4;
+        const __nv_bfloat16* row = src + (long)r * stride;
+        const float2* tr = turn + (long)r * half;
+        sink(r, c, r < nt ? make_float4(turned(row, c, rot_dims, layout, tr), turned(row, c + 1, rot_dims, layout, tr), turned(row, c + 2, rot_dims, layout, tr), turned(row, c + 3, rot_dims, layout, tr)) : zero);
     }
+}
+// four columns times w as two bf16 terms, the low ones `low` elements behind the high ones
+__device__ __forceinline__ void put_split(__nv_bfloat16* hi, int low, float4 v, float w) {
+    uint32_t h0, l0, h1, l1;
+    split2(v.x * w, v.y * w, h0, l0);
+    split2(v.z * w, v.w * w, h1, l1);
+    *reinterpret_cast<uint2*>(hi) = make_uint2(h0, h1);
+    *reinterpret_cast<uint2*>(hi + low) = make_uint2(l0, l1);
 }
 __device__ __forceinline__ void fetch_rows(__nv_bfloat16* dst, int ld, const __nv_bfloat16* __restrict__ src, long stride, int nt, int n) {      // nt of 64 rows of n columns, the rest zeros
     const int pieces = n >> 3;
@@ -272,7 +262,7 @@ __device__ __forceinline__ void fetch_rows(__nv_bfloat16* dst, int ld, const __n
 }
 
 // grid (spans, heads), 8 warps; a unit of work is 16 key rows x up to 64 value columns of U, at most two per warp
-__global__ void __launch_bounds__(256, 2) retention_chunk_state_kernel(const Retention a, float* __restrict__ ws) {
+__global__ void __launch_bounds__(256, 2) retention_chunk_state_kernel(const Retention a, float* __restrict__ ws, __nv_bfloat16* __restrict__ q_rows, __nv_bfloat16* __restrict__ k_rows) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ int info[4];
     __shared__ float row_w[kRetSpan];
@@ -301,7 +291,15 @@ __global__ void __launch_bounds__(256, 2) retention_chunk_state_kernel(const Ret
         const int nt = min(kRetQ, n - part * kRetQ), k16 = (nt + 15) >> 4;
         __syncthreads();      // row_w is there; the first half is consumed
         fetch_rows(Vs, ldv, proj + t1 * a.stride + a.v_off + (long)h * dv, a.stride, nt, dv);
-        stage_turned(Kh, Kl, ldk, proj + t1 * a.stride + a.k_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, a.turn + t1 * (a.rot_dims >> 1), a.k_scale, row_w + part * kRetQ);
+        const float2* turn = a.turn + t1 * (a.rot_dims >> 1);
+        const __nv_bfloat16* rows = proj + t1 * a.stride + (long)h * d;
+        turned_rows<2>(rows + a.k_off, a.stride, nt, d, a.rot_dims, a.layout, turn, [&](int r, int c, float4 v) {
+            if (r < nt) put_split(k_rows + ((t1 + r) * a.H + h) * (2L * d) + c, d, v, a.k_scale);
+            put_split(Kh + r * ldk + c, kRetQ * ldk, v, r < nt ? a.k_scale * row_w[part * kRetQ + r] : 0.f);
+        });
+        turned_rows<2>(rows + a.q_off, a.stride, nt, d, a.rot_dims, a.layout, turn, [&](int r, int c, float4 v) {
+            if (r < nt) put_split(q_rows + ((t1 + r) * a.H + h) * (2L * d) + c, d, v, 1.0f);
+        });
         cp_async_wait_all();
         __syncthreads();
 #pragma unroll
@@ -398,16 +396,18 @@ __global__ void __launch_bounds__(128) retention_carry_kernel(const Retention a,
     }
 }
 
-// grid (chunks, heads), 8 warps: warp w has the chunk's tokens 16 (w & 3) .. + 15 and one half of the value columns.  Shared memory: Q hi, lo | V |
-// K hi, lo, and before that the state in pieces of 64 key rows | weighted scores hi, lo.  The score tiles of 16 tokens are shared out between their two
-// warps and pass through shared memory.
+// grid (chunks, heads), 8 warps: warp w has the chunk's tokens 16 (w & 3) .. + 15 and one half of the value columns.  Shared memory: Q hi, lo | K hi,
+// lo | V | weighted scores hi, lo; ahead of the keys the state's first 64 key rows where K goes and the others where V and the scores go.  The score
+// tiles of 16 tokens are shared out between their two warps and pass through shared memory.
 constexpr int kRetLdA = kRetQ + 8;
+__host__ __device__ static inline int ret_k_elems(int d, int dv) { return 2 * kRetQ * ((d > dv ? d : dv) + 8); }      // (K rows are d columns, state rows dv)
 static size_t ret_out_smem(int d, int dv) {
-    const int wide = d > dv ? d : dv;      // (K rows are d columns, state rows dv)
-    return ((size_t)2 * kRetQ * (d + 8) + (size_t)kRetQ * (dv + 8) + (size_t)2 * kRetQ * (wide + 8) + (size_t)2 * kRetQ * kRetLdA) * sizeof(__nv_bfloat16);
+    const size_t va = (size_t)kRetQ * (dv + 8) + 2 * kRetQ * kRetLdA, state = (size_t)2 * kRetQ * (dv + 8);
+    return ((size_t)2 * kRetQ * (d + 8) + ret_k_elems(d, dv) + (d > kRetQ && state > va ? state : va)) * sizeof(__nv_bfloat16);
 }
 template <int D16MAX, int DV16MAX>
-__global__ void __launch_bounds__(256, 2) retention_chunk_out_kernel(const Retention a, const float* __restrict__ ws, __nv_bfloat16* __restrict__ out) {
+__global__ void __launch_bounds__(256, 2) retention_chunk_out_kernel(const Retention a, const float* __restrict__ ws, const __nv_bfloat16* __restrict__ q_rows,
+                                                                      const __nv_bfloat16* __restrict__ k_rows, __nv_bfloat16* __restrict__ out) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     constexpr int VT = (DV16MAX + 1) / 2;      // 16-column tiles per warp
     __shared__ int info[4];
@@ -423,27 +423,32 @@ __global__ void __launch_bounds__(256, 2) retention_chunk_out_kernel(const Reten
     const bool has_state = info[1] >= kRetSpan || a.seqs[2 * a.seqs_stride + info[0]] >= 0;
     __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(smem_raw);
     __nv_bfloat16* Ql = Qh + kRetQ * ldk;
-    __nv_bfloat16* Vs = Ql + kRetQ * ldk;
-    __nv_bfloat16* Kh = Vs + kRetQ * ldv;
+    __nv_bfloat16* Kh = Ql + kRetQ * ldk;
     __nv_bfloat16* Kl = Kh + kRetQ * ldk;
-    __nv_bfloat16 *Sh = Kh, *Sl = Kh + kRetQ * ldv;
-    __nv_bfloat16* Ah = Kh + 2 * kRetQ * ((d > dv ? d : dv) + 8);
+    __nv_bfloat16* Vs = Kh + ret_k_elems(d, dv);
+    __nv_bfloat16* Ah = Vs + kRetQ * ldv;
     __nv_bfloat16* Al = Ah + kRetQ * kRetLdA;
     const __nv_bfloat16* proj = (const __nv_bfloat16*)a.proj;
-    const __nv_bfloat16* Sg = reinterpret_cast<const __nv_bfloat16*>(ws + (((long)info[3] + info[1] / kRetSpan) * a.H + h) * d * dv);
-    const int groups = dv >> 3;
-    auto fetch_state = [&](int r0) {      // key rows r0 .. r0 + 63, groups of 8 columns [8 hi | 8 lo]
-        const int rows = min(kRetQ, d - r0);
-        for (int i = tid; i < rows * groups; i += 256) {
+    const int groups = dv >> 3, kp = d >> 3;
+    if (has_state) {      // key rows in pieces of 64, groups of 8 columns [8 hi | 8 lo]
+        const __nv_bfloat16* Sg = reinterpret_cast<const __nv_bfloat16*>(ws + (((long)info[3] + info[1] / kRetSpan) * a.H + h) * d * dv);
+        for (int i = tid; i < d * groups; i += 256) {
             const int r = i / groups, g = i - r * groups;
-            const __nv_bfloat16* src = Sg + ((long)(r0 + r) * dv + g * 8) * 2;
-            cp_async16(Sh + r * ldv + g * 8, src, true);
-            cp_async16(Sl + r * ldv + g * 8, src + 8, true);
+            const __nv_bfloat16* src = Sg + (long)i * 16;
+            __nv_bfloat16* dst = (r < kRetQ ? Kh : Vs) + (r & (kRetQ - 1)) * ldv + g * 8;
+            cp_async16(dst, src, true);
+            cp_async16(dst + kRetQ * ldv, src + 8, true);
+        }
+    }
+    auto fetch_planes = [&](__nv_bfloat16* hi, const __nv_bfloat16* rows, int n) {      // n of 64 rows [d hi | d lo], the rest zeros
+        for (int i = tid; i < kRetQ * kp; i += 256) {
+            const int r = i / kp, c = (i - r * kp) * 8;
+            const __nv_bfloat16* src = rows + (long)(r < n ? r : 0) * a.H * (2 * d) + c;
+            cp_async16(hi + r * ldk + c, src, r < n);
+            cp_async16(hi + (kRetQ + r) * ldk + c, src + d, r < n);
         }
     };
-    if (has_state) fetch_state(0);
-    const float2* turn = a.turn + t0 * (a.rot_dims >> 1);
-    stage_turned(Qh, Ql, ldk, proj + t0 * a.stride + a.q_off + (long)h * d, a.stride, nt, d, a.rot_dims, a.layout, turn, 1.0f, nullptr);
+    fetch_planes(Qh, q_rows + (t0 * a.H + h) * (2L * d), nt);
     const bool live = rg * 16 < nt;
     const int v0 = side * ((dv16 + 1) >> 1), v1 = side ? dv16 : (dv16 + 1) >> 1;      // this warp's column tiles
     float Y[2 * VT][4];
@@ -454,34 +459,27 @@ __global__ void __launch_bounds__(256, 2) retention_chunk_out_kernel(const Reten
     const int qat = (rg * 16 + (lane & 15)) * ldk + 8 * (lane >> 4);
     const int iA = rg * 16 + gq, iB = iA + 8;
     if (has_state) {
-        for (int r0 = 0; r0 < d; r0 += kRetQ) {
-            if (r0) {
-                __syncthreads();      // the previous piece is consumed
-                fetch_state(r0);
-            }
-            cp_async_wait_all();
-            __syncthreads();
-            if (live) {
-                const int k16 = min(4, (d - r0) >> 4);
+        cp_async_wait_all();
+        __syncthreads();
+        if (live) {
 #pragma unroll 2
-                for (int kk = 0; kk < k16; kk++) {
-                    uint32_t qh[4], ql[4];
-                    ldmatrix_x4(qh, Qh + qat + r0 + kk * 16);
-                    ldmatrix_x4(ql, Ql + qat + r0 + kk * 16);
+            for (int kk = 0; kk < d16; kk++) {
+                uint32_t qh[4], ql[4];
+                ldmatrix_x4(qh, Qh + qat + kk * 16);
+                ldmatrix_x4(ql, Ql + qat + kk * 16);
+                const __nv_bfloat16* Sk = (kk < 4 ? Kh : Vs) + ((kk & 3) * 16 + (lane & 15)) * ldv + 8 * (lane >> 4);
 #pragma unroll
-                    for (int vp = 0; vp < VT; vp++) {
-                        if (v0 + vp < v1) {
-                            uint32_t bh[4], bl[4];
-                            const int at = (kk * 16 + (lane & 15)) * ldv + (v0 + vp) * 16 + 8 * (lane >> 4);
-                            ldmatrix_x4_trans(bh, Sh + at);
-                            ldmatrix_x4_trans(bl, Sl + at);
-                            mma_bf16_16816(Y[2 * vp], qh, bh[0], bh[1]);
-                            mma_bf16_16816(Y[2 * vp + 1], qh, bh[2], bh[3]);
-                            mma_bf16_16816(Y[2 * vp], ql, bh[0], bh[1]);
-                            mma_bf16_16816(Y[2 * vp + 1], ql, bh[2], bh[3]);
-                            mma_bf16_16816(Y[2 * vp], qh, bl[0], bl[1]);
-                            mma_bf16_16816(Y[2 * vp + 1], qh, bl[2], bl[3]);
-                        }
+                for (int vp = 0; vp < VT; vp++) {
+                    if (v0 + vp < v1) {
+                        uint32_t bh[4], bl[4];
+                        ldmatrix_x4_trans(bh, Sk + (v0 + vp) * 16);
+                        ldmatrix_x4_trans(bl, Sk + kRetQ * ldv + (v0 + vp) * 16);
+                        mma_bf16_16816(Y[2 * vp], qh, bh[0], bh[1]);
+                        mma_bf16_16816(Y[2 * vp + 1], qh, bh[2], bh[3]);
+                        mma_bf16_16816(Y[2 * vp], ql, bh[0], bh[1]);
+                        mma_bf16_16816(Y[2 * vp + 1], ql, bh[2], bh[3]);
+                        mma_bf16_16816(Y[2 * vp], qh, bl[0], bl[1]);
+                        mma_bf16_16816(Y[2 * vp + 1], qh, bl[2], bl[3]);
                     }
                 }
             }
@@ -499,9 +497,9 @@ __global__ void __launch_bounds__(256, 2) retention_chunk_out_kernel(const Reten
     for (int back = behind; back >= 0; back -= kRetQ) {
         const long t1 = t0 - back;
         const int kt = back ? kRetQ : nt;
-        __syncthreads();      // the state's last piece, or the keys and scores ahead, are consumed
+        if (has_state || back != behind) __syncthreads();      // the state, or the keys and scores ahead, are consumed
         fetch_rows(Vs, ldv, proj + t1 * a.stride + a.v_off + (long)h * dv, a.stride, kt, dv);
-        stage_turned(Kh, Kl, ldk, proj + t1 * a.stride + a.k_off + (long)h * d, a.stride, kt, d, a.rot_dims, a.layout, a.turn + t1 * (a.rot_dims >> 1), a.k_scale, nullptr);
+        fetch_planes(Kh, k_rows + (t1 * a.H + h) * (2L * d), kt);
         cp_async_wait_all();
         __syncthreads();
         const int tiles = back ? kRetQ / 16 : rg + 1;      // key tiles of 16 that the warp's tokens see
@@ -762,7 +760,7 @@ extern "C" int ktb200_retention_chunk_supported(int dim, int vdim, int dtype) {
 }
 static long ret_tiles(int n_tokens, int n_seqs, int per) { return n_tokens / per + n_seqs; }      // (an upper bound: whole tiles and one partial per portion)
 extern "C" size_t ktb200_retention_chunk_workspace(int heads, int dim, int vdim, int n_tokens, int n_seqs) {
-    return (size_t)ret_tiles(n_tokens, n_seqs, kRetSpan) * heads * dim * vdim * sizeof(float);
+    return (size_t)ret_tiles(n_tokens, n_seqs, kRetSpan) * heads * dim * vdim * sizeof(float) + (size_t)n_tokens * heads * dim * 4 * sizeof(__nv_bfloat16);
 }
 
 extern "C" int ktb200_retention_chunk(const ktb200_retention_params* c, void* out, int n_tokens, void* workspace, size_t workspace_bytes, int dtype, void* stream) {
@@ -775,11 +773,13 @@ extern "C" int ktb200_retention_chunk(const ktb200_retention_params* c, void* ou
     if (n_tokens <= 0 || c->n_seqs <= 0) return KTB200_OK;
     const Retention a = ret_args(c);
     float* ws = (float*)workspace;
+    __nv_bfloat16* q_rows = reinterpret_cast<__nv_bfloat16*>(ws + (size_t)ret_tiles(n_tokens, c->n_seqs, kRetSpan) * c->heads * c->dim * c->vdim);
+    __nv_bfloat16* k_rows = q_rows + (size_t)n_tokens * c->heads * c->dim * 2;
     cudaStream_t st = (cudaStream_t)stream;
     const dim3 spans((unsigned)ret_tiles(n_tokens, c->n_seqs, kRetSpan), c->heads), chunks((unsigned)ret_tiles(n_tokens, c->n_seqs, kRetQ), c->heads);
     const size_t s1 = ((size_t)2 * kRetQ * (c->dim + 8) + (size_t)kRetQ * (c->vdim + 8)) * sizeof(__nv_bfloat16);
     GRANT_SMEM(retention_chunk_state_kernel, s1);
-    retention_chunk_state_kernel<<<spans, 256, s1, st>>>(a, ws);
+    retention_chunk_state_kernel<<<spans, 256, s1, st>>>(a, ws, q_rows, k_rows);
     KTB_LAUNCH_CHECK();
     retention_carry_kernel<<<dim3((c->dim * c->vdim / 8 + 127) / 128, c->heads, c->n_seqs), 128, 0, st>>>(a, ws);
     KTB_LAUNCH_CHECK();
@@ -787,7 +787,7 @@ extern "C" int ktb200_retention_chunk(const ktb200_retention_params* c, void* ou
 #define OUT_LAUNCH(DK, DV)                                                                                      \
     do {                                                                                                        \
         GRANT_SMEM((retention_chunk_out_kernel<DK, DV>), s3);                                                   \
-        retention_chunk_out_kernel<DK, DV><<<chunks, 256, s3, st>>>(a, ws, (__nv_bfloat16*)out);                  \
+        retention_chunk_out_kernel<DK, DV><<<chunks, 256, s3, st>>>(a, ws, q_rows, k_rows, (__nv_bfloat16*)out);                  \
     } while (0)
     if (c->dim <= 64 && c->vdim <= 64) OUT_LAUNCH(4, 4);
     else if (c->vdim <= 64) OUT_LAUNCH(8, 4);

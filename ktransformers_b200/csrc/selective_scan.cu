@@ -91,6 +91,15 @@ template <> struct RawVec<__nv_bfloat16, 4> { using type = uint2; };
 template <> struct RawVec<__nv_bfloat16, 1> { using type = __nv_bfloat16; };
 template <> struct RawVec<float, 4> { using type = float4; };
 template <> struct RawVec<float, 1> { using type = float; };
+// (volatile: issued where they stand, ahead of the tokens that run meanwhile)
+__device__ __forceinline__ void load_ahead(uint2& r, const void* p) { asm volatile("ld.global.nc.v2.u32 {%0, %1}, [%2];" : "=r"(r.x), "=r"(r.y) : "l"(p)); }
+__device__ __forceinline__ void load_ahead(float4& r, const void* p) { asm volatile("ld.global.nc.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(r.x), "=f"(r.y), "=f"(r.z), "=f"(r.w) : "l"(p)); }
+__device__ __forceinline__ void load_ahead(float& r, const void* p) { asm volatile("ld.global.nc.f32 %0, [%1];" : "=f"(r) : "l"(p)); }
+__device__ __forceinline__ void load_ahead(__nv_bfloat16& r, const void* p) {
+    unsigned short u;
+    asm volatile("ld.global.nc.u16 %0, [%1];" : "=h"(u) : "l"(p));
+    r = __ushort_as_bfloat16(u);
+}
 template <typename T, int VEC> __device__ __forceinline__ void unpack(float (&v)[VEC], const typename RawVec<T, VEC>::type& r) {
     const T* p = reinterpret_cast<const T*>(&r);
 #pragma unroll
@@ -162,9 +171,9 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const SelScan a, T*
             rx[e] = rdt[e] = rz[e] = RX{};
             if (tt < nt && sok) {
                 const long t = t0 + tt;
-                rx[e] = *reinterpret_cast<const RX*>(xp + t * inner);
-                rdt[e] = *reinterpret_cast<const RX*>(dp + t * a.dt_stride);
-                rz[e] = *reinterpret_cast<const RX*>(zp + t * a.z_stride);
+                load_ahead(rx[e], xp + t * inner);
+                load_ahead(rdt[e], dp + t * a.dt_stride);
+                load_ahead(rz[e], zp + t * a.z_stride);
             }
         }
 #pragma unroll
@@ -173,8 +182,8 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const SelScan a, T*
             rb[e] = rc[e] = RB{};
             if (tt < nt && n < N) {
                 const long t = start + t0 + tt;
-                rb[e] = *reinterpret_cast<const RB*>((const T*)a.B + t * a.bc_stride + n);
-                rc[e] = *reinterpret_cast<const RB*>((const T*)a.C + t * a.bc_stride + n);
+                load_ahead(rb[e], (const T*)a.B + t * a.bc_stride + n);
+                load_ahead(rc[e], (const T*)a.C + t * a.bc_stride + n);
             }
         }
     };
