@@ -225,6 +225,27 @@ def test_grouped_softmax_router(outputs, top, groups, keep, width, n, shift):
     assert top == outputs or n < 100 or plain.tolist() != want_ids.tolist()
 
 
+@gpu
+@pytest.mark.parametrize("outputs,top,groups,keep", [(13, 3, 1, 1), (24, 5, 4, 2), (320, 8, 8, 3)])
+@pytest.mark.parametrize("n", [1, 6, 200])
+@pytest.mark.parametrize("width", [64, 72, 1024, 50])
+def test_router_on_bf16_rows(outputs, top, groups, keep, n, width):
+    """bf16 rows and bf16 router weights: one GEMM with exact products and fp32 sums at every batch size; weights that are no bf16 numbers, or a
+    width the GEMM does not take, keep to fp32 products"""
+    from ktransformers_b200.operators.gate import KGroupedSoftmaxGate
+    g = torch.Generator().manual_seed(n + outputs)
+    x, corr = torch.randn(n, width, generator=g).bfloat16(), torch.randn(outputs, generator=g) * 0.3
+    for rounded in (True, False):
+        W = torch.randn(outputs, width, generator=g) * 3.0 / width ** 0.5
+        W = W.bfloat16() if rounded else W
+        op = KGroupedSoftmaxGate(width, outputs, top, groups, keep, 1.5)
+        op.load(DictLoader({"r": W, "c": corr}), "r", "c")
+        assert (op.weight_bf16 is not None) == (rounded and width % 8 == 0)
+        ids, wts = op(x.cuda())
+        want_ids, want_w = O.grouped_softmax_router(x.double(), W.double(), corr.double(), top, groups, keep, 1.5)
+        assert ids.cpu().tolist() == want_ids.tolist() and rel(wts, want_w) < 1e-5
+
+
 def test_router_refuses_impossible_sizes():
     from ktransformers_b200.operators.gate import KGroupedSoftmaxGate
     for outputs, top, groups, keep in ((7, 1, 2, 1), (8, 5, 2, 1), (8, 2, 2, 3), (8, 2, 2, 0), (600, 2, 2, 1), (64, 33, 1, 1)):
