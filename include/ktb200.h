@@ -666,7 +666,7 @@ typedef struct {
 } ktb200_selective_scan_params;
 int ktb200_conv_silu(const void* in, long in_stride, const void* conv_w, const void* conv_b, int taps, int channels, const int* seq_of, const int* seqs,
                      int seqs_stride, float* state, long state_stride, long conv_off, void* out, int n_tokens, int n_seqs, int dtype, void* stream);
-int ktb200_selective_scan(const ktb200_selective_scan_params* params, void* out, int dtype, void* stream);
+int ktb200_selective_scan(const ktb200_selective_scan_params* params, void* out, int n_tokens, int dtype, void* stream);
 
 /* Diagnostics (bench.py --probe): time a plain read-only stream over `bytes` of device memory.
  * mode 0 = grid-stride coalesced 16-byte loads; mode 1 = every warp reads chunk_bytes pieces at hashed offsets

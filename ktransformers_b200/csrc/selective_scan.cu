@@ -2,7 +2,7 @@
 //
 //   dt = softplus(dt_logit + dt_bias_c) ;  S_cn <- exp(dt a_cn) S_cn + dt x_c B_n ;  y_c = sum_n S_cn C_n + D_c x_c ;  out_c = y_c silu(z_c)
 //
-//   ktb200_selective_scan   prompt portions and decode steps alike, one launch (its x: ktb200_conv_silu, csrc/ssd.cu)
+//   ktb200_selective_scan   steps, recurrence, skip and gate of prompt portions or of decode steps in one launch (its x: ktb200_conv_silu, csrc/ssd.cu)
 //
 // State row of a sequence and layer (fp32): [ S inner x state_size | filter inputs (taps - 1) x inner, oldest first ], read from the row seqs[2][s] (or
 // zeros when -1) and written to the row seqs[3][s].  Storage type T (bf16 or float) for projections, the filtered channels and the output; steps,
@@ -111,7 +111,7 @@ template <typename T, int VEC> __device__ __forceinline__ void unpack(float (&v)
 // at a time are added over the lanes of a channel so that every shuffle halves the tokens a lane still holds.  VX, VB: values per access of the
 // rows of x, dt, z (out) and of B, C.
 template <typename T, int SPT, int L, int VX, int VB>
-__global__ void __launch_bounds__(128) selective_scan_kernel(const SelScan a, T* __restrict__ out) {
+__global__ void __launch_bounds__(128, 4) selective_scan_kernel(const SelScan a, T* __restrict__ out) {
     using M = ScanMath<T>;
     constexpr int CH = 128 / L, CP = CH + 8, NP = SPT * L, TC = L <= 2 ? 16 : (NP <= 64 ? 32 : (NP <= 128 ? 16 : 8));
     constexpr int GX = CH / VX, GB = NP / VB;      // accesses per token
@@ -300,6 +300,66 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const SelScan a, T*
     }
 }
 
+// One token per portion: grid (blocks of channels x L lanes, portions), no shared memory.  L lanes (a power of two) share a channel, four neighbouring
+// states each at a time; what a channel needs besides is read by all of its lanes.
+constexpr int kStepThreads = 128;
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kStepThreads) selective_scan_step_kernel(const SelScan a, int L, T* __restrict__ out) {
+    using M = ScanMath<T>;
+    const long i = blockIdx.x * (long)kStepThreads + threadIdx.x;
+    const int s = blockIdx.y, N = a.N, l = (int)(i % L), ch = (int)min(i / L, (long)a.inner - 1);      // (lanes behind the last channel repeat it, and store nothing)
+    const bool live = i / L < a.inner;
+    const long t = a.seqs[s], at = (long)ch * N;
+    const int rd = a.seqs[2 * a.seqs_stride + s], wr = a.seqs[3 * a.seqs_stride + s];
+    const float x = to_f(((const T*)a.x)[t * a.inner + ch]), z = to_f(((const T*)a.z)[t * a.z_stride + ch]);
+    const float dt = M::softplus(to_f(((const T*)a.dt)[t * a.dt_stride + ch]) + a.dt_bias[ch]), dx = dt * x;
+    const T *B = (const T*)a.B + t * a.bc_stride, *Cv = (const T*)a.C + t * a.bc_stride;
+    const float* Sr = a.state + (long)rd * a.state_stride + at;
+    float* Sw = a.state + (long)wr * a.state_stride + at;
+    uint64_t y = 0;      // (two zeros)
+    for (int n = 4 * l; n < N; n += 4 * L) {
+        float4 f, v = make_float4(0.f, 0.f, 0.f, 0.f), b = v, c = v;
+        if (VEC) {
+            f = load4(a.A + at + n);
+            if (rd >= 0) v = load4(Sr + n);
+            b = load4(B + n);
+            c = load4(Cv + n);
+        } else {
+            float u[4][4];
+#pragma unroll
+            for (int k = 0; k < 4; k++) {
+                const bool in = n + k < N;
+                u[0][k] = in ? a.A[at + n + k] : 0.f;
+                u[1][k] = in && rd >= 0 ? Sr[n + k] : 0.f;
+                u[2][k] = in ? to_f(B[n + k]) : 0.f;
+                u[3][k] = in ? to_f(Cv[n + k]) : 0.f;
+            }
+            f = make_float4(u[0][0], u[0][1], u[0][2], u[0][3]);
+            v = make_float4(u[1][0], u[1][1], u[1][2], u[1][3]);
+            b = make_float4(u[2][0], u[2][1], u[2][2], u[2][3]);
+            c = make_float4(u[3][0], u[3][1], u[3][2], u[3][3]);
+        }
+        uint64_t S0 = pair_of(v.x, v.y), S1 = pair_of(v.z, v.w);
+        M::step(S0, pair_of(M::factor(f.x), M::factor(f.y)), dt, dx, make_float2(b.x, b.y), make_float2(c.x, c.y), y);
+        M::step(S1, pair_of(M::factor(f.z), M::factor(f.w)), dt, dx, make_float2(b.z, b.w), make_float2(c.z, c.w), y);
+        if (wr >= 0 && live) {
+            const float2 p = halves_of(S0), q = halves_of(S1);
+            if (VEC) {
+                store4(Sw + n, make_float4(p.x, p.y, q.x, q.y));
+            } else {
+                const float w[4] = {p.x, p.y, q.x, q.y};
+#pragma unroll
+                for (int k = 0; k < 4; k++)
+                    if (n + k < N) Sw[n + k] = w[k];
+            }
+        }
+    }
+    const float2 two = halves_of(y);
+    float sum = two.x + two.y;
+    for (int o = 1; o < L; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    if (live && l == 0) out[t * a.inner + ch] = from_f<T>(fmaf(a.D[ch], x, sum) * silu_for<T>(z));
+}
+
 }  // namespace ktb
 
 using namespace ktb;
@@ -311,13 +371,13 @@ using namespace ktb;
         else { set_error("dtype must be bf16 or f32"); return KTB200_EINVAL; }             \
     } while (0)
 
-extern "C" int ktb200_selective_scan(const ktb200_selective_scan_params* c, void* out, int dtype, void* stream) {
+extern "C" int ktb200_selective_scan(const ktb200_selective_scan_params* c, void* out, int n_tokens, int dtype, void* stream) {
     if (!c || !c->x || !c->dt_logit || !c->b || !c->c || !c->z || !c->dt_bias || !c->a || !c->d_skip || !c->seqs || !c->state || !out || c->inner <= 0 || c->state_size <= 0 ||
         c->state_size > 256) {
         set_error("selective_scan: bad argument (state size <= 256)");
         return KTB200_EINVAL;
     }
-    if (c->n_seqs <= 0) return KTB200_OK;
+    if (c->n_seqs <= 0 || n_tokens <= 0) return KTB200_OK;
     const int N = c->state_size;
     const size_t esz = dtype == KTB200_TYPE_BF16 ? 2 : 4;
     auto al = [](const void* p, size_t b) { return (reinterpret_cast<uintptr_t>(p) & (b - 1)) == 0; };
@@ -327,6 +387,17 @@ extern "C" int ktb200_selective_scan(const ktb200_selective_scan_params* c, void
     const bool vec = c->inner % 4 == 0 && N % 4 == 0 && c->dt_stride % 4 == 0 && c->z_stride % 4 == 0 && c->bc_stride % 4 == 0 && al(c->x, 4 * esz) && al(c->dt_logit, 4 * esz) &&
                      al(c->z, 4 * esz) && al(c->b, 4 * esz) && al(c->c, 4 * esz) && al(out, 4 * esz);
     const cudaStream_t st = (cudaStream_t)stream;
+    if (n_tokens == c->n_seqs) {
+        int L = 1;
+        while (L < 32 && 4 * L < N) L <<= 1;
+        const dim3 grid((unsigned)(((long)c->inner * L + kStepThreads - 1) / kStepThreads), c->n_seqs);
+        SEQ_DISPATCH(dtype, {
+            if (vec && a.vec_state) selective_scan_step_kernel<T, true><<<grid, kStepThreads, 0, st>>>(a, L, (T*)out);
+            else selective_scan_step_kernel<T, false><<<grid, kStepThreads, 0, st>>>(a, L, (T*)out);
+        });
+        KTB_LAUNCH_CHECK();
+        return KTB200_OK;
+    }
 #define SCAN_LAUNCH(SPT, L)                                                                                     \
     SEQ_DISPATCH(dtype, {                                                                                       \
         const dim3 grid((c->inner + 128 / (L) - 1) / (128 / (L)), c->n_seqs);                                   \

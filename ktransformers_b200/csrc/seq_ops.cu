@@ -294,11 +294,14 @@ __global__ void __launch_bounds__(NV == 0 ? 256 : (NV > 4 ? 512 : 1024)) sum_rms
     const T *w = (const T*)p.w, *dw = (const T*)p.dot_w;
     T* h_out = (T*)p.h_out;
     float xs = p.x_scale;
-    if (p.ids)
-        for (int j = 0; j < p.top; j++) {      // (the same few numbers for every thread)
-            const float iw = p.id_w[row * p.top + j];
-            if (p.ids[row * p.top + j] >= p.first_identity) xs += iw;
+    if (p.ids) {      // the row's choices over the lanes of every warp
+        float iw = 0.f;
+        for (int j = tid & 31; j < p.top; j += 32) {
+            const float w_j = p.id_w[row * p.top + j];
+            if (p.ids[row * p.top + j] >= p.first_identity) iw += w_j;
         }
+        xs += warp_sum(iw);
+    }
     const float bs = p.b && p.b_scale ? p.b_scale[row] : 1.0f;
     float dot = 0.f;
     if (NV > 0) {

@@ -200,7 +200,7 @@ SEQ_SYMBOLS = {
     "ktb200_retention_scan": (_I, [C.POINTER(RetentionParams), _VP, _I, _VP]),
     "ktb200_retention_step_max_vdim": (_I, []),
     "ktb200_retention_step": (_I, [C.POINTER(RetentionParams), _VP, _I, _VP]),
-    "ktb200_selective_scan": (_I, [C.POINTER(SelectiveScanParams), _VP, _I, _VP]),
+    "ktb200_selective_scan": (_I, [C.POINTER(SelectiveScanParams), _VP, _I, _I, _VP]),
     # csrc/ssd.cu
     "ktb200_conv_silu": (_I, [_VP, _L, _VP, _VP, _I, _I, _VP, _VP, _I, _VP, _L, _L, _VP, _I, _I, _I, _VP]),
     "ktb200_ssd_conv": (_I, [C.POINTER(SsdParams), _VP, _I, _I, _VP]),

@@ -355,5 +355,5 @@ class KSelectiveScan(nn.Module):
                                        d_skip=self.d_skip.data_ptr(), inner=s.inner, state_size=s.state_size, seqs=batch.seqs.data_ptr(), seqs_stride=batch.seqs.stride(0),
                                        n_seqs=batch.n_seqs, state=state.data_ptr(), state_stride=state.stride(0))
         y = torch.empty((T, s.inner), dtype=dt, device=dev)
-        native.check_seq(lib.ktb200_selective_scan(C.byref(a), y.data_ptr(), code, st))
+        native.check_seq(lib.ktb200_selective_scan(C.byref(a), y.data_ptr(), T, code, st))
         return nn.functional.linear(y, self.o)

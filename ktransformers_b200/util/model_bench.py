@@ -1212,7 +1212,7 @@ def lipadra_kernel_leg(flush, peak_gbs, peak_tf):
     bias, A, Dk = rn(I, dt=f32) - 3.0, -torch.arange(1, N1 + 1, device=dev, dtype=f32).repeat(I, 1).contiguous(), rn(I, dt=f32)
     props = torch.cuda.get_device_properties(0)
     ex_per_s = props.multi_processor_count * 16 * 1.965e9
-    for B, T in ((1, 1), (8, 1), (1, 2048), (8, 256)):
+    for B, T in ((1, 1), (8, 1), (32, 1), (1, 2048), (8, 256)):      # (32 sequences hold as many state bytes as eight of the state-space layer's)
         bt = KernelBatch([T] * B, max(T, 64), dev)
         n, it = B * T, 5 if T > 1 else 10
         proj, p, step, x, y = rn(n, 2 * I), rn(n, bcw), rn(n, I), torch.empty(n, I, dtype=bf, device=dev), torch.empty(n, I, dtype=bf, device=dev)
@@ -1225,7 +1225,7 @@ def lipadra_kernel_leg(flush, peak_gbs, peak_tf):
         a = native.SelectiveScanParams(x=x.data_ptr(), dt_logit=step.data_ptr(), b=p[:, R_:].data_ptr(), c=p[:, R_ + N1:].data_ptr(), z=proj[:, I:].data_ptr(), dt_stride=I, bc_stride=bcw, z_stride=2 * I,
                                        dt_bias=bias.data_ptr(), a=A.data_ptr(), d_skip=Dk.data_ptr(), inner=I, state_size=N1, seqs=bt.seqs.data_ptr(), seqs_stride=B, n_seqs=B, state=state.data_ptr(),
                                        state_stride=state.stride(0))
-        ms = timed(lambda: ok(seq.ktb200_selective_scan(C.byref(a), y.data_ptr(), 30, S())), flush, iters=it)
+        ms = timed(lambda: ok(seq.ktb200_selective_scan(C.byref(a), y.data_ptr(), n, 30, S())), flush, iters=it)
         sproj, sstate = rn(n, s_in), torch.zeros(2 * B, sw, device=dev)
         xbc, sy = torch.empty(n, C_, dtype=bf, device=dev), torch.empty(n, inner2, device=dev)
         sa = native.SsdParams(proj=sproj.data_ptr(), proj_stride=s_in, xbc_off=inner2, dt_off=inner2 + C_, conv_w=scw.data_ptr(), conv_b=scb.data_ptr(), taps=taps, dt_bias=dtb.data_ptr(),

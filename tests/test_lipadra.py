@@ -636,34 +636,36 @@ def test_selective_scan_alone(dtype, tol, desc):
 
 @gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("I,N", [(37, 16), (64, 5), (200, 1), (16, 128), (5, 200), (300, 32)])
+@pytest.mark.parametrize("I,N", [(37, 16), (64, 16), (64, 5), (200, 1), (16, 128), (5, 200), (8, 200), (300, 32), (36, 8), (132, 4), (20, 64)])
+@pytest.mark.parametrize("portions", [True, False])
 @pytest.mark.parametrize("rate", [-7.0, 0.0, 3.0])
-def test_selective_scan_kernel_on_rows(dtype, I, N, rate):
+def test_selective_scan_kernel_on_rows(dtype, I, N, rate, portions):
     """the recurrence, skip and gate against the restatement, outputs and states: portions on, before and after the staging edge, one starting from a
     state; decays from almost one to almost zero, steps from almost none to past the soft-plus's straight part"""
     from ktransformers_b200 import native
-    lib, lens, g = native.seq_lib(), [16, 17, 70, 1, 3, 32], torch.Generator().manual_seed(I * N)
+    lib, lens, g = native.seq_lib(), [16, 17, 70, 1, 3, 32] if portions else [1] * 6, torch.Generator().manual_seed(I * N)
     T, code = sum(lens), 30 if dtype == torch.bfloat16 else 0
     rn = lambda *s: torch.randn(*s, generator=g)
-    x, dtl, bc, z = rn(T, I).to(dtype), (2.0 * rn(T, I)).to(dtype), rn(T, 2 * N + 3).to(dtype), rn(T, I + 2).to(dtype)
+    pad, lo_b = (4, 4) if I % 4 == 0 and N % 4 == 0 else (3, 1)      # rows in groups of four, or not
+    x, dtl, bc, z = rn(T, I).to(dtype), (2.0 * rn(T, I)).to(dtype), rn(T, 2 * N + pad).to(dtype), rn(T, I + pad).to(dtype)
     dtl[::7], dtl[3::11] = -9.0, 25.0
     bias, al, D, before = rn(I), torch.full((I, N), rate) + 0.3 * rn(I, N), rn(I), rn(I, N)
     starts = [sum(lens[:i]) for i in range(len(lens))]
     seqs = torch.tensor([starts, lens, [-1, 2, -1, -1, -1, -1], [7 + i for i in range(len(lens))]], dtype=torch.int32).cuda()
-    state = torch.zeros(20, I * N + 3)
+    state = torch.zeros(20, I * N + pad)
     state[2, :I * N] = before.reshape(-1)
     dev = [t.cuda() for t in (x, dtl, bc, z, bias, -torch.exp(al), D, state)]
     y = torch.full((T, I), float("nan"), dtype=dtype, device="cuda")
-    a = native.SelectiveScanParams(x=dev[0].data_ptr(), dt_logit=dev[1].data_ptr(), b=dev[2][:, 1:].data_ptr(), c=dev[2][:, N + 1:].data_ptr(), z=dev[3].data_ptr(), dt_stride=I,
-                                   bc_stride=2 * N + 3, z_stride=I + 2, dt_bias=dev[4].data_ptr(), a=dev[5].data_ptr(), d_skip=dev[6].data_ptr(), inner=I, state_size=N, seqs=seqs.data_ptr(),
+    a = native.SelectiveScanParams(x=dev[0].data_ptr(), dt_logit=dev[1].data_ptr(), b=dev[2][:, lo_b:].data_ptr(), c=dev[2][:, N + lo_b:].data_ptr(), z=dev[3].data_ptr(), dt_stride=I,
+                                   bc_stride=2 * N + pad, z_stride=I + pad, dt_bias=dev[4].data_ptr(), a=dev[5].data_ptr(), d_skip=dev[6].data_ptr(), inner=I, state_size=N, seqs=seqs.data_ptr(),
                                    seqs_stride=len(lens), n_seqs=len(lens), state=dev[7].data_ptr(), state_stride=dev[7].stride(0))
-    native.check_seq(lib.ktb200_selective_scan(C.byref(a), y.data_ptr(), code, torch.cuda.current_stream().cuda_stream))
+    native.check_seq(lib.ktb200_selective_scan(C.byref(a), y.data_ptr(), T, code, torch.cuda.current_stream().cuda_stream))
     xd, bcd = x.double(), bc.double()
     dt = O.softplus(dtl.double() + bias.double())
     for i, (lo, n) in enumerate(zip(starts, lens)):
         r = slice(lo, lo + n)
         S0 = before.double() if i == 1 else torch.zeros(I, N).double()
-        want, st = O.selective_scan(xd[r], dt[r], -torch.exp(al.double()), bcd[r, 1:N + 1], bcd[r, N + 1:2 * N + 1], D.double(), S0)
+        want, st = O.selective_scan(xd[r], dt[r], -torch.exp(al.double()), bcd[r, lo_b:N + lo_b], bcd[r, N + lo_b:2 * N + lo_b], D.double(), S0)
         want = want * O.silu(z[r, :I].double())
         assert rel(y[r], want) < (1e-2 if dtype == torch.bfloat16 else 2e-5)
         assert rel(dev[7][7 + i, :I * N], st.reshape(-1)) < 2e-5
