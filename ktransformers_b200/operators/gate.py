@@ -240,11 +240,12 @@ class KGroupedSoftmaxGate(nn.Module):
     times `out_scale`, not normalised: the router kernel's `scoring = softmax, topk_method = biased_group_max` case.
 
     Logits: for bf16 activations and router weights that are bf16 numbers (as checkpoints ship them) every product is exact in fp32, and the
-    library's tensor-core GEMM with fp32 accumulation and fp32 output makes the fp32 logits at any batch size.  Otherwise, as for
-    KGroupedSigmoidGate: decode-sized batches run the one-launch kernel, batches from `gemm_min_tokens` tokens an fp32 library GEMM (TF32 off).
-    The selection behind a GEMM is `ktb200_moe_gate_select`."""
+    library's tensor-core GEMM with fp32 accumulation and fp32 output makes the fp32 logits from `bf16_min_tokens` tokens on.  Otherwise, as
+    for KGroupedSigmoidGate: decode-sized batches run the one-launch kernel, batches from `gemm_min_tokens` tokens an fp32 library GEMM (TF32
+    off).  The selection behind a GEMM is `ktb200_moe_gate_select`."""
 
     gemm_min_tokens = 48
+    bf16_min_tokens = 4
 
     def __init__(self, width: int, outputs: int, top: int, groups: int, keep_groups: int, out_scale: float, device="cuda"):
         super().__init__()
@@ -273,7 +274,7 @@ class KGroupedSoftmaxGate(nn.Module):
         cfg = native.GateConfig(self.outputs, self.width, self.top, self.groups, self.keep_groups, _SCORING["softmax"], _TOPK["biased_group_max"], 0, self.out_scale,
                                 self.weight.data_ptr(), self.correction.data_ptr(), TORCH_TO_GGML_HIDDEN[x.dtype])
         st = torch.cuda.current_stream(x.device).cuda_stream
-        if x.dtype == torch.bfloat16 and self.weight_bf16 is not None:
+        if n >= self.bf16_min_tokens and x.dtype == torch.bfloat16 and self.weight_bf16 is not None:
             logits = torch.mm(x, self.weight_bf16.t(), out_dtype=torch.float32)
             native.check_seq(native.seq_lib().ktb200_moe_gate_select(C.byref(cfg), n, logits.data_ptr(), idx.data_ptr(), wt.data_ptr(), st))
         elif n >= self.gemm_min_tokens or self.width % 4:

@@ -1245,6 +1245,7 @@ def lipadra_kernel_leg(flush, peak_gbs, peak_tf):
     mine, theirs = KGroupedSoftmaxGate(D, E, top, 8, 4, 2.0), KGroupedSigmoidGate(D, E, top, 8, 4, 2.0)
     mine.weight.data.copy_((rn(E, D, dt=f32) * D ** -0.5).bfloat16().float())
     theirs.weight.data.copy_(mine.weight.data)
+    mine.bf16_min_tokens = 1
     for T in (1, 8, 2048):
         x, nb = rn(T, D), E * D * 4 + T * D * 2
         peer = K.measure("grouped sigmoid: " + ("gate_kernel" if T < mine.gemm_min_tokens else "fp32 GEMM + gate_select_kernel"), timed(lambda: theirs(x), flush), nb)

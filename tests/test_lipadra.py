@@ -230,7 +230,7 @@ def test_grouped_softmax_router(outputs, top, groups, keep, width, n, shift):
 @pytest.mark.parametrize("n", [1, 6, 200])
 @pytest.mark.parametrize("width", [64, 72, 1024, 50])
 def test_router_on_bf16_rows(outputs, top, groups, keep, n, width):
-    """bf16 rows and bf16 router weights: one GEMM with exact products and fp32 sums at every batch size; weights that are no bf16 numbers, or a
+    """bf16 rows and bf16 router weights: one GEMM with exact products and fp32 sums beyond a few tokens; weights that are no bf16 numbers, or a
     width the GEMM does not take, keep to fp32 products"""
     from ktransformers_b200.operators.gate import KGroupedSoftmaxGate
     g = torch.Generator().manual_seed(n + outputs)
